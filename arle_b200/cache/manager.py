@@ -200,17 +200,16 @@ class CacheManager:
             self._tokens[rid] = new_total
 
     def release_passed(self, rid) -> int:
-        """Give back the pages of window groups that no later query of rid can see:
-        a query at position p >= tokens sees keys >= p - window + 1, so a page whose
-        last token lies before tokens - window + 1 is done; the pages of the first tokens
-        that the group's need keeps visible stay.  Returns pages freed."""
+        """Give back the pages of window and chunk groups that no later query of rid can see:
+        a query at position p >= tokens sees keys >= p - window + 1 (or from the start of its
+        chunk on), so a page whose last token lies before that of p = tokens is done; the pages
+        of the first tokens that the group's need keeps visible stay.  Returns pages freed."""
         slot, n = self._slot_of[rid], self._tokens[rid]
         freed = 0
         for g in self.groups:
-            w = g.need.window
-            if w is None:
+            if g.need.window is None and g.need.chunk is None:
                 continue
-            first_needed_token = max(0, n - w + 1)
+            first_needed_token = g.need.first_needed(n)
             upto = min(first_needed_token // g.page_size, int(g.num_logical[slot]))
             lo = max(int(g.first_held[slot]), min(g.kept_pages, int(g.num_logical[slot])))
             if upto > lo:

@@ -1,4 +1,5 @@
 from .model_spec import ModelSpec, ScheduleEntry
+from .dabilorn import DabilornConfig
 from .kolodra import KolodraConfig
 from .lasupel import LasupelConfig
 from .lukinex import LukinexConfig
@@ -12,6 +13,7 @@ register_architecture(KolodraConfig.architecture, KolodraConfig)
 register_architecture(ZuderaxConfig.architecture, ZuderaxConfig)
 register_architecture(LasupelConfig.architecture, LasupelConfig)
 register_architecture(LukinexConfig.architecture, LukinexConfig)
+register_architecture(DabilornConfig.architecture, DabilornConfig)
 
-__all__ = ["ModelSpec", "ScheduleEntry", "ConfigError", "Qwen3Config", "KolodraConfig", "ZuderaxConfig", "LasupelConfig", "LukinexConfig", "UnknownArchitecture", "config_class_for",
+__all__ = ["ModelSpec", "ScheduleEntry", "ConfigError", "Qwen3Config", "KolodraConfig", "ZuderaxConfig", "LasupelConfig", "LukinexConfig", "DabilornConfig", "UnknownArchitecture", "config_class_for",
            "config_from_dict", "load_config", "register_architecture", "registered_architectures"]

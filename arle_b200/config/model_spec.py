@@ -40,6 +40,7 @@ class ModelSpec:
     embed_scale: float = 1.0                  # the embedding row is multiplied by this
     logit_cap: Optional[float] = None         # logits <- cap * tanh(logits / cap)
     logit_scale: float = 1.0                  # logits <- logits * this (before a cap)
+    embed_norm: Optional[object] = None       # norm spec: the embedding row is normed before the first block
 
     def validate(self) -> None:
         if not self.blocks or not self.schedule:

@@ -23,6 +23,8 @@
 // With keep_first > 0 the keys below keep_first that the window has passed are visible too: they stand in front of the
 // window's keys as whole tiles (the last one padded with masked places), so that no tile holds keys of both runs and the
 // splits cut the joined run.  With a cap, a score s (after the scale) becomes cap * tanh(s / cap) (tanh as 1 - 2 / (1 + e^(2x))).
+// With chunks a row's key range starts at its token's chunk (counted from position 0).  With sigmoid weights a key's weight is
+// sigmoid(score + pb[head]); nothing is normalised: every part counts with factor one (m = 0, and l = 1 says that it has keys).
 #include "common.cuh"
 #include "mma_utils.cuh"
 using namespace arle;
@@ -36,16 +38,19 @@ __device__ __forceinline__ float tanh_by_exp(float x) { return 1.0f - __fdividef
 constexpr int kThreads = 128;
 constexpr int kTile = 64;   // keys per tile
 
-template <int HD, bool EXT>
+// FORM 0: the usual one; 1: with kept first keys and a score cap; 2: sigmoid weights, with chunks or a window.
+template <int HD, int FORM>
 __global__ void __launch_bounds__(kThreads) paged_decode_kernel(
     const __nv_bfloat16* __restrict__ q, int q_row_stride, __nv_bfloat16* __restrict__ out,
     const __nv_bfloat16* __restrict__ k_cache, const __nv_bfloat16* __restrict__ v_cache,
     const int* __restrict__ q_indptr, const int* __restrict__ kv_lens, const int* __restrict__ block_table,
     int bt_stride, float* __restrict__ part_o, float* __restrict__ part_ml, int* __restrict__ counters, int nq, int nkv,
     int page_size, int ps_shift, float scale_log2, float sink_log2, int window, int splits, int keep_first, float cap_arg,
-    float scale_over_cap) {
+    float scale_over_cap, int chunk_arg, const float* __restrict__ pb) {
   pdl_launch_dependents();
   pdl_wait();
+  constexpr bool EXT = FORM == 1, SIG = FORM == 2;
+  const int chunk_size = SIG ? chunk_arg : 0;
   const float cap_log2 = EXT ? cap_arg : 0.f;
   constexpr int ROW = HD + 8;                 // padded row, in elements: 16 B more keeps ldmatrix conflict-free
   constexpr int CHUNKS = HD / 8;              // 16-byte chunks per row
@@ -60,7 +65,7 @@ __global__ void __launch_bounds__(kThreads) paged_decode_kernel(
   const int t = q_indptr[r];
   if (q_indptr[r + 1] - t != 1) return;
   const int kv_len = kv_lens[r];
-  const int lo = (window > 0 && kv_len > window) ? kv_len - window : 0;
+  const int lo = first_visible_key(kv_len - 1, window, chunk_size);
   // places: [0, kap) the kept first keys (key = place, those from ka on masked), then the window's keys (key = lo + place - kap)
   const int ka = EXT ? min(keep_first, lo) : 0;
   const int kap = (ka + kTile - 1) / kTile * kTile;
@@ -150,6 +155,12 @@ __global__ void __launch_bounds__(kThreads) paged_decode_kernel(
 #pragma unroll
   for (int i = 0; i < HD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;   // rows g and g+8
+  float npb0 = 0.f, npb1 = 0.f;
+  if (SIG) {
+    m0 = m1 = 0.f;
+    if (g < G) npb0 = -pb[kvh * G + g] * 1.4426950408889634f;
+    if (g + 8 < G) npb1 = -pb[kvh * G + g + 8] * 1.4426950408889634f;
+  }
 
   for (int tile = 0; tile < ntiles; ++tile) {
     const int stage = tile & 1;
@@ -182,7 +193,7 @@ __global__ void __launch_bounds__(kThreads) paged_decode_kernel(
         if (cap_log2 > 0.f) {
 #pragma unroll
           for (int e = 0; e < 4; ++e) s[n][e] = cap_log2 * tanh_by_exp(s[n][e] * scale_over_cap);
-        } else {
+        } else if (!SIG) {
 #pragma unroll
           for (int e = 0; e < 4; ++e) s[n][e] *= scale_log2;
         }
@@ -193,16 +204,27 @@ __global__ void __launch_bounds__(kThreads) paged_decode_kernel(
         mx0 = fmaxf(mx0, fmaxf(s[n][0], s[n][1]));
         mx1 = fmaxf(mx1, fmaxf(s[n][2], s[n][3]));
       }
+      uint32_t pa[4];
+      float p[2][4];
+      float c0 = 1.f, c1 = 1.f;
+      if (SIG) {
+        // sigmoid(z) = 1 / (1 + 2^(-z log2 e)); a masked score is -inf and gives no weight
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float w = __fdividef(1.0f, 1.0f + exp2f(fminf(fmaf(s[n][e], -scale_log2, e < 2 ? npb0 : npb1), 126.0f)));
+            p[n][e] = s[n][e] == -INFINITY ? 0.f : w;
+          }
+      } else {
       mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
       mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
       mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
       mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
       const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);   // finite: key kbeg is valid
-      const float c0 = exp2f(m0 - mn0), c1 = exp2f(m1 - mn1);
+      c0 = exp2f(m0 - mn0), c1 = exp2f(m1 - mn1);
       m0 = mn0;
       m1 = mn1;
-      uint32_t pa[4];
-      float p[2][4];
 #pragma unroll
       for (int n = 0; n < 2; ++n) {
         p[n][0] = exp2f(s[n][0] - mn0);
@@ -212,14 +234,17 @@ __global__ void __launch_bounds__(kThreads) paged_decode_kernel(
       }
       l0 = l0 * c0 + p[0][0] + p[0][1] + p[1][0] + p[1][1];
       l1 = l1 * c1 + p[0][2] + p[0][3] + p[1][2] + p[1][3];
+      }
       pa[0] = pack_bf16(p[0][0], p[0][1]);
       pa[1] = pack_bf16(p[0][2], p[0][3]);
       pa[2] = pack_bf16(p[1][0], p[1][1]);
       pa[3] = pack_bf16(p[1][2], p[1][3]);
 #pragma unroll
       for (int dn = 0; dn < HD / 16; ++dn) {
-        o[2 * dn][0] *= c0; o[2 * dn][1] *= c0; o[2 * dn][2] *= c1; o[2 * dn][3] *= c1;
-        o[2 * dn + 1][0] *= c0; o[2 * dn + 1][1] *= c0; o[2 * dn + 1][2] *= c1; o[2 * dn + 1][3] *= c1;
+        if (!SIG) {
+          o[2 * dn][0] *= c0; o[2 * dn][1] *= c0; o[2 * dn][2] *= c1; o[2 * dn][3] *= c1;
+          o[2 * dn + 1][0] *= c0; o[2 * dn + 1][1] *= c0; o[2 * dn + 1][2] *= c1; o[2 * dn + 1][3] *= c1;
+        }
         uint32_t b0, b1, b2, b3;
         ldsm_x4_t(smem_u32(vt + (((lane >> 3) & 1) * 8 + (lane & 7)) * ROW + dn * 16 + (lane >> 4) * 8), b0, b1, b2, b3);
         mma_bf16(o[2 * dn], pa, b0, b1);
@@ -262,8 +287,9 @@ __global__ void __launch_bounds__(kThreads) paged_decode_kernel(
       O += mo[(w * 16 + row) * HD + d] * f;
     }
     const int head = kvh * G + row;
+    if (SIG) L = 1.f;
     if (splits == 1) {
-      out[((size_t)t * nq + head) * HD + d] = __float2bfloat16_rn(O / (L + exp2f(sink_log2 - M)));      // sink_log2 -inf: no sink
+      out[((size_t)t * nq + head) * HD + d] = __float2bfloat16_rn(SIG ? O : O / (L + exp2f(sink_log2 - M)));      // sink_log2 -inf: no sink
     } else {
       const size_t pidx = ((size_t)r * nq + head) * splits + split;
       part_o[pidx * HD + d] = O;
@@ -306,7 +332,7 @@ __global__ void __launch_bounds__(kThreads) paged_decode_kernel(
       fac[tid * 64 + sp] = f;
       L += l * f;
     }
-    invl[tid] = 1.0f / (L + exp2f(sink_log2 - M));
+    invl[tid] = SIG ? 1.0f : 1.0f / (L + exp2f(sink_log2 - M));
   }
   __syncthreads();
   for (int i = tid; i < G * HD; i += kThreads) {
@@ -326,7 +352,7 @@ template <int HD>
 int launch_decode(const void* q, int q_row_stride, void* out, const void* k_cache, const void* v_cache,
                   const int* q_indptr, const int* kv_lens, const int* block_table, int bt_stride, float* part_o,
                   float* part_ml, int* counters, int nq, int nkv, int page_size, float scale, float sink, int window, int rows,
-                  int splits, int keep_first, float softcap, cudaStream_t s) {
+                  int splits, int keep_first, float softcap, int chunk, const float* pb, cudaStream_t s) {
   constexpr int ROW = HD + 8;
   int ps_shift = -1;
   if ((page_size & (page_size - 1)) == 0)
@@ -334,20 +360,20 @@ int launch_decode(const void* q, int q_row_stride, void* out, const void* k_cach
   const size_t tiles = (size_t)(4 * kTile + 16) * ROW * sizeof(__nv_bfloat16);
   const size_t merge = (size_t)(4 * 16 * HD + 128) * sizeof(float);
   const size_t smem = tiles > merge ? tiles : merge;
-  const bool ext = (window > 0 && keep_first > 0) || softcap > 0.f;
-  auto kernel = ext ? paged_decode_kernel<HD, true> : paged_decode_kernel<HD, false>;
-  static bool configured[2] = {false, false};
-  if (!configured[ext]) {
+  const int form = pb ? 2 : ((window > 0 && keep_first > 0) || softcap > 0.f) ? 1 : 0;
+  auto kernel = form == 2 ? paged_decode_kernel<HD, 2> : form == 1 ? paged_decode_kernel<HD, 1> : paged_decode_kernel<HD, 0>;
+  static bool configured[3] = {false, false, false};
+  if (!configured[form]) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    configured[ext] = true;
+    configured[form] = true;
   }
   dim3 grid(rows, nkv, splits);
   launch_kernel(kernel, dim3(grid), dim3(kThreads), smem, s, 1, 
       (const __nv_bfloat16*)q, q_row_stride, (__nv_bfloat16*)out, (const __nv_bfloat16*)k_cache,
       (const __nv_bfloat16*)v_cache, q_indptr, kv_lens, block_table, bt_stride, part_o, part_ml, counters, nq, nkv,
       page_size, ps_shift, scale * 1.4426950408889634f, sink * 1.4426950408889634f, window, splits, window > 0 ? keep_first : 0,
-      softcap > 0.f ? softcap * 1.4426950408889634f : 0.f, softcap > 0.f ? scale / softcap : 0.f);
+      softcap > 0.f ? softcap * 1.4426950408889634f : 0.f, softcap > 0.f ? scale / softcap : 0.f, chunk, pb);
   return launch_status();
 }
 
@@ -359,18 +385,19 @@ ARLE_API int arle_paged_attention_decode(const void* q, int q_row_stride, void* 
                                          const void* v_cache, const int* q_indptr, const int* kv_lens,
                                          const int* block_table, int bt_stride, float* part_o, float* part_ml,
                                          int* counters, int nq, int nkv, int hd, int page_size, float scale, float sink, int window,
-                                         int rows, int splits, int keep_first, float softcap, cudaStream_t s) {
+                                         int rows, int splits, int keep_first, float softcap, int chunk, const float* pb, cudaStream_t s) {
   if (rows <= 0) return 0;
   if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || nq / nkv > 16 || page_size <= 0) return ARLE_E_UNSUPPORTED;
   if (splits < 1 || splits > 64 || nkv > 65535) return ARLE_E_UNSUPPORTED;
   if (splits > 1 && (!part_o || !part_ml || !counters)) return ARLE_E_BADARG;
   if ((q_row_stride % 8) != 0) return ARLE_E_UNSUPPORTED;     // 16-byte loads of q rows
-  if (keep_first < 0 || softcap < 0.f) return ARLE_E_BADARG;
+  if (keep_first < 0 || softcap < 0.f || chunk < 0 || (chunk > 0 && window > 0)) return ARLE_E_BADARG;
+  if (pb ? (keep_first > 0 || softcap > 0.f) : chunk > 0) return ARLE_E_UNSUPPORTED;      // the sigmoid form has neither; only it has chunks
   if (hd == 128)
     return launch_decode<128>(q, q_row_stride, out, k_cache, v_cache, q_indptr, kv_lens, block_table, bt_stride, part_o,
-                              part_ml, counters, nq, nkv, page_size, scale, sink, window, rows, splits, keep_first, softcap, s);
+                              part_ml, counters, nq, nkv, page_size, scale, sink, window, rows, splits, keep_first, softcap, chunk, pb, s);
   if (hd == 64)
     return launch_decode<64>(q, q_row_stride, out, k_cache, v_cache, q_indptr, kv_lens, block_table, bt_stride, part_o,
-                             part_ml, counters, nq, nkv, page_size, scale, sink, window, rows, splits, keep_first, softcap, s);
+                             part_ml, counters, nq, nkv, page_size, scale, sink, window, rows, splits, keep_first, softcap, chunk, pb, s);
   return ARLE_E_UNSUPPORTED;
 }

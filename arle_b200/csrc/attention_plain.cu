@@ -14,6 +14,10 @@
 // Values may have another width than keys (vd; the value cache is [page][kv_head][slot][vd]).  With a sink the
 // softmax has one more term in its denominator, exp(sink_logit), that carries no value:
 // p_j = exp(s_j) / (exp(sink_logit) + sum exp(s_j)).
+//
+// With sigmoid weights (pb: one number per query head, added to the scaled score) there is no softmax: a visible key's weight
+// is sigmoid(score + pb[h]) as it is, and the values' weighted sum is the result.  With chunks a query sees only the keys of
+// its own chunk of positions (counted from position 0).
 #include "common.cuh"
 using namespace arle;
 
@@ -27,7 +31,7 @@ __global__ void paged_attention_plain_kernel(const T* __restrict__ q, int q_row_
                                              const int* __restrict__ row_of_token,
                                              const int* __restrict__ block_table, int bt_stride, int nq,
                                              int nkv, int hd, int vd, int page_size, float scale, int window, int has_sink,
-                                             float sink_logit, int keep_first, float softcap) {
+                                             float sink_logit, int keep_first, float softcap, int chunk, const float* __restrict__ pb) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float qs[256];
@@ -38,7 +42,7 @@ __global__ void paged_attention_plain_kernel(const T* __restrict__ q, int q_row_
   const int kvh = h / (nq / nkv);
   const int pos = positions[t];
   const int* bt = block_table + (size_t)row_of_token[t] * bt_stride;
-  const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+  const int lo = first_visible_key(pos, window, chunk);
   const int ka = min(keep_first, lo);                // kept first keys outside the window
   const int nvis = ka + pos - lo + 1;                // visible keys: index i is key i (i < ka) or key lo + i - ka
 
@@ -64,14 +68,20 @@ __global__ void paged_attention_plain_kernel(const T* __restrict__ q, int q_row_
       for (int e = 0; e < hd; ++e) d = fmaf(qs[e], to_f32(kp[e]), d);
       sc = softcap > 0.f ? softcap * tanhf(d / softcap) : d;
     }
-    const float mt = warp_max(sc);
-    const float m_new = fmaxf(m, mt);
-    const float p = iv < nvis ? expf(sc - m_new) : 0.f;
-    const float corr = expf(m - m_new);
-    l = l * corr + warp_sum(p);
+    float p;
+    if (pb) {
+      p = iv < nvis ? 1.0f / (1.0f + expf(-(sc + pb[h]))) : 0.f;
+      m = 0.f;                                       // every warp's sums count as they are
+    } else {
+      const float mt = warp_max(sc);
+      const float m_new = fmaxf(m, mt);
+      p = iv < nvis ? expf(sc - m_new) : 0.f;
+      const float corr = expf(m - m_new);
+      l = l * corr + warp_sum(p);
 #pragma unroll
-    for (int i = 0; i < kAttnMaxD; ++i) acc[i] *= corr;
-    m = m_new;
+      for (int i = 0; i < kAttnMaxD; ++i) acc[i] *= corr;
+      m = m_new;
+    }
     const int nvalid = min(32, nvis - i0);
     for (int jj = 0; jj < nvalid; ++jj) {
       const float pj = __shfl_sync(0xffffffffu, p, jj);
@@ -102,6 +112,7 @@ __global__ void paged_attention_plain_kernel(const T* __restrict__ q, int q_row_
     f[i] = expf(m_s[i] - mm);  // a warp without keys has m = -inf, so f = 0
     ll += l_s[i] * f[i];
   }
+  if (pb) ll = 1.f;
   T* op = out + ((size_t)t * nq + h) * vd;
   for (int d = threadIdx.x; d < vd; d += blockDim.x) {
     float o = 0.f;
@@ -114,8 +125,9 @@ ARLE_API int arle_paged_attention_plain(const void* q, int q_row_stride, void* o
                                         const void* v_cache, int dtype, const int* positions,
                                         const int* row_of_token, const int* block_table, int bt_stride,
                                         int nq, int nkv, int hd, int vd, int page_size, float scale, int window,
-                                        int has_sink, float sink_logit, int keep_first, float softcap, int num_tokens, cudaStream_t s) {
+                                        int has_sink, float sink_logit, int keep_first, float softcap, int chunk, const float* pb, int num_tokens, cudaStream_t s) {
   if (num_tokens <= 0) return 0;
+  if (chunk < 0 || (chunk > 0 && window > 0) || (pb && has_sink)) return ARLE_E_BADARG;
   if (vd <= 0 || vd > 256) return ARLE_E_UNSUPPORTED;
   if (hd <= 0 || hd > 256 || nq <= 0 || nkv <= 0 || nq % nkv != 0 || page_size <= 0) return ARLE_E_UNSUPPORTED;
   if (nq > 65535) return ARLE_E_UNSUPPORTED;
@@ -124,12 +136,12 @@ ARLE_API int arle_paged_attention_plain(const void* q, int q_row_stride, void* o
   if (dtype == 0)
     launch_kernel(paged_attention_plain_kernel<float>, dim3(grid), dim3(kAttnWarps * 32), 0, s, 1, 
         (const float*)q, q_row_stride, (float*)out, (const float*)k_cache, (const float*)v_cache, positions,
-        row_of_token, block_table, bt_stride, nq, nkv, hd, vd, page_size, scale, window, has_sink, sink_logit, keep_first, softcap);
+        row_of_token, block_table, bt_stride, nq, nkv, hd, vd, page_size, scale, window, has_sink, sink_logit, keep_first, softcap, chunk, pb);
   else if (dtype == 1)
     launch_kernel(paged_attention_plain_kernel<__nv_bfloat16>, dim3(grid), dim3(kAttnWarps * 32), 0, s, 1, 
         (const __nv_bfloat16*)q, q_row_stride, (__nv_bfloat16*)out, (const __nv_bfloat16*)k_cache,
         (const __nv_bfloat16*)v_cache, positions, row_of_token, block_table, bt_stride, nq, nkv, hd, vd,
-        page_size, scale, window, has_sink, sink_logit, keep_first, softcap);
+        page_size, scale, window, has_sink, sink_logit, keep_first, softcap, chunk, pb);
   else
     return ARLE_E_BADARG;
   return launch_status();

@@ -17,6 +17,8 @@
 // With keep_first > 0 a windowed query also sees the keys below keep_first: the tiles that hold them (counted from key 0)
 // run before the window's tiles, under the same mask.  With a cap, a score s (after the scale) becomes cap * tanh(s / cap)
 // before the softmax (tanh as 1 - 2 / (1 + e^(2x)), not the approximate tanh instruction, whose error the cap would multiply).
+// With chunks a query sees only the keys of its own chunk of positions (counted from position 0).  With sigmoid weights a
+// visible key's weight is sigmoid(score + pb[head]), nothing is normalised and no maximum is kept.
 #include "common.cuh"
 #include "mma_utils.cuh"
 using namespace arle;
@@ -31,16 +33,18 @@ constexpr int kThreads = 128;
 constexpr int kBlockM = 64;
 constexpr int kTile = 64;
 
-// EXT: with kept first keys and a score cap (the usual form compiles without either).
-template <int HD, bool EXT>
+// FORM 0: the usual one; 1: with kept first keys and a score cap; 2: sigmoid weights, with chunks or a window.
+template <int HD, int FORM>
 __global__ void __launch_bounds__(kThreads, 3) paged_prefill_kernel(
     const __nv_bfloat16* __restrict__ q, int q_row_stride, __nv_bfloat16* __restrict__ out,
     const __nv_bfloat16* __restrict__ k_cache, const __nv_bfloat16* __restrict__ v_cache,
     const int* __restrict__ q_indptr, const int* __restrict__ kv_lens, const int* __restrict__ block_table,
     int bt_stride, int nq, int nkv, int page_size, int ps_shift, float scale_log2, float sink_log2, int window, int skip_single,
-    int keep_first_arg, float cap_arg, float scale_over_cap) {
+    int keep_first_arg, float cap_arg, float scale_over_cap, int chunk_arg, const float* __restrict__ pb) {
   pdl_launch_dependents();
   pdl_wait();
+  constexpr bool EXT = FORM == 1, SIG = FORM == 2;
+  const int chunk = SIG ? chunk_arg : 0;
   const int keep_first = EXT ? keep_first_arg : 0;
   const float cap_log2 = EXT ? cap_arg : 0.f;
   constexpr int ROW = HD + 8;
@@ -60,7 +64,7 @@ __global__ void __launch_bounds__(kThreads, 3) paged_prefill_kernel(
   const int pos0 = kv_len - qlen;                       // position of the row's first query
   const int rows_here = min(kBlockM, qlen - mbeg);
   const int p_first = pos0 + mbeg, p_last = pos0 + mbeg + rows_here - 1;
-  const int lo = (window > 0 && p_first - window + 1 > 0) ? p_first - window + 1 : 0;
+  const int lo = first_visible_key(p_first, window, chunk);
   const int kb = lo / kTile * kTile;
   const int nk = (min(keep_first, kb) + kTile - 1) / kTile;     // tiles of kept first keys that lie before the window's first tile
   const int ntiles = nk + (p_last - kb) / kTile + 1;
@@ -140,10 +144,11 @@ __global__ void __launch_bounds__(kThreads, 3) paged_prefill_kernel(
   // positions of this thread's two query rows; rows past the portion's end copy the last one
   const int prow0 = min(pos0 + mbeg + warp * 16 + g, p_last);
   const int prow1 = min(pos0 + mbeg + warp * 16 + g + 8, p_last);
-  const int plo0 = window > 0 ? prow0 - window + 1 : 0;
-  const int plo1 = window > 0 ? prow1 - window + 1 : 0;
+  const int plo0 = SIG ? first_visible_key(prow0, window, chunk) : window > 0 ? prow0 - window + 1 : 0;
+  const int plo1 = SIG ? first_visible_key(prow1, window, chunk) : window > 0 ? prow1 - window + 1 : 0;
   const int warp_last = min(pos0 + mbeg + warp * 16 + 15, p_last);   // last key any row of this warp may see
-  const int warp_first = window > 0 ? max(0, min(pos0 + mbeg + warp * 16, p_last) - window + 1) : 0;
+  const int warp_first = first_visible_key(min(pos0 + mbeg + warp * 16, p_last), window, chunk);
+  const float npb = SIG ? -pb[h] * 1.4426950408889634f : 0.f;
 
   float o[HD / 8][4];
 #pragma unroll
@@ -185,7 +190,7 @@ __global__ void __launch_bounds__(kThreads, 3) paged_prefill_kernel(
         if (cap_log2 > 0.f) {
 #pragma unroll
           for (int e = 0; e < 4; ++e) s[n][e] = cap_log2 * tanh_by_exp(s[n][e] * scale_over_cap);
-        } else {
+        } else if (!SIG) {
 #pragma unroll
           for (int e = 0; e < 4; ++e) s[n][e] *= scale_log2;
         }
@@ -193,9 +198,18 @@ __global__ void __launch_bounds__(kThreads, 3) paged_prefill_kernel(
         s[n][1] = (kj + 1 <= prow0 && (kj + 1 >= plo0 || kj + 1 < keep_first)) ? s[n][1] : -INFINITY;
         s[n][2] = (kj <= prow1 && (kj >= plo1 || kj < keep_first)) ? s[n][2] : -INFINITY;
         s[n][3] = (kj + 1 <= prow1 && (kj + 1 >= plo1 || kj + 1 < keep_first)) ? s[n][3] : -INFINITY;
+        if (SIG) {
+          // sigmoid(z) = 1 / (1 + 2^(-z log2 e)); a masked score (-inf) gives no weight
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float wgt = __fdividef(1.0f, 1.0f + exp2f(fminf(fmaf(s[n][e], -scale_log2, npb), 126.0f)));
+            s[n][e] = s[n][e] == -INFINITY ? 0.f : wgt;
+          }
+        }
         mx0 = fmaxf(mx0, fmaxf(s[n][0], s[n][1]));
         mx1 = fmaxf(mx1, fmaxf(s[n][2], s[n][3]));
       }
+      if (!SIG) {
       mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
       mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
       mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
@@ -222,6 +236,7 @@ __global__ void __launch_bounds__(kThreads, 3) paged_prefill_kernel(
       for (int i = 0; i < HD / 8; ++i) {
         o[i][0] *= c0; o[i][1] *= c0; o[i][2] *= c1; o[i][3] *= c1;
       }
+      }
 #pragma unroll
       for (int kk = 0; kk < 4; ++kk) {          // 16 keys per step of P.V
         uint32_t pa[4];
@@ -245,7 +260,7 @@ __global__ void __launch_bounds__(kThreads, 3) paged_prefill_kernel(
   l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
   // a sink's term in the denominator (its score in log2 units; -inf: none, and the sums stay as they are)
-  const float inv0 = 1.0f / (l0 + exp2f(sink_log2 - m0)), inv1 = 1.0f / (l1 + exp2f(sink_log2 - m1));
+  const float inv0 = SIG ? 1.0f : 1.0f / (l0 + exp2f(sink_log2 - m0)), inv1 = SIG ? 1.0f : 1.0f / (l1 + exp2f(sink_log2 - m1));
   const int row0 = mbeg + warp * 16 + g, row1 = row0 + 8;
 #pragma unroll
   for (int i = 0; i < HD / 8; ++i) {
@@ -264,26 +279,26 @@ template <int HD>
 int launch_prefill(const void* q, int q_row_stride, void* out, const void* k_cache, const void* v_cache,
                    const int* q_indptr, const int* kv_lens, const int* block_table, int bt_stride, int nq, int nkv,
                    int page_size, float scale, float sink, int window, int rows, int max_q_len, int skip_single, int keep_first, float softcap,
-                   cudaStream_t s) {
+                   int chunk, const float* pb, cudaStream_t s) {
   constexpr int ROW = HD + 8;
   int ps_shift = -1;
   if ((page_size & (page_size - 1)) == 0)
     for (ps_shift = 0; (1 << ps_shift) < page_size; ++ps_shift) {}
   const size_t smem = (size_t)(4 * kTile) * ROW * sizeof(__nv_bfloat16);
-  const bool ext = (window > 0 && keep_first > 0) || softcap > 0.f;
-  auto kernel = ext ? paged_prefill_kernel<HD, true> : paged_prefill_kernel<HD, false>;
-  static bool configured[2] = {false, false};
-  if (!configured[ext]) {
+  const int form = pb ? 2 : ((window > 0 && keep_first > 0) || softcap > 0.f) ? 1 : 0;
+  auto kernel = form == 2 ? paged_prefill_kernel<HD, 2> : form == 1 ? paged_prefill_kernel<HD, 1> : paged_prefill_kernel<HD, 0>;
+  static bool configured[3] = {false, false, false};
+  if (!configured[form]) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    configured[ext] = true;
+    configured[form] = true;
   }
   dim3 grid((max_q_len + kBlockM - 1) / kBlockM, nq, rows);
   launch_kernel(kernel, dim3(grid), dim3(kThreads), smem, s, 1, 
       (const __nv_bfloat16*)q, q_row_stride, (__nv_bfloat16*)out, (const __nv_bfloat16*)k_cache,
       (const __nv_bfloat16*)v_cache, q_indptr, kv_lens, block_table, bt_stride, nq, nkv, page_size, ps_shift,
       scale * 1.4426950408889634f, sink * 1.4426950408889634f, window, skip_single, window > 0 ? keep_first : 0,
-      softcap > 0.f ? softcap * 1.4426950408889634f : 0.f, softcap > 0.f ? scale / softcap : 0.f);
+      softcap > 0.f ? softcap * 1.4426950408889634f : 0.f, softcap > 0.f ? scale / softcap : 0.f, chunk, pb);
   return launch_status();
 }
 
@@ -293,16 +308,17 @@ ARLE_API int arle_paged_attention_prefill(const void* q, int q_row_stride, void*
                                           const void* v_cache, const int* q_indptr, const int* kv_lens,
                                           const int* block_table, int bt_stride, int nq, int nkv, int hd, int page_size,
                                           float scale, float sink, int window, int rows, int max_q_len, int skip_single,
-                                          int keep_first, float softcap, cudaStream_t s) {
+                                          int keep_first, float softcap, int chunk, const float* pb, cudaStream_t s) {
   if (rows <= 0 || max_q_len <= 0) return 0;
   if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || page_size <= 0 || nq > 65535 || rows > 65535) return ARLE_E_UNSUPPORTED;
   if ((q_row_stride % 8) != 0) return ARLE_E_UNSUPPORTED;
-  if (keep_first < 0 || softcap < 0.f) return ARLE_E_BADARG;
+  if (keep_first < 0 || softcap < 0.f || chunk < 0 || (chunk > 0 && window > 0)) return ARLE_E_BADARG;
+  if (pb ? (keep_first > 0 || softcap > 0.f) : chunk > 0) return ARLE_E_UNSUPPORTED;      // the sigmoid form has neither; only it has chunks
   if (hd == 128)
     return launch_prefill<128>(q, q_row_stride, out, k_cache, v_cache, q_indptr, kv_lens, block_table, bt_stride, nq,
-                               nkv, page_size, scale, sink, window, rows, max_q_len, skip_single, keep_first, softcap, s);
+                               nkv, page_size, scale, sink, window, rows, max_q_len, skip_single, keep_first, softcap, chunk, pb, s);
   if (hd == 64)
     return launch_prefill<64>(q, q_row_stride, out, k_cache, v_cache, q_indptr, kv_lens, block_table, bt_stride, nq,
-                              nkv, page_size, scale, sink, window, rows, max_q_len, skip_single, keep_first, softcap, s);
+                              nkv, page_size, scale, sink, window, rows, max_q_len, skip_single, keep_first, softcap, chunk, pb, s);
   return ARLE_E_UNSUPPORTED;
 }

@@ -43,6 +43,9 @@
 // Q as soon as this block's last S product is done, and the tensor core has the next block's first scores
 // ready when the softmax warps have normalised and stored this block's output (the next block's first
 // product with the values waits until they have taken O out of tensor memory).
+// A third form has sigmoid weights, sigmoid(score + pb[head]), in the softmax's place, and chunks (a query sees only the keys
+// of its own chunk of positions, counted from 0) or a window: no maximum, no sum and no rescaling; two scores share one
+// reciprocal, since the special-function unit is what bounds the softmax warps.
 // Scores, maxima, sums and the accumulators are float32.  Every mbarrier wait is bounded; when one runs
 // out the kernel raises the error flag, stops, draws the remaining tickets so that the counter ends at
 // zero, frees its TMEM and returns.
@@ -138,7 +141,7 @@ struct Block {
   int nk, keep;      // key tiles of kept first keys in front of the window's tiles (tile j < nk starts at key j * BKV), and how many keys are kept
   // false: the block is beyond the request's queries (or the request is one that the decode kernel serves)
   __device__ bool init(int b, int nq, int nkv, int nyb, const int* q_indptr, const int* kv_lens, int window, int skip_single,
-                       int keep_first) {
+                       int keep_first, int chunk) {
     h = b % nq;
     const int y = (b / nq) % nyb;
     r = b / (nq * nyb);
@@ -160,7 +163,7 @@ struct Block {
     for (int x = 0; x < 2; ++x) {
       pf_x[x] = pos0 + mbeg + x * BQ;
       pl_x[x] = pf_x[x] + max(rows_x[x], 1) - 1;
-      lo_x[x] = (window > 0 && pf_x[x] - window + 1 > 0) ? pf_x[x] - window + 1 : 0;
+      lo_x[x] = first_visible_key(pf_x[x], window, chunk);
     }
     kb = lo_x[0] / BKV * BKV;
     // Kept first keys (a windowed query sees the keys below keep_first too): the tiles that hold those before kb run first.
@@ -187,16 +190,18 @@ struct Block {
 
 constexpr int kWorkReaders = 11;             // who reads a drawn ticket: the two loader warps, the MMA thread, eight softmax warps
 
-// EXT: with kept first keys and a score cap (the usual form compiles without either).
-template <bool EXT>
+// FORM 0: the usual one; 1: with kept first keys and a score cap; 2: sigmoid weights, with chunks or a window.
+template <int FORM>
 __global__ void __launch_bounds__(kThreads, 1) paged_prefill_tc_kernel(
     const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
     const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* __restrict__ out, const int* __restrict__ q_indptr,
     const int* __restrict__ kv_lens, const int* __restrict__ block_table, int bt_stride, int bt_width, int nq, int nkv,
     int page_size, float scale_log2, float sink_log2, int window, int skip_single, int nyb, int nblocks, int ticket_slot, int* __restrict__ err,
-    int keep_arg, float cap_arg, float scale_over_cap) {
+    int keep_arg, float cap_arg, float scale_over_cap, int chunk_arg, const float* __restrict__ pb) {
   pdl_launch_dependents();
   pdl_wait();
+  constexpr bool EXT = FORM == 1, SIG = FORM == 2;
+  const int chunk = SIG ? chunk_arg : 0;
   const int keep_first = EXT ? keep_arg : 0;
   const float cap_log2 = EXT ? cap_arg : 0.f;
   const float cap_c1 = scale_over_cap * 2.8853900817779268f, cap_c2 = -2.0f * cap_log2;      // e^(2z) as a power of two; -2 cap
@@ -216,7 +221,7 @@ __global__ void __launch_bounds__(kThreads, 1) paged_prefill_tc_kernel(
   // the CTA's first block is the one of its own index: its shape is worked out while the rest is set up
   bool first_has_queries = false;
   if (warp == kKeyWarp && lane == 0)
-    first_has_queries = work_blk[0].init((int)blockIdx.x, nq, nkv, nyb, q_indptr, kv_lens, window, skip_single, keep_first);
+    first_has_queries = work_blk[0].init((int)blockIdx.x, nq, nkv, nyb, q_indptr, kv_lens, window, skip_single, keep_first, chunk);
   if (threadIdx.x == 0) {
     mbar_init(smem_addr(&q_full), 1);
     mbar_init(smem_addr(&q_empty), 1);
@@ -284,7 +289,7 @@ __global__ void __launch_bounds__(kThreads, 1) paged_prefill_tc_kernel(
             if (!*aborted) {
               const unsigned int tk = draw_ticket(nblocks, ticket_slot);
               if (tk < (unsigned int)nblocks) b = (int)tk; else ended = true;
-              if (b >= 0 && !work_blk[it & 1].init(b, nq, nkv, nyb, q_indptr, kv_lens, window, skip_single, keep_first)) b = -2;
+              if (b >= 0 && !work_blk[it & 1].init(b, nq, nkv, nyb, q_indptr, kv_lens, window, skip_single, keep_first, chunk)) b = -2;
             }
           } else {
             abort_flag = 1;
@@ -495,13 +500,16 @@ __global__ void __launch_bounds__(kThreads, 1) paged_prefill_tc_kernel(
       const int kb = blk.kb;
       const int keep = EXT ? blk.keep : 0, nk = EXT ? blk.nk : 0;      // without kept keys both are zero when the kernel is compiled
       const int p_row = min(p_first + row, pl);
-      const int lo_row = window > 0 ? p_row - window + 1 : 0;
+      const int lo_row = SIG ? first_visible_key(p_row, window, chunk) : window > 0 ? p_row - window + 1 : 0;
+      const int lo_last = SIG ? first_visible_key(pl, window, chunk) : 0;
+      const float npb = SIG ? -pb[blk.h] * 1.4426950408889634f : 0.f;
       float m_used = -INFINITY, l = 0.f;
       int n = 0;
       for (int j = (EXT && rows_here > 0 && nk > 0) ? 0 : jlo; j < jhi; ++j) {
         if (EXT && j >= nk && j < jlo) continue;               // between the kept tiles and this query tile's first
         const int k0 = (EXT && j < nk) ? j * BKV : kb + (j - nk) * BKV;
-        const bool full_tile = (EXT && j < nk) ? k0 + BKV <= keep : (k0 + BKV - 1 <= p_first && (window <= 0 || k0 >= pl - window + 1));
+        const bool full_tile = (EXT && j < nk) ? k0 + BKV <= keep
+                               : SIG ? (k0 + BKV - 1 <= p_first && k0 >= lo_last) : (k0 + BKV - 1 <= p_first && (window <= 0 || k0 >= pl - window + 1));
         bool ready = mbar_wait_bounded(smem_addr(&s_full[x]), (uint32_t)(n_all & 1), aborted);
         if (__any_sync(0xffffffffu, !ready)) { ok = false; break; }
         tc_fence_after();
@@ -510,6 +518,32 @@ __global__ void __launch_bounds__(kThreads, 1) paged_prefill_tc_kernel(
 #pragma unroll
         for (int c = 0; c < 4; ++c) tmem_ld32(tmem_s + lane_addr + (uint32_t)(c * 32), sv[c]);
         tmem_ld_wait();
+        if constexpr (SIG) {
+          // sigmoid(z) = 1 / (1 + t), t = 2^(-z log2 e).  Two neighbours share a reciprocal: 1 / a = b / (a b); t is kept below 2^60
+          // so that the product stays finite.
+#pragma unroll
+          for (int h2 = 0; h2 < 2; ++h2) {
+            uint32_t packed[32];                                  // 64 keys of this row as bfloat16 pairs
+#pragma unroll
+            for (int c = 0; c < 2; ++c)
+#pragma unroll
+              for (int i = 0; i < 32; i += 2) {
+                const float s0 = __uint_as_float(sv[2 * h2 + c][i]), s1 = __uint_as_float(sv[2 * h2 + c][i + 1]);
+                const float a0 = 1.0f + ex2_fast(fminf(fmaf(s0, -scale_log2, npb), 60.0f));
+                const float a1 = 1.0f + ex2_fast(fminf(fmaf(s1, -scale_log2, npb), 60.0f));
+                const float rr = rcp_fast(a0 * a1);
+                float e0 = rr * a1, e1 = rr * a0;
+                if (!full_tile) {
+                  const int kj = k0 + (2 * h2 + c) * 32 + i;
+                  e0 = (kj <= p_row && kj >= lo_row) ? e0 : 0.f;
+                  e1 = (kj + 1 <= p_row && kj + 1 >= lo_row) ? e1 : 0.f;
+                }
+                packed[c * 16 + (i >> 1)] = pack_bf16x2(e0, e1);
+              }
+            tmem_st32(tmem_s + lane_addr + (uint32_t)(h2 * 32), packed);
+          }
+          tmem_st_wait();
+        } else {
         // the row maximum (raw scores; the scale is positive, so it is applied to the maximum
         // alone).  Four running maxima keep the chain of dependent instructions short.
         float mx;
@@ -592,6 +626,7 @@ __global__ void __launch_bounds__(kThreads, 1) paged_prefill_tc_kernel(
         }
         tmem_st_wait();
         l += (l4[0] + l4[1]) + (l4[2] + l4[3]);
+        }
         tc_fence_before();
         __syncwarp();
         if (lane == 0) mbar_arrive(smem_addr(&p_full[x]));
@@ -606,7 +641,7 @@ __global__ void __launch_bounds__(kThreads, 1) paged_prefill_tc_kernel(
         ++o_all;
         tc_fence_after();
         // a sink's term in the denominator (its score in log2 units; -inf: none, and the sum stays as it is)
-        const float inv = 1.0f / (l + exp2f(sink_log2 - (m_used == -INFINITY ? 0.f : m_used)));
+        const float inv = SIG ? 1.0f : 1.0f / (l + exp2f(sink_log2 - (m_used == -INFINITY ? 0.f : m_used)));
         __nv_bfloat16* orow = out + ((size_t)(blk.t0 + blk.mbeg + x * BQ + row) * nq + blk.h) * HD;
 #pragma unroll 1
         for (int c = 0; c < 4; ++c) {
@@ -653,7 +688,7 @@ ARLE_API int arle_paged_attention_prefill_tc(const void* q, int q_row_stride, in
                                              const void* v_cache, long long cache_pages, const int* q_indptr,
                                              const int* kv_lens, const int* block_table, int bt_stride, int bt_width, int nq, int nkv,
                                              int hd, int page_size, float scale, float sink, int window, int rows, int max_q_len,
-                                             int skip_single, int* err, int keep_first, float softcap, cudaStream_t s) {
+                                             int skip_single, int* err, int keep_first, float softcap, int chunk, const float* pb, cudaStream_t s) {
   if (rows <= 0 || max_q_len <= 0) return 0;
   if (bt_width < 1) return ARLE_E_BADARG;
   if (hd != HD || page_size % 16 != 0 || nq <= 0 || nkv <= 0 || nq % nkv != 0 || rows > 65535 || (max_q_len + BQ2 - 1) / BQ2 > 65535)
@@ -669,14 +704,15 @@ ARLE_API int arle_paged_attention_prefill_tc(const void* q, int q_row_stride, in
   rc = tensor_map_2d_bf16(v_cache, cache_rows, HD, HD, 16, &mv);
   if (rc) return rc;
   const size_t smem = (2 + 2 * kStages) * (size_t)TILE + 1024;
-  if (keep_first < 0 || softcap < 0.f) return ARLE_E_BADARG;
-  const bool ext = (window > 0 && keep_first > 0) || softcap > 0.f;
-  auto kernel = ext ? paged_prefill_tc_kernel<true> : paged_prefill_tc_kernel<false>;
-  static bool configured[2] = {false, false};
-  if (!configured[ext]) {
+  if (keep_first < 0 || softcap < 0.f || chunk < 0 || (chunk > 0 && window > 0)) return ARLE_E_BADARG;
+  if (pb ? (keep_first > 0 || softcap > 0.f) : chunk > 0) return ARLE_E_UNSUPPORTED;      // the sigmoid form has neither; only it has chunks
+  const int form = pb ? 2 : ((window > 0 && keep_first > 0) || softcap > 0.f) ? 1 : 0;
+  auto kernel = form == 2 ? paged_prefill_tc_kernel<2> : form == 1 ? paged_prefill_tc_kernel<1> : paged_prefill_tc_kernel<0>;
+  static bool configured[3] = {false, false, false};
+  if (!configured[form]) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    configured[ext] = true;
+    configured[form] = true;
   }
   // CTAs stay resident and draw blocks (a query head, 256 queries of a request) from a counter, the heaviest first
   const int nyb = (max_q_len + BQ2 - 1) / BQ2;
@@ -692,7 +728,7 @@ ARLE_API int arle_paged_attention_prefill_tc(const void* q, int q_row_stride, in
                                 q_indptr, kv_lens, block_table, bt_stride, bt_width, nq, nkv, page_size,
                                 scale * 1.4426950408889634f, sink * 1.4426950408889634f, window, skip_single, nyb, (int)nblocks, ticket_slot, err,
                                 window > 0 ? keep_first : 0, softcap > 0.f ? softcap * 1.4426950408889634f : 0.f,
-                                softcap > 0.f ? scale / softcap : 0.f);
+                                softcap > 0.f ? scale / softcap : 0.f, chunk, pb);
   if (e != cudaSuccess) return (int)e;
   return launch_status();
 }

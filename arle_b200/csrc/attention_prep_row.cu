@@ -8,13 +8,13 @@
 //   k: the same over the nkv*hd elements with k_weight, rotate, store into k_cache at the
 //      token's slot;
 //   v: with values_are_keys the row of k as projected (before norm and rotation) goes into
-//      v_cache unchanged; otherwise the v heads that follow the k heads in the row do.
+//      v_cache unchanged; otherwise the v heads (nkv * vd) that follow the k heads in the row do.
 // Rotation, within the first rotary_dim elements of each head: pairing 0 turns element i with
 // i + rotary_dim/2 ("half split"), pairing 1 turns element 2i with 2i + 1 ("interleaved"); the
 // pair (u, v) becomes (u cos a - v sin a, v cos a + u sin a) with a = position * inv_freq[i],
 // in float32 (sincosf), or with the cosines and sines of a table [T][rotary_dim/2] of (cos, sin) that was filled the
 // same way once for the step (the same bits).  Norm statistics and products are float32.
-// Cache layout: [page][kv_head][slot_in_page][head_dim]; slot_mapping[t] < 0: no store.
+// Cache layout: [page][kv_head][slot_in_page][head_dim] (vd for the values); slot_mapping[t] < 0: no store.
 #include "common.cuh"
 using namespace arle;
 
@@ -24,7 +24,7 @@ __global__ void attention_prep_row_kernel(T* __restrict__ qk, int row_stride, co
                                           const float* __restrict__ k_weight, float eps,
                                           const float* __restrict__ inv_freq, const float2* __restrict__ angles,
                                           int rotary_dim, int pairing, int values_are_keys, T* __restrict__ k_cache, T* __restrict__ v_cache,
-                                          int nq, int nkv, int hd, int page_size, int vec8) {
+                                          int nq, int nkv, int hd, int vd, int page_size, int vec8) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float row[];                 // (nq + nkv) * hd floats: x * weight, still without the row's factor
@@ -83,7 +83,7 @@ __global__ void attention_prep_row_kernel(T* __restrict__ qk, int row_stride, co
   const float inv_q = q_weight ? 1.0f / sqrtf(sq / (float)nqe + eps) : 1.0f;
   const float inv_k = k_weight ? 1.0f / sqrtf(sk / (float)(nke > 0 ? nke : 1) + eps) : 1.0f;
   const int page = slot >= 0 ? slot / page_size : 0, off = slot >= 0 ? slot - page * page_size : 0;
-  const int half = rotary_dim >> 1, hd2 = hd >> 1;
+  const int half = rotary_dim >> 1, hd2 = (hd + 1) >> 1;
   const float2* ang = angles ? angles + (size_t)t * half : nullptr;
   // a thread takes a pair of elements: the two that turn together, or two neighbours past rotary_dim
   for (int p = threadIdx.x; p < (nq + nkv) * hd2; p += blockDim.x) {
@@ -107,7 +107,7 @@ __global__ void attention_prep_row_kernel(T* __restrict__ qk, int row_stride, co
     } else {
       const float inv = head < nq ? inv_q : inv_k;
       e0 = head * hd + rotary_dim + 2 * (d2 - half);
-      e1 = e0 + 1;
+      e1 = 2 * d2 + 1 < hd ? e0 + 1 : e0;            // the last number of an odd head stands alone
       o0 = row[e0] * inv, o1 = row[e1] * inv;
     }
     const bool pair = sizeof(T) == 2 && vec8 && e1 == e0 + 1;      // neighbours: one 4-byte access for both
@@ -120,16 +120,23 @@ __global__ void attention_prep_row_kernel(T* __restrict__ qk, int row_stride, co
       }
     } else if (slot >= 0) {
       const size_t base = (((size_t)page * nkv + (head - nq)) * page_size + off) * hd - (size_t)head * hd;
-      const T* vsrc = values_are_keys ? src : src + nke;
       if (pair) {
         *reinterpret_cast<__nv_bfloat162*>(k_cache + base + e0) = __floats2bfloat162_rn(o0, o1);
-        *reinterpret_cast<uint32_t*>(v_cache + base + e0) = *reinterpret_cast<const uint32_t*>(vsrc + e0);
       } else {
         k_cache[base + e0] = from_f32<T>(o0);
         k_cache[base + e1] = from_f32<T>(o1);
-        v_cache[base + e0] = vsrc[e0];
-        v_cache[base + e1] = vsrc[e1];
       }
+    }
+  }
+  if (nkv > 0 && slot >= 0) {
+    const T* vsrc = src + nqe + (values_are_keys ? 0 : nke);
+    const int nve = nkv * vd;
+    T* vdst = v_cache + ((size_t)page * nkv * page_size + off) * vd;      // head 0; the heads stand page_size rows apart
+    if (sizeof(T) == 2 && vec8 && vd % 8 == 0) {
+      for (int e = threadIdx.x * 8; e < nve; e += blockDim.x * 8)
+        *reinterpret_cast<uint4*>(vdst + (size_t)(e / vd) * (page_size - 1) * vd + e) = *reinterpret_cast<const uint4*>(vsrc + e);
+    } else {
+      for (int e = threadIdx.x; e < nve; e += blockDim.x) vdst[(size_t)(e / vd) * (page_size - 1) * vd + e] = vsrc[e];
     }
   }
 }
@@ -137,9 +144,9 @@ __global__ void attention_prep_row_kernel(T* __restrict__ qk, int row_stride, co
 ARLE_API int arle_attention_prep_row(void* qk, int dtype, int row_stride, const int* positions, const int* slot_mapping,
                                      const float* q_weight, const float* k_weight, float eps, const float* inv_freq,
                                      const float* angles, int rotary_dim, int pairing, int values_are_keys, void* k_cache, void* v_cache, int nq,
-                                     int nkv, int hd, int page_size, int num_tokens, cudaStream_t s) {
+                                     int nkv, int hd, int vd, int page_size, int num_tokens, cudaStream_t s) {
   if (num_tokens <= 0) return 0;
-  if (hd & 1) return ARLE_E_UNSUPPORTED;
+  if (nkv > 0 && (vd <= 0 || (values_are_keys && vd != hd))) return ARLE_E_BADARG;
   if (hd <= 0 || nq <= 0 || nkv < 0 || page_size <= 0 || rotary_dim < 0 || rotary_dim > hd || (rotary_dim & 1)) return ARLE_E_BADARG;
   if (pairing != 0 && pairing != 1) return ARLE_E_BADARG;
   if (rotary_dim > 0 && !inv_freq) return ARLE_E_BADARG;
@@ -149,21 +156,21 @@ ARLE_API int arle_attention_prep_row(void* qk, int dtype, int row_stride, const 
   const int n = (nq + nkv) * hd;
   const int threads = n >= 512 ? 256 : 128;
   // wide accesses: every row, head and cache entry starts on a 16-byte boundary (even head sizes keep pairs on 4)
-  const int vec8 = dtype == 1 && (nq * hd) % 8 == 0 && (nkv * hd) % 8 == 0 && row_stride % 8 == 0 && ((uintptr_t)qk % 16) == 0 &&
+  const int vec8 = dtype == 1 && hd % 2 == 0 && (nq * hd) % 8 == 0 && (nkv * hd) % 8 == 0 && row_stride % 8 == 0 && ((uintptr_t)qk % 16) == 0 &&
                    ((uintptr_t)k_cache % 16) == 0 && ((uintptr_t)v_cache % 16) == 0 && ((uintptr_t)q_weight % 16) == 0 &&
                    ((uintptr_t)k_weight % 16) == 0;
   if (dtype == 0) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(attention_prep_row_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     launch_kernel(attention_prep_row_kernel<float>, dim3(num_tokens), dim3(threads), smem, s, 1, (float*)qk, row_stride, positions,
                   slot_mapping, q_weight, k_weight, eps, inv_freq, (const float2*)angles, rotary_dim, pairing, values_are_keys, (float*)k_cache,
-                  (float*)v_cache, nq, nkv, hd, page_size, vec8);
+                  (float*)v_cache, nq, nkv, hd, vd, page_size, vec8);
   } else if (dtype == 1) {
     if (smem > 48 * 1024)
       cudaFuncSetAttribute(attention_prep_row_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     launch_kernel(attention_prep_row_kernel<__nv_bfloat16>, dim3(num_tokens), dim3(threads), smem, s, 1, (__nv_bfloat16*)qk,
                   row_stride, positions, slot_mapping, q_weight, k_weight, eps, inv_freq, (const float2*)angles, rotary_dim, pairing,
                   values_are_keys,
-                  (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, nq, nkv, hd, page_size, vec8);
+                  (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, nq, nkv, hd, vd, page_size, vec8);
   } else {
     return ARLE_E_BADARG;
   }

@@ -98,6 +98,13 @@ __device__ __forceinline__ float block_max(float v, float* scratch) {
   return scratch[32];
 }
 
+// The first key a query at position pos sees: the start of its chunk (chunks counted from position 0), or the first key of a
+// sliding window, or key 0.
+__device__ __forceinline__ int first_visible_key(int pos, int window, int chunk) {
+  if (chunk > 0) return pos - pos % chunk;
+  return (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+}
+
 // Programmatic dependent launch.  Every kernel of this library starts with
 // pdl_launch_dependents() (the next kernel of the stream may be scheduled as soon as
 // all CTAs of this one have started) and calls pdl_wait() before it first touches

@@ -3,6 +3,9 @@
 //  * head_gate: out[t, h, :] = x[t, h, :] * sigmoid(g[t, h]) * scale, one gate number per (token, head)
 //    taken from a wider row (the packed input projection; no gate pointer: a scaled copy); float32 arithmetic, rounded once.  The
 //    output may be a slice of a wider buffer (row stride given).
+//  * gate_mul: out[t, i] = x[t, i] * sigmoid(g[t, i]), one gate number per element (columns of a wider row are fine; out may
+//    be x).
+//  * square_relu: out = max(x, 0)^2.
 //  * weighted_sum: out = a * x + b * y in float32, rounded once (the outputs of two mixers that were
 //    projected separately).
 //  * logit_cap: y <- cap * tanh(y / cap), in place on float32 logits.
@@ -86,6 +89,79 @@ ARLE_API int arle_head_gate(const void* x, int x_stride, const void* g, int g_st
                   x_stride, (const __nv_bfloat16*)g, g_stride, scale, (__nv_bfloat16*)out, out_stride, heads, hd, total);
   else
     return ARLE_E_BADARG;
+  return launch_status();
+}
+
+// VEC consecutive elements a thread.
+template <typename T, int VEC>
+__global__ void gate_mul_kernel(const T* x, int x_stride, const T* __restrict__ g, int g_stride, T* out, int out_stride, int width, size_t total) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int wv = width / VEC;
+  for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
+    const size_t t = idx / wv;
+    const int e = (int)(idx - t * wv) * VEC;
+    float a[VEC], b[VEC];
+    load_vec<T, VEC>(x + t * x_stride + e, a);
+    load_vec<T, VEC>(g + t * g_stride + e, b);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) a[i] *= sizeof(T) == 2 ? __fdividef(1.0f, 1.0f + __expf(-b[i])) : 1.0f / (1.0f + expf(-b[i]));
+    store_vec<T, VEC>(out + t * out_stride + e, a);
+  }
+}
+
+template <typename T, int VEC>
+__global__ void square_relu_kernel(const T* x, int x_stride, T* out, int out_stride, int width, size_t total) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int wv = width / VEC;
+  for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
+    const size_t t = idx / wv;
+    const int e = (int)(idx - t * wv) * VEC;
+    float a[VEC];
+    load_vec<T, VEC>(x + t * x_stride + e, a);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+      const float r = fmaxf(a[i], 0.f);
+      a[i] = r * r;
+    }
+    store_vec<T, VEC>(out + t * out_stride + e, a);
+  }
+}
+
+ARLE_API int arle_gate_mul(const void* x, int x_stride, const void* g, int g_stride, void* out, int out_stride, int dtype, int num_tokens, int width,
+                           cudaStream_t s) {
+  if (num_tokens <= 0) return 0;
+  if (width <= 0 || (dtype != 0 && dtype != 1)) return ARLE_E_BADARG;
+  const size_t total = (size_t)num_tokens * width, eb = dtype == 0 ? 4 : 2;
+  const int n = dtype == 0 ? 4 : 8;
+  const bool vec = width % n == 0 && x_stride % n == 0 && g_stride % n == 0 && out_stride % n == 0 && ((uintptr_t)x % (n * eb)) == 0 &&
+                   ((uintptr_t)g % (n * eb)) == 0 && ((uintptr_t)out % (n * eb)) == 0;
+  const size_t work = vec ? total / n : total;
+  const dim3 grid(blocks_for(work, 256)), block(256);
+  if (dtype == 0)
+    launch_kernel(vec ? gate_mul_kernel<float, 4> : gate_mul_kernel<float, 1>, grid, block, 0, s, 1, (const float*)x, x_stride, (const float*)g,
+                  g_stride, (float*)out, out_stride, width, work);
+  else
+    launch_kernel(vec ? gate_mul_kernel<__nv_bfloat16, 8> : gate_mul_kernel<__nv_bfloat16, 1>, grid, block, 0, s, 1, (const __nv_bfloat16*)x,
+                  x_stride, (const __nv_bfloat16*)g, g_stride, (__nv_bfloat16*)out, out_stride, width, work);
+  return launch_status();
+}
+
+ARLE_API int arle_square_relu(const void* x, int x_stride, void* out, int out_stride, int dtype, int num_tokens, int width, cudaStream_t s) {
+  if (num_tokens <= 0) return 0;
+  if (width <= 0 || (dtype != 0 && dtype != 1)) return ARLE_E_BADARG;
+  const size_t total = (size_t)num_tokens * width, eb = dtype == 0 ? 4 : 2;
+  const int n = dtype == 0 ? 4 : 8;
+  const bool vec = width % n == 0 && x_stride % n == 0 && out_stride % n == 0 && ((uintptr_t)x % (n * eb)) == 0 && ((uintptr_t)out % (n * eb)) == 0;
+  const size_t work = vec ? total / n : total;
+  const dim3 grid(blocks_for(work, 256)), block(256);
+  if (dtype == 0)
+    launch_kernel(vec ? square_relu_kernel<float, 4> : square_relu_kernel<float, 1>, grid, block, 0, s, 1, (const float*)x, x_stride, (float*)out,
+                  out_stride, width, work);
+  else
+    launch_kernel(vec ? square_relu_kernel<__nv_bfloat16, 8> : square_relu_kernel<__nv_bfloat16, 1>, grid, block, 0, s, 1, (const __nv_bfloat16*)x,
+                  x_stride, (__nv_bfloat16*)out, out_stride, width, work);
   return launch_status();
 }
 

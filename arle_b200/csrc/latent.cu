@@ -7,7 +7,8 @@
 // the whole record and whose values are the record's first `rank` elements.
 //
 //  * latent_prep: per token, RMSNorm of the latent part with its weight, rotation of the shared key part
-//    (element i with i + rot_dims/2, angle position * inv_freq[i] in float32, elements past rot_dims pass),
+//    (element i with i + rot_dims/2, or 2i with 2i + 1; angle position * inv_freq[i] in float32, cosine and sine times a
+//    constant; elements past rot_dims pass),
 //    the record's store into the paged cache, and the rotation of every head's rotated query part into the
 //    folded queries' last `rot` columns.
 //  * latent_attention: one block per (token, group of heads).  A tile of 32 records is staged in shared
@@ -30,13 +31,29 @@ template <typename T>
 __global__ void latent_prep_kernel(const T* __restrict__ q, int q_stride, const T* __restrict__ dkv, int dkv_stride,
                                    const int* __restrict__ positions, const int* __restrict__ slot_mapping,
                                    const float* __restrict__ c_weight, float eps, const float* __restrict__ inv_freq,
-                                   int rot_dims, T* __restrict__ cache, T* __restrict__ q_abs, int H, int dn, int dr, int rank) {
+                                   int rot_dims, int pairing, float amplitude, T* __restrict__ cache, T* __restrict__ q_abs, int H, int dn, int dr, int rank) {
   pdl_launch_dependents();
   pdl_wait();
+  extern __shared__ float2 turn[];                 // (cos, sin) of the token's angles, evaluated once for the key and all heads
   __shared__ float red[33];
   const int t = blockIdx.x;
   const float pos = (float)positions[t];
   const int kd = rank + dr, half = rot_dims >> 1;
+  for (int j = threadIdx.x; j < half; j += blockDim.x) {
+    float sn, cs;
+    sincosf(pos * inv_freq[j], &sn, &cs);
+    turn[j] = make_float2(cs * amplitude, sn * amplitude);
+  }
+  __syncthreads();
+  // number i of a rotated vector p, turned with its partner (pairing 0: i and i + half; 1: neighbours 2j and 2j + 1)
+  auto turned = [&](const T* p, int i) -> float {
+    if (i >= rot_dims) return to_f32(p[i]);
+    const int j = pairing ? i >> 1 : (i < half ? i : i - half);
+    const bool first = pairing ? (i & 1) == 0 : i < half;
+    const float cs = turn[j].x, sn = turn[j].y;
+    const float u = to_f32(p[pairing ? 2 * j : j]), v = to_f32(p[pairing ? 2 * j + 1 : j + half]);
+    return first ? u * cs - v * sn : v * cs + u * sn;
+  };
   const T* kv = dkv + (size_t)t * dkv_stride;
   if (cache != nullptr) {
     float ss = 0.f;
@@ -48,49 +65,29 @@ __global__ void latent_prep_kernel(const T* __restrict__ q, int q_stride, const 
     const float inv = 1.0f / sqrtf(total / (float)rank + eps);
     T* dst = cache + (size_t)slot_mapping[t] * kd;
     for (int c = threadIdx.x; c < rank; c += blockDim.x) dst[c] = from_f32<T>(to_f32(kv[c]) * inv * c_weight[c]);
-    for (int i = threadIdx.x; i < dr; i += blockDim.x) {
-      float o;
-      if (i < rot_dims) {
-        const int p = i < half ? i : i - half;
-        float sn, cs;
-        sincosf(pos * inv_freq[p], &sn, &cs);
-        const float u = to_f32(kv[rank + p]), v = to_f32(kv[rank + p + half]);
-        o = i < half ? u * cs - v * sn : v * cs + u * sn;
-      } else {
-        o = to_f32(kv[rank + i]);
-      }
-      dst[rank + i] = from_f32<T>(o);
-    }
+    for (int i = threadIdx.x; i < dr; i += blockDim.x) dst[rank + i] = from_f32<T>(turned(kv + rank, i));
   }
   for (int idx = threadIdx.x; idx < H * dr; idx += blockDim.x) {
     const int h = idx / dr, i = idx - h * dr;
     const T* qp = q + (size_t)t * q_stride + (size_t)h * (dn + dr) + dn;
-    float o;
-    if (i < rot_dims) {
-      const int p = i < half ? i : i - half;
-      float sn, cs;
-      sincosf(pos * inv_freq[p], &sn, &cs);
-      const float u = to_f32(qp[p]), v = to_f32(qp[p + half]);
-      o = i < half ? u * cs - v * sn : v * cs + u * sn;
-    } else {
-      o = to_f32(qp[i]);
-    }
-    q_abs[((size_t)t * H + h) * kd + rank + i] = from_f32<T>(o);
+    q_abs[((size_t)t * H + h) * kd + rank + i] = from_f32<T>(turned(qp, i));
   }
 }
 
 ARLE_API int arle_latent_prep(const void* q, int q_stride, const void* dkv, int dkv_stride, int dtype, const int* positions,
-                              const int* slot_mapping, const float* c_weight, float eps, const float* inv_freq, int rot_dims,
+                              const int* slot_mapping, const float* c_weight, float eps, const float* inv_freq, int rot_dims, int pairing, float amplitude,
                               void* cache, void* q_abs, int H, int dn, int dr, int rank, int num_tokens, cudaStream_t s) {
   if (num_tokens <= 0) return 0;
-  if (H <= 0 || dn < 0 || dr < 0 || rank <= 0 || rot_dims < 0 || rot_dims > dr || (rot_dims & 1)) return ARLE_E_BADARG;
+  if (H <= 0 || dn < 0 || dr < 0 || rank <= 0 || rot_dims < 0 || rot_dims > dr || (rot_dims & 1) || (pairing != 0 && pairing != 1)) return ARLE_E_BADARG;
   const int threads = 128;
+  const size_t smem = (size_t)rot_dims / 2 * sizeof(float2);
+  if (smem > 40 * 1024) return ARLE_E_UNSUPPORTED;
   if (dtype == 0)
-    launch_kernel(latent_prep_kernel<float>, dim3(num_tokens), dim3(threads), 0, s, 1, (const float*)q, q_stride, (const float*)dkv,
-                  dkv_stride, positions, slot_mapping, c_weight, eps, inv_freq, rot_dims, (float*)cache, (float*)q_abs, H, dn, dr, rank);
+    launch_kernel(latent_prep_kernel<float>, dim3(num_tokens), dim3(threads), smem, s, 1, (const float*)q, q_stride, (const float*)dkv,
+                  dkv_stride, positions, slot_mapping, c_weight, eps, inv_freq, rot_dims, pairing, amplitude, (float*)cache, (float*)q_abs, H, dn, dr, rank);
   else if (dtype == 1)
-    launch_kernel(latent_prep_kernel<__nv_bfloat16>, dim3(num_tokens), dim3(threads), 0, s, 1, (const __nv_bfloat16*)q, q_stride,
-                  (const __nv_bfloat16*)dkv, dkv_stride, positions, slot_mapping, c_weight, eps, inv_freq, rot_dims,
+    launch_kernel(latent_prep_kernel<__nv_bfloat16>, dim3(num_tokens), dim3(threads), smem, s, 1, (const __nv_bfloat16*)q, q_stride,
+                  (const __nv_bfloat16*)dkv, dkv_stride, positions, slot_mapping, c_weight, eps, inv_freq, rot_dims, pairing, amplitude,
                   (__nv_bfloat16*)cache, (__nv_bfloat16*)q_abs, H, dn, dr, rank);
   else
     return ARLE_E_BADARG;

@@ -8,6 +8,8 @@
 //  * gla_decay: alpha[t, c] = sigmoid(z)^(1/tau), z = b[c] + sum_r low[t, r] * w2[c, r], the second
 //    half of a low-rank gate (low = W_a1 x comes from the packed input projection).  Evaluated as
 //    exp(-softplus(-z) / tau) in float32; a block takes sixteen tokens and 256 channels, r ascending.
+//    A second form has tanh between the two matrices and another decay: alpha = exp(-exp(z)), z = b[c] + sum_r
+//    tanh(low[t, r]) * w2[c, r].
 //  * gla_scan: the recurrence over this step's tokens of every request row, from the state that the
 //    request's slot holds, which is left updated.  Float32 throughout; q, k, v are read in the
 //    activation type.  One block of 128 threads per (columns of vdim, head, row); a thread keeps four
@@ -16,8 +18,12 @@
 //    q, k, alpha and v are staged in shared memory a chunk of tokens at a time, and o_t[j] is the sum
 //    over the column's lanes.  The order of every sum depends on (dim, vdim) only: a token's result
 //    does not depend on how the prompt was cut or on what else is in the batch.
-//  * gla_out: per head, o / sqrt(mean(o^2) + eps) * weight (shared by the heads), times silu(gate) (or sigmoid(gate)),
+//    With a bonus u (one number per head and key channel) the read-out comes before the update and sees the current
+//    token through u instead: o_t = (S_(t-1) + diag(u) k_t v_t^T)^T q_t.
+//  * gla_out: per head, o / sqrt(mean(o^2) + eps) * weight (shared by the heads, or one of all heads' size), times silu(gate) (or sigmoid(gate)),
 //    times a constant, rounded once into the activation type (a row of a wider buffer may be given).
+#include <initializer_list>
+
 #include "common.cuh"
 using namespace arle;
 
@@ -27,7 +33,7 @@ constexpr int kDecayTokens = 16;                 // tokens a block of the decay 
 constexpr int kDecayBatch = 16;                  // weights a thread asks for before it uses the first
 
 // w2t is the second matrix of the gate transposed, [rank][channels]: consecutive threads read consecutive floats.
-template <typename T>
+template <typename T, bool DOUBLE_EXP>
 __global__ void __launch_bounds__(256) gla_decay_kernel(const T* __restrict__ low, int low_stride, const float* __restrict__ w2t,
                                                         const float* __restrict__ bias, float inv_tau, float* __restrict__ alpha,
                                                         int num_tokens, int channels, int rank) {
@@ -38,7 +44,8 @@ __global__ void __launch_bounds__(256) gla_decay_kernel(const T* __restrict__ lo
   const int n = min(kDecayTokens, num_tokens - t0);
   for (int i = threadIdx.x; i < kDecayTokens * rank; i += blockDim.x) {
     const int tt = i / rank, r = i - tt * rank;
-    lo_s[i] = tt < n ? to_f32(low[(size_t)(t0 + tt) * low_stride + r]) : 0.f;
+    const float v = tt < n ? to_f32(low[(size_t)(t0 + tt) * low_stride + r]) : 0.f;
+    lo_s[i] = DOUBLE_EXP ? tanhf(v) : v;
   }
   __syncthreads();
   const int c = blockIdx.y * blockDim.x + threadIdx.x;
@@ -61,6 +68,10 @@ __global__ void __launch_bounds__(256) gla_decay_kernel(const T* __restrict__ lo
 #pragma unroll
   for (int tt = 0; tt < kDecayTokens; ++tt) {
     if (tt >= n) break;
+    if (DOUBLE_EXP) {
+      alpha[(size_t)(t0 + tt) * channels + c] = expf(-expf(z[tt] + b));
+      continue;
+    }
     const float y = -(z[tt] + b);                // softplus(y) = log(1 + e^y), the stable way
     const float sp = y > 0.f ? y + log1pf(expf(-y)) : log1pf(expf(y));
     alpha[(size_t)(t0 + tt) * channels + c] = expf(-sp * inv_tau);
@@ -85,10 +96,11 @@ template <> struct Raw4<__nv_bfloat16, true> { using type = uint2; };
 // worked on, the next chunk's q, k, alpha and v are already on their way into registers.  Every number of q, k and
 // alpha that a thread reads from shared memory serves four columns: with one column a thread the kernel was bound by
 // shared-memory bandwidth.
-template <typename T, int DPT, int LPC, bool VEC>
+// BONUS: the read-out before the update, with the current token weighted by u.
+template <typename T, int DPT, int LPC, bool VEC, bool BONUS>
 __global__ void __launch_bounds__(kScanThreads) gla_scan_kernel(
     const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, int in_stride,
-    const float* __restrict__ alpha, float* __restrict__ state, const int* __restrict__ q_indptr,
+    const float* __restrict__ alpha, const float* __restrict__ bonus, float* __restrict__ state, long slot_stride, const int* __restrict__ q_indptr,
     const int* __restrict__ state_slots, float* __restrict__ out, int heads, int dim, int vdim, float q_scale) {
   pdl_launch_dependents();
   pdl_wait();
@@ -108,8 +120,13 @@ __global__ void __launch_bounds__(kScanThreads) gla_scan_kernel(
   const int jb = j0 + jl * CPT;                  // this thread's first column
   const int t_begin = q_indptr[r], t_end = q_indptr[r + 1];
   // the state of a head is kept as [vdim][dim]: a thread's channels of a column are contiguous
-  float* S_g = state + (((size_t)state_slots[r] * heads + h) * vdim) * dim + l * DPT;
-  const bool vec_state = (dim & 3) == 0;
+  float* S_g = state + (size_t)state_slots[r] * slot_stride + ((size_t)h * vdim) * dim + l * DPT;
+  const bool vec_state = (dim & 3) == 0 && (slot_stride & 3) == 0 && ((uintptr_t)state & 15) == 0;
+  float u[BONUS ? DPT : 1];
+  if constexpr (BONUS) {
+#pragma unroll
+    for (int i = 0; i < DPT; ++i) u[i] = l * DPT + i < dim ? bonus[(size_t)h * dim + l * DPT + i] : 0.f;
+  }
   float S[CPT][DPT];
 #pragma unroll
   for (int cc = 0; cc < CPT; ++cc) {
@@ -216,6 +233,17 @@ __global__ void __launch_bounds__(kScanThreads) gla_scan_kernel(
         const float4 a4 = at[i], k4 = kt[i], q4 = qt[i];
 #pragma unroll
         for (int cc = 0; cc < CPT; ++cc) {
+          if constexpr (BONUS) {
+            const float kv0 = k4.x * vj[cc], kv1 = k4.y * vj[cc], kv2 = k4.z * vj[cc], kv3 = k4.w * vj[cc];
+            const float lo = fmaf(fmaf(u[4 * i], kv0, S[cc][4 * i]), q4.x, fmaf(u[4 * i + 1], kv1, S[cc][4 * i + 1]) * q4.y);
+            const float hi = fmaf(fmaf(u[4 * i + 2], kv2, S[cc][4 * i + 2]), q4.z, fmaf(u[4 * i + 3], kv3, S[cc][4 * i + 3]) * q4.w);
+            o[cc] += lo + hi;
+            S[cc][4 * i] = fmaf(a4.x, S[cc][4 * i], kv0);
+            S[cc][4 * i + 1] = fmaf(a4.y, S[cc][4 * i + 1], kv1);
+            S[cc][4 * i + 2] = fmaf(a4.z, S[cc][4 * i + 2], kv2);
+            S[cc][4 * i + 3] = fmaf(a4.w, S[cc][4 * i + 3], kv3);
+            continue;
+          }
           S[cc][4 * i] = fmaf(a4.x, S[cc][4 * i], k4.x * vj[cc]);
           S[cc][4 * i + 1] = fmaf(a4.y, S[cc][4 * i + 1], k4.y * vj[cc]);
           S[cc][4 * i + 2] = fmaf(a4.z, S[cc][4 * i + 2], k4.z * vj[cc]);
@@ -279,7 +307,7 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float a, float b, float
 template <typename T, bool VEC4>
 __global__ void gla_out_kernel(const float* __restrict__ o, const T* __restrict__ gate, int gate_stride,
                                const float* __restrict__ weight, float eps, float scale, T* __restrict__ out,
-                               int out_stride, int heads, int vdim, long long units, int sigmoid_gate) {
+                               int out_stride, int heads, int vdim, long long units, int sigmoid_gate, int weight_stride) {
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31;
@@ -288,6 +316,7 @@ __global__ void gla_out_kernel(const float* __restrict__ o, const T* __restrict_
   const long long t = unit / heads;
   const int h = (int)(unit - t * heads);
   const float* src = o + ((size_t)t * heads + h) * vdim;
+  if (weight) weight += (size_t)h * weight_stride;
   float ss = 0.f;
   if constexpr (VEC4) {                          // vdim a multiple of 4, rows on 16-byte (8-byte for bfloat16) boundaries
     const T* gp = gate ? gate + (size_t)t * gate_stride + (size_t)h * vdim : nullptr;
@@ -334,19 +363,26 @@ __global__ void gla_out_kernel(const float* __restrict__ o, const T* __restrict_
 }
 
 ARLE_API int arle_gla_decay(const void* low, int dtype, int low_stride, const float* w2t, const float* bias, float tau,
-                            float* alpha, int num_tokens, int channels, int rank, cudaStream_t s) {
+                            float* alpha, int num_tokens, int channels, int rank, int double_exp, cudaStream_t s) {
   if (num_tokens <= 0) return 0;
   if (channels <= 0 || rank <= 0 || !(tau > 0.f) || rank > 1024) return ARLE_E_BADARG;
   const int threads = 256;
   dim3 grid((num_tokens + kDecayTokens - 1) / kDecayTokens, (channels + threads - 1) / threads);
   if (grid.y > 65535) return ARLE_E_UNSUPPORTED;
   const size_t smem = (size_t)kDecayTokens * rank * sizeof(float);
+  if (smem > 40 * 1024) {
+    for (auto k : {(const void*)gla_decay_kernel<float, false>, (const void*)gla_decay_kernel<float, true>,
+                   (const void*)gla_decay_kernel<__nv_bfloat16, false>, (const void*)gla_decay_kernel<__nv_bfloat16, true>}) {
+      cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      if (e != cudaSuccess) return (int)e;
+    }
+  }
   if (dtype == 0)
-    launch_kernel(gla_decay_kernel<float>, grid, dim3(threads), smem, s, 1, (const float*)low, low_stride, w2t, bias, 1.0f / tau, alpha,
-                  num_tokens, channels, rank);
+    launch_kernel(double_exp ? gla_decay_kernel<float, true> : gla_decay_kernel<float, false>, grid, dim3(threads), smem, s, 1, (const float*)low,
+                  low_stride, w2t, bias, 1.0f / tau, alpha, num_tokens, channels, rank);
   else if (dtype == 1)
-    launch_kernel(gla_decay_kernel<__nv_bfloat16>, grid, dim3(threads), smem, s, 1, (const __nv_bfloat16*)low, low_stride, w2t, bias,
-                  1.0f / tau, alpha, num_tokens, channels, rank);
+    launch_kernel(double_exp ? gla_decay_kernel<__nv_bfloat16, true> : gla_decay_kernel<__nv_bfloat16, false>, grid, dim3(threads), smem, s, 1,
+                  (const __nv_bfloat16*)low, low_stride, w2t, bias, 1.0f / tau, alpha, num_tokens, channels, rank);
   else
     return ARLE_E_BADARG;
   return launch_status();
@@ -355,30 +391,28 @@ ARLE_API int arle_gla_decay(const void* low, int dtype, int low_stride, const fl
 namespace {
 
 template <typename T, int DPT, int LPC>
-int scan_launch(const void* q, const void* k, const void* v, int in_stride, const float* alpha, float* state, const int* q_indptr,
+int scan_launch(const void* q, const void* k, const void* v, int in_stride, const float* alpha, const float* bonus, float* state, long slot_stride, const int* q_indptr,
                 const int* state_slots, float* out, int rows, int heads, int dim, int vdim, float q_scale, cudaStream_t s) {
   constexpr int COLS = kScanThreads / LPC * kScanCpt;
   dim3 grid((vdim + COLS - 1) / COLS, heads, rows);
   const size_t eb = sizeof(T) * 4;               // bytes of four elements of q or k
   const bool vec = dim % 4 == 0 && in_stride % 4 == 0 && ((uintptr_t)q % eb) == 0 && ((uintptr_t)k % eb) == 0 &&
                    ((uintptr_t)alpha % 16) == 0;
-  if (vec)
-    launch_kernel(gla_scan_kernel<T, DPT, LPC, true>, grid, dim3(kScanThreads), 0, s, 1, (const T*)q, (const T*)k, (const T*)v,
-                  in_stride, alpha, state, q_indptr, state_slots, out, heads, dim, vdim, q_scale);
-  else
-    launch_kernel(gla_scan_kernel<T, DPT, LPC, false>, grid, dim3(kScanThreads), 0, s, 1, (const T*)q, (const T*)k, (const T*)v,
-                  in_stride, alpha, state, q_indptr, state_slots, out, heads, dim, vdim, q_scale);
+  auto kernel = bonus ? (vec ? gla_scan_kernel<T, DPT, LPC, true, true> : gla_scan_kernel<T, DPT, LPC, false, true>)
+                      : (vec ? gla_scan_kernel<T, DPT, LPC, true, false> : gla_scan_kernel<T, DPT, LPC, false, false>);
+  launch_kernel(kernel, grid, dim3(kScanThreads), 0, s, 1, (const T*)q, (const T*)k, (const T*)v, in_stride, alpha, bonus, state, slot_stride,
+                q_indptr, state_slots, out, heads, dim, vdim, q_scale);
   return launch_status();
 }
 
 // The split of the key channels among threads depends on dim alone, so the order of a token's sums does too: four
 // channels a thread up to 128 channels (as many lanes as that takes, a power of two), then 8 and 16 on 32 lanes.
 template <typename T>
-int scan_dispatch(const void* q, const void* k, const void* v, int in_stride, const float* alpha, float* state,
-                  const int* q_indptr, const int* state_slots, float* out, int rows, int heads, int dim, int vdim, float q_scale,
+int scan_dispatch(const void* q, const void* k, const void* v, int in_stride, const float* alpha, const float* bonus, float* state,
+                  long slot_stride, const int* q_indptr, const int* state_slots, float* out, int rows, int heads, int dim, int vdim, float q_scale,
                   cudaStream_t s) {
 #define ARLE_SCAN(D, L) \
-  return scan_launch<T, D, L>(q, k, v, in_stride, alpha, state, q_indptr, state_slots, out, rows, heads, dim, vdim, q_scale, s)
+  return scan_launch<T, D, L>(q, k, v, in_stride, alpha, bonus, state, slot_stride, q_indptr, state_slots, out, rows, heads, dim, vdim, q_scale, s)
   if (dim <= 4) ARLE_SCAN(4, 1);
   if (dim <= 8) ARLE_SCAN(4, 2);
   if (dim <= 16) ARLE_SCAN(4, 4);
@@ -393,21 +427,21 @@ int scan_dispatch(const void* q, const void* k, const void* v, int in_stride, co
 
 }  // namespace
 
-ARLE_API int arle_gla_scan(const void* q, const void* k, const void* v, int dtype, int in_stride, const float* alpha,
-                           float* state, const int* q_indptr, const int* state_slots, float* out, int rows, int heads,
+ARLE_API int arle_gla_scan(const void* q, const void* k, const void* v, int dtype, int in_stride, const float* alpha, const float* bonus,
+                           float* state, long slot_stride, const int* q_indptr, const int* state_slots, float* out, int rows, int heads,
                            int dim, int vdim, float q_scale, int max_q_len, cudaStream_t s) {
   if (rows <= 0) return 0;
-  if (heads <= 0 || dim <= 0 || vdim <= 0 || max_q_len <= 0) return ARLE_E_BADARG;
+  if (heads <= 0 || dim <= 0 || vdim <= 0 || max_q_len <= 0 || slot_stride < (long)heads * vdim * dim) return ARLE_E_BADARG;
   if (dim > 512 || heads > 65535 || rows > 65535) return ARLE_E_UNSUPPORTED;
   if (dtype == 0)
-    return scan_dispatch<float>(q, k, v, in_stride, alpha, state, q_indptr, state_slots, out, rows, heads, dim, vdim, q_scale, s);
+    return scan_dispatch<float>(q, k, v, in_stride, alpha, bonus, state, slot_stride, q_indptr, state_slots, out, rows, heads, dim, vdim, q_scale, s);
   if (dtype == 1)
-    return scan_dispatch<__nv_bfloat16>(q, k, v, in_stride, alpha, state, q_indptr, state_slots, out, rows, heads, dim, vdim, q_scale, s);
+    return scan_dispatch<__nv_bfloat16>(q, k, v, in_stride, alpha, bonus, state, slot_stride, q_indptr, state_slots, out, rows, heads, dim, vdim, q_scale, s);
   return ARLE_E_BADARG;
 }
 
 ARLE_API int arle_gla_out(const float* o, const void* gate, int dtype, int gate_stride, const float* weight, float eps,
-                          float scale, void* out, int out_stride, int num_tokens, int heads, int vdim, int sigmoid_gate, cudaStream_t s) {
+                          float scale, void* out, int out_stride, int num_tokens, int heads, int vdim, int sigmoid_gate, int weight_stride, cudaStream_t s) {
   if (num_tokens <= 0) return 0;
   if (heads <= 0 || vdim <= 0) return ARLE_E_BADARG;
   const long long units = (long long)num_tokens * heads;
@@ -416,15 +450,15 @@ ARLE_API int arle_gla_out(const float* o, const void* gate, int dtype, int gate_
   if (blocks > 0x7fffffffLL) return ARLE_E_UNSUPPORTED;
   const size_t eb = dtype == 0 ? 16 : 8;         // bytes of four elements of gate and out
   const bool vec = vdim % 4 == 0 && gate_stride % 4 == 0 && out_stride % 4 == 0 && ((uintptr_t)o % 16) == 0 &&
-                   ((uintptr_t)gate % eb) == 0 && ((uintptr_t)out % eb) == 0 && ((uintptr_t)weight % 16) == 0;
+                   ((uintptr_t)gate % eb) == 0 && ((uintptr_t)out % eb) == 0 && ((uintptr_t)weight % 16) == 0 && weight_stride % 4 == 0;
   if (dtype == 0) {
     auto kern = vec ? gla_out_kernel<float, true> : gla_out_kernel<float, false>;
     launch_kernel(kern, dim3((unsigned)blocks), dim3(warps * 32), 0, s, 1, o, (const float*)gate, gate_stride, weight, eps, scale,
-                  (float*)out, out_stride, heads, vdim, units, sigmoid_gate);
+                  (float*)out, out_stride, heads, vdim, units, sigmoid_gate, weight_stride);
   } else if (dtype == 1) {
     auto kern = vec ? gla_out_kernel<__nv_bfloat16, true> : gla_out_kernel<__nv_bfloat16, false>;
     launch_kernel(kern, dim3((unsigned)blocks), dim3(warps * 32), 0, s, 1, o, (const __nv_bfloat16*)gate, gate_stride, weight, eps,
-                  scale, (__nv_bfloat16*)out, out_stride, heads, vdim, units, sigmoid_gate);
+                  scale, (__nv_bfloat16*)out, out_stride, heads, vdim, units, sigmoid_gate, weight_stride);
   } else {
     return ARLE_E_BADARG;
   }

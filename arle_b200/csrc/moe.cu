@@ -18,7 +18,9 @@
 //    columns, mma.sync with float32 sums, operands brought in by cp.async in three stages), and a step of few pairs
 //    (decoding) runs it as one dot product a warp (moe_gemv: every chosen expert's rows are streamed once, 16 bytes
 //    a lane and load), since a tile of 64 places would be all but empty.
-//  * moe_combine: out[t] = sum_k weight[t, k] * Y[place(t, k)] (k ascending) + sigmoid(gate[t]) * shared[t].
+//    The sums may be finished before they are stored: times a number per place (the choice's weight, when it multiplies the
+//    expert's input: W (w x) = w (W x)), then through an activation (the square of relu).
+//  * moe_combine: out[t] = sum_k weight[t, k] * Y[place(t, k)] (k ascending; no weights: ones) + sigmoid(gate[t]) * shared[t].
 #include "common.cuh"
 #include "mma_utils.cuh"
 using namespace arle;
@@ -110,7 +112,8 @@ constexpr int kMoeMaxExperts = 1024;
 
 // plan (int32): [0, E] offsets of the experts' runs; [E + 1] tiles in use; then per tile (expert, first place, places).
 __global__ void __launch_bounds__(1024) moe_plan_kernel(const int* __restrict__ ids, int pairs, int top, int E, int* __restrict__ plan,
-                                                        int* __restrict__ place_of_pair, int* __restrict__ row_of_place, int max_tiles) {
+                                                        int* __restrict__ place_of_pair, int* __restrict__ row_of_place, int max_tiles,
+                                                        const float* __restrict__ wts, float* __restrict__ weight_of_place) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ int count[kMoeMaxExperts], offset[kMoeMaxExperts + 1], cursor[kMoeMaxExperts];
@@ -141,18 +144,30 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const int* __restrict__ 
     const int place = offset[e] + atomicAdd(&cursor[e], 1);
     place_of_pair[p] = place;
     row_of_place[place] = p / top;
+    if (wts) weight_of_place[place] = wts[p];
   }
 }
 
 ARLE_API int arle_moe_plan_ints(int E, int pairs) { return E + 2 + 3 * (pairs / kMoeTile + E + 1); }
 
 ARLE_API int arle_moe_plan(const int* ids, int pairs, int top, int E, int* plan, int* place_of_pair, int* row_of_place,
-                           cudaStream_t s) {
+                           const float* wts, float* weight_of_place, cudaStream_t s) {
   if (pairs <= 0) return 0;
   if (E <= 0 || E > kMoeMaxExperts || top <= 0) return ARLE_E_UNSUPPORTED;
+  if ((wts == nullptr) != (weight_of_place == nullptr)) return ARLE_E_BADARG;
   launch_kernel(moe_plan_kernel, dim3(1), dim3(1024), 0, s, 1, ids, pairs, top, E, plan, place_of_pair, row_of_place,
-                pairs / kMoeTile + E + 1);
+                pairs / kMoeTile + E + 1, wts, weight_of_place);
   return launch_status();
+}
+
+// What happens to a grouped product's sum before it is stored.  act 1: the square of relu.
+__device__ __forceinline__ float finish_sum(float v, float place_scale, int act) {
+  v *= place_scale;
+  if (act == 1) {
+    v = fmaxf(v, 0.f);
+    v *= v;
+  }
+  return v;
 }
 
 constexpr int GM = 64, GN = 64, GK = 16;
@@ -160,7 +175,8 @@ constexpr int GM = 64, GN = 64, GK = 16;
 template <typename TA, typename TW, typename TC>
 __global__ void __launch_bounds__(256) moe_gemm_kernel(const TA* __restrict__ A, int lda, const int* __restrict__ rows,
                                                        const TW* __restrict__ W, int ldw, long w_expert, TC* __restrict__ C, int ldc,
-                                                       const int* __restrict__ plan, int E, int N, int K) {
+                                                       const int* __restrict__ plan, int E, int N, int K,
+                                                       const float* __restrict__ place_scale, int act) {
   pdl_launch_dependents();
   pdl_wait();
   const int tile = blockIdx.y;
@@ -210,10 +226,11 @@ __global__ void __launch_bounds__(256) moe_gemm_kernel(const TA* __restrict__ A,
   for (int i = 0; i < 4; ++i) {
     const int m = ty * 4 + i;
     if (m >= M) continue;
+    const float ps = place_scale ? place_scale[p0 + m] : 1.f;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int gn = n0 + tx * 4 + j;
-      if (gn < N) C[(size_t)(p0 + m) * ldc + gn] = from_f32<TC>(acc[i][j]);
+      if (gn < N) C[(size_t)(p0 + m) * ldc + gn] = from_f32<TC>(finish_sum(acc[i][j], ps, act));
     }
   }
 }
@@ -222,10 +239,11 @@ constexpr int TM = 64, TN = 128, TK = 32, TPITCH = 40, kStages = 3;
 
 // A tile of 64 rows x 128 columns of C = A . W^T on the tensor cores: row r of the tile is row arow[r] of A (-1: none) and
 // row crow0 + r of C; M rows are live.  Three stages of cp.async, one barrier a stage, eight warps of 32 x 32, mma.sync with float32 sums.
-template <typename TC>
+// finish(v, row of C, column): what is stored for the sum v.
+template <typename TC, typename FINISH>
 __device__ __forceinline__ void mma_tile_64x128(const __nv_bfloat16* __restrict__ A, int lda, const int* arow, const __nv_bfloat16* __restrict__ W,
                                                 int ldw, TC* __restrict__ C, int ldc, size_t crow0, int M, int n0, int N, int K,
-                                                __nv_bfloat16 (*As)[TM * TPITCH], __nv_bfloat16 (*Ws)[TN * TPITCH]) {
+                                                __nv_bfloat16 (*As)[TM * TPITCH], __nv_bfloat16 (*Ws)[TN * TPITCH], FINISH finish) {
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int wm = warp & 1, wn = warp >> 1;
   auto load = [&](int stage, int k0) {
@@ -291,15 +309,15 @@ __device__ __forceinline__ void mma_tile_64x128(const __nv_bfloat16* __restrict_
         const int col = n0 + wn * 32 + nt * 8 + 2 * t4;
         if (m >= M) continue;
         TC* cp = C + (crow0 + m) * ldc + col;
-        if (col < N) cp[0] = from_f32<TC>(acc[mt][nt][2 * half]);
-        if (col + 1 < N) cp[1] = from_f32<TC>(acc[mt][nt][2 * half + 1]);
+        if (col < N) cp[0] = from_f32<TC>(finish(acc[mt][nt][2 * half], crow0 + m, col));
+        if (col + 1 < N) cp[1] = from_f32<TC>(finish(acc[mt][nt][2 * half + 1], crow0 + m, col + 1));
       }
 }
 
 __global__ void __launch_bounds__(256) moe_gemm_mma_kernel(const __nv_bfloat16* __restrict__ A, int lda, const int* __restrict__ rows,
                                                            const __nv_bfloat16* __restrict__ W, int ldw, long w_expert,
                                                            __nv_bfloat16* __restrict__ C, int ldc, const int* __restrict__ plan, int E,
-                                                           int N, int K) {
+                                                           int N, int K, const float* __restrict__ place_scale, int act) {
   pdl_launch_dependents();
   pdl_wait();
   const int tile = blockIdx.y;
@@ -311,15 +329,17 @@ __global__ void __launch_bounds__(256) moe_gemm_mma_kernel(const __nv_bfloat16* 
   __shared__ int arow[TM];
   if (threadIdx.x < TM) arow[threadIdx.x] = (int)threadIdx.x < M ? (rows ? rows[p0 + threadIdx.x] : p0 + (int)threadIdx.x) : -1;
   __syncthreads();
-  mma_tile_64x128(A, lda, arow, W + (size_t)expert * w_expert, ldw, C, ldc, (size_t)p0, M, blockIdx.x * TN, N, K, As, Ws);
+  mma_tile_64x128(A, lda, arow, W + (size_t)expert * w_expert, ldw, C, ldc, (size_t)p0, M, blockIdx.x * TN, N, K, As, Ws,
+                  [&](float v, size_t row, int) { return finish_sum(v, place_scale ? place_scale[row] : 1.f, act); });
 }
 
 // The same tile for one matrix per head, heads side by side in the rows of A and C (see arle_gemm_heads): grid (column
-// tiles, row tiles, heads).
+// tiles, row tiles, heads).  With a gate [M][heads * N] a sum is multiplied by sigmoid(gate) before it is stored.
 template <typename TC>
 __global__ void __launch_bounds__(256) gemm_heads_mma_kernel(const __nv_bfloat16* __restrict__ A, int lda, int a_head,
                                                              const __nv_bfloat16* __restrict__ W, int ldw, long w_head,
-                                                             TC* __restrict__ C, int ldc, int c_head, int M, int N, int K) {
+                                                             TC* __restrict__ C, int ldc, int c_head, int M, int N, int K,
+                                                             const __nv_bfloat16* __restrict__ gate, int gate_stride) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ __align__(16) __nv_bfloat16 As[kStages][TM * TPITCH];
@@ -329,12 +349,14 @@ __global__ void __launch_bounds__(256) gemm_heads_mma_kernel(const __nv_bfloat16
   if (threadIdx.x < TM) arow[threadIdx.x] = m0 + (int)threadIdx.x < M ? m0 + (int)threadIdx.x : -1;
   __syncthreads();
   mma_tile_64x128(A + (size_t)head * a_head, lda, arow, W + (size_t)head * w_head, ldw, C + (size_t)head * c_head, ldc, (size_t)m0,
-                  min(TM, M - m0), blockIdx.x * TN, N, K, As, Ws);
+                  min(TM, M - m0), blockIdx.x * TN, N, K, As, Ws, [&](float v, size_t row, int col) {
+                    return gate ? v * __fdividef(1.0f, 1.0f + __expf(-__bfloat162float(gate[row * gate_stride + (size_t)head * N + col]))) : v;
+                  });
 }
 
 // bfloat16 A and W, K and every stride a multiple of 8 elements, bases on 16-byte boundaries; C bfloat16 or (c_dtype 0) float32.
 ARLE_API int arle_gemm_heads_mma(const void* A, const void* W, void* C, int c_dtype, int M, int N, int K, int heads, int lda, int ldw, int ldc,
-                                 int a_head, long w_head, int c_head, cudaStream_t s) {
+                                 int a_head, long w_head, int c_head, const void* gate, int gate_stride, cudaStream_t s) {
   if (M <= 0 || N <= 0 || heads <= 0) return 0;
   if (K <= 0) return ARLE_E_BADARG;
   if (K % 8 || lda % 8 || ldw % 8 || a_head % 8 || w_head % 8 || ((uintptr_t)A & 15) || ((uintptr_t)W & 15)) return ARLE_E_UNSUPPORTED;
@@ -342,10 +364,10 @@ ARLE_API int arle_gemm_heads_mma(const void* A, const void* W, void* C, int c_dt
   if (grid.y > 65535 || heads > 65535) return ARLE_E_UNSUPPORTED;
   if (c_dtype == 0)
     launch_kernel(gemm_heads_mma_kernel<float>, dim3(grid), dim3(256), 0, s, 1, (const __nv_bfloat16*)A, lda, a_head, (const __nv_bfloat16*)W,
-                  ldw, w_head, (float*)C, ldc, c_head, M, N, K);
+                  ldw, w_head, (float*)C, ldc, c_head, M, N, K, (const __nv_bfloat16*)gate, gate_stride);
   else
     launch_kernel(gemm_heads_mma_kernel<__nv_bfloat16>, dim3(grid), dim3(256), 0, s, 1, (const __nv_bfloat16*)A, lda, a_head,
-                  (const __nv_bfloat16*)W, ldw, w_head, (__nv_bfloat16*)C, ldc, c_head, M, N, K);
+                  (const __nv_bfloat16*)W, ldw, w_head, (__nv_bfloat16*)C, ldc, c_head, M, N, K, (const __nv_bfloat16*)gate, gate_stride);
   return launch_status();
 }
 
@@ -354,7 +376,7 @@ ARLE_API int arle_gemm_heads_mma(const void* A, const void* W, void* C, int c_dt
 __global__ void __launch_bounds__(256) moe_gemv_kernel(const __nv_bfloat16* __restrict__ A, int lda, const int* __restrict__ rows,
                                                        const __nv_bfloat16* __restrict__ W, int ldw, long w_expert,
                                                        __nv_bfloat16* __restrict__ C, int ldc, const int* __restrict__ plan, int E, int N,
-                                                       int K) {
+                                                       int K, const float* __restrict__ place_scale, int act) {
   pdl_launch_dependents();
   pdl_wait();
   const int place = blockIdx.y;
@@ -379,38 +401,40 @@ __global__ void __launch_bounds__(256) moe_gemv_kernel(const __nv_bfloat16* __re
     }
   }
   acc = warp_sum(acc);
-  if (lane == 0) C[(size_t)place * ldc + n] = __float2bfloat16_rn(acc);
+  if (lane == 0) C[(size_t)place * ldc + n] = __float2bfloat16_rn(finish_sum(acc, place_scale ? place_scale[place] : 1.f, act));
 }
 
 // dtype: type of A and C; w_dtype: type of W [E][N][K] (an expert every w_expert elements).  pairs: places in all.
+// place_scale float32 [pairs] or null, act 0 none / 1 square of relu: see finish_sum.
 // fast: bfloat16 operands with aligned rows may take the tensor-core tiles or, for few pairs, the dot products.
 ARLE_API int arle_moe_gemm(const void* A, int lda, const int* rows, const void* W, int ldw, long w_expert, void* C, int ldc,
-                           int dtype, int w_dtype, const int* plan, int E, int pairs, int N, int K, int fast, cudaStream_t s) {
+                           int dtype, int w_dtype, const int* plan, int E, int pairs, int N, int K, int fast,
+                           const float* place_scale, int act, cudaStream_t s) {
   if (pairs <= 0 || N <= 0) return 0;
-  if (K <= 0 || E <= 0) return ARLE_E_BADARG;
+  if (K <= 0 || E <= 0 || (act != 0 && act != 1)) return ARLE_E_BADARG;
   const int max_tiles = pairs / kMoeTile + E + 1;
   if (max_tiles > 65535) return ARLE_E_UNSUPPORTED;
   if (fast && dtype == 1 && w_dtype == 1 && K % 8 == 0 && lda % 8 == 0 && ldw % 8 == 0 && w_expert % 8 == 0 &&
       ((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0) {
     if (pairs <= 128) {
       launch_kernel(moe_gemv_kernel, dim3((N + 7) / 8, pairs), dim3(256), 0, s, 1, (const __nv_bfloat16*)A, lda, rows,
-                    (const __nv_bfloat16*)W, ldw, w_expert, (__nv_bfloat16*)C, ldc, plan, E, N, K);
+                    (const __nv_bfloat16*)W, ldw, w_expert, (__nv_bfloat16*)C, ldc, plan, E, N, K, place_scale, act);
     } else {
       launch_kernel(moe_gemm_mma_kernel, dim3((N + TN - 1) / TN, max_tiles), dim3(256), 0, s, 1, (const __nv_bfloat16*)A, lda, rows,
-                    (const __nv_bfloat16*)W, ldw, w_expert, (__nv_bfloat16*)C, ldc, plan, E, N, K);
+                    (const __nv_bfloat16*)W, ldw, w_expert, (__nv_bfloat16*)C, ldc, plan, E, N, K, place_scale, act);
     }
     return launch_status();
   }
   dim3 grid((N + GN - 1) / GN, max_tiles);
   if (dtype == 0 && w_dtype == 0)
     launch_kernel(moe_gemm_kernel<float, float, float>, dim3(grid), dim3(256), 0, s, 1, (const float*)A, lda, rows, (const float*)W, ldw,
-                  w_expert, (float*)C, ldc, plan, E, N, K);
+                  w_expert, (float*)C, ldc, plan, E, N, K, place_scale, act);
   else if (dtype == 0 && w_dtype == 1)
     launch_kernel(moe_gemm_kernel<float, __nv_bfloat16, float>, dim3(grid), dim3(256), 0, s, 1, (const float*)A, lda, rows,
-                  (const __nv_bfloat16*)W, ldw, w_expert, (float*)C, ldc, plan, E, N, K);
+                  (const __nv_bfloat16*)W, ldw, w_expert, (float*)C, ldc, plan, E, N, K, place_scale, act);
   else if (dtype == 1 && w_dtype == 1)
     launch_kernel(moe_gemm_kernel<__nv_bfloat16, __nv_bfloat16, __nv_bfloat16>, dim3(grid), dim3(256), 0, s, 1, (const __nv_bfloat16*)A,
-                  lda, rows, (const __nv_bfloat16*)W, ldw, w_expert, (__nv_bfloat16*)C, ldc, plan, E, N, K);
+                  lda, rows, (const __nv_bfloat16*)W, ldw, w_expert, (__nv_bfloat16*)C, ldc, plan, E, N, K, place_scale, act);
   else
     return ARLE_E_BADARG;
   return launch_status();
@@ -428,7 +452,7 @@ __global__ void moe_combine_kernel(const T* __restrict__ y, int y_stride, const 
   for (int c = threadIdx.x; c < width; c += blockDim.x) {
     float acc = 0.f;
     for (int k = 0; k < top; ++k)
-      acc = fmaf(wts[(size_t)t * top + k], to_f32(y[(size_t)place_of_pair[(size_t)t * top + k] * y_stride + c]), acc);
+      acc = fmaf(wts ? wts[(size_t)t * top + k] : 1.f, to_f32(y[(size_t)place_of_pair[(size_t)t * top + k] * y_stride + c]), acc);
     if (shared) acc = fmaf(g, to_f32(shared[(size_t)t * shared_stride + c]), acc);
     out[(size_t)t * out_stride + c] = from_f32<T>(acc);
   }

@@ -44,16 +44,16 @@ _SIGNATURES = {
     "arle_residual_add": [_P, _P, _I, _I, _I, _P],
     "arle_silu_mul": [_P, _P, _I, _I, _I, _P],
     "arle_act_mul": [_P, _P, _I, _I, _I, _I, _I, _P],
-    "arle_attention_prep_row": [_P, _I, _I, _P, _P, _P, _P, _F, _P, _P, _I, _I, _I, _P, _P, _I, _I, _I, _I, _I, _P],
+    "arle_attention_prep_row": [_P, _I, _I, _P, _P, _P, _P, _F, _P, _P, _I, _I, _I, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     "arle_head_gate": [_P, _I, _P, _I, _F, _P, _I, _I, _I, _I, _I, _P],
     "arle_weighted_sum": [_P, _F, _P, _F, _P, _I, ctypes.c_longlong, _P],
     "arle_logit_cap": [_P, _F, ctypes.c_longlong, _P],
-    "arle_gla_decay": [_P, _I, _I, _P, _P, _F, _P, _I, _I, _I, _P],
-    "arle_gla_scan": [_P, _P, _P, _I, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _P],
-    "arle_gla_out": [_P, _P, _I, _I, _P, _F, _F, _P, _I, _I, _I, _I, _I, _P],
+    "arle_gla_decay": [_P, _I, _I, _P, _P, _F, _P, _I, _I, _I, _I, _P],
+    "arle_gla_scan": [_P, _P, _P, _I, _I, _P, _P, _P, ctypes.c_long, _P, _P, _P, _I, _I, _I, _I, _F, _I, _P],
+    "arle_gla_out": [_P, _P, _I, _I, _P, _F, _F, _P, _I, _I, _I, _I, _I, _I, _P],
     "arle_attention_prep": [_P, _I, _I, _P, _P, _P, _P, _F, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P],
     "arle_rotary_angles": [_P, _P, _P, _I, _I, _P],
-    "arle_paged_attention_plain": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _F, _I, _F, _I, _P],
+    "arle_paged_attention_plain": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _F, _I, _F, _I, _P, _I, _P],
     "arle_attention_prep_post": [_P, _I, _I, _P, _P, _P, _P, _F, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
     "arle_branch_norm_add": [_P, _P, _I, _P, _P, _I, _I, _I, _F, _P],
     "arle_branch_norm_add_norm": [_P, _P, _I, _P, _P, _P, _I, _I, _I, _F, _F, _P],
@@ -65,16 +65,16 @@ _SIGNATURES = {
     "arle_delta_gates": [_P, _I, _P, _P, _P, _P, _I, _I, _P],
     "arle_delta_scan": [_P, _P, _P, _I, _I, _I, _I, _P, _P, _P, ctypes.c_long, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _P],
     "arle_clamped_glu": [_P, _P, _I, _I, _I, _I, _F, _F, _P],
-    "arle_paged_attention_decode": [_P, _I, _P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _F, _F, _I, _I, _I, _I, _F, _P],
+    "arle_paged_attention_decode": [_P, _I, _P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _F, _F, _I, _I, _I, _I, _F, _I, _P, _P],
     "arle_paged_attention_decode_stream": [_P, _I, _P, _P, _P, ctypes.c_longlong, _P, _P, _P, _I, _I, _P, _P, _P, _I, _I, _I, _I,
                                            _F, _F, _I, _I, _I, _P, _P],
     "arle_paged_attention_decode_stream_prep": [_P, _I, _P, _P, _P, ctypes.c_longlong, _P, _P, _P, _I, _I, _P, _P, _P, _I, _I, _I, _I,
                                                 _F, _F, _I, _I, _I, _I, _P, _P, _P, _F, _P, _P, _P, _P],
     "arle_decode_stream_plan_ints": [_I, _I],
     "arle_decode_stream_plan": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P],
-    "arle_paged_attention_prefill": [_P, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _I, _I, _I, _I, _I, _F, _P],
+    "arle_paged_attention_prefill": [_P, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _I, _I, _I, _I, _I, _F, _I, _P, _P],
     "arle_paged_attention_prefill_tc": [_P, _I, _I, _P, _P, _P, ctypes.c_longlong, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _I,
-                                        _I, _I, _I, _P, _I, _F, _P],
+                                        _I, _I, _I, _P, _I, _F, _I, _P, _P],
     "arle_gemm_f32": [_P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _P],
     "arle_gemm_plain_bf16": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
     "arle_gemm_skinny": [_P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _P, _P],
@@ -86,9 +86,9 @@ _SIGNATURES = {
     "arle_scatter_tokens": [_P, _P, _P, _I, _P],
     "arle_sample": [_P, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P, _P],
     "arle_dyt_norm": [_P, _P, _P, _P, _P, _F, _P, _I, _I, _I, _I, _P],
-    "arle_gemm_heads_mma": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, ctypes.c_long, _I, _P],
+    "arle_gemm_heads_mma": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, ctypes.c_long, _I, _P, _I, _P],
     "arle_gemm_heads": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, ctypes.c_long, _I, _P],
-    "arle_latent_prep": [_P, _I, _P, _I, _I, _P, _P, _P, _F, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P],
+    "arle_latent_prep": [_P, _I, _P, _I, _I, _P, _P, _P, _F, _P, _I, _I, _F, _P, _P, _I, _I, _I, _I, _I, _P],
     "arle_latent_attention_mma": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P],
     "arle_latent_attention": [_P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P],
     "arle_decay_scan": [_P, _P, _P, _I, _I, _I, _I, _P, _P, _P, ctypes.c_long, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P],
@@ -98,8 +98,14 @@ _SIGNATURES = {
     "arle_conv_silu": [_P, _I, _I, _P, _P, _P, ctypes.c_long, ctypes.c_long, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P],
     "arle_gated_group_norm": [_P, _P, _I, _I, _P, _I, _P, _I, _P, _F, _P, _I, _I, _I, _I, _P],
     "arle_moe_select": [_P, _I, _P, _P, _I, _I, _I, _I, _F, _I, _P, _P, _I, _P],
-    "arle_moe_plan": [_P, _I, _I, _I, _P, _P, _P, _P],
-    "arle_moe_gemm": [_P, _I, _P, _P, _I, ctypes.c_long, _P, _I, _I, _I, _P, _I, _I, _I, _I, _I, _P],
+    "arle_moe_plan": [_P, _I, _I, _I, _P, _P, _P, _P, _P, _P],
+    "arle_moe_gemm": [_P, _I, _P, _P, _I, ctypes.c_long, _P, _I, _I, _I, _P, _I, _I, _I, _I, _I, _P, _I, _P],
+    "arle_layernorm": [_P, _P, _P, _P, _P, _I, _I, _I, _F, _I, _P],
+    "arle_branch_layernorm_add": [_P, _P, _I, _P, _P, _I, _I, _I, _F, _P, _I, _P, ctypes.c_long, _P, _P, _P],
+    "arle_input_conv": [_P, _P, _P, ctypes.c_long, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
+    "arle_token_shift": [_P, _I, _I, _P, _I, _P, ctypes.c_long, _P, _P, _P, _P, ctypes.c_long, _I, _I, _I, _I, _P],
+    "arle_gate_mul": [_P, _I, _P, _I, _P, _I, _I, _I, _I, _P],
+    "arle_square_relu": [_P, _I, _P, _I, _I, _I, _I, _P],
     "arle_moe_combine": [_P, _I, _P, _P, _I, _P, _I, _P, _I, _P, _I, _I, _I, _I, _P],
 }
 
@@ -526,8 +532,11 @@ def attention_prep(qkv, positions, slot_mapping, q_weight, k_weight, eps, inv_fr
 
 def paged_attention(q, out, k_cache, v_cache, positions, row_of_token, block_table, nq: int, nkv: int, hd: int,
                     page_size: int, scale: float, window, batch=None, vd: int = None, sink: float = None, keep_first: int = 0,
-                    softcap: float = None) -> None:
+                    softcap: float = None, chunk: int = None, score_bias=None) -> None:
     """Causal attention of this step's queries over the paged cache.
+
+    ``chunk``: a query sees only the keys of its own chunk of that many positions, counted from position 0 (in a window's
+    place).  ``score_bias`` (float32 [nq]): no softmax, a visible key's weight is sigmoid(score + score_bias[head]) as it is.
 
     ``keep_first``: with a window, the keys j < keep_first stay visible (at their true places) after the window has
     passed them.  ``softcap``: a score s becomes softcap * tanh(s / softcap) before the softmax.
@@ -558,13 +567,20 @@ def paged_attention(q, out, k_cache, v_cache, positions, row_of_token, block_tab
     if block_table.stride(1) != 1:
         raise KernelError("paged_attention: block table rows must be contiguous")
     keep_first = int(keep_first or 0) if window else 0
-    if batch is not None and _KERNEL_SET == "fast" and vd == hd and fast_attention_supported(q, nq, nkv, hd):
+    chunk = int(chunk or 0)
+    if chunk < 0 or (chunk and window) or (score_bias is not None and (sink is not None or score_bias.dtype != torch.float32
+                                                                      or score_bias.numel() != nq or not score_bias.is_contiguous())):
+        raise KernelError("paged_attention: chunks or a window, not both; score_bias must be float32 [nq] and goes without a sink")
+    # chunks are in the sigmoid forms of the fast kernels, kept first keys and the cap in the softmax forms
+    fast_form = not (keep_first or softcap) if score_bias is not None else not chunk
+    if batch is not None and _KERNEL_SET == "fast" and vd == hd and fast_form and fast_attention_supported(q, nq, nkv, hd):
         # kept first keys and capped scores are in both prompt kernels and in the split-KV decode kernel (not the streaming one)
-        extended = bool(keep_first or softcap)
+        extended = bool(keep_first or softcap or score_bias is not None)
         if batch.max_q_len > 1:
             prefill = paged_attention_prefill_tc if tc_attention_supported(q, hd, page_size) else paged_attention_prefill
             prefill(q, out, k_cache, v_cache, batch.q_indptr, batch.kv_lens, block_table, nq, nkv, hd, page_size, scale,
-                    window, batch.max_q_len, skip_single=batch.num_single > 0, sink=sink, keep_first=keep_first, softcap=softcap)
+                    window, batch.max_q_len, skip_single=batch.num_single > 0, sink=sink, keep_first=keep_first, softcap=softcap, chunk=chunk,
+                    score_bias=score_bias)
         if batch.num_single > 0 and not extended and stream_decode_supported(batch.num_rows, page_size, nq // nkv):
             ctas = sm_count(q.device)
             slots = (ctas + batch.num_rows * nkv) * (nq // nkv)
@@ -577,6 +593,8 @@ def paged_attention(q, out, k_cache, v_cache, positions, row_of_token, block_tab
             bound = block_table.shape[1] * page_size
             if window:
                 bound = min(bound, int(window) + keep_first + 63)
+            if chunk:
+                bound = min(bound, chunk)
             splits = decode_splits(batch.num_rows, nkv, bound, q.device)
             part_o = part_ml = counters = None
             if splits > 1:
@@ -585,12 +603,13 @@ def paged_attention(q, out, k_cache, v_cache, positions, row_of_token, block_tab
                 counters = batch.ws.get_zeroed("attn_split_counters", (batch.num_rows * nkv,), torch.int32)
             paged_attention_decode(q, out, k_cache, v_cache, batch.q_indptr, batch.kv_lens, block_table, nq, nkv, hd,
                                    page_size, scale, window, splits, part_o, part_ml, counters, sink=sink, keep_first=keep_first,
-                                   softcap=softcap)
+                                   softcap=softcap, chunk=chunk, score_bias=score_bias)
         return
     _check(library().arle_paged_attention_plain(
         _ptr(q), q.stride(0), _ptr(out), _ptr(k_cache), _ptr(v_cache), _dt(q), _ptr(positions), _ptr(row_of_token),
         _ptr(block_table), block_table.stride(0), nq, nkv, hd, vd, page_size, float(scale),
-        int(window) if window else 0, int(sink is not None), float(sink or 0.0), keep_first, float(softcap or 0.0), T, _stream()),
+        int(window) if window else 0, int(sink is not None), float(sink or 0.0), keep_first, float(softcap or 0.0), chunk,
+        _ptr(score_bias), T, _stream()),
         "paged_attention")
 
 
@@ -614,7 +633,7 @@ def tc_attention_supported(q, hd: int, page_size: int) -> bool:
 
 def paged_attention_prefill_tc(q, out, k_cache, v_cache, q_indptr, kv_lens, block_table, nq, nkv, hd, page_size, scale,
                                window, max_q_len: int, skip_single: bool = False, sink: float = None, keep_first: int = 0,
-                               softcap: float = None) -> None:
+                               softcap: float = None, chunk: int = 0, score_bias=None) -> None:
     """Flash attention over the paged cache on the tcgen05 tensor cores (TMA-fed, scores
     and output in tensor memory) for rows with several queries."""
     R = kv_lens.numel()
@@ -625,7 +644,7 @@ def paged_attention_prefill_tc(q, out, k_cache, v_cache, q_indptr, kv_lens, bloc
         _ptr(q), q.stride(0), q.shape[0], _ptr(out), _ptr(k_cache), _ptr(v_cache), k_cache.shape[0], _ptr(q_indptr),
         _ptr(kv_lens), _ptr(block_table), block_table.stride(0), block_table.shape[1], nq, nkv, hd, page_size, float(scale),
         _sink_arg(sink), int(window) if window else 0, R, int(max_q_len), int(bool(skip_single)), _ptr(error_flag(q.device)),
-        int(keep_first or 0), float(softcap or 0.0), _stream()), "paged_attention_prefill_tc")
+        int(keep_first or 0), float(softcap or 0.0), int(chunk or 0), _ptr(score_bias), _stream()), "paged_attention_prefill_tc")
 
 
 _SM_COUNT: dict = {}
@@ -744,7 +763,7 @@ def decode_splits(rows: int, nkv: int, kv_bound: int, device=None) -> int:
 
 def paged_attention_decode(q, out, k_cache, v_cache, q_indptr, kv_lens, block_table, nq, nkv, hd, page_size, scale,
                            window, splits: int, part_o=None, part_ml=None, counters=None, sink: float = None, keep_first: int = 0,
-                           softcap: float = None) -> None:
+                           softcap: float = None, chunk: int = 0, score_bias=None) -> None:
     """Split-KV attention of the rows that have exactly one query (others are
     skipped).  q_indptr int32 [R+1], kv_lens int32 [R] (keys after this step).
     When splits > 1: part_o / part_ml are float32 scratch of R*nq*splits*hd and
@@ -760,12 +779,12 @@ def paged_attention_decode(q, out, k_cache, v_cache, q_indptr, kv_lens, block_ta
         _ptr(q), q.stride(0), _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(q_indptr), _ptr(kv_lens),
         _ptr(block_table), block_table.stride(0), _ptr(part_o), _ptr(part_ml), _ptr(counters), nq, nkv, hd, page_size,
         float(scale), _sink_arg(sink), int(window) if window else 0, R, int(splits), int(keep_first or 0), float(softcap or 0.0),
-        _stream()), "paged_attention_decode")
+        int(chunk or 0), _ptr(score_bias), _stream()), "paged_attention_decode")
 
 
 def paged_attention_prefill(q, out, k_cache, v_cache, q_indptr, kv_lens, block_table, nq, nkv, hd, page_size, scale,
                             window, max_q_len: int, skip_single: bool = False, sink: float = None, keep_first: int = 0,
-                            softcap: float = None) -> None:
+                            softcap: float = None, chunk: int = 0, score_bias=None) -> None:
     """Flash-attention over the paged cache for rows with several queries (and,
     unless skip_single, for single-query rows too)."""
     R = kv_lens.numel()
@@ -774,7 +793,7 @@ def paged_attention_prefill(q, out, k_cache, v_cache, q_indptr, kv_lens, block_t
         _ptr(q), q.stride(0), _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(q_indptr), _ptr(kv_lens),
         _ptr(block_table), block_table.stride(0), nq, nkv, hd, page_size, float(scale),
         _sink_arg(sink), int(window) if window else 0, R, int(max_q_len), int(bool(skip_single)), int(keep_first or 0),
-        float(softcap or 0.0), _stream()), "paged_attention_prefill")
+        float(softcap or 0.0), int(chunk or 0), _ptr(score_bias), _stream()), "paged_attention_prefill")
 
 
 # ------------------------------------------------------------------ activation
@@ -932,18 +951,20 @@ ROTARY_PAIRINGS = {"half": 0, "interleaved": 1}
 
 
 def attention_prep_row(qk, positions, slot_mapping, q_weight, k_weight, eps: float, inv_freq, rotary_dim: int, pairing: str,
-                       values_are_keys: bool, k_cache, v_cache, nq: int, nkv: int, hd: int, page_size: int, angles=None) -> None:
+                       values_are_keys: bool, k_cache, v_cache, nq: int, nkv: int, hd: int, page_size: int, angles=None,
+                       vd: int = None) -> None:
     """RMSNorm of q and of k over their whole projected rows (weights float32 [nq*hd], [nkv*hd], or None: no
     norm), rotation of the first ``rotary_dim`` elements of every head (``pairing`` "half": element i with
     i + rotary_dim/2; "interleaved": 2i with 2i + 1), q stored in place on qk [T, >= (nq + nkv) hd], k into the
-    paged k_cache; v_cache gets the keys as projected (``values_are_keys``) or the v heads that follow the k
-    heads in the row.  nkv = 0: queries only, nothing stored.  ``angles``: the table of ``rotary_angles`` for these
+    paged k_cache; v_cache gets the keys as projected (``values_are_keys``) or the v heads (``vd`` numbers each, hd when
+    None) that follow the k heads in the row.  nkv = 0: queries only, nothing stored.  ``angles``: the table of ``rotary_angles`` for these
     positions and inv_freq (float32 [T, rotary_dim / 2, 2]), or None: the kernel evaluates them itself (the same bits)."""
     T = qk.shape[0]
     if angles is not None and (angles.dtype != torch.float32 or tuple(angles.shape) != (T, rotary_dim // 2, 2)
                                or not angles.is_contiguous()):
         raise KernelError("attention_prep_row: angles must be contiguous float32 [T, rotary_dim / 2, 2]")
-    need = (nq + (nkv if values_are_keys else 2 * nkv)) * hd
+    vd = hd if vd is None else int(vd)
+    need = (nq + nkv) * hd + (0 if values_are_keys else nkv * vd)
     if qk.stride(1) != 1 or qk.shape[1] < need:
         raise KernelError(f"attention_prep_row: qk must be [T, >= {need}] with unit inner stride")
     if pairing not in ROTARY_PAIRINGS:
@@ -954,9 +975,10 @@ def attention_prep_row(qk, positions, slot_mapping, q_weight, k_weight, eps: flo
     if nkv > 0:
         if k_cache.dtype != qk.dtype or v_cache.dtype != qk.dtype:
             raise KernelError("attention_prep_row: cache type differs from activation type")
-        if tuple(k_cache.shape[1:]) != (nkv, page_size, hd) or k_cache.shape != v_cache.shape or not (
-                k_cache.is_contiguous() and v_cache.is_contiguous()):
-            raise KernelError(f"attention_prep_row: cache shape {tuple(k_cache.shape)} is not [pages, {nkv}, {page_size}, {hd}]")
+        if (tuple(k_cache.shape[1:]) != (nkv, page_size, hd) or tuple(v_cache.shape[1:]) != (nkv, page_size, vd) or not (
+                k_cache.is_contiguous() and v_cache.is_contiguous())):
+            raise KernelError(f"attention_prep_row: cache shapes {tuple(k_cache.shape)}, {tuple(v_cache.shape)} are not "
+                              f"[pages, {nkv}, {page_size}, {hd}] and [pages, {nkv}, {page_size}, {vd}]")
         _i32(slot_mapping, "slot_mapping")
     _i32(positions, "positions")
     if rotary_dim and (inv_freq.dtype != torch.float32 or inv_freq.numel() != rotary_dim // 2):
@@ -965,7 +987,7 @@ def attention_prep_row(qk, positions, slot_mapping, q_weight, k_weight, eps: flo
         _ptr(qk), _dt(qk), qk.stride(0), _ptr(positions), _ptr(slot_mapping) if nkv else None, _ptr(q_weight), _ptr(k_weight),
         float(eps), _ptr(inv_freq) if rotary_dim else None, _ptr(angles) if rotary_dim else None, int(rotary_dim),
         ROTARY_PAIRINGS[pairing], int(bool(values_are_keys)),
-        _ptr(k_cache) if nkv else None, _ptr(v_cache) if nkv else None, nq, nkv, hd, page_size, T, _stream()),
+        _ptr(k_cache) if nkv else None, _ptr(v_cache) if nkv else None, nq, nkv, hd, vd, page_size, T, _stream()),
         "attention_prep_row")
 
 
@@ -998,28 +1020,33 @@ def logit_cap(logits, cap: float) -> None:
 
 
 # ------------------------------------------------------------ gated linear attention
-def gla_decay(low, w2t, bias, tau: float, alpha) -> None:
-    """alpha[t, c] = sigmoid(bias[c] + sum_r low[t, r] * w2t[r, c]) ^ (1 / tau), float32 [T, channels].  ``low``
+def gla_decay(low, w2t, bias, tau: float, alpha, form: str = "sigmoid_root") -> None:
+    """alpha[t, c] = sigmoid(bias[c] + sum_r low[t, r] * w2t[r, c]) ^ (1 / tau), float32 [T, channels] (``form`` "double_exp":
+    exp(-exp(bias[c] + sum_r tanh(low[t, r]) * w2t[r, c])), tau is not used).  ``low``
     [T, rank] in the activation type (a slice of a wider row is fine), w2t float32 [rank, channels] (the gate's
     second matrix transposed), bias float32 [channels] or None."""
     T, rank = low.shape
     C = w2t.shape[1]
     w2 = w2t
+    if form not in ("sigmoid_root", "double_exp"):
+        raise KernelError(f"gla_decay: form {form!r} (sigmoid_root, double_exp)")
     if (w2.dtype != torch.float32 or w2.shape[0] != rank or not w2.is_contiguous() or alpha.dtype != torch.float32
             or tuple(alpha.shape) != (T, C) or not alpha.is_contiguous() or low.stride(1) != 1):
         raise KernelError(f"gla_decay: shapes low {tuple(low.shape)} w2t {tuple(w2.shape)} alpha {tuple(alpha.shape)}")
     if bias is not None and (bias.dtype != torch.float32 or bias.numel() != C):
         raise KernelError("gla_decay: bias must be float32 [channels]")
     _check(library().arle_gla_decay(_ptr(low), _dt(low), low.stride(0), _ptr(w2), _ptr(bias), float(tau), _ptr(alpha), T, C,
-                                    rank, _stream()), "gla_decay")
+                                    rank, int(form == "double_exp"), _stream()), "gla_decay")
 
 
 def gla_scan(q, k, v, alpha, state, q_indptr, state_slots, out, heads: int, dim: int, vdim: int, q_scale: float,
-             max_q_len: int) -> None:
-    """The recurrence S <- diag(alpha_t) S + k_t v_t^T, o_t = S^T (q_t * q_scale) over the tokens of every row of
+             max_q_len: int, bonus=None) -> None:
+    """``bonus`` (float32 [heads*dim]): the read-out comes before the update, o_t = (S + diag(bonus) k_t v_t^T)^T (q_t *
+    q_scale).  Without it: the recurrence S <- diag(alpha_t) S + k_t v_t^T, o_t = S^T (q_t * q_scale) over the tokens of every row of
     the step (row r owns tokens q_indptr[r] .. q_indptr[r+1]-1), from and into state[state_slots[r]].
     q, k [T, heads*dim] and v [T, heads*vdim]: slices of one wider buffer (same row stride, unit inner stride);
-    alpha float32 [T, heads*dim]; state float32 [slots, heads, vdim, dim] (a head's state transposed);
+    alpha float32 [T, heads*dim]; state float32 [slots, heads, vdim, dim] (a head's state transposed) or [slots, n] whose
+    first heads*vdim*dim numbers are that (any slot stride);
     out float32 [T, heads*vdim]."""
     T = q.shape[0]
     R = state_slots.numel()
@@ -1029,15 +1056,18 @@ def gla_scan(q, k, v, alpha, state, q_indptr, state_slots, out, heads: int, dim:
         raise KernelError("gla_scan: q, k, v must be slices of one buffer: [T, heads*dim], [T, heads*dim], [T, heads*vdim]")
     if alpha.dtype != torch.float32 or tuple(alpha.shape) != (T, heads * dim) or not alpha.is_contiguous():
         raise KernelError("gla_scan: alpha must be contiguous float32 [T, heads*dim]")
-    if (state.dtype != torch.float32 or tuple(state.shape[1:]) != (heads, vdim, dim) or not state.is_contiguous()):
-        raise KernelError(f"gla_scan: state {tuple(state.shape)} is not float32 [slots, {heads}, {vdim}, {dim}]")
+    flat = state.dim() == 2 and state.shape[1] >= heads * vdim * dim and state.stride(1) == 1
+    if state.dtype != torch.float32 or not (flat or (tuple(state.shape[1:]) == (heads, vdim, dim) and state.is_contiguous())):
+        raise KernelError(f"gla_scan: state {tuple(state.shape)} is not float32 [slots, {heads}, {vdim}, {dim}] or flat rows of as many")
+    if bonus is not None and (bonus.dtype != torch.float32 or bonus.numel() != heads * dim or not bonus.is_contiguous()):
+        raise KernelError("gla_scan: bonus must be contiguous float32 [heads*dim]")
     if out.dtype != torch.float32 or tuple(out.shape) != (T, heads * vdim) or not out.is_contiguous():
         raise KernelError("gla_scan: out must be contiguous float32 [T, heads*vdim]")
     _i32(q_indptr, "q_indptr"), _i32(state_slots, "state_slots")
     if q_indptr.numel() != R + 1:
         raise KernelError("gla_scan: q_indptr must have one entry more than state_slots")
-    _check(library().arle_gla_scan(_ptr(q), _ptr(k), _ptr(v), _dt(q), q.stride(0), _ptr(alpha), _ptr(state), _ptr(q_indptr),
-                                   _ptr(state_slots), _ptr(out), R, heads, dim, vdim, float(q_scale), int(max_q_len), _stream()),
+    _check(library().arle_gla_scan(_ptr(q), _ptr(k), _ptr(v), _dt(q), q.stride(0), _ptr(alpha), _ptr(bonus), _ptr(state),
+                                   state.stride(0), _ptr(q_indptr), _ptr(state_slots), _ptr(out), R, heads, dim, vdim, float(q_scale), int(max_q_len), _stream()),
            "gla_scan")
 
 
@@ -1045,19 +1075,20 @@ def gla_out(o, gate, weight, eps: float, scale: float, out, heads: int, vdim: in
     """out[t, h, :] = o[t, h, :] / sqrt(mean(o[t, h, :]^2) + eps) * weight * silu(gate[t, h, :]) * scale (``gate_act`` "sigmoid": times
     sigmoid(gate) instead).
     o float32 [T, heads*vdim] contiguous; gate (activation type, or None) and out may be slices of wider rows;
-    weight float32 [vdim] or None."""
+    weight float32 [vdim] (shared by the heads) or [heads*vdim], or None."""
     T = o.shape[0]
     if o.dtype != torch.float32 or tuple(o.shape) != (T, heads * vdim) or not o.is_contiguous():
         raise KernelError("gla_out: o must be contiguous float32 [T, heads*vdim]")
     if out.shape != o.shape or out.stride(1) != 1 or (gate is not None and (gate.shape != o.shape or gate.stride(1) != 1
                                                                           or gate.dtype != out.dtype)):
         raise KernelError("gla_out: gate and out must be [T, heads*vdim] of one type with unit inner stride")
-    if weight is not None and (weight.dtype != torch.float32 or weight.numel() != vdim):
-        raise KernelError("gla_out: weight must be float32 [vdim]")
+    if weight is not None and (weight.dtype != torch.float32 or weight.numel() not in (vdim, heads * vdim)):
+        raise KernelError("gla_out: weight must be float32 [vdim] or [heads*vdim]")
+    per_head = weight is not None and weight.numel() != vdim
     if gate_act not in ("silu", "sigmoid"):
         raise KernelError(f"gla_out: gate_act {gate_act!r} (silu, sigmoid)")
     _check(library().arle_gla_out(_ptr(o), _ptr(gate), _dt(out), gate.stride(0) if gate is not None else 0, _ptr(weight),
-                                  float(eps), float(scale), _ptr(out), out.stride(0), T, heads, vdim, int(gate_act == "sigmoid"), _stream()),
+                                  float(eps), float(scale), _ptr(out), out.stride(0), T, heads, vdim, int(gate_act == "sigmoid"), vdim if per_head else 0, _stream()),
            "gla_out")
 
 
@@ -1086,11 +1117,12 @@ def dyt_norm(resid, delta, rows, weight, bias, alpha: float, out, write_resid: b
 
 
 # ------------------------------------------------------------------ attention over latent vectors
-def gemm_heads(x, w, out) -> None:
+def gemm_heads(x, w, out, gate=None) -> None:
     """out[m, h, :] = x[m, h, :] . w[h]^T for every head h: x [M, heads, K], w [heads, N, K] contiguous, out [M, heads, N].
     x and out may be views into wider rows (any row stride and head stride, unit inner stride).  float32 sums; k ascending
     in the general kernel, tensor-core tiles for bfloat16 rows on 16-byte boundaries (fast kernel set).  ``out`` has x's
-    type, or is float32 (the sums as they are) for bfloat16 rows."""
+    type, or is float32 (the sums as they are) for bfloat16 rows.  ``gate`` [M, heads*N] in x's type (unit inner stride; columns
+    of a wider row are fine): the result is multiplied by sigmoid(gate), on the float32 sums where the tensor cores form them."""
     M, heads, K = x.shape
     N = w.shape[1]
     if (w.shape[0] != heads or w.shape[2] != K or tuple(out.shape) != (M, heads, N) or not w.is_contiguous()
@@ -1098,26 +1130,36 @@ def gemm_heads(x, w, out) -> None:
         raise KernelError(f"gemm_heads: shapes x {tuple(x.shape)} w {tuple(w.shape)} out {tuple(out.shape)}")
     if x.dtype == torch.bfloat16 and w.dtype != torch.bfloat16:
         raise KernelError("gemm_heads: bfloat16 rows need bfloat16 matrices")
+    if gate is not None and (tuple(gate.shape) != (M, heads * N) or gate.dtype != x.dtype or gate.stride(1) != 1 or not out.is_contiguous()
+                             or out.dtype != x.dtype):
+        raise KernelError(f"gemm_heads: gate {tuple(gate.shape)} must be [M, heads*N] of x's type and out contiguous of that type")
     if (_KERNEL_SET == "fast" and x.dtype == torch.bfloat16 and K % 8 == 0 and x.stride(0) % 8 == 0 and x.stride(1) % 8 == 0
             and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0):
         # the same sums on the tensor cores (tiles of 64 rows x 128 columns)
         _check(library().arle_gemm_heads_mma(_ptr(x), _ptr(w), _ptr(out), _dt(out), M, N, K, heads, x.stride(0), K, out.stride(0), x.stride(1),
-                                             N * K, out.stride(1), _stream()), "gemm_heads_mma")
+                                                 N * K, out.stride(1), _ptr(gate), gate.stride(0) if gate is not None else 0, _stream()),
+               "gemm_heads_mma")
         return
     _check(library().arle_gemm_heads(_ptr(x), _ptr(w), _ptr(out), _dt(x), _dt(w), _dt(out), M, N, K, heads, x.stride(0), K, out.stride(0),
                                      x.stride(1), N * K, out.stride(1), _stream()), "gemm_heads")
+    if gate is not None:
+        flat = out.view(M, heads * N)
+        gate_mul(flat, gate, flat)
 
 
 def latent_prep(q, dkv, positions, slot_mapping, c_weight, eps: float, inv_freq, rot_dims: int, cache, q_abs, heads: int,
-                dn: int, dr: int, rank: int) -> None:
+                dn: int, dr: int, rank: int, pairing: str = "half", amplitude: float = 1.0) -> None:
     """The per-token preparation of an attention whose cache holds one record [latent | rotated key part] per token.
     dkv [T, >= rank + dr]: its first ``rank`` numbers are RMS-normed with ``c_weight`` (float32 [rank]), its next ``dr``
-    numbers are rotated (the first ``rot_dims`` of them, element i with i + rot_dims / 2, by position * inv_freq[i]);
+    numbers are rotated (the first ``rot_dims`` of them, element i with i + rot_dims / 2 or, ``pairing`` "interleaved", 2i with
+    2i + 1, by position * inv_freq[i], cosine and sine times ``amplitude``);
     both go to cache[slot_mapping[t]] (cache [pages, 1, page_size, rank + dr]; None: nothing is stored).  q [T, >= heads
     * (dn + dr)]: every head's last ``dr`` numbers are rotated the same way into q_abs[t, h, rank:] (q_abs [T, heads,
     rank + dr], contiguous)."""
     T = q.shape[0]
     kd = rank + dr
+    if pairing not in ROTARY_PAIRINGS:
+        raise KernelError(f"latent_prep: pairing {pairing!r} (known: {', '.join(ROTARY_PAIRINGS)})")
     if cache is None and dkv is None:               # nothing to store: only the queries' rotated numbers are prepared
         dkv, c_weight = q, None
     elif dkv is None or c_weight is None:
@@ -1136,8 +1178,8 @@ def latent_prep(q, dkv, positions, slot_mapping, c_weight, eps: float, inv_freq,
     _i32(positions, "positions")
     _check(library().arle_latent_prep(_ptr(q), q.stride(0), _ptr(dkv), dkv.stride(0), _dt(q), _ptr(positions),
                                       _ptr(slot_mapping) if cache is not None else None, _ptr(c_weight), float(eps),
-                                      _ptr(inv_freq) if rot_dims else None, int(rot_dims), _ptr(cache), _ptr(q_abs), heads, dn, dr,
-                                      rank, T, _stream()), "latent_prep")
+                                      _ptr(inv_freq) if rot_dims else None, int(rot_dims), ROTARY_PAIRINGS[pairing], float(amplitude),
+                                      _ptr(cache), _ptr(q_abs), heads, dn, dr, rank, T, _stream()), "latent_prep")
 
 
 def latent_mma_supported(q_abs, rank: int) -> bool:
@@ -1360,22 +1402,29 @@ def moe_plan_size(experts: int, pairs: int) -> int:
     return int(lib.arle_moe_plan_ints(int(experts), int(pairs)))
 
 
-def moe_plan(ids, experts: int, plan, place_of_pair, row_of_place) -> None:
+def moe_plan(ids, experts: int, plan, place_of_pair, row_of_place, weights=None, weight_of_place=None) -> None:
     """Sorts the pairs (token, choice) of ids [T, top] by expert, on the device: plan (int32, ``moe_plan_size`` entries: the
     experts' runs and the tiles the grouped product runs), place_of_pair int32 [T*top], row_of_place int32 [T*top] (the
-    token of the pair at each place)."""
+    token of the pair at each place).  ``weights`` float32 [T, top] go to ``weight_of_place`` float32 [T*top] in the same order."""
     T, top = ids.shape
     pairs = T * top
     if (ids.dtype != torch.int32 or not ids.is_contiguous() or plan.dtype != torch.int32 or plan.numel() < moe_plan_size(experts, pairs)
             or place_of_pair.dtype != torch.int32 or place_of_pair.numel() < pairs or row_of_place.dtype != torch.int32
             or row_of_place.numel() < pairs):
         raise KernelError("moe_plan: int32 tables of the sizes moe_plan_size gives")
-    _check(library().arle_moe_plan(_ptr(ids), pairs, top, experts, _ptr(plan), _ptr(place_of_pair), _ptr(row_of_place), _stream()),
-           "moe_plan")
+    for t_ in (weights, weight_of_place):
+        if t_ is not None and (t_.dtype != torch.float32 or t_.numel() < pairs or not t_.is_contiguous()):
+            raise KernelError("moe_plan: weights and weight_of_place must be contiguous float32 with one entry per pair")
+    _check(library().arle_moe_plan(_ptr(ids), pairs, top, experts, _ptr(plan), _ptr(place_of_pair), _ptr(row_of_place),
+                                   _ptr(weights), _ptr(weight_of_place), _stream()), "moe_plan")
 
 
-def moe_gemm(x, rows, w, out, plan, experts: int) -> None:
-    """out[place] = x[rows[place]] . w[expert of place]^T for every place of the plan (rows None: x is in place order).
+MOE_ACTS = {"none": 0, "square_relu": 1}
+
+
+def moe_gemm(x, rows, w, out, plan, experts: int, place_scale=None, act: str = "none") -> None:
+    """out[place] = act(place_scale[place] * x[rows[place]] . w[expert of place]^T) for every place of the plan (rows None: x is
+    in place order; place_scale float32 [pairs] or None: ones; ``act`` "none" or "square_relu", on the float32 sums).
     x [*, K], w [experts, N, K] contiguous, out [pairs, N] in x's type; float32 sums, k ascending.  With the fast kernel
     set, bfloat16 operands with rows on 16-byte boundaries run on the tensor cores (many pairs) or as one dot product a
     warp (up to 128 pairs: a decode step)."""
@@ -1384,19 +1433,23 @@ def moe_gemm(x, rows, w, out, plan, experts: int) -> None:
     if (w.dim() != 3 or w.shape[0] != experts or w.shape[1] != N or w.shape[2] != K or not w.is_contiguous() or x.stride(1) != 1
             or out.stride(1) != 1 or x.dtype != out.dtype or (x.dtype == torch.bfloat16 and w.dtype != torch.bfloat16)):
         raise KernelError(f"moe_gemm: shapes x {tuple(x.shape)} w {tuple(w.shape)} out {tuple(out.shape)}")
+    if act not in MOE_ACTS or (place_scale is not None and (place_scale.dtype != torch.float32 or place_scale.numel() < pairs)):
+        raise KernelError(f"moe_gemm: act {act!r} (known: {', '.join(MOE_ACTS)}); place_scale must be float32 [pairs]")
     _i32(rows, "rows"), _i32(plan, "plan")
     _check(library().arle_moe_gemm(_ptr(x), x.stride(0), _ptr(rows), _ptr(w), K, N * K, _ptr(out), out.stride(0), _dt(x), _dt(w),
-                                   _ptr(plan), experts, pairs, N, K, int(_KERNEL_SET == "fast"), _stream()), "moe_gemm")
+                                   _ptr(plan), experts, pairs, N, K, int(_KERNEL_SET == "fast"), _ptr(place_scale), MOE_ACTS[act], _stream()),
+           "moe_gemm")
 
 
-def moe_combine(y, place_of_pair, weights, shared, gate, out) -> None:
+def moe_combine(y, place_of_pair, weights, shared, gate, out, top: int = None) -> None:
     """out[t] = sum_k weights[t, k] * y[place_of_pair[t*top + k]] (k ascending, float32) + sigmoid(gate[t]) * shared[t].
     y [pairs, width]; shared [T, width] or None; gate float32 [T] (any stride) or None (the shared rows are added as
-    they are); out [T, width] (unit inner stride)."""
-    T, top = weights.shape
-    width = out.shape[1]
-    if (y.shape[1] != width or y.stride(1) != 1 or out.stride(1) != 1 or y.dtype != out.dtype or weights.dtype != torch.float32
-            or not weights.is_contiguous() or out.shape[0] != T):
+    they are); out [T, width] (unit inner stride).  ``weights`` None: ones, with ``top`` choices per token."""
+    T, width = out.shape
+    if weights is not None:
+        top = weights.shape[1]
+    if (y.shape[1] != width or y.stride(1) != 1 or out.stride(1) != 1 or y.dtype != out.dtype or not top
+            or (weights is not None and (weights.dtype != torch.float32 or not weights.is_contiguous() or weights.shape[0] != T))):
         raise KernelError("moe_combine: y [pairs, width] and out [T, width] of one type, weights float32 [T, top]")
     if shared is not None and (tuple(shared.shape) != (T, width) or shared.stride(1) != 1 or shared.dtype != out.dtype):
         raise KernelError("moe_combine: shared must be [T, width] in the activation type")
@@ -1629,3 +1682,119 @@ def delta_scan(q, k, v, beta, decay, state, q_indptr, state_slots, out, heads: i
     _check(library().arle_delta_scan(_ptr(q), _ptr(k), _ptr(v), _dt(q), q.stride(0), k.stride(0), v.stride(0), _ptr(beta), _ptr(decay),
                                      _ptr(state), state.stride(0), _ptr(q_indptr), _ptr(state_slots), _ptr(out), T, R, heads, kq_heads,
                                      dim, vdim, float(q_scale), float(unit_eps), _stream()), "delta_scan")
+
+
+def gate_mul(x, gate, out) -> None:
+    """out[t, i] = x[t, i] * sigmoid(gate[t, i]): one gate number per element; [T, width] of one type, columns of wider rows are
+    fine, out may be x.  float32 arithmetic, rounded once."""
+    T, width = x.shape
+    if gate.shape != x.shape or out.shape != x.shape or gate.dtype != x.dtype or out.dtype != x.dtype or any(
+            t_.stride(1) != 1 for t_ in (x, gate, out)):
+        raise KernelError("gate_mul: x, gate and out must be [T, width] of one type with unit inner stride")
+    _check(library().arle_gate_mul(_ptr(x), x.stride(0), _ptr(gate), gate.stride(0), _ptr(out), out.stride(0), _dt(x), T, width, _stream()),
+           "gate_mul")
+
+
+def square_relu(x, out) -> None:
+    """out = max(x, 0)^2, [T, width] of one type (columns of wider rows are fine, out may be x)."""
+    T, width = x.shape
+    if out.shape != x.shape or out.dtype != x.dtype or x.stride(1) != 1 or out.stride(1) != 1:
+        raise KernelError("square_relu: x and out must be [T, width] of one type with unit inner stride")
+    _check(library().arle_square_relu(_ptr(x), x.stride(0), _ptr(out), out.stride(0), _dt(x), T, width, _stream()), "square_relu")
+
+
+def layernorm(resid, delta, rows, weight, eps: float, out, write_resid: bool) -> None:
+    """For output row i (source row r = rows[i], or i): x = resid[r] (+ delta[r]); resid[r] = x when write_resid; out[i] =
+    (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps) * weight.  resid float32 [N, H]; delta and out in the activation type
+    (out may be resid itself when that is float32 and no rows are listed); weight float32 [H]."""
+    H = resid.shape[1]
+    n_out = out.shape[0]
+    if resid.dtype != torch.float32 or weight.dtype != torch.float32:
+        raise KernelError("layernorm: residual and weight must be float32")
+    if not (resid.is_contiguous() and out.is_contiguous()) or out.shape[1] != H or weight.numel() != H:
+        raise KernelError("layernorm: bad shapes or strides")
+    if delta is not None and (delta.dtype != out.dtype or delta.shape != resid.shape or not delta.is_contiguous()):
+        raise KernelError("layernorm: delta must match the residual's shape and the output's type")
+    if rows is not None:
+        _i32(rows, "rows")
+        if rows.numel() != n_out:
+            raise KernelError("layernorm: one output row per entry of rows")
+    elif n_out != resid.shape[0]:
+        raise KernelError("layernorm: output rows must match residual rows when no row list is given")
+    _check(library().arle_layernorm(_ptr(resid), _ptr(delta), _ptr(rows), _ptr(weight), _ptr(out), _dt(out), n_out, H, float(eps),
+                                    int(bool(write_resid)), _stream()), "layernorm")
+
+
+def branch_layernorm_add(resid, branch, weight, eps: float, copy, conv=None) -> None:
+    """resid += (branch - mean) / sqrt(variance + eps) * weight per row, in float32; ``copy`` (or None) gets the new residual in
+    its own type.  resid float32 [T, H] contiguous; branch [T, H] (unit inner stride) and copy [T, H] contiguous in the
+    activation type; weight float32 [H].  ``conv`` (for steps in which row t is one token): (weight float32 [taps, H], state
+    float32 [slots, >= H * (taps - 1)], state_slots int32 [T], out [T, H] in the branch's type): the next block's input
+    convolution of the new residual, see ``input_conv``."""
+    T, H = resid.shape
+    if resid.dtype != torch.float32 or not resid.is_contiguous():
+        raise KernelError("branch_layernorm_add: the residual must be contiguous float32")
+    if tuple(branch.shape) != (T, H) or branch.stride(1) != 1 or weight.dtype != torch.float32 or weight.numel() != H:
+        raise KernelError("branch_layernorm_add: branch [T, H] with unit inner stride and weight float32 [H]")
+    if copy is not None and (tuple(copy.shape) != (T, H) or not copy.is_contiguous() or copy.dtype != branch.dtype):
+        raise KernelError("branch_layernorm_add: copy must be contiguous [T, H] of branch's type")
+    cw = st = slots = cout = None
+    taps = 0
+    if conv is not None:
+        cw, st, slots, cout = conv
+        taps = cw.shape[0]
+        _check_conv("branch_layernorm_add", cw, st, H, cout)
+        if slots.numel() != T or cout.dtype != branch.dtype or tuple(cout.shape) != (T, H):
+            raise KernelError("branch_layernorm_add: a convolution here takes one token per row, into [T, H] of branch's type")
+        _i32(slots, "state_slots")
+    _check(library().arle_branch_layernorm_add(_ptr(resid), _ptr(branch), branch.stride(0), _ptr(weight), _ptr(copy), _dt(branch), T, H, float(eps),
+                                               _ptr(cw), taps, _ptr(st), st.stride(0) if st is not None else 0, _ptr(slots), _ptr(cout),
+                                               _stream()), "branch_layernorm_add")
+
+
+def _check_conv(what: str, weight, state, C: int, out) -> None:
+    taps = weight.shape[0]
+    if weight.dtype != torch.float32 or tuple(weight.shape) != (taps, C) or not weight.is_contiguous() or not out.is_contiguous():
+        raise KernelError(f"{what}: the convolution's weight must be contiguous float32 [taps, C] and its output contiguous")
+    if taps > 1 and (state is None or state.dtype != torch.float32 or state.dim() != 2 or state.shape[1] < C * (taps - 1) or state.stride(1) != 1):
+        raise KernelError(f"{what}: state must be float32 [slots, n] with room for C * (taps - 1) numbers")
+
+
+def input_conv(x, weight, state, q_indptr, row_of_token, state_slots, out, max_q_len: int) -> None:
+    """out[t, c] = sum_j weight[j, c] * x[t - (taps - 1) + j, c] over the tokens of t's row, zeros before a request's first; x is
+    the float32 residual [T, C], weight float32 [taps, C] (a block that adds its convolution to its input adds one to the last
+    row), out [T, C] float32 or bfloat16.  The request's last taps - 1 inputs are kept at state[slot, j * C + c] (oldest first;
+    zero for a new request) and brought up to date."""
+    T, C = x.shape
+    R = state_slots.numel()
+    if x.dtype != torch.float32 or not x.is_contiguous() or tuple(out.shape) != (T, C):
+        raise KernelError("input_conv: x must be contiguous float32 [T, C] and out [T, C]")
+    _check_conv("input_conv", weight, state, C, out)
+    _i32(q_indptr, "q_indptr"), _i32(row_of_token, "row_of_token"), _i32(state_slots, "state_slots")
+    taps = weight.shape[0]
+    single = int(max_q_len == 1)
+    _check(library().arle_input_conv(_ptr(x), _ptr(weight), _ptr(state), state.stride(0) if state is not None else 0, _ptr(q_indptr),
+                                     _ptr(row_of_token), _ptr(state_slots), _ptr(out), _dt(out), T, R, C, taps, single, _stream()), "input_conv")
+    if taps > 1 and not single:
+        add_launches(1)
+
+
+def token_shift(h, mu, state, q_indptr, row_of_token, state_slots, out, max_q_len: int) -> None:
+    """out[s, t] = h[t] + (h[t - 1] - h[t]) * mu[s] for every mix s, the previous token's row taken from state[slot, :C] before a
+    row's first token (zero for a new request); the state is left holding the row's last h.  h [T, C] (unit inner stride) and
+    out [S, T, C] (contiguous) in the activation type; mu float32 [S, C]; state float32 [slots, >= C]."""
+    T, C = h.shape
+    S = mu.shape[0]
+    R = state_slots.numel()
+    if h.stride(1) != 1 or tuple(out.shape) != (S, T, C) or not out.is_contiguous() or out.dtype != h.dtype:
+        raise KernelError("token_shift: h [T, C] with unit inner stride, out contiguous [S, T, C] of its type")
+    if mu.dtype != torch.float32 or mu.shape[1] != C or not mu.is_contiguous():
+        raise KernelError("token_shift: mu must be contiguous float32 [S, C]")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.shape[1] < C or state.stride(1) != 1:
+        raise KernelError("token_shift: state must be float32 [slots, >= C]")
+    _i32(q_indptr, "q_indptr"), _i32(row_of_token, "row_of_token"), _i32(state_slots, "state_slots")
+    single = int(max_q_len == 1)
+    _check(library().arle_token_shift(_ptr(h), _dt(h), h.stride(0), _ptr(mu), S, _ptr(state), state.stride(0), _ptr(q_indptr), _ptr(row_of_token),
+                                      _ptr(state_slots), _ptr(out), T * C, T, R, C, single, _stream()), "token_shift")
+    if not single:
+        add_launches(1)

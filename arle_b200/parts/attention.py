@@ -28,6 +28,11 @@ and output projections (tensor name + ``bias_suffix``); ``conv_taps`` runs a sho
 channel of q, k and v right after the projection (weights [channels, taps] under tensor name + ``conv_suffix``, zeros
 before a sequence's start; the last taps - 1 projected rows of a request are its state).  Its order is projection (+ bias)
 -> convolution -> per-head norm -> rotation -> cache -> attention -> output projection (+ bias).
+
+With ``qk_norm`` "row": ``weights`` "sigmoid" has no softmax, a visible key's weight is sigmoid(score + b_h) with a stored number
+per query head (tensor ``score_bias``); ``chunk`` lets a position see only its own chunk of that many positions, counted from 0;
+``out_gate`` multiplies the heads' outputs number by number with sigmoid(W_g x) (rows of the packed input projection);
+``value_dim`` may differ from ``head_dim`` when values are projected.
 """
 from __future__ import annotations
 
@@ -67,11 +72,14 @@ class AttentionSpec:
     conv_taps: int = 0              # a short causal convolution on q, k and v (0: none)
     bias_suffix: str = ".b"
     conv_suffix: str = ".conv"
+    weights: str = "softmax"        # "sigmoid": sigmoid(score + b_h) per key, not normalised
+    chunk: Optional[int] = None     # a position sees its own chunk of this many positions only
+    out_gate: bool = False          # the heads' outputs times sigmoid(W_g x), number by number
     kind: ClassVar[str] = "attention"
 
 
 DEFAULT_NAMES = (("q", "q_proj.weight"), ("k", "k_proj.weight"), ("v", "v_proj.weight"), ("o", "o_proj.weight"),
-                 ("q_norm", "q_norm.weight"), ("k_norm", "k_norm.weight"), ("gate", "g_proj.weight"))
+                 ("q_norm", "q_norm.weight"), ("k_norm", "k_norm.weight"), ("gate", "g_proj.weight"), ("score_bias", "score_bias"))
 
 
 class Attention(Mixer):
@@ -91,11 +99,19 @@ class Attention(Mixer):
             raise ValueError("attention: cache_window goes with a window and is at least as long")
         if spec.keep_first < 0 or spec.conv_taps < 0 or (spec.softcap is not None and not spec.softcap > 0):
             raise ValueError("attention: keep_first and conv_taps cannot be negative, softcap must be positive")
+        if spec.weights not in ("softmax", "sigmoid") or (spec.chunk is not None and (spec.chunk <= 0 or spec.window is not None)):
+            raise ValueError(f"attention: weights {spec.weights!r} (softmax, sigmoid); a chunk is positive and goes without a window")
+        if spec.head_gate and spec.out_gate:
+            raise ValueError("attention: a gate per head or one per number, not both")
+        # sigmoid weights, chunks, a gate per number: with the norm over the whole row
+        self.row_form = spec.weights == "sigmoid" or spec.chunk is not None or spec.out_gate
+        if self.row_form and spec.qk_norm != "row":
+            raise ValueError("attention: sigmoid weights, chunks and a gate per number go with qk_norm 'row'")
         self.spec = spec
         self.own_keys = spec.own_keys
         self.general_form = bool(spec.keep_first or spec.softcap is not None or spec.bias or spec.conv_taps
                                  or (spec.qk_norm == "head" and (self.vd != spec.head_dim or spec.head_dim % 2)))
-        if spec.head_dim % 2 and not self.general_form:
+        if spec.head_dim % 2 and not self.general_form and spec.qk_norm != "row":
             raise ValueError(f"head_dim {spec.head_dim} not supported by this form of attention (even sizes only)")
         if self.general_form and (spec.qk_norm != "head" or spec.values != "projected" or spec.head_gate or spec.sink is not None
                                   or not spec.own_keys or not spec.qk_norm_weight):
@@ -105,10 +121,13 @@ class Attention(Mixer):
         self.post_form = spec.qk_norm == "head_after_rotation"
         if self.post_form and (spec.values != "projected" or spec.head_gate):
             raise ValueError("attention: a norm after the rotation goes with projected values and no gate")
-        if not self.post_form and not self.general_form and (self.vd != spec.head_dim or spec.sink is not None or not spec.qk_norm_weight or not spec.own_keys):
+        own_width = self.vd != spec.head_dim and not (spec.qk_norm == "row" and spec.values == "projected" and not spec.head_gate)
+        if not self.post_form and not self.general_form and (own_width or spec.sink is not None or not spec.qk_norm_weight or not spec.own_keys):
             raise ValueError("attention: value_dim, sink, a norm without weight and a run without keys of its own need qk_norm 'head_after_rotation'")
         self.position = build_part(spec.position) if spec.position is not None else None
         self.pairing = getattr(self.position, "pairing", "half")
+        if getattr(self.position, "amplitude", 1.0) != 1.0:
+            raise ValueError("attention: a stretched rotation with an amplitude is not applied by this mixer's preparation kernels")
         # the form the first kernels of this package were written for; everything else takes the general preparation
         if (self.post_form or self.general_form) and self.pairing != "half":
             raise ValueError("attention: a norm after the rotation, and the general form, go with half-split rotation")
@@ -120,7 +139,7 @@ class Attention(Mixer):
         self.names.update(dict(spec.names or ()))
         self.w_qkv = self.w_o = self.q_norm = self.k_norm = None
         self.gate_at = None             # column of the packed projection where the gate numbers start
-        self.b_qkv = self.b_o = self.w_conv = None
+        self.b_qkv = self.b_o = self.w_conv = self.score_bias = None
         self.channels = spec.num_heads * spec.head_dim + spec.num_kv_heads * (spec.head_dim + self.vd)   # q | k | v
 
     # ---------------------------------------------------------------- weights
@@ -154,8 +173,12 @@ class Attention(Mixer):
             return tuple(decls)
         decls = [WeightDecl(self._name("q"), (dq, s.hidden_size)), WeightDecl(self._name("k"), (dkv, s.hidden_size))]
         if s.values == "projected":
-            decls.append(WeightDecl(self._name("v"), (dkv, s.hidden_size)))
-        decls.append(WeightDecl(self._name("o"), (s.hidden_size, dq)))
+            decls.append(WeightDecl(self._name("v"), (s.num_kv_heads * self.vd, s.hidden_size)))
+        decls.append(WeightDecl(self._name("o"), (s.hidden_size, s.num_heads * self.vd)))
+        if s.weights == "sigmoid":
+            decls.append(WeightDecl(self._name("score_bias"), (s.num_heads,), init="around_zero"))
+        if s.out_gate:
+            decls.append(WeightDecl(self._name("gate"), (s.num_heads * self.vd, s.hidden_size)))
         if s.qk_norm_eps is not None:
             nq_, nk_ = ((s.head_dim,), (s.head_dim,)) if s.qk_norm == "head" else ((dq,), (dkv,))
             decls += [WeightDecl(self._name("q_norm"), nq_, init="gain"), WeightDecl(self._name("k_norm"), nk_, init="gain")]
@@ -169,7 +192,10 @@ class Attention(Mixer):
         if self.post_form and not self.own_keys:
             roles = ("q",)
         mats = [tensors[self._name(n)] for n in roles]
-        if s.head_gate:
+        if s.head_gate or s.out_gate:
+            gap = -sum(m.shape[0] for m in mats) % 8 if s.out_gate else 0
+            if gap:
+                mats.append(torch.zeros((gap, s.hidden_size), dtype=mats[0].dtype))
             self.gate_at = sum(m.shape[0] for m in mats)
             mats.append(tensors[self._name("gate")])
             pad = -sum(m.shape[0] for m in mats) % 8       # rows of the packed output start on 16-byte boundaries
@@ -183,6 +209,8 @@ class Attention(Mixer):
             self.q_norm = tensors[self._name("q_norm")].to(device=device, dtype=torch.float32).contiguous()
             if self.own_keys:
                 self.k_norm = tensors[self._name("k_norm")].to(device=device, dtype=torch.float32).contiguous()
+        if s.weights == "sigmoid":
+            self.score_bias = tensors[self._name("score_bias")].to(device=device, dtype=torch.float32).contiguous()
         if self.position is not None:
             self.position.load(tensors, dtype, device)
         if s.bias:
@@ -205,8 +233,8 @@ class Attention(Mixer):
         window = s.cache_window if s.cache_window is not None else s.window
         keep = s.keep_first if window is not None else 0
         if self.vd != s.head_dim:
-            return CacheNeed(streams=((s.num_kv_heads, s.head_dim), (s.num_kv_heads, self.vd)), window=window, keep_first=keep)
-        return CacheNeed(s.num_kv_heads, s.head_dim, window, keep_first=keep)
+            return CacheNeed(streams=((s.num_kv_heads, s.head_dim), (s.num_kv_heads, self.vd)), window=window, keep_first=keep, chunk=s.chunk)
+        return CacheNeed(s.num_kv_heads, s.head_dim, window, keep_first=keep, chunk=s.chunk)
 
     def state_need(self):
         """The convolution's memory: a request's last taps - 1 projected rows of q | k | v, float32."""
@@ -293,7 +321,7 @@ class Attention(Mixer):
 
     # ------------------------------------------------- the general form, up to the output projection
     def pre_output_width(self):
-        return None if self.general_form else self.spec.num_heads * self.vd
+        return None if self.general_form or self.spec.out_gate else self.spec.num_heads * self.vd
 
     def output_weight(self):
         return self.w_o
@@ -303,7 +331,7 @@ class Attention(Mixer):
         heads' outputs [T, heads*head_dim] and the packed projection (whose gate columns the caller reads)."""
         s = self.spec
         T = x.shape[0]
-        nq, nkv, hd = s.num_heads, s.num_kv_heads, s.head_dim
+        nq, nkv, hd, vd = s.num_heads, s.num_kv_heads, s.head_dim, self.vd
         rot = self.position.rotary() if self.position is not None else None
         inv_freq, rdim = rot if rot is not None else (None, 0)
         eps = s.qk_norm_eps if s.qk_norm_eps is not None else 0.0
@@ -318,10 +346,11 @@ class Attention(Mixer):
             ops.attention_prep_row(proj, ctx.positions, cache.slot_mapping if kv else None, self.q_norm,
                                    self.k_norm if kv else None, eps, inv_freq, rdim, self.pairing, s.values == "keys",
                                    cache.k if kv else None, cache.v if kv else None, nq, kv, hd, cache.page_size,
-                                   angles=self._angles(proj, ctx, inv_freq, rdim, general=True))
-        attn = ctx.ws.get("attn_out", (T, nq * hd), x.dtype)
+                                   angles=self._angles(proj, ctx, inv_freq, rdim, general=True), vd=vd)
+        attn = ctx.ws.get("attn_out", (T, nq * vd), x.dtype)
         ops.paged_attention(proj[:, : nq * hd], attn, cache.k, cache.v, ctx.positions, ctx.row_of_token,
-                            cache.block_table, nq, nkv, hd, cache.page_size, s.scale, s.window, batch=ctx)
+                            cache.block_table, nq, nkv, hd, cache.page_size, s.scale, s.window, batch=ctx, vd=vd, chunk=s.chunk,
+                            score_bias=self.score_bias)
         return attn, proj
 
     def forward_pre(self, x, ctx, cache, state, into, scale):
@@ -344,6 +373,8 @@ class Attention(Mixer):
                 gated = ctx.ws.get("attn_gated", tuple(attn.shape), x.dtype)
                 ops.head_gate(attn, proj[:, self.gate_at: self.gate_at + s.num_heads], 1.0, gated, s.num_heads, s.head_dim)
                 attn = gated
+            if s.out_gate:
+                ops.gate_mul(attn, proj[:, self.gate_at: self.gate_at + s.num_heads * self.vd], attn)
             out = ctx.ws.get("mixer_out", (T, s.hidden_size), x.dtype)
             return None if ops.gemm(attn, self.w_o, out, sink=sink) else out
         nq, nkv, hd = s.num_heads, s.num_kv_heads, s.head_dim

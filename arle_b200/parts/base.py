@@ -60,13 +60,22 @@ class CacheNeed:
     ``window`` None keeps every token; an integer keeps only what the last
     ``window`` positions can still see, so older pages go back to the pool.
     ``keep_first``: with a window, the first ``keep_first`` tokens of a request stay
-    visible for its whole life, so the pages that hold them are never given back."""
+    visible for its whole life, so the pages that hold them are never given back.
+    ``chunk`` (in a window's place): a position sees only its own chunk of that many
+    positions, counted from 0, so the pages before the next token's chunk go back."""
 
     num_kv_heads: int = 0
     head_dim: int = 0
     window: Optional[int] = None
     streams: Optional[Tuple[Tuple[int, int], ...]] = None
     keep_first: int = 0
+    chunk: Optional[int] = None
+
+    def first_needed(self, tokens: int) -> int:
+        """The first token that a query at position ``tokens`` or later can still see (kept first tokens aside)."""
+        if self.chunk is not None:
+            return tokens // self.chunk * self.chunk
+        return max(0, tokens - self.window + 1) if self.window is not None else 0
 
     def arrays(self) -> Tuple[Tuple[int, int], ...]:
         if self.streams is not None:
@@ -77,7 +86,7 @@ class CacheNeed:
         return sum(h * w for h, w in self.arrays())
 
     def group_key(self):
-        return (self.arrays(), self.window, self.keep_first if self.window is not None else 0)
+        return (self.arrays(), self.window, self.keep_first if self.window is not None else 0, self.chunk)
 
 
 @dataclass(frozen=True)
@@ -193,9 +202,13 @@ class FeedForward(Part):
 
 
 class Block(Part):
-    """Arrangement of norms, mixer and feed-forward around the residual stream."""
+    """Arrangement of norms, mixer and feed-forward around the residual stream.  What it keeps per token and per request
+    is its mixer's, unless the arrangement itself has a memory (a convolution in front of the mixer)."""
 
     mixer: Mixer
+
+    def state_need(self) -> Optional[StateNeed]:
+        return self.mixer.state_need()
 
     def forward(self, stream, ctx, cache, state) -> None:
         raise NotImplementedError
@@ -204,4 +217,10 @@ class Block(Part):
         """(the norm this block applies first, the part that reads its output), or None: lets the
         block that runs before this one fold its last residual sum and this norm into its last
         product."""
+        return None
+
+    def input_conv(self, state):
+        """(weight [taps, hidden], this request's memory of it: columns of ``state``) when the block convolves the residual
+        before its mixer reads it, else None: lets the block that runs before this one do that in its last kernel, in steps
+        in which every row is one token."""
         return None

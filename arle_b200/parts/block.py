@@ -9,7 +9,9 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import ClassVar
 
-from .base import Block
+import torch
+
+from .base import Block, StateNeed, WeightDecl
 from .registry import build_part, register_part
 
 
@@ -83,17 +85,26 @@ register_part(PreNormBlockSpec.kind, PreNormBlock)
 @dataclass(frozen=True)
 class OutputNormBlockSpec:
     """x <- x + norm(mixer(x)); x <- x + norm(ffn(x)): the norms stand on the sublayers' outputs, the sublayers read the
-    residual as it is (the second half is absent when the spec names no feed-forward)."""
+    residual as it is (the second half is absent when the spec names no feed-forward).  With ``conv_taps`` the mixer reads
+    x + conv(x) instead, a causal convolution over time on every channel (stored weight ``conv_name`` [size, taps], no bias,
+    zeros before a sequence's start)."""
     mixer_norm: object
     mixer: object
     ffn_norm: object = None
     ffn: object = None
+    conv_taps: int = 0              # 0: no convolution
+    conv_name: str = ""
+    conv_size: int = 0              # the model width, with a convolution
     kind: ClassVar[str] = "outnorm_block"
 
 
 class OutputNormBlock(Block):
     """The norm needs ``add_normed(resid, branch, copy)`` (``RmsNorm`` has it): the branch's norm, the sum into the 32-bit
-    residual and the rounded copy that the next sublayer reads are one kernel."""
+    residual and the rounded copy that the next sublayer reads are one kernel.
+
+    The input convolution reads the 32-bit residual itself.  Its memory, a request's last taps - 1 residual rows in float32,
+    stands in front of the mixer's state in one row per request slot (a mixer behind a convolution keeps a flat float32
+    state).  In a step of decoded tokens only it runs inside the kernel that ends the block before."""
 
     def __init__(self, spec: OutputNormBlockSpec):
         self.spec = spec
@@ -107,13 +118,37 @@ class OutputNormBlock(Block):
         for n in (self.mixer_norm, self.ffn_norm):
             if n is not None and not hasattr(n, "add_normed"):
                 raise ValueError(f"norm {type(n).__name__} cannot stand on a branch's output (no add_normed)")
+        if spec.conv_taps < 0 or (spec.conv_taps and (spec.conv_size <= 0 or not spec.conv_name)):
+            raise ValueError("a block's input convolution needs taps, a size and its weight's name")
+        self.conv = None
+        n = spec.conv_size * (spec.conv_taps - 1) if spec.conv_taps else 0
+        self.conv_state = -(-n // 4) * 4                # columns of the state row that belong to the convolution
+        self._mixer_state = self.mixer.state_need()
+        if spec.conv_taps and self._mixer_state is not None and (self._mixer_state.dtype != torch.float32 or len(self._mixer_state.shape) != 1):
+            raise ValueError("a mixer behind an input convolution needs a flat float32 state")
 
     def weight_decls(self):
-        return tuple(d for p in self._parts for d in p.weight_decls())
+        s = self.spec
+        own = (WeightDecl(s.conv_name, (s.conv_size, s.conv_taps), init="around_zero"),) if s.conv_taps else ()
+        return tuple(d for p in self._parts for d in p.weight_decls()) + own
 
     def load(self, tensors, dtype, device):
         for p in self._parts:
             p.load(tensors, dtype, device)
+        if self.spec.conv_taps:
+            w = tensors[self.spec.conv_name].to(device=device, dtype=torch.float32).t().contiguous().clone()        # [taps, size]
+            w[-1] += 1.0                                # x + conv(x) as one sum
+            self.conv = w
+
+    def state_need(self):
+        if not self.conv_state:
+            return self._mixer_state
+        return StateNeed((self.conv_state + (self._mixer_state.shape[0] if self._mixer_state is not None else 0),), torch.float32)
+
+    def input_conv(self, state):
+        if self.conv is None:
+            return None
+        return self.conv, (state[:, : self.spec.conv_size * (self.spec.conv_taps - 1)] if self.conv_state else None)
 
     def weight_bytes(self):
         return sum(p.weight_bytes() for p in self._parts)
@@ -123,11 +158,22 @@ class OutputNormBlock(Block):
         return 2 * width + max(self.mixer.scratch_elements_per_token(), self.ffn.scratch_elements_per_token() if self.ffn is not None else 0)
 
     def forward(self, stream, ctx, cache, state):
-        h = stream.plain("plain_a")
-        stream.add_normed(self.mixer_norm, self.mixer.forward(h, ctx, cache, state), "plain_b")
-        if self.ffn is not None:
-            h = stream.plain("plain_b")
-            stream.add_normed(self.ffn_norm, self.ffn.forward(h, ctx), "plain_a")
+        conv = self.input_conv(state)
+        h = stream.plain("plain_a") if conv is None else stream.convolved(conv, ctx, "convolved")
+        if self.conv_state:
+            state = state[:, self.conv_state:] if self._mixer_state is not None else None
+        branch = self.mixer.forward(h, ctx, cache, state)
+        # what the next block reads: the residual's convolution (then no rounded copy of the residual is wanted), or its copy
+        leaves = None if stream.next_conv is not None else "plain_a"
+        if self.ffn is None:
+            if not stream.add_normed_then_conv(self.mixer_norm, branch, ctx, "convolved"):
+                stream.add_normed(self.mixer_norm, branch, leaves)
+            return
+        stream.add_normed(self.mixer_norm, branch, "plain_b")
+        h = stream.plain("plain_b")
+        branch = self.ffn.forward(h, ctx)
+        if not stream.add_normed_then_conv(self.ffn_norm, branch, ctx, "convolved"):
+            stream.add_normed(self.ffn_norm, branch, leaves)
 
 
 register_part(OutputNormBlockSpec.kind, OutputNormBlock)

@@ -9,12 +9,15 @@ Only c and k_rot are cached: one record of rank + dr numbers per token, one stre
 cache.  The keys and values are never built.  Since q_nope . (W_uk[h] c) = (W_uk[h]^T q_nope) . c, the heads' key
 maps are folded into the queries (one small product per head), every head then attends over the same records with
 keys [c | k_rot] and values c, and W_uv[h] is applied to the head's weighted sum of latents afterwards.  The
-position encoding is the rotary part's (pairing "half"); it turns the first ``rotary_dim`` of the dr numbers.
+position encoding is the rotary part's (either pairing, with its amplitude); it turns the first ``rotary_dim`` of the dr
+numbers.
 A ``window`` keeps the last ``window`` positions visible (itself included) and lets older pages go back.
 
 ``q_rank``: the queries go through a latent of their own, c_q = rmsnorm(W_dq x) * weight, q = W_uq c_q (tensors ``dq``,
 ``dq.norm``, ``uq`` instead of ``q``).  ``own_latent`` False: the layer has no W_dkv and no latent norm; it reads the
 records another layer stored (the schedule names that layer) with its own key and value maps, queries and window.
+``out_gate``: the heads' outputs side by side are multiplied number by number with sigmoid(W_g x) before the output projection
+(W_g's rows ride in the first product; the gate is applied to the sums of the per-head value products).
 """
 from __future__ import annotations
 
@@ -44,11 +47,12 @@ class LatentAttentionSpec:
     names: Optional[Tuple[Tuple[str, str], ...]] = None    # (role, name after the prefix); see DEFAULT_NAMES
     q_rank: Optional[int] = None    # size of the queries' latent (None: q = W_q x)
     own_latent: bool = True         # False: no down-projection of its own; every run reads another run's records
+    out_gate: bool = False          # the heads' outputs times sigmoid(W_g x), number by number
     kind: ClassVar[str] = "latent_attention"
 
 
 DEFAULT_NAMES = (("q", "q"), ("dkv", "dkv"), ("latent_norm", "dkv.norm"), ("uk", "uk"), ("uv", "uv"), ("o", "o"), ("dq", "dq"),
-                 ("q_latent_norm", "dq.norm"), ("uq", "uq"))
+                 ("q_latent_norm", "dq.norm"), ("uq", "uq"), ("gate", "g"))
 
 
 class LatentAttention(Mixer):
@@ -61,9 +65,8 @@ class LatentAttention(Mixer):
             raise ValueError("window must be positive")
         self.spec = spec
         self.position = build_part(spec.position) if spec.position is not None else None
-        if self.position is not None and (getattr(self.position, "pairing", "half") != "half"
-                                          or self.position.spec.rotary_dim > spec.rope_dim):
-            raise ValueError("latent attention: the rotation pairs element i with i + dims/2 and turns at most rope_dim numbers")
+        if self.position is not None and self.position.spec.rotary_dim > spec.rope_dim:
+            raise ValueError("latent attention: the rotation turns at most rope_dim numbers")
         self.names = dict(DEFAULT_NAMES)
         self.names.update(dict(spec.names or ()))
         if spec.q_rank is not None and spec.q_rank <= 0:
@@ -72,6 +75,9 @@ class LatentAttention(Mixer):
         self.record = spec.kv_rank + spec.rope_dim
         self.first = spec.q_rank if spec.q_rank is not None else self.q_width      # rows of the first product that belong to the queries
         self.rows = -(-(self.first + (self.record if spec.own_latent else 0)) // 8) * 8
+        self.gate_at = self.rows                        # the gate's columns, on a 16-byte boundary
+        if spec.out_gate:
+            self.rows += -(-spec.num_heads * spec.value_dim // 8) * 8
         self.w_in = self.w_uk_t = self.w_uv = self.w_o = self.latent_norm = self.w_uq = self.q_latent_norm = None
 
     def _name(self, role: str) -> str:
@@ -87,6 +93,8 @@ class LatentAttention(Mixer):
             decls = [WeightDecl(self._name("q"), (self.q_width, s.hidden_size))]
         if s.own_latent:
             decls += [WeightDecl(self._name("dkv"), (self.record, s.hidden_size)), WeightDecl(self._name("latent_norm"), (s.kv_rank,), init="gain")]
+        if s.out_gate:
+            decls.append(WeightDecl(self._name("gate"), (s.num_heads * s.value_dim, s.hidden_size)))
         return tuple(decls) + (WeightDecl(self._name("uk"), (s.num_heads * s.nope_dim, s.kv_rank)),
                                WeightDecl(self._name("uv"), (s.num_heads * s.value_dim, s.kv_rank)),
                                WeightDecl(self._name("o"), (s.hidden_size, s.num_heads * s.value_dim)))
@@ -94,6 +102,9 @@ class LatentAttention(Mixer):
     def load(self, tensors, dtype, device):
         s = self.spec
         mats = [tensors[self._name("dq" if s.q_rank is not None else "q")]] + ([tensors[self._name("dkv")]] if s.own_latent else [])
+        if s.out_gate:
+            gap = self.gate_at - sum(m.shape[0] for m in mats)
+            mats += ([torch.zeros((gap, s.hidden_size), dtype=mats[0].dtype)] if gap else []) + [tensors[self._name("gate")]]
         pad = self.rows - sum(m.shape[0] for m in mats)
         if pad:
             mats.append(torch.zeros((pad, s.hidden_size), dtype=mats[0].dtype))
@@ -153,7 +164,8 @@ class LatentAttention(Mixer):
         stores = cache.writable and s.own_latent
         if stores or dr:
             ops.latent_prep(q, proj[:, self.first: self.first + self.record] if s.own_latent else None, ctx.positions, cache.slot_mapping,
-                            self.latent_norm, s.norm_eps, inv_freq, rdim, records if stores else None, q_abs, H, dn, dr, rank)
+                            self.latent_norm, s.norm_eps, inv_freq, rdim, records if stores else None, q_abs, H, dn, dr, rank,
+                            pairing=getattr(self.position, "pairing", "half"), amplitude=getattr(self.position, "amplitude", 1.0))
         if dn:
             ops.gemm_heads(q.unflatten(1, (H, dn + dr))[:, :, :dn], self.w_uk_t, q_abs[:, :, :rank])
         else:
@@ -162,7 +174,7 @@ class LatentAttention(Mixer):
         ops.latent_attention(q_abs, o_lat, records, ctx.positions, ctx.row_of_token, cache.block_table, rank, cache.page_size,
                              s.scale, s.window, batch=ctx)
         heads_out = ctx.ws.get("attn_out", (T, H, s.value_dim), x.dtype)
-        ops.gemm_heads(o_lat, self.w_uv, heads_out)
+        ops.gemm_heads(o_lat, self.w_uv, heads_out, gate=proj[:, self.gate_at: self.gate_at + H * s.value_dim] if s.out_gate else None)
         out = ctx.ws.get("mixer_out", (T, s.hidden_size), x.dtype)
         return None if ops.gemm(heads_out.view(T, H * s.value_dim), self.w_o, out, sink=sink) else out
 

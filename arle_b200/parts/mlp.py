@@ -94,3 +94,52 @@ class GatedMlp(FeedForward):
 
 
 register_part(GatedMlpSpec.kind, GatedMlp)
+
+
+@dataclass(frozen=True)
+class UngatedMlpSpec:
+    """down(act(up(x))), no biases; ``activation`` "square_relu": max(z, 0)^2."""
+    prefix: str
+    hidden_size: int
+    intermediate_size: int
+    activation: str = "square_relu"
+    names: Tuple[str, str] = ("up_proj.weight", "down_proj.weight")     # after the prefix
+    kind: ClassVar[str] = "ungated_mlp"
+
+
+class UngatedMlp(FeedForward):
+    def __init__(self, spec: UngatedMlpSpec):
+        if spec.activation != "square_relu":
+            raise ValueError(f"activation {spec.activation!r} not supported by the ungated feed-forward (square_relu)")
+        self.spec = spec
+        self.w_up = self.w_down = None
+
+    def weight_decls(self):
+        s = self.spec
+        return (WeightDecl(s.prefix + s.names[0], (s.intermediate_size, s.hidden_size)),
+                WeightDecl(s.prefix + s.names[1], (s.hidden_size, s.intermediate_size)))
+
+    def load(self, tensors, dtype, device):
+        up, down = (tensors[self.spec.prefix + n] for n in self.spec.names)
+        self.w_up, self.w_down = (t.to(device=device, dtype=dtype if dtype == torch.bfloat16 else t.dtype).contiguous() for t in (up, down))
+
+    def weight_bytes(self):
+        return sum(t.numel() * t.element_size() for t in (self.w_up, self.w_down))
+
+    def scratch_elements_per_token(self):
+        return self.spec.intermediate_size + self.spec.hidden_size
+
+    def can_sink(self, num_rows):
+        return ops.fused_gemm_shape_ok(num_rows, self.w_down)
+
+    def forward(self, x, ctx, sink=None):
+        s = self.spec
+        T = x.shape[0]
+        act = ctx.ws.get("ffn_act", (T, s.intermediate_size), x.dtype)
+        ops.gemm(x, self.w_up, act)
+        ops.square_relu(act, act)
+        out = ctx.ws.get("ffn_out", (T, s.hidden_size), x.dtype)
+        return None if ops.gemm(act, self.w_down, out, sink=sink) else out
+
+
+register_part(UngatedMlpSpec.kind, UngatedMlp)

@@ -41,6 +41,8 @@ class ResidualStream:
         self._sinks_made = 0
         self._copy: Optional[torch.Tensor] = None       # the residual as it stands, in the activation type (or None)
         self._normed_branch = None                      # (norm, branch): resid += norm(branch) still to be done
+        self.next_conv = None                           # the next block's input convolution and its memory (or None), set by the model
+        self._convolved = None                          # (weight, output): already done by the kernel of the sum before it
 
     def _settle(self) -> None:
         """Whatever ``add_normed_before_norm`` left to the next norm is summed into the residual now."""
@@ -86,13 +88,49 @@ class ResidualStream:
             ops.branch_norm_add(self.resid, None, None, 0.0, self._copy)
         return self._copy
 
-    def add_normed(self, norm, branch: torch.Tensor, buffer_name: str) -> None:
-        """resid += norm(branch), and the rounded residual for whoever reads it next, in one kernel."""
+    def convolved(self, conv, ctx, buffer_name: str) -> torch.Tensor:
+        """The causal convolution of the residual over time that a block puts before its mixer; ``conv`` is what the block's
+        ``input_conv`` returned."""
+        weight, memory = conv
+        if self._convolved is not None:
+            done_for, out = self._convolved
+            self._convolved = None
+            if done_for is not weight:
+                raise RuntimeError("an input convolution was run for another block than the one that runs next")
+            return out
         self._settle()
         if self.pending is not None:
             ops.residual_add(self.resid, self.pending)
             self.pending = None
-        copy = None if self.act_dtype == torch.float32 else self.ws.get(buffer_name, tuple(self.resid.shape), self.act_dtype)
+            self._copy = None
+        out = self.ws.get(buffer_name, tuple(self.resid.shape), self.act_dtype)
+        ops.input_conv(self.resid, weight, memory, ctx.q_indptr, ctx.row_of_token, ctx.state_slots, out, ctx.max_q_len)
+        return out
+
+    def add_normed_then_conv(self, norm, branch: torch.Tensor, ctx, buffer_name: str) -> bool:
+        """resid += norm(branch) as a block's last act, with the next block's input convolution in the same kernel where that
+        can be (every row of the step one token, a norm that knows how).  False: nothing was done."""
+        if self.next_conv is None or ctx.max_q_len != 1 or not hasattr(norm, "add_normed_conv"):
+            return False
+        self._settle()
+        if self.pending is not None:
+            ops.residual_add(self.resid, self.pending)
+            self.pending = None
+        weight, memory = self.next_conv
+        out = self.ws.get(buffer_name, tuple(self.resid.shape), self.act_dtype)
+        norm.add_normed_conv(self.resid, branch, weight, memory, ctx.state_slots, out)
+        self._copy = None
+        self._convolved = (weight, out)
+        return True
+
+    def add_normed(self, norm, branch: torch.Tensor, buffer_name: Optional[str]) -> None:
+        """resid += norm(branch), and the rounded residual for whoever reads it next (no buffer name: nobody does), in one
+        kernel."""
+        self._settle()
+        if self.pending is not None:
+            ops.residual_add(self.resid, self.pending)
+            self.pending = None
+        copy = None if self.act_dtype == torch.float32 or buffer_name is None else self.ws.get(buffer_name, tuple(self.resid.shape), self.act_dtype)
         norm.add_normed(self.resid, branch, copy)
         self._copy = copy
 
@@ -148,6 +186,8 @@ class ResidualStream:
 def declared_weights(spec: ModelSpec) -> List[WeightDecl]:
     """Every tensor a checkpoint of this model must hold."""
     decls = [WeightDecl(spec.embed_name, (spec.vocab_size, spec.hidden_size))]
+    if spec.embed_norm is not None:
+        decls.extend(build_part(spec.embed_norm).weight_decls())
     for b in spec.blocks:
         decls.extend(build_part(b).weight_decls())
     decls.extend(build_part(spec.final_norm).weight_decls())
@@ -166,6 +206,7 @@ class DecoderModel:
         self.spec = spec
         self.blocks = [build_part(b) for b in spec.blocks]
         self.final_norm = build_part(spec.final_norm)
+        self.embed_norm = build_part(spec.embed_norm) if spec.embed_norm is not None else None
         self.embed = self.head = None
         self.dtype = None
         # cache layers: one per schedule entry that keeps keys of its own
@@ -187,7 +228,7 @@ class DecoderModel:
                 self.cache_needs.append(need)
             else:
                 self.entry_cache_layer.append(None)
-            sneed = mixer.state_need()
+            sneed = self.blocks[e.block].state_need()
             if sneed is not None:
                 self.entry_state.append(len(self.state_needs))
                 self.state_needs.append(sneed)
@@ -212,6 +253,8 @@ class DecoderModel:
         for b in self.blocks:
             b.load(tensors, dtype, device)
         self.final_norm.load(tensors, dtype, device)
+        if self.embed_norm is not None:
+            self.embed_norm.load(tensors, dtype, device)
         return self
 
     def weight_bytes_per_step(self) -> int:
@@ -230,15 +273,23 @@ class DecoderModel:
         resid = ctx.ws.get("residual", (ctx.num_tokens, self.spec.hidden_size), torch.float32)
         ops.embedding(ctx.token_ids, self.embed, resid, None, getattr(ctx, "last_token", None),
                       getattr(ctx, "slot_of_token", None), scale=self.spec.embed_scale)
+        if self.embed_norm is not None:
+            self.embed_norm.apply(resid, None, None, resid, write_resid=False)       # in place: the residual starts normed, in float32
         return resid
 
     def run_blocks(self, stream: ResidualStream, ctx) -> None:
         order = self.spec.schedule
+
+        def state_of(i):
+            return ctx.state_view(self.entry_state[i]) if self.entry_state[i] is not None else None
+
         for i, e in enumerate(order):
-            stream.next_entry = self.blocks[order[i + 1].block].entry() if i + 1 < len(order) else None
+            after = self.blocks[order[i + 1].block] if i + 1 < len(order) else None
+            stream.next_entry = after.entry() if after is not None else None
+            stream.next_conv = after.input_conv(state_of(i + 1)) if after is not None else None
             cl = self.entry_cache_layer[i]
             cache = ctx.cache_view(cl, writable=e.keys_of is None) if cl is not None else None
-            st = ctx.state_view(self.entry_state[i]) if self.entry_state[i] is not None else None
+            st = state_of(i)
             self.blocks[e.block].forward(stream, ctx, cache, st)
 
     def logits_at_wanted(self, stream: ResidualStream, ctx) -> torch.Tensor:

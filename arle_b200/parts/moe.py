@@ -10,7 +10,10 @@ sigmoid(w_sg . x), one number per token, when it has such a gate.
 Variants, each a field of the spec: ``scores`` "softmax" takes the scores as a softmax over all experts; "softmax_chosen"
 chooses the experts with the largest router sums and weights them by the softmax over the chosen sums alone; ``group_score``
 "max" scores a group by its largest choice score alone; ``activation`` "clamped_glu" makes an expert
-down(g * sigmoid(act_alpha * g) * (u + 1)) with g = min(gate x, act_limit) and u = up x clamped to +-act_limit.
+down(g * sigmoid(act_alpha * g) * (u + 1)) with g = min(gate x, act_limit) and u = up x clamped to +-act_limit; ``gated`` False
+makes it down(act(up x)) with ``activation`` "square_relu"; ``weight_on`` "input" multiplies the expert's input by its weight
+instead of its output, expert(w x): the first product is linear, so the weight goes onto its float32 sums, and the outputs are
+added as they are.
 
 The step's (token, choice) pairs are sorted by expert on the device and the experts' products run as grouped tiles over
 the sorted places, so nothing depends on the host knowing how many tokens an expert got (a decode step stays capturable).
@@ -47,6 +50,8 @@ class RoutedExpertsSpec:
     group_score: str = "top2_sum"    # or "max"
     act_limit: Optional[float] = None    # of the "clamped_glu" activation
     act_alpha: float = 1.702
+    gated: bool = True               # False: down(act(up x))
+    weight_on: str = "output"        # "input": an expert runs on its weight times x
     kind: ClassVar[str] = "routed_experts"
 
 
@@ -61,8 +66,9 @@ class RoutedExperts(FeedForward):
             raise ValueError("routed experts: experts must split into the groups, of which at most all are kept")
         if spec.top > spec.keep * per or E > 1024:
             raise ValueError("routed experts: more experts chosen than the kept groups hold, or more than 1,024 experts")
-        if spec.activation not in ops.ACTIVATIONS and spec.activation != "clamped_glu":
-            raise ValueError(f"routed experts: activation {spec.activation!r}")
+        known = tuple(ops.ACTIVATIONS) + ("clamped_glu",) if spec.gated else ("square_relu",)
+        if spec.activation not in known or spec.weight_on not in ("output", "input"):
+            raise ValueError(f"routed experts: activation {spec.activation!r} ({', '.join(known)}) / weight_on {spec.weight_on!r} (output, input)")
         if spec.activation == "clamped_glu" and not (spec.act_limit is not None and spec.act_limit > 0):
             raise ValueError("routed experts: the clamped activation needs a positive act_limit")
         if spec.scores not in ("sigmoid", "softmax", "softmax_chosen") or spec.group_score not in ("top2_sum", "max"):
@@ -73,7 +79,8 @@ class RoutedExperts(FeedForward):
         self.names = dict(DEFAULT_NAMES)
         self.names.update(dict(spec.names or ()))
         self.shared = build_part(spec.shared) if spec.shared is not None else None
-        self.w_router = self.correction = self.w_gate_up = self.w_down = None
+        self.w_router = self.correction = self.w_gate_up = self.w_down = None     # w_gate_up: the up matrices alone without gates
+        self.first_rows = (2 if spec.gated else 1) * spec.expert_ff
 
     def _name(self, role: str, expert: int = None) -> str:
         if expert is None:
@@ -86,8 +93,8 @@ class RoutedExperts(FeedForward):
         if s.correction:
             decls.append(WeightDecl(self._name("correction"), (s.num_experts,), init="around_zero"))
         for e in range(s.num_experts):
-            decls += [WeightDecl(self._name("gate", e), (s.expert_ff, s.hidden_size)), WeightDecl(self._name("up", e), (s.expert_ff, s.hidden_size)),
-                      WeightDecl(self._name("down", e), (s.hidden_size, s.expert_ff))]
+            decls += [WeightDecl(self._name(n, e), (s.expert_ff, s.hidden_size)) for n in (("gate", "up") if s.gated else ("up",))]
+            decls.append(WeightDecl(self._name("down", e), (s.hidden_size, s.expert_ff)))
         if self.shared is not None:
             decls += list(self.shared.weight_decls())
         if s.shared_gate:
@@ -106,8 +113,10 @@ class RoutedExperts(FeedForward):
             self.correction = tensors[self._name("correction")].to(device=device, dtype=torch.float32).contiguous()
         gu, dn = [], []
         for e in range(s.num_experts):
-            g, u, d = (tensors[self._name(n, e)] for n in ("gate", "up", "down"))
-            gu.append(torch.stack([g, u], dim=1).reshape(2 * s.expert_ff, s.hidden_size))      # rows 2i, 2i + 1: gate_i, up_i
+            u, d = (tensors[self._name(n, e)] for n in ("up", "down"))
+            if s.gated:
+                u = torch.stack([tensors[self._name("gate", e)], u], dim=1).reshape(2 * s.expert_ff, s.hidden_size)      # rows 2i, 2i + 1: gate_i, up_i
+            gu.append(u)
             dn.append(d)
         self.w_gate_up = torch.stack(gu).to(device=device, dtype=kept(gu)).contiguous()
         self.w_down = torch.stack(dn).to(device=device, dtype=kept(dn)).contiguous()
@@ -138,19 +147,24 @@ class RoutedExperts(FeedForward):
         plan = ctx.ws.get("moe_plan", (ops.moe_plan_size(E, pairs),), torch.int32)
         place_of_pair = ctx.ws.get("moe_place", (pairs,), torch.int32)
         row_of_place = ctx.ws.get("moe_row", (pairs,), torch.int32)
-        ops.moe_plan(ids, E, plan, place_of_pair, row_of_place)
-        gu = ctx.ws.get("moe_gate_up", (pairs, 2 * ff), x.dtype)
-        ops.moe_gemm(x, row_of_place, self.w_gate_up, gu, plan, E)
-        act = ctx.ws.get("moe_act", (pairs, ff), x.dtype)
-        if s.activation == "clamped_glu":
-            ops.clamped_glu(gu, act, s.act_limit, s.act_alpha)
+        on_input = s.weight_on == "input"
+        of_place = ctx.ws.get("moe_weight_of_place", (pairs,), torch.float32) if on_input else None
+        ops.moe_plan(ids, E, plan, place_of_pair, row_of_place, weights if on_input else None, of_place)
+        gu = ctx.ws.get("moe_gate_up", (pairs, self.first_rows), x.dtype)
+        ops.moe_gemm(x, row_of_place, self.w_gate_up, gu, plan, E, place_scale=of_place, act="none" if s.gated else s.activation)
+        if not s.gated:
+            act = gu                                    # the activation is the product's last act
         else:
-            ops.act_mul(gu, act, s.activation)
+            act = ctx.ws.get("moe_act", (pairs, ff), x.dtype)
+            if s.activation == "clamped_glu":
+                ops.clamped_glu(gu, act, s.act_limit, s.act_alpha)
+            else:
+                ops.act_mul(gu, act, s.activation)
         y = ctx.ws.get("moe_y", (pairs, s.hidden_size), x.dtype)
         ops.moe_gemm(act, None, self.w_down, y, plan, E)
         shared = self.shared.forward(x, ctx) if self.shared is not None else None
         out = ctx.ws.get("moe_out", (T, s.hidden_size), x.dtype)
-        ops.moe_combine(y, place_of_pair, weights, shared, z[:, E] if s.shared_gate else None, out)
+        ops.moe_combine(y, place_of_pair, None if on_input else weights, shared, z[:, E] if s.shared_gate else None, out, top=top)
         return out
 
 

@@ -5,7 +5,11 @@ With ``one_plus`` the checkpoint stores the gain around zero and the norm multip
 
 Dynamic Tanh stands where a norm stands but forms no mean and no variance: y = tanh(alpha * x) * weight + bias, element
 by element, with a stored scalar alpha and a stored bias vector ("<name>.alpha", "<name>.b" beside the weight).  It has no
-per-row factor, so it cannot be deferred into the product that follows (``deferred()`` is None)."""
+per-row factor, so it cannot be deferred into the product that follows (``deferred()`` is None).
+
+Layer norm: y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight, no bias, statistics in float32.  With ``scale_name`` a
+second stored vector multiplies the result element by element (a layer scale behind the norm on a branch's output); the two
+vectors are multiplied once at load, in float32."""
 from __future__ import annotations
 
 from dataclasses import dataclass
@@ -69,6 +73,52 @@ class RmsNorm(Norm):
 
 
 register_part(RmsNormSpec.kind, RmsNorm)
+
+
+@dataclass(frozen=True)
+class LayerNormSpec:
+    weight_name: str
+    size: int
+    eps: float
+    scale_name: str = ""            # a second vector the result is multiplied by ("": none)
+    kind: ClassVar[str] = "layernorm"
+
+
+class LayerNorm(Norm):
+    def __init__(self, spec: LayerNormSpec):
+        self.spec = spec
+        self.eps = spec.eps
+        self.weight = None
+
+    def weight_decls(self):
+        names = [self.spec.weight_name] + ([self.spec.scale_name] if self.spec.scale_name else [])
+        return tuple(WeightDecl(n, (self.spec.size,), init="gain") for n in names)
+
+    def load(self, tensors, dtype, device):
+        w = tensors[self.spec.weight_name].to(device=device, dtype=torch.float32)
+        if self.spec.scale_name:
+            w = w * tensors[self.spec.scale_name].to(device=device, dtype=torch.float32)
+        self.weight = w.contiguous()
+
+    def weight_bytes(self):
+        return self.weight.numel() * 4
+
+    def scratch_elements_per_token(self):
+        return self.spec.size
+
+    def apply(self, resid, delta, rows, out, write_resid: bool):
+        ops.layernorm(resid, delta, rows, self.weight, self.eps, out, write_resid)
+        return out
+
+    def add_normed(self, resid, branch, copy):
+        ops.branch_layernorm_add(resid, branch, self.weight, self.eps, copy)
+
+    def add_normed_conv(self, resid, branch, conv_weight, conv_memory, state_slots, out):
+        """resid += norm(branch), and the next block's input convolution of it, for rows of one token each."""
+        ops.branch_layernorm_add(resid, branch, self.weight, self.eps, None, conv=(conv_weight, conv_memory, state_slots, out))
+
+
+register_part(LayerNormSpec.kind, LayerNorm)
 
 
 @dataclass(frozen=True)
