@@ -87,13 +87,13 @@ def attention_prep(qkv, positions, slot_mapping, q_weight, k_weight, eps, inv_fr
 
 
 def paged_attention(q, out, k_cache, v_cache, positions, row_of_token, block_table, nq, nkv, hd, page_size, scale,
-                    window, batch=None, vd=None, sink=None, keep_first=0, softcap=None):
+                    window, batch=None, vd=None, sink=None, keep_first=0, softcap=None, chunk=None, score_bias=None):
     T = q.shape[0]
     g = nq // nkv
     vd = hd if vd is None else vd
     for t in range(T):
         p = int(positions[t])
-        lo = max(0, p - window + 1) if window else 0
+        lo = p - p % chunk if chunk else max(0, p - window + 1) if window else 0
         js = torch.cat([torch.arange(0, min(int(keep_first or 0), lo)), torch.arange(lo, p + 1)])
         pages = block_table[int(row_of_token[t]), js // page_size].long()
         offs = js % page_size
@@ -104,7 +104,9 @@ def paged_attention(q, out, k_cache, v_cache, positions, row_of_token, block_tab
             s = (k[:, h // g] @ qt[h]) * scale
             if softcap:
                 s = softcap * torch.tanh(s / softcap)
-            if sink is None:
+            if score_bias is not None:                       # no softmax: a weight per key as it is
+                pr = torch.sigmoid(s + score_bias[h])
+            elif sink is None:
                 pr = torch.softmax(s, dim=0)
             else:                                            # one more term in the denominator, without a value
                 pr = torch.softmax(torch.cat([s, torch.tensor([float(sink)])]), dim=0)[:-1]
@@ -177,8 +179,9 @@ def gemm_act_mul(x, w, gate_up, out, activation="silu"):
 
 
 def attention_prep_row(qk, positions, slot_mapping, q_weight, k_weight, eps, inv_freq, rotary_dim, pairing, values_are_keys,
-                       k_cache, v_cache, nq, nkv, hd, page_size, angles=None):
+                       k_cache, v_cache, nq, nkv, hd, page_size, angles=None, vd=None):
     T = qk.shape[0]
+    vd = hd if vd is None else vd
 
     def norm_rope(x, w, heads):
         x = x.to(F32)
@@ -200,7 +203,7 @@ def attention_prep_row(qk, positions, slot_mapping, q_weight, k_weight, eps, inv
     q = norm_rope(qk[:, : nq * hd], q_weight, nq)
     if nkv:
         k = norm_rope(qk[:, nq * hd:(nq + nkv) * hd], k_weight, nkv).to(qk.dtype)
-        v = raw_k if values_are_keys else qk[:, (nq + nkv) * hd:(nq + 2 * nkv) * hd].view(T, nkv, hd)
+        v = raw_k if values_are_keys else qk[:, (nq + nkv) * hd:(nq + nkv) * hd + nkv * vd].view(T, nkv, vd)
         keep = slot_mapping >= 0
         page = (slot_mapping[keep] // page_size).long()
         off = (slot_mapping[keep] % page_size).long()
@@ -225,20 +228,28 @@ def logit_cap(logits, cap):
     logits.copy_(cap * torch.tanh(logits / cap))
 
 
-def gla_decay(low, w2t, bias, tau, alpha):
-    z = low.to(F32) @ w2t
+def gla_decay(low, w2t, bias, tau, alpha, form="sigmoid_root"):
+    z = (torch.tanh(low.to(F32)) if form == "double_exp" else low.to(F32)) @ w2t
     if bias is not None:
         z = z + bias
+    if form == "double_exp":
+        alpha.copy_(torch.exp(-torch.exp(z)))
+        return
     alpha.copy_(torch.exp(-torch.nn.functional.softplus(-z) / tau))
 
 
-def gla_scan(q, k, v, alpha, state, q_indptr, state_slots, out, heads, dim, vdim, q_scale, max_q_len):
+def gla_scan(q, k, v, alpha, state, q_indptr, state_slots, out, heads, dim, vdim, q_scale, max_q_len, bonus=None):
     for r in range(state_slots.numel()):
-        S = state[int(state_slots[r])]                                   # [heads, vdim, dim]
+        S = state[int(state_slots[r])].reshape(-1)[: heads * vdim * dim].view(heads, vdim, dim)
         for t in range(int(q_indptr[r]), int(q_indptr[r + 1])):
             qt = q[t].to(F32).view(heads, dim) * q_scale
             kt, vt, at = k[t].to(F32).view(heads, dim), v[t].to(F32).view(heads, vdim), alpha[t].view(heads, dim)
-            S.copy_(S * at[:, None, :] + vt[:, :, None] * kt[:, None, :])
+            kv = vt[:, :, None] * kt[:, None, :]
+            if bonus is not None:
+                out[t] = torch.einsum("hvd,hd->hv", S + bonus.view(heads, 1, dim) * kv, qt).reshape(-1)
+                S.copy_(S * at[:, None, :] + kv)
+                continue
+            S.copy_(S * at[:, None, :] + kv)
             out[t] = torch.einsum("hvd,hd->hv", S, qt).reshape(-1)
 
 
@@ -247,7 +258,7 @@ def gla_out(o, gate, weight, eps, scale, out, heads, vdim, gate_act="silu"):
     y = o.view(T, heads, vdim)
     y = y * (1.0 / torch.sqrt((y * y).mean(dim=-1, keepdim=True) + eps))
     if weight is not None:
-        y = y * weight
+        y = y * (weight if weight.numel() == vdim else weight.view(heads, vdim))
     y = y.reshape(T, heads * vdim)
     if gate is not None:
         g = gate.to(F32)
@@ -273,8 +284,11 @@ def dyt_norm(resid, delta, rows, weight, bias, alpha, out, write_resid):
 
 
 # ---------------------------------------------------------------- attention over latent vectors
-def gemm_heads(x, w, out):
-    out.copy_(torch.einsum("mhk,hnk->mhn", x.to(F32), w.to(F32)).to(out.dtype))
+def gemm_heads(x, w, out, gate=None):
+    y = torch.einsum("mhk,hnk->mhn", x.to(F32), w.to(F32))
+    if gate is not None:
+        y = y * torch.sigmoid(gate.to(F32)).reshape(y.shape)
+    out.copy_(y.to(out.dtype))
 
 
 def _turn_half(x, pos, inv_freq, dims):
@@ -290,18 +304,31 @@ def _turn_half(x, pos, inv_freq, dims):
     return torch.cat([u * c - v * s_, v * c + u * s_, x[..., dims:]], dim=-1)
 
 
-def latent_prep(q, dkv, positions, slot_mapping, c_weight, eps, inv_freq, rot_dims, cache, q_abs, heads, dn, dr, rank):
+def latent_prep(q, dkv, positions, slot_mapping, c_weight, eps, inv_freq, rot_dims, cache, q_abs, heads, dn, dr, rank, pairing="half",
+                amplitude=1.0):
     T = q.shape[0]
+
+    def turn(x):
+        if pairing == "half" and amplitude == 1.0:
+            return _turn_half(x, positions, inv_freq, rot_dims)
+        y = x.clone()
+        for i in range(rot_dims // 2):
+            a, b = (2 * i, 2 * i + 1) if pairing == "interleaved" else (i, i + rot_dims // 2)
+            ang = (positions.to(F32) * inv_freq[i]).view([T] + [1] * (x.dim() - 2))
+            c, s_ = amplitude * torch.cos(ang), amplitude * torch.sin(ang)
+            y[..., a], y[..., b] = x[..., a] * c - x[..., b] * s_, x[..., b] * c + x[..., a] * s_
+        return y
+
     if cache is not None:
         kv = dkv[:, : rank + dr].to(F32)
         c = kv[:, :rank]
         c = c * (1.0 / torch.sqrt((c * c).mean(dim=-1, keepdim=True) + eps)) * c_weight
-        rec = torch.cat([c, _turn_half(kv[:, rank:], positions, inv_freq, rot_dims)], dim=-1).to(cache.dtype)
+        rec = torch.cat([c, turn(kv[:, rank:])], dim=-1).to(cache.dtype)
         page_size = cache.shape[2]
         sm = slot_mapping.long()
         cache[sm // page_size, 0, sm % page_size] = rec
     qr = q[:, : heads * (dn + dr)].to(F32).view(T, heads, dn + dr)[:, :, dn:]
-    q_abs[:, :, rank:] = _turn_half(qr, positions, inv_freq, rot_dims).to(q_abs.dtype)
+    q_abs[:, :, rank:] = turn(qr).to(q_abs.dtype)
 
 
 def latent_attention(q_abs, out, cache, positions, row_of_token, block_table, rank, page_size, scale, window, batch=None):
@@ -412,29 +439,37 @@ def moe_plan_size(experts, pairs):
     return experts + 2 + 3 * (pairs // 64 + experts + 1)
 
 
-def moe_plan(ids, experts, plan, place_of_pair, row_of_place):
+def moe_plan(ids, experts, plan, place_of_pair, row_of_place, weights=None, weight_of_place=None):
     T, top = ids.shape
     flat = ids.reshape(-1).long()
     order = torch.argsort(flat, stable=True)
     place_of_pair[order] = torch.arange(T * top, dtype=torch.int32)
     row_of_place[: T * top] = (order // top).to(torch.int32)
+    if weights is not None:
+        weight_of_place[: T * top] = weights.reshape(-1)[order]
     counts = torch.bincount(flat, minlength=experts)
     plan[:experts] = (torch.cumsum(counts, 0) - counts).to(torch.int32)
     plan[experts] = T * top
     plan[experts + 1] = -1                      # no tiles: the plain statement of the grouped product reads the runs
 
 
-def moe_gemm(x, rows, w, out, plan, experts):
+def moe_gemm(x, rows, w, out, plan, experts, place_scale=None, act="none"):
     pairs = out.shape[0]
     bounds = plan[: experts + 1].tolist()
     for e in range(experts):
         lo, hi = bounds[e], bounds[e + 1]
         if hi > lo:
             src = x[rows[lo:hi].long()] if rows is not None else x[lo:hi]
-            out[lo:hi] = (src.to(F32) @ w[e].to(F32).t()).to(out.dtype)
+            y = src.to(F32) @ w[e].to(F32).t()
+            if place_scale is not None:
+                y = y * place_scale[lo:hi, None]
+            out[lo:hi] = (y.clamp(min=0.0) ** 2 if act == "square_relu" else y).to(out.dtype)
 
 
-def moe_combine(y, place_of_pair, weights, shared, gate, out):
+def moe_combine(y, place_of_pair, weights, shared, gate, out, top=None):
+    T = out.shape[0]
+    if weights is None:
+        weights = torch.ones(T, top)
     T, top = weights.shape
     acc = (weights[:, :, None] * y[place_of_pair[: T * top].long()].to(F32).view(T, top, -1)).sum(1)
     if shared is not None:
@@ -570,9 +605,73 @@ def delta_scan(q, k, v, beta, decay, state, q_indptr, state_slots, out, heads, k
                 out[t, h] = Sh @ qq[t, g]
 
 
+def gate_mul(x, gate, out):
+    out.copy_((x.to(F32) * torch.sigmoid(gate.to(F32))).to(out.dtype))
+
+
+def square_relu(x, out):
+    out.copy_((x.to(F32).clamp(min=0.0) ** 2).to(out.dtype))
+
+
+def _ln(x, weight, eps):
+    d = x - x.mean(-1, keepdim=True)
+    return d / torch.sqrt((d * d).mean(-1, keepdim=True) + eps) * weight
+
+
+def layernorm(resid, delta, rows, weight, eps, out, write_resid):
+    idx = rows.long() if rows is not None else torch.arange(resid.shape[0], device=resid.device)
+    x = resid[idx].to(F32)
+    if delta is not None:
+        x = x + delta[idx].to(F32)
+    if write_resid:
+        resid[idx] = x
+    out.copy_(_ln(x, weight, eps).to(out.dtype))
+
+
+def branch_layernorm_add(resid, branch, weight, eps, copy, conv=None):
+    resid += _ln(branch.to(F32), weight, eps)
+    if copy is not None:
+        copy.copy_(resid.to(copy.dtype))
+    if conv is not None:
+        cw, state, slots, out = conv
+        T = resid.shape[0]
+        input_conv(resid, cw, state, torch.arange(T + 1), torch.arange(T), slots, out, 1)
+
+
+def input_conv(x, weight, state, q_indptr, row_of_token, state_slots, out, max_q_len):
+    taps, C = weight.shape
+    for r in range(state_slots.numel()):
+        beg, end = int(q_indptr[r]), int(q_indptr[r + 1])
+        if end == beg:
+            continue
+        slot = int(state_slots[r])
+        hist = state[slot, : C * (taps - 1)].view(taps - 1, C) if taps > 1 else torch.zeros(0, C)
+        seq = torch.cat([hist, x[beg:end]], dim=0)
+        acc = torch.zeros(end - beg, C)
+        for j in range(taps):
+            acc = acc + seq[j: j + end - beg] * weight[j][None, :]
+        out[beg:end] = acc.to(out.dtype)
+        if taps > 1:
+            hist.copy_(seq[seq.shape[0] - (taps - 1):].clone())
+
+
+def token_shift(h, mu, state, q_indptr, row_of_token, state_slots, out, max_q_len):
+    C = h.shape[1]
+    for r in range(state_slots.numel()):
+        beg, end = int(q_indptr[r]), int(q_indptr[r + 1])
+        if end == beg:
+            continue
+        slot = int(state_slots[r])
+        x = h[beg:end].to(F32)
+        before = torch.cat([state[slot, :C][None], x[:-1]], dim=0)
+        for s_ in range(mu.shape[0]):
+            out[s_, beg:end] = (x + (before - x) * mu[s_][None, :]).to(out.dtype)
+        state[slot, :C] = x[-1]
+
+
 ALL = ("rotary_angles", "embedding", "rmsnorm", "residual_add", "gemm", "fused_gemm_shape_ok", "fused_decode_supported", "attention_prep_takes_angles", "attention_prep", "paged_attention", "silu_mul", "gemm_silu_mul", "argmax", "scatter_tokens", "sample",
        "act_mul", "gemm_act_mul", "attention_prep_row", "head_gate", "weighted_sum", "logit_cap", "gla_decay", "gla_scan", "gla_out",
        "dyt_norm", "gemm_heads", "latent_prep", "latent_attention", "decay_scan", "mlstm_gates", "mlstm_out", "ssm_gates", "conv_silu",
        "gated_group_norm", "moe_select", "moe_plan_size", "moe_plan", "moe_gemm", "moe_combine", "clamped_glu", "branch_norm_add",
        "attention_prep_post", "causal_conv", "rglru_scan", "delta_gates", "delta_scan", "branch_norm_add_norm", "rms_rows", "normed_sum",
-       "bias_add")
+       "bias_add", "gate_mul", "square_relu", "layernorm", "branch_layernorm_add", "input_conv", "token_shift")
