@@ -22,6 +22,8 @@ every second feed-forward one of routed experts) beside Kolodra and Qwen3 layers
 ``--design lukinex`` does the same for Lukinex layers (an attention whose window keeps the first tokens, two latent attentions
 of which the second reads the first one's latents, and a parallel mixer of a capped attention with biases and a short
 convolution beside a memory with constant decays, all with routed feed-forwards) beside Lasupel and Zuderax layers.
+``--design dabilorn`` does the same for Dabilorn layers (a latent attention with stretched rotation and an output gate, a chunked
+attention with sigmoid weights, RWKV-style time mixing, in turn, all with routed feed-forwards) beside Lukinex and Kolodra layers.
 ``--design lasupel`` does the same for Lasupel layers (an attention with a sliding window and a sink, an RG-LRU layer, an
 attention that reads the first one's keys and values, a gated delta rule layer, in turn; the first feed-forward of four
 dense, the others routed experts) beside Zuderax and Qwen3 layers of equal width.
@@ -245,6 +247,27 @@ def lukinex_config(z, kk, L, window):
     return {"architecture": "Lukinex", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "layers": layers}
 
 
+# Mixer sizes for ``--design dabilorn`` at the same widths: the latent attention is Lukinex's with 32 / 64 rotated numbers
+# (stretched) on top, the chunked attention has the Qwen3 layer's heads (chunks of three fifths of the benchmark's context, the whole head
+# rotated), the time mixing has Kolodra's memories of 128 x 128 and decay rank, the chosen experts together with the shared one
+# are as wide as the dense feed-forward.
+DABILORN_SIZES = {"0.6b": dict(latent=(16, 64, 32, 64, 256, 512), experts=16, top=3),
+                  "8b": dict(latent=(32, 128, 64, 128, 512, 1536), experts=32, top=3)}
+
+
+def dabilorn_config(z, dd, L, chunk):
+    routed = {"kind": "moe", "expert": {"ff": z["ff"] // (dd["top"] + 1)}, "shared": {"ff": z["ff"] // (dd["top"] + 1)},
+              "router": {"experts": dd["experts"], "top": dd["top"]}}
+    h, dk, dr, dv, rank, qrank = dd["latent"]
+    mixers = [("latent_attention", {"heads": h, "dim": dk, "rot_dim": dr, "vdim": dv, "kv_rank": rank, "q_rank": qrank, "scale": (dk + dr) ** -0.5,
+                                    "rot": {"base": 1e6, "dims": dr, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}),
+              ("attention", {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["hd"], "vdim": z["hd"], "scale": z["hd"] ** -0.5,
+                             "mask": {"size": chunk}, "rot": {"base": 1e6, "dims": z["hd"]}}),
+              ("wkv", {"heads": z["rheads"], "dim": 128, "decay_rank": z["rank"]})]
+    layers = [{"type": mixers[i % 3][0], "mixer": dict(mixers[i % 3][1]), "mlp": routed} for i in range(L)]
+    return {"architecture": "Dabilorn", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "canon": {"taps": 4}, "layers": layers}
+
+
 def design_table(args, torch, ops, pk) -> int:
     """``--design kolodra``: prefill and decode throughput of a few Kolodra layers beside the same number of Qwen3
     layers of equal width, heads and feed-forward, with the device time of every kernel of one step (profiler
@@ -254,7 +277,7 @@ def design_table(args, torch, ops, pk) -> int:
     from arle_b200.engine import ModelRunner, StepEntry, random_model
 
     dev = torch.device("cuda:0")
-    L, T, C = args.layers or (6 if args.design == "zuderax" else (8 if args.design in ("lasupel", "lukinex") else 4)), args.prefill_tokens, args.context
+    L, T, C = args.layers or (6 if args.design == "zuderax" else 12 if args.design == "dabilorn" else (8 if args.design in ("lasupel", "lukinex") else 4)), args.prefill_tokens, args.context
     gen = torch.Generator().manual_seed(1)
     out = {"design": args.design, "layers": L, "prefill_tokens": T, "context": C, "dtype": "bf16", "peaks": pk, "sizes": {}}
 
@@ -368,6 +391,14 @@ def design_table(args, torch, ops, pk) -> int:
             if not args.design_alone:
                 out["sizes"][name].update({"lasupel": measure(lasupel_config(z, LASUPEL_SIZES[name], L, max(C // 2, 16))),
                                            "zuderax": measure(zuderax_config(z, ZUDERAX_SIZES[name], L, max(C // 2, 16)))})
+        elif args.design == "dabilorn":
+            out["sizes"][name]["mixers"] = DABILORN_SIZES[name]
+            # chunks of three fifths of the context: the decoded tokens stand in the middle of the second one
+            out["sizes"][name]["dabilorn"] = measure(dabilorn_config(z, DABILORN_SIZES[name], L, max(3 * C // 5, 16)))
+            if not args.design_alone:
+                # twelve layers by default: whole rounds of Dabilorn's three kinds of layers and of Lukinex's four
+                out["sizes"][name].update({"lukinex": measure(lukinex_config(z, LUKINEX_SIZES[name], L, max(C // 2, 16))),
+                                           "kolodra": measure(kolodra_config(z))})
         elif not args.design_alone:
             out["sizes"][name].update({"kolodra": measure(kolodra_config(z)), "qwen3": measure(qwen_config(z))})
     print(json.dumps(out))
@@ -396,8 +427,8 @@ def main() -> int:
     ap.add_argument("--no-cuda-graph", action="store_true")
     ap.add_argument("--no-kernel-times", action="store_true",
                     help="with --design: leave out the per-kernel times (they come from torch's profiler, which cannot run under another profiler)")
-    ap.add_argument("--design-alone", action="store_true", help="with --design zuderax, lasupel or lukinex: leave out the models it stands beside")
-    ap.add_argument("--design", default=None, choices=["kolodra", "zuderax", "lasupel", "lukinex"],
+    ap.add_argument("--design-alone", action="store_true", help="with --design zuderax, lasupel, lukinex or dabilorn: leave out the models it stands beside")
+    ap.add_argument("--design", default=None, choices=["kolodra", "zuderax", "lasupel", "lukinex", "dabilorn"],
                     help="instead of the default workload: a few layers of this design beside as many Qwen3 layers of equal "
                          "sizes, prefill and decode, with every kernel's time (uses --layers, --steps, --context, --prefill-tokens)")
     ap.add_argument("--timeline", action="store_true",
