@@ -45,14 +45,19 @@ __global__ void latent_prep_kernel(const T* __restrict__ q, int q_stride, const 
     turn[j] = make_float2(cs * amplitude, sn * amplitude);
   }
   __syncthreads();
-  // number i of a rotated vector p, turned with its partner (pairing 0: i and i + half; 1: neighbours 2j and 2j + 1)
-  auto turned = [&](const T* p, int i) -> float {
-    if (i >= rot_dims) return to_f32(p[i]);
-    const int j = pairing ? i >> 1 : (i < half ? i : i - half);
-    const bool first = pairing ? (i & 1) == 0 : i < half;
-    const float cs = turn[j].x, sn = turn[j].y;
-    const float u = to_f32(p[pairing ? 2 * j : j]), v = to_f32(p[pairing ? 2 * j + 1 : j + half]);
-    return first ? u * cs - v * sn : v * cs + u * sn;
+  // unit i of a rotated vector p into o: the pair i (pairing 0: numbers i and i + half; 1: neighbours 2i and 2i + 1), or past the
+  // pairs one of the numbers that pass
+  const int units = half + dr - rot_dims;
+  auto turned = [&](const T* p, T* o, int i) {
+    if (i >= half) {
+      o[i - half + rot_dims] = p[i - half + rot_dims];
+      return;
+    }
+    const int e0 = pairing ? 2 * i : i, e1 = pairing ? 2 * i + 1 : i + half;
+    const float cs = turn[i].x, sn = turn[i].y;
+    const float u = to_f32(p[e0]), v = to_f32(p[e1]);
+    o[e0] = from_f32<T>(u * cs - v * sn);
+    o[e1] = from_f32<T>(v * cs + u * sn);
   };
   const T* kv = dkv + (size_t)t * dkv_stride;
   if (cache != nullptr) {
@@ -65,12 +70,12 @@ __global__ void latent_prep_kernel(const T* __restrict__ q, int q_stride, const 
     const float inv = 1.0f / sqrtf(total / (float)rank + eps);
     T* dst = cache + (size_t)slot_mapping[t] * kd;
     for (int c = threadIdx.x; c < rank; c += blockDim.x) dst[c] = from_f32<T>(to_f32(kv[c]) * inv * c_weight[c]);
-    for (int i = threadIdx.x; i < dr; i += blockDim.x) dst[rank + i] = from_f32<T>(turned(kv + rank, i));
+    for (int i = threadIdx.x; i < units; i += blockDim.x) turned(kv + rank, dst + rank, i);
   }
-  for (int idx = threadIdx.x; idx < H * dr; idx += blockDim.x) {
-    const int h = idx / dr, i = idx - h * dr;
-    const T* qp = q + (size_t)t * q_stride + (size_t)h * (dn + dr) + dn;
-    q_abs[((size_t)t * H + h) * kd + rank + i] = from_f32<T>(turned(qp, i));
+#pragma unroll 4
+  for (int idx = threadIdx.x; idx < H * units; idx += blockDim.x) {
+    const int h = idx / units, i = idx - h * units;
+    turned(q + (size_t)t * q_stride + (size_t)h * (dn + dr) + dn, q_abs + ((size_t)t * H + h) * kd + rank, i);
   }
 }
 
@@ -79,7 +84,7 @@ ARLE_API int arle_latent_prep(const void* q, int q_stride, const void* dkv, int 
                               void* cache, void* q_abs, int H, int dn, int dr, int rank, int num_tokens, cudaStream_t s) {
   if (num_tokens <= 0) return 0;
   if (H <= 0 || dn < 0 || dr < 0 || rank <= 0 || rot_dims < 0 || rot_dims > dr || (rot_dims & 1) || (pairing != 0 && pairing != 1)) return ARLE_E_BADARG;
-  const int threads = 128;
+  const int threads = H * dr >= 1024 ? 256 : 128;
   const size_t smem = (size_t)rot_dims / 2 * sizeof(float2);
   if (smem > 40 * 1024) return ARLE_E_UNSUPPORTED;
   if (dtype == 0)
@@ -362,19 +367,38 @@ __global__ void latent_merge_kernel(const float* __restrict__ part_o, const floa
                                     int rank, int splits) {
   pdl_launch_dependents();
   pdl_wait();
+  __shared__ float fac[64], inv_s;                // a part's factor (zero for a part without keys), and 1 / the sum
   const size_t th = blockIdx.x;
-  const float* ml = part_ml + th * splits * 2;
-  float M = -INFINITY;
-  for (int s = 0; s < splits; ++s)
-    if (ml[2 * s + 1] > 0.f) M = fmaxf(M, ml[2 * s]);
-  float den = 0.f;
-  for (int s = 0; s < splits; ++s)
-    if (ml[2 * s + 1] > 0.f) den += expf(ml[2 * s] - M) * ml[2 * s + 1];
-  const float inv = 1.0f / den;
+  if (threadIdx.x < 32) {
+    const float2* ml = reinterpret_cast<const float2*>(part_ml) + th * splits;
+    float2 p[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int s = threadIdx.x + 32 * i;
+      p[i] = s < splits ? ml[s] : make_float2(-INFINITY, 0.f);
+    }
+    const float M = warp_max(fmaxf(p[0].y > 0.f ? p[0].x : -INFINITY, p[1].y > 0.f ? p[1].x : -INFINITY));
+    float den = 0.f;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const float f = p[i].y > 0.f ? expf(p[i].x - M) : 0.f;
+      fac[threadIdx.x + 32 * i] = f;
+      den += f * p[i].y;
+    }
+    den = warp_sum(den);
+    if (threadIdx.x == 0) inv_s = 1.0f / den;
+  }
+  __syncthreads();
+  const float inv = inv_s;
   for (int c = threadIdx.x; c < rank; c += blockDim.x) {
     float acc = 0.f;
-    for (int s = 0; s < splits; ++s)
-      if (ml[2 * s + 1] > 0.f) acc = fmaf(expf(ml[2 * s] - M), part_o[(th * splits + s) * rank + c], acc);
+    const float* po = part_o + th * splits * rank + c;
+#pragma unroll 8
+    for (int s = 0; s < splits; ++s) {
+      const float f = fac[s];
+      const float v = po[(size_t)s * rank];       // a part without keys holds zeros
+      acc = fmaf(f, v, acc);
+    }
     out[th * rank + c] = __float2bfloat16_rn(acc * inv);
   }
 }
@@ -392,7 +416,7 @@ static int launch_latent_mma(const void* q_abs, void* out, float* part_o, float*
                 part_o, part_ml, (const __nv_bfloat16*)cache, positions, row_of_token, block_table, bt_stride, H, kd, page_size, scale,
                 window, splits);
   if (splits > 1)
-    launch_kernel(latent_merge_kernel, dim3(num_tokens * H), dim3(64 * R64 >= 256 ? 128 : 64), 0, s, 1, (const float*)part_o,
+    launch_kernel(latent_merge_kernel, dim3(num_tokens * H), dim3(64 * R64 >= 256 ? 256 : 64), 0, s, 1, (const float*)part_o,
                   (const float*)part_ml, (__nv_bfloat16*)out, 64 * R64, splits);
   return launch_status();
 }
@@ -404,7 +428,7 @@ ARLE_API int arle_latent_attention_mma(const void* q_abs, void* out, float* part
                                        int rank, int kd, int page_size, float scale, int window, int num_tokens, int splits,
                                        cudaStream_t s) {
   if (num_tokens <= 0) return 0;
-  if (H <= 0 || kd < rank || (kd - rank) % 16 || page_size <= 0 || splits < 1 || splits > 65535 || (H + 15) / 16 > 65535 ||
+  if (H <= 0 || kd < rank || (kd - rank) % 16 || page_size <= 0 || splits < 1 || splits > 65535 || splits > 64 || (H + 15) / 16 > 65535 ||
       (splits > 1 && (!part_o || !part_ml)))
     return ARLE_E_BADARG;
 #define ARLE_LAT(R) \

@@ -186,7 +186,14 @@ __global__ void input_conv_state_kernel(const float* __restrict__ x, float* __re
 
 namespace {
 
-int row_threads(int hidden, int per) { return hidden >= 2048 * per ? 512 : (hidden >= 512 * per ? 256 : 128); }
+// Threads a row: with few rows (a decode step) as many as the row has accesses, so that every loop over it is one round.
+int row_threads(int hidden, int per, int rows) {
+  if (rows <= 296) {
+    const int n = ((hidden + per - 1) / per + 31) / 32 * 32;
+    return n < 64 ? 64 : (n > 1024 ? 1024 : n);
+  }
+  return hidden >= 2048 * per ? 512 : (hidden >= 512 * per ? 256 : 128);
+}
 
 template <typename TA>
 int launch_layernorm(float* resid, const void* delta, const int* rows, const float* weight, void* out, int n_out, int hidden, float eps,
@@ -199,7 +206,7 @@ int launch_layernorm(float* resid, const void* delta, const int* rows, const flo
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
-  launch_kernel(kernel, dim3(n_out), dim3(row_threads(hidden, vec ? 4 : 1)), smem, s, 1, resid, (const TA*)delta, rows, weight, (TA*)out, hidden,
+  launch_kernel(kernel, dim3(n_out), dim3(row_threads(hidden, vec ? 4 : 1, n_out)), smem, s, 1, resid, (const TA*)delta, rows, weight, (TA*)out, hidden,
                 eps, write_resid);
   return launch_status();
 }
@@ -218,7 +225,7 @@ int launch_branch_layernorm(float* resid, const void* branch, int branch_stride,
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
-  launch_kernel(kernel, dim3(num_tokens), dim3(row_threads(hidden, vec ? 4 : 1)), smem, s, 1, resid, (const TA*)branch, branch_stride, weight,
+  launch_kernel(kernel, dim3(num_tokens), dim3(row_threads(hidden, vec ? 4 : 1, num_tokens)), smem, s, 1, resid, (const TA*)branch, branch_stride, weight,
                 (TA*)copy, hidden, eps, conv_w, taps, state, slot_stride, state_slots, (TA*)conv_out);
   return launch_status();
 }

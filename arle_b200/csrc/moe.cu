@@ -4,7 +4,7 @@
 //    stand in `groups` equal groups of neighbours, a group's score is the sum of its two largest choice scores (its one
 //    score when a group is a single expert), only experts of the `keep` best groups can be chosen (the others count as
 //    minus infinity); the `top` largest choice scores are chosen and weighted with s * scale (no renormalisation).
-//    Ties go to the lower index.  One thread per token, everything float32.  `mode` bit 0: the scores are a softmax
+//    Ties go to the lower index.  One thread per token (a warp per token where there are no groups), everything float32.  `mode` bit 0: the scores are a softmax
 //    over all experts instead of sigmoids; bit 1: a group's score is its largest choice score alone; bit 2: the sums z
 //    themselves are the choice scores and the weights are the softmax over the chosen sums alone (times scale).
 //  * moe_plan: sorts the step's (token, choice) pairs by expert (counts, offsets, a place for every pair) and lists
@@ -98,10 +98,73 @@ __global__ void moe_select_kernel(const float* __restrict__ z, int z_stride, con
   }
 }
 
+// The same without groups and softmax over all experts, for the usual sizes: a warp per token, a lane keeps the choice scores of
+// the experts lane, lane + 32, ...; the largest is found by exchanges, ties to the lower index.
+template <int PER>
+__global__ void moe_select_warp_kernel(const float* __restrict__ z, int z_stride, const float* __restrict__ correction, int E, int top, float scale,
+                                       int mode, int* __restrict__ ids, float* __restrict__ wts, int num_tokens) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (t >= num_tokens) return;
+  const float* zr = z + (size_t)t * z_stride;
+  float zv[PER], ch[PER];
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int e = lane + 32 * i;
+    zv[i] = e < E ? zr[e] : 0.f;
+    ch[i] = ((mode & 4) ? zv[i] : 1.0f / (1.0f + expf(-zv[i]))) + (correction && e < E ? correction[e] : 0.f);
+  }
+  unsigned taken = 0;                                   // this lane's experts that are chosen, or not experts at all
+#pragma unroll
+  for (int i = 0; i < PER; ++i)
+    if (lane + 32 * i >= E) taken |= 1u << i;
+  float cm = 0.f, cs = 0.f;
+  for (int it = 0; it < top; ++it) {
+    float bv = -INFINITY, bz = 0.f;
+    int bi = 0x7fffffff;
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+      if (!((taken >> i) & 1) && (bi == 0x7fffffff || ch[i] > bv)) {
+        bv = ch[i];
+        bz = zv[i];
+        bi = lane + 32 * i;
+      }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, bv, o), oz = __shfl_xor_sync(0xffffffffu, bz, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (oi != 0x7fffffff && (bi == 0x7fffffff || ov > bv || (ov == bv && oi < bi))) {
+        bv = ov;
+        bz = oz;
+        bi = oi;
+      }
+    }
+    if ((bi & 31) == lane) taken |= 1u << (bi >> 5);
+    if (it == 0) cm = bz;
+    const float w = (mode & 4) ? expf(bz - cm) : scale / (1.0f + expf(-bz));
+    cs += w;
+    if (lane == 0) {
+      ids[(size_t)t * top + it] = bi;
+      wts[(size_t)t * top + it] = w;
+    }
+  }
+  if ((mode & 4) && lane == 0)                          // softmax over the chosen sums, in choice order
+    for (int it = 0; it < top; ++it) wts[(size_t)t * top + it] = scale * (wts[(size_t)t * top + it] / cs);
+}
+
 ARLE_API int arle_moe_select(const float* z, int z_stride, const float* correction, float* scratch, int E, int top, int groups,
                              int keep, float scale, int mode, int* ids, float* wts, int num_tokens, cudaStream_t s) {
   if (num_tokens <= 0) return 0;
   if (E <= 0 || top <= 0 || groups <= 0 || E % groups || keep <= 0 || keep > groups || top > keep * (E / groups)) return ARLE_E_BADARG;
+  if (groups == 1 && !(mode & 1) && E <= 256 && !((mode & 4) && correction)) {
+    auto kernel = E <= 32 ? moe_select_warp_kernel<1> : E <= 64 ? moe_select_warp_kernel<2> : moe_select_warp_kernel<8>;
+    const int warps = num_tokens <= 592 ? 1 : 4;
+    launch_kernel(kernel, dim3((num_tokens + warps - 1) / warps), dim3(32 * warps), 0, s, 1, z, z_stride, correction, E, top, scale, mode, ids, wts,
+                  num_tokens);
+    return launch_status();
+  }
   launch_kernel(moe_select_kernel, dim3((num_tokens + 63) / 64), dim3(64), 0, s, 1, z, z_stride, correction, scratch, E, top, groups,
                 keep, scale, mode, ids, wts, num_tokens);
   return launch_status();
@@ -309,6 +372,10 @@ __device__ __forceinline__ void mma_tile_64x128(const __nv_bfloat16* __restrict_
         const int col = n0 + wn * 32 + nt * 8 + 2 * t4;
         if (m >= M) continue;
         TC* cp = C + (crow0 + m) * ldc + col;
+        if (sizeof(TC) == 2 && col + 1 < N && ((uintptr_t)cp & 3) == 0) {      // both numbers in one store
+          *reinterpret_cast<uint32_t*>(cp) = pack_bf16(finish(acc[mt][nt][2 * half], crow0 + m, col), finish(acc[mt][nt][2 * half + 1], crow0 + m, col + 1));
+          continue;
+        }
         if (col < N) cp[0] = from_f32<TC>(finish(acc[mt][nt][2 * half], crow0 + m, col));
         if (col + 1 < N) cp[1] = from_f32<TC>(finish(acc[mt][nt][2 * half + 1], crow0 + m, col + 1));
       }
@@ -440,22 +507,33 @@ ARLE_API int arle_moe_gemm(const void* A, int lda, const int* rows, const void* 
   return launch_status();
 }
 
-template <typename T>
+// VEC columns a thread, one column tile of a token a block: every load of a thread is asked for before the sum is formed.
+template <typename T, int VEC>
 __global__ void moe_combine_kernel(const T* __restrict__ y, int y_stride, const int* __restrict__ place_of_pair,
                                    const float* __restrict__ wts, int top, const T* __restrict__ shared, int shared_stride,
                                    const float* __restrict__ gate, int gate_stride, T* __restrict__ out, int out_stride, int width) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
-  float g = 1.f;
-  if (shared && gate) g = 1.0f / (1.0f + expf(-gate[(size_t)t * gate_stride]));
-  for (int c = threadIdx.x; c < width; c += blockDim.x) {
-    float acc = 0.f;
-    for (int k = 0; k < top; ++k)
-      acc = fmaf(wts ? wts[(size_t)t * top + k] : 1.f, to_f32(y[(size_t)place_of_pair[(size_t)t * top + k] * y_stride + c]), acc);
-    if (shared) acc = fmaf(g, to_f32(shared[(size_t)t * shared_stride + c]), acc);
-    out[(size_t)t * out_stride + c] = from_f32<T>(acc);
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
+  if (c >= width) return;
+  float acc[VEC], v[VEC];
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) acc[i] = 0.f;
+#pragma unroll 4
+  for (int k = 0; k < top; ++k) {
+    const float w = wts ? wts[(size_t)t * top + k] : 1.f;
+    load_vec<T, VEC>(y + (size_t)place_of_pair[(size_t)t * top + k] * y_stride + c, v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) acc[i] = fmaf(w, v[i], acc[i]);
   }
+  if (shared) {
+    const float g = gate ? 1.0f / (1.0f + expf(-gate[(size_t)t * gate_stride])) : 1.f;
+    load_vec<T, VEC>(shared + (size_t)t * shared_stride + c, v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) acc[i] = fmaf(g, v[i], acc[i]);
+  }
+  store_vec<T, VEC>(out + (size_t)t * out_stride + c, acc);
 }
 
 ARLE_API int arle_moe_combine(const void* y, int y_stride, const int* place_of_pair, const float* wts, int top, const void* shared,
@@ -463,12 +541,17 @@ ARLE_API int arle_moe_combine(const void* y, int y_stride, const int* place_of_p
                               int num_tokens, int width, cudaStream_t s) {
   if (num_tokens <= 0) return 0;
   if (width <= 0 || top <= 0) return ARLE_E_BADARG;
-  const int threads = width >= 1024 ? 256 : 128;
+  const int threads = 128, n = dtype == 0 ? 4 : 8;
+  const size_t eb = dtype == 0 ? 4 : 2;
+  const bool vec = width % n == 0 && y_stride % n == 0 && shared_stride % n == 0 && out_stride % n == 0 && ((uintptr_t)y % (n * eb)) == 0 &&
+                   ((uintptr_t)shared % (n * eb)) == 0 && ((uintptr_t)out % (n * eb)) == 0;
+  const int per = threads * (vec ? n : 1);
+  const dim3 grid(num_tokens, (width + per - 1) / per);
   if (dtype == 0)
-    launch_kernel(moe_combine_kernel<float>, dim3(num_tokens), dim3(threads), 0, s, 1, (const float*)y, y_stride, place_of_pair, wts, top,
+    launch_kernel(vec ? moe_combine_kernel<float, 4> : moe_combine_kernel<float, 1>, grid, dim3(threads), 0, s, 1, (const float*)y, y_stride, place_of_pair, wts, top,
                   (const float*)shared, shared_stride, gate, gate_stride, (float*)out, out_stride, width);
   else if (dtype == 1)
-    launch_kernel(moe_combine_kernel<__nv_bfloat16>, dim3(num_tokens), dim3(threads), 0, s, 1, (const __nv_bfloat16*)y, y_stride,
+    launch_kernel(vec ? moe_combine_kernel<__nv_bfloat16, 8> : moe_combine_kernel<__nv_bfloat16, 1>, grid, dim3(threads), 0, s, 1, (const __nv_bfloat16*)y, y_stride,
                   place_of_pair, wts, top, (const __nv_bfloat16*)shared, shared_stride, gate, gate_stride, (__nv_bfloat16*)out,
                   out_stride, width);
   else

@@ -108,6 +108,9 @@ class RoutedExperts(FeedForward):
             return dtype if dtype == torch.bfloat16 else (torch.float32 if any(t.dtype == torch.float32 for t in ts) else torch.bfloat16)
 
         rows = [tensors[self._name("router")]] + ([tensors[self._name("shared_gate")]] if s.shared_gate else [])
+        n = sum(r.shape[0] for r in rows)
+        if n % 8:                                       # the sums' rows on 16-byte boundaries
+            rows.append(torch.zeros((-n % 8, s.hidden_size), dtype=rows[0].dtype))
         self.w_router = torch.cat([r.to(device=device, dtype=kept(rows)) for r in rows], dim=0).contiguous()
         if s.correction:
             self.correction = tensors[self._name("correction")].to(device=device, dtype=torch.float32).contiguous()
