@@ -70,6 +70,7 @@ struct Fusion {
   __nv_bfloat16* xs;           // [M, ldxs]
   int ldxs;
   float* out_ss;               // [kSsRows][kSsSlots]: this launch fills every slot (zeros beyond its own CTAs)
+  int act;                     // 1: the sums go through the square of relu on their way to out (not with resid)
 };
 
 __device__ __forceinline__ void mbar_init(uint32_t bar, uint32_t count) {
@@ -272,6 +273,10 @@ __global__ void __launch_bounds__(kThreads, 1) skinny_gemm_kernel(
   };
   auto finish = [&](float v, int m, int n, bool valid, float r_old, float gn) -> float {
     if (!fu.resid) {
+      if (fu.act) {
+        v = fmaxf(v, 0.f);
+        v *= v;
+      }
       if (valid) store_out<OutT>(out + (size_t)m * ldo + n, v);
       return 0.f;
     }
@@ -557,7 +562,7 @@ ARLE_API int arle_gemm_skinny_gated(const void* x, int ldx, const void* W, int l
 // The same two products with the fusions described at the top of the file.
 //  in_ss (may be null): float32 [16][192], sums of squares of x's rows as left by an earlier launch
 //    with a sink; the sums of this product are multiplied by rsqrt(sum(in_ss[m, :]) * inv_width + eps).
-//  gated: 0 plain product; 1 the gate is silu; 2 the gate is the tanh form of gelu.
+//  gated: 0 plain product; 1 the gate is silu; 2 the gate is the tanh form of gelu; 3 no gate, out = max(sum, 0)^2.
 //  resid (may be null; not with gated): float32 [M, ldr].  When given, nothing goes to out (it may be
 //    null): resid[m, n] += sum, xs[m, n] = bfloat16(resid[m, n] * gamma[n]), and out_ss [16][192] gets
 //    the sums of squares of the new residual rows, every slot written.
@@ -565,6 +570,8 @@ ARLE_API int arle_gemm_skinny_fused(const void* x, int ldx, const void* W, int l
                                     int N, int K, int gated, const float* in_ss, float inv_width, float eps, float* resid,
                                     int ldr, const float* gamma, void* xs, int ldxs, float* out_ss, int* err,
                                     cudaStream_t s) {
-  Fusion fu{in_ss, inv_width, eps, resid, ldr, gamma, (__nv_bfloat16*)xs, ldxs, out_ss};
+  if (gated == 3 && resid) return ARLE_E_BADARG;
+  Fusion fu{in_ss, inv_width, eps, resid, ldr, gamma, (__nv_bfloat16*)xs, ldxs, out_ss, gated == 3 ? 1 : 0};
+  if (gated == 3) gated = 0;
   return skinny_entry(x, ldx, W, ldw, out, out_dtype, ldo, M, N, K, gated, fu, err, s);
 }

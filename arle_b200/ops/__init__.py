@@ -1703,6 +1703,16 @@ def square_relu(x, out) -> None:
     _check(library().arle_square_relu(_ptr(x), x.stride(0), _ptr(out), out.stride(0), _dt(x), T, width, _stream()), "square_relu")
 
 
+def gemm_square_relu(x, w: torch.Tensor, out: torch.Tensor) -> None:
+    """out = max(x . w^T, 0)^2: the first half of an ungated feed-forward.  Few rows of x take one launch of the
+    weight-streaming kernel (the activation on its float32 sums); otherwise the product is followed by the activation."""
+    if fused_gemm_supported(x, w) and skinny_gemm_supported(x, w, out) and w.shape[1] == x.shape[1] and tuple(out.shape) == (x.shape[0], w.shape[0]):
+        _fused_gemm(x, w, out, 3, None, None)
+        return
+    gemm(x, w, out)
+    square_relu(out, out)
+
+
 def layernorm(resid, delta, rows, weight, eps: float, out, write_resid: bool) -> None:
     """For output row i (source row r = rows[i], or i): x = resid[r] (+ delta[r]); resid[r] = x when write_resid; out[i] =
     (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps) * weight.  resid float32 [N, H]; delta and out in the activation type

@@ -136,8 +136,7 @@ class UngatedMlp(FeedForward):
         s = self.spec
         T = x.shape[0]
         act = ctx.ws.get("ffn_act", (T, s.intermediate_size), x.dtype)
-        ops.gemm(x, self.w_up, act)
-        ops.square_relu(act, act)
+        ops.gemm_square_relu(x, self.w_up, act)
         out = ctx.ws.get("ffn_out", (T, s.hidden_size), x.dtype)
         return None if ops.gemm(act, self.w_down, out, sink=sink) else out
 

@@ -613,6 +613,11 @@ def square_relu(x, out):
     out.copy_((x.to(F32).clamp(min=0.0) ** 2).to(out.dtype))
 
 
+def gemm_square_relu(x, w, out):
+    gemm(x, w, out)
+    square_relu(out, out)
+
+
 def _ln(x, weight, eps):
     d = x - x.mean(-1, keepdim=True)
     return d / torch.sqrt((d * d).mean(-1, keepdim=True) + eps) * weight
@@ -674,4 +679,4 @@ ALL = ("rotary_angles", "embedding", "rmsnorm", "residual_add", "gemm", "fused_g
        "dyt_norm", "gemm_heads", "latent_prep", "latent_attention", "decay_scan", "mlstm_gates", "mlstm_out", "ssm_gates", "conv_silu",
        "gated_group_norm", "moe_select", "moe_plan_size", "moe_plan", "moe_gemm", "moe_combine", "clamped_glu", "branch_norm_add",
        "attention_prep_post", "causal_conv", "rglru_scan", "delta_gates", "delta_scan", "branch_norm_add_norm", "rms_rows", "normed_sum",
-       "bias_add", "gate_mul", "square_relu", "layernorm", "branch_layernorm_add", "input_conv", "token_shift")
+       "bias_add", "gate_mul", "square_relu", "gemm_square_relu", "layernorm", "branch_layernorm_add", "input_conv", "token_shift")

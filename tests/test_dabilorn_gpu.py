@@ -310,6 +310,9 @@ def test_gates_per_number_and_the_square_of_relu(dtype):
         gate = torch.randn(T, n + 16, generator=g).to(dtype)[:, 8: n + 8] * 3
         _close(_both("gate_mul", [x, gate, torch.zeros(T, n, dtype=dtype)], [2]), dtype)
         _close(_both("square_relu", [x, torch.zeros(T, n, dtype=dtype)], [1]), dtype)
+    for M, K, N in ((1, 64, 40), (8, 4096, 136), (5, 8192, 24), (30, 96, 64), (3, 20, 12)):         # one CTA's sums, a cluster's, many rows
+        x, w = torch.randn(M, K, generator=g).to(dtype), (torch.randn(N, K, generator=g) * K ** -0.5).to(dtype)
+        _close(_both("gemm_square_relu", [x, w, torch.zeros(M, N, dtype=dtype)], [2]), dtype)
     for M, heads, K, N in ((7, 3, 24, 20), (130, 4, 64, 32), (5, 2, 9, 11), (70, 2, 256, 136)):
         x = torch.randn(M, heads, K, generator=g).to(dtype)
         w = (torch.randn(heads, N, K, generator=g) * K ** -0.5).to(dtype)
