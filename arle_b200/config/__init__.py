@@ -4,6 +4,7 @@ from .kolodra import KolodraConfig
 from .lasupel import LasupelConfig
 from .lukinex import LukinexConfig
 from .qwen3 import ConfigError, Qwen3Config
+from .virorax import ViroraxConfig
 from .zuderax import ZuderaxConfig
 from .registry import (UnknownArchitecture, config_class_for, config_from_dict, load_config,
                        register_architecture, registered_architectures)
@@ -14,6 +15,7 @@ register_architecture(ZuderaxConfig.architecture, ZuderaxConfig)
 register_architecture(LasupelConfig.architecture, LasupelConfig)
 register_architecture(LukinexConfig.architecture, LukinexConfig)
 register_architecture(DabilornConfig.architecture, DabilornConfig)
+register_architecture(ViroraxConfig.architecture, ViroraxConfig)
 
-__all__ = ["ModelSpec", "ScheduleEntry", "ConfigError", "Qwen3Config", "KolodraConfig", "ZuderaxConfig", "LasupelConfig", "LukinexConfig", "DabilornConfig", "UnknownArchitecture", "config_class_for",
+__all__ = ["ModelSpec", "ScheduleEntry", "ConfigError", "Qwen3Config", "KolodraConfig", "ZuderaxConfig", "LasupelConfig", "LukinexConfig", "DabilornConfig", "ViroraxConfig", "UnknownArchitecture", "config_class_for",
            "config_from_dict", "load_config", "register_architecture", "registered_architectures"]

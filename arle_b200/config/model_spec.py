@@ -16,10 +16,12 @@ class ScheduleEntry:
     ``block`` indexes ``ModelSpec.blocks`` (the same block, hence the same
     weights, may be named by several entries).  ``keys_of`` is None when the run
     keeps a cache of its own, or the index of an earlier schedule entry whose
-    cache this run reads instead of writing one."""
+    cache this run reads instead of writing one.  ``add_embedding``: the residual as it was before
+    the first run is added to it right before this one."""
 
     block: int
     keys_of: Optional[int] = None
+    add_embedding: bool = False               # the embedding output is added to the residual right before this run
 
 
 @dataclass(frozen=True)
@@ -41,6 +43,8 @@ class ModelSpec:
     logit_cap: Optional[float] = None         # logits <- cap * tanh(logits / cap)
     logit_scale: float = 1.0                  # logits <- logits * this (before a cap)
     embed_norm: Optional[object] = None       # norm spec: the embedding row is normed before the first block
+    position_name: Optional[str] = None       # a learned vector per position, [max_position, hidden], added to the (scaled) embedding row
+    branch_scale: float = 1.0                 # every sublayer's output is multiplied by this before it is added to the residual
 
     def validate(self) -> None:
         if not self.blocks or not self.schedule:

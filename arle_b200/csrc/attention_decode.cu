@@ -45,7 +45,7 @@ __global__ void __launch_bounds__(kThreads) paged_decode_kernel(
     const __nv_bfloat16* __restrict__ k_cache, const __nv_bfloat16* __restrict__ v_cache,
     const int* __restrict__ q_indptr, const int* __restrict__ kv_lens, const int* __restrict__ block_table,
     int bt_stride, float* __restrict__ part_o, float* __restrict__ part_ml, int* __restrict__ counters, int nq, int nkv,
-    int page_size, int ps_shift, float scale_log2, float sink_log2, int window, int splits, int keep_first, float cap_arg,
+    int page_size, int ps_shift, float scale_log2, HeadTail<__nv_bfloat16> tail, int window, int splits, int keep_first, float cap_arg,
     float scale_over_cap, int chunk_arg, const float* __restrict__ pb) {
   pdl_launch_dependents();
   pdl_wait();
@@ -289,7 +289,7 @@ __global__ void __launch_bounds__(kThreads) paged_decode_kernel(
     const int head = kvh * G + row;
     if (SIG) L = 1.f;
     if (splits == 1) {
-      out[((size_t)t * nq + head) * HD + d] = __float2bfloat16_rn(SIG ? O : O / (L + exp2f(sink_log2 - M)));      // sink_log2 -inf: no sink
+      out[((size_t)t * nq + head) * HD + d] = __float2bfloat16_rn((SIG ? O : O / (L + exp2f(tail.sink_log2(head) - M))) * tail.gate_of(t, head));
     } else {
       const size_t pidx = ((size_t)r * nq + head) * splits + split;
       part_o[pidx * HD + d] = O;
@@ -332,7 +332,7 @@ __global__ void __launch_bounds__(kThreads) paged_decode_kernel(
       fac[tid * 64 + sp] = f;
       L += l * f;
     }
-    invl[tid] = SIG ? 1.0f : 1.0f / (L + exp2f(sink_log2 - M));
+    invl[tid] = (SIG ? 1.0f : 1.0f / (L + exp2f(tail.sink_log2(kvh * G + tid) - M))) * tail.gate_of(t, kvh * G + tid);
   }
   __syncthreads();
   for (int i = tid; i < G * HD; i += kThreads) {
@@ -351,7 +351,7 @@ __global__ void __launch_bounds__(kThreads) paged_decode_kernel(
 template <int HD>
 int launch_decode(const void* q, int q_row_stride, void* out, const void* k_cache, const void* v_cache,
                   const int* q_indptr, const int* kv_lens, const int* block_table, int bt_stride, float* part_o,
-                  float* part_ml, int* counters, int nq, int nkv, int page_size, float scale, float sink, int window, int rows,
+                  float* part_ml, int* counters, int nq, int nkv, int page_size, float scale, HeadTail<__nv_bfloat16> tail, int window, int rows,
                   int splits, int keep_first, float softcap, int chunk, const float* pb, cudaStream_t s) {
   constexpr int ROW = HD + 8;
   int ps_shift = -1;
@@ -372,7 +372,7 @@ int launch_decode(const void* q, int q_row_stride, void* out, const void* k_cach
   launch_kernel(kernel, dim3(grid), dim3(kThreads), smem, s, 1, 
       (const __nv_bfloat16*)q, q_row_stride, (__nv_bfloat16*)out, (const __nv_bfloat16*)k_cache,
       (const __nv_bfloat16*)v_cache, q_indptr, kv_lens, block_table, bt_stride, part_o, part_ml, counters, nq, nkv,
-      page_size, ps_shift, scale * 1.4426950408889634f, sink * 1.4426950408889634f, window, splits, window > 0 ? keep_first : 0,
+      page_size, ps_shift, scale * 1.4426950408889634f, tail, window, splits, window > 0 ? keep_first : 0,
       softcap > 0.f ? softcap * 1.4426950408889634f : 0.f, softcap > 0.f ? scale / softcap : 0.f, chunk, pb);
   return launch_status();
 }
@@ -384,8 +384,8 @@ int launch_decode(const void* q, int q_row_stride, void* out, const void* k_cach
 ARLE_API int arle_paged_attention_decode(const void* q, int q_row_stride, void* out, const void* k_cache,
                                          const void* v_cache, const int* q_indptr, const int* kv_lens,
                                          const int* block_table, int bt_stride, float* part_o, float* part_ml,
-                                         int* counters, int nq, int nkv, int hd, int page_size, float scale, float sink, int window,
-                                         int rows, int splits, int keep_first, float softcap, int chunk, const float* pb, cudaStream_t s) {
+                                         int* counters, int nq, int nkv, int hd, int page_size, float scale, const float* sinks,
+                                         const void* gate, int gate_stride, int window, int rows, int splits, int keep_first, float softcap, int chunk, const float* pb, cudaStream_t s) {
   if (rows <= 0) return 0;
   if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || nq / nkv > 16 || page_size <= 0) return ARLE_E_UNSUPPORTED;
   if (splits < 1 || splits > 64 || nkv > 65535) return ARLE_E_UNSUPPORTED;
@@ -393,11 +393,12 @@ ARLE_API int arle_paged_attention_decode(const void* q, int q_row_stride, void* 
   if ((q_row_stride % 8) != 0) return ARLE_E_UNSUPPORTED;     // 16-byte loads of q rows
   if (keep_first < 0 || softcap < 0.f || chunk < 0 || (chunk > 0 && window > 0)) return ARLE_E_BADARG;
   if (pb ? (keep_first > 0 || softcap > 0.f) : chunk > 0) return ARLE_E_UNSUPPORTED;      // the sigmoid form has neither; only it has chunks
+  const HeadTail<__nv_bfloat16> tail{sinks, (const __nv_bfloat16*)gate, gate_stride};
   if (hd == 128)
     return launch_decode<128>(q, q_row_stride, out, k_cache, v_cache, q_indptr, kv_lens, block_table, bt_stride, part_o,
-                              part_ml, counters, nq, nkv, page_size, scale, sink, window, rows, splits, keep_first, softcap, chunk, pb, s);
+                              part_ml, counters, nq, nkv, page_size, scale, tail, window, rows, splits, keep_first, softcap, chunk, pb, s);
   if (hd == 64)
     return launch_decode<64>(q, q_row_stride, out, k_cache, v_cache, q_indptr, kv_lens, block_table, bt_stride, part_o,
-                             part_ml, counters, nq, nkv, page_size, scale, sink, window, rows, splits, keep_first, softcap, chunk, pb, s);
+                             part_ml, counters, nq, nkv, page_size, scale, tail, window, rows, splits, keep_first, softcap, chunk, pb, s);
   return ARLE_E_UNSUPPORTED;
 }

@@ -49,7 +49,7 @@ constexpr int kConsumers = kConsumerWarps * 32;
 constexpr int kThreads = kConsumers + 64;          // two producer warps: keys, values
 constexpr int kTile = 64;                          // keys per unit
 constexpr int kMaxStages = 8;
-constexpr int kStaticSmem = 2 * kMaxStages * 8 + 32;   // bytes of __shared__ variables in the kernel: the barriers, six words
+constexpr int kStaticSmem = 2 * kMaxStages * 8 + 32 + 128;   // bytes of __shared__ variables in the kernel: the barriers, six words, 32 numbers
 
 __device__ __forceinline__ void mbar_arrive_one(uint32_t bar) {
   asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(bar) : "memory");
@@ -86,20 +86,23 @@ struct Prep {
   const float* q_weight;        // [HD] or null: no norm
   const float* k_weight;
   float eps;
-  const float* inv_freq;        // [HD / 2] or null: no rotation
+  const float* inv_freq;        // [rotary_dim / 2] or null: no rotation
+  int rotary_dim;               // the first numbers of a head that turn; a multiple of 2 HD / 32
+  const float* bias;            // float32 [(nq + 2 nkv) * HD] added to the projection's sums, or null
   __nv_bfloat16* k_cache;
   __nv_bfloat16* v_cache;
 };
 
 // One head of HD elements, lane l holding elements l * HD / 32 ..: RMSNorm over the head (if w), then the
-// half-split rotation by pos (if inv_freq); the same arithmetic, in the same order, as the preparation kernel.
+// half-split rotation of the first rotary_dim elements by pos (if inv_freq); the same arithmetic, in the same order, as the
+// preparation kernel.  A bias (if given) is added before everything else.
 template <int HD>
-__device__ __forceinline__ void prep_head(const __nv_bfloat16* src, const float* w, float eps, const float* inv_freq,
-                                          float pos, int lane, __nv_bfloat16* dst) {
+__device__ __forceinline__ void prep_head(const __nv_bfloat16* src, const float* bias, const float* w, float eps, const float* inv_freq,
+                                          int rotary_dim, float pos, int lane, __nv_bfloat16* dst) {
   constexpr int VE = HD / 32;
   float x[VE];
 #pragma unroll
-  for (int i = 0; i < VE; ++i) x[i] = __bfloat162float(src[lane * VE + i]);
+  for (int i = 0; i < VE; ++i) x[i] = __bfloat162float(src[lane * VE + i]) + (bias ? bias[lane * VE + i] : 0.f);
   if (w) {
     float ss = 0.f;
 #pragma unroll
@@ -109,14 +112,18 @@ __device__ __forceinline__ void prep_head(const __nv_bfloat16* src, const float*
 #pragma unroll
     for (int i = 0; i < VE; ++i) x[i] = x[i] * inv * w[lane * VE + i];
   }
+  const int hl = rotary_dim / (2 * VE);                   // lanes that hold the first halves of the pairs; the next hl hold the second
+  const bool first = lane < hl, turns = lane < 2 * hl;
 #pragma unroll
   for (int i = 0; i < VE; ++i) {
     float o = x[i];
     if (inv_freq) {
-      const float other = __shfl_xor_sync(0xffffffffu, x[i], 16);
-      float sn, cs;
-      sincosf(pos * inv_freq[(lane & 15) * VE + i], &sn, &cs);
-      o = lane < 16 ? x[i] * cs - other * sn : other * sn + x[i] * cs;
+      const float other = __shfl_sync(0xffffffffu, x[i], first ? lane + hl : turns ? lane - hl : lane);
+      if (turns) {
+        float sn, cs;
+        sincosf(pos * inv_freq[(first ? lane : lane - hl) * VE + i], &sn, &cs);
+        o = first ? x[i] * cs - other * sn : other * sn + x[i] * cs;
+      }
     }
     dst[lane * VE + i] = __float2bfloat16_rn(o);
   }
@@ -266,7 +273,7 @@ __global__ void __launch_bounds__(kThreads, 1) decode_stream_kernel(
     const __nv_bfloat16* __restrict__ q, int q_row_stride, __nv_bfloat16* __restrict__ out,
     const int* __restrict__ q_indptr, const int* __restrict__ kv_lens, const int* __restrict__ block_table, int bt_stride,
     float* __restrict__ part_o, float* __restrict__ part_ml, int* __restrict__ counters, int R, int nq, int nkv,
-    int bt_width, int page_size, int ps_shift, float scale_log2, float sink_log2, int window, int stages, Prep prep, const int* __restrict__ plan,
+    int bt_width, int page_size, int ps_shift, float scale_log2, HeadTail<__nv_bfloat16> tail, int window, int stages, Prep prep, const int* __restrict__ plan,
     int* __restrict__ err) {
   pdl_launch_dependents();
   pdl_wait();
@@ -288,6 +295,7 @@ __global__ void __launch_bounds__(kThreads, 1) decode_stream_kernel(
   __nv_bfloat16* heads = reinterpret_cast<__nv_bfloat16*>(mlv + kConsumerWarps * 16 + ((3 * R + 1 + 3) & ~3));   // [18][HD]: 16 query heads, new key, new value
   __shared__ __align__(8) uint64_t full[kMaxStages], empty[kMaxStages];
   __shared__ int abort_flag, is_last;
+  __shared__ float tail_sink[16], tail_gate[16];            // of the piece's query heads: the sink's score (log2 units), the output gate
   __shared__ int own_row, own_first, own_k, by_pair;        // the CTA's place when pairs are shared out whole (below)
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -422,6 +430,8 @@ __global__ void __launch_bounds__(kThreads, 1) decode_stream_kernel(
       const int ntile = pe - u;
       const int t = tok[r];
 
+      // read behind the merge's barrier, written behind the last piece's
+      if (tid < G) tail_sink[tid] = tail.sink_log2(kvh * G + tid), tail_gate[tid] = tail.gate_of(t, kvh * G + tid);
       // the G query heads of this kv head as the A operand: rows 0..G-1 of 16, the rest zero
       uint32_t qa[HD / 16][4];
       const bool has_last = prep.on && pair_begin + T <= u1;      // this piece holds the pair's last tile, hence the new key
@@ -431,11 +441,14 @@ __global__ void __launch_bounds__(kThreads, 1) decode_stream_kernel(
         const float pos = (float)(kv_len - 1);
         for (int hh = warp; hh < G + (has_last ? 2 : 0); hh += kConsumerWarps) {
           if (hh < G)
-            prep_head<HD>(row + (size_t)(kvh * G + hh) * HD, prep.q_weight, prep.eps, prep.inv_freq, pos, lane, heads + hh * HD);
+            prep_head<HD>(row + (size_t)(kvh * G + hh) * HD, prep.bias ? prep.bias + (kvh * G + hh) * HD : nullptr, prep.q_weight, prep.eps,
+                          prep.inv_freq, prep.rotary_dim, pos, lane, heads + hh * HD);
           else if (hh == G)
-            prep_head<HD>(row + (size_t)(nq + kvh) * HD, prep.k_weight, prep.eps, prep.inv_freq, pos, lane, heads + 16 * HD);
+            prep_head<HD>(row + (size_t)(nq + kvh) * HD, prep.bias ? prep.bias + (nq + kvh) * HD : nullptr, prep.k_weight, prep.eps,
+                          prep.inv_freq, prep.rotary_dim, pos, lane, heads + 16 * HD);
           else
-            prep_head<HD>(row + (size_t)(nq + nkv + kvh) * HD, nullptr, 0.f, nullptr, 0.f, lane, heads + 17 * HD);
+            prep_head<HD>(row + (size_t)(nq + nkv + kvh) * HD, prep.bias ? prep.bias + (nq + nkv + kvh) * HD : nullptr, nullptr, 0.f, nullptr, 0,
+                          0.f, lane, heads + 17 * HD);
         }
         consumer_sync();
       }
@@ -611,7 +624,7 @@ __global__ void __launch_bounds__(kThreads, 1) decode_stream_kernel(
           O += mo[(w * G + row) * HD + d] * f;
         }
         if (pieces == 1) {
-          out[((size_t)t * nq + kvh * G + row) * HD + d] = __float2bfloat16_rn(O / (L + exp2f(sink_log2 - M)));   // sink_log2 -inf: no sink
+          out[((size_t)t * nq + kvh * G + row) * HD + d] = __float2bfloat16_rn(O / (L + exp2f(tail_sink[row] - M)) * tail_gate[row]);
         } else {
           part_o[((size_t)slot * G + row) * HD + d] = O;
           if (d == 0) {
@@ -660,7 +673,7 @@ __global__ void __launch_bounds__(kThreads, 1) decode_stream_kernel(
                 }
               }
             }
-            const float inv = 1.0f / (L + exp2f(sink_log2 - M));
+            const float inv = tail_gate[row] / (L + exp2f(tail_sink[row] - M));
             *reinterpret_cast<__nv_bfloat162*>(out + ((size_t)t * nq + kvh * G + row) * HD + d) = __floats2bfloat162_rn(O0 * inv, O1 * inv);
           }
         }
@@ -682,7 +695,7 @@ size_t fixed_smem(int G, int hd, int ctas, int R) {
 template <int HD>
 int launch_stream(const CUtensorMap& mk, const CUtensorMap& mv, const void* q, int q_row_stride, void* out,
                   const int* q_indptr, const int* kv_lens, const int* block_table, int bt_stride, float* part_o,
-                  float* part_ml, int* counters, int rows, int nq, int nkv, int bt_width, int page_size, float scale, float sink, int window,
+                  float* part_ml, int* counters, int rows, int nq, int nkv, int bt_width, int page_size, float scale, HeadTail<__nv_bfloat16> tail, int window,
                   int ctas, const Prep& prep, const int* plan, int* err, cudaStream_t s) {
   int ps_shift = -1;
   if ((page_size & (page_size - 1)) == 0)
@@ -709,7 +722,7 @@ int launch_stream(const CUtensorMap& mk, const CUtensorMap& mv, const void* q, i
   if (e != cudaSuccess) return (int)e;
   e = launch_kernel(decode_stream_kernel<HD>, dim3(ctas), dim3(kThreads), smem, s, 1, mk, mv, (const __nv_bfloat16*)q,
                     q_row_stride, (__nv_bfloat16*)out, q_indptr, kv_lens, block_table, bt_stride, part_o, part_ml, counters,
-                    rows, nq, nkv, bt_width, page_size, ps_shift, scale * 1.4426950408889634f, sink * 1.4426950408889634f, window, stages, prep, plan, err);
+                    rows, nq, nkv, bt_width, page_size, ps_shift, scale * 1.4426950408889634f, tail, window, stages, prep, plan, err);
   if (e != cudaSuccess) return (int)e;
   return launch_status();
 }
@@ -720,9 +733,11 @@ ARLE_API int arle_paged_attention_decode_stream_prep(const void* q, int q_row_st
                                                      const void* v_cache, long long cache_pages, const int* q_indptr,
                                                      const int* kv_lens, const int* block_table, int bt_stride, int bt_width,
                                                      float* part_o, float* part_ml, int* counters, int nq, int nkv, int hd,
-                                                     int page_size, float scale, float sink, int window, int rows, int ctas, int fused,
+                                                     int page_size, float scale, const float* sinks, const void* gate, int gate_stride,
+                                                     int window, int rows, int ctas, int fused,
                                                      const int* slot_mapping, const float* q_weight, const float* k_weight,
-                                                     float eps, const float* inv_freq, const int* plan, int* err, cudaStream_t s);
+                                                     float eps, const float* inv_freq, int rotary_dim, const float* bias, const int* plan, int* err,
+                                                     cudaStream_t s);
 
 // k_cache / v_cache: [cache_pages, nkv, page_size, hd].  Scratch: part_o float32
 // [(ctas + rows * nkv) * (nq / nkv) * hd], part_ml float32 [(ctas + rows * nkv) * (nq / nkv) * 2], counters
@@ -733,12 +748,13 @@ ARLE_API int arle_paged_attention_decode_stream(const void* q, int q_row_stride,
                                                 const void* v_cache, long long cache_pages, const int* q_indptr,
                                                 const int* kv_lens, const int* block_table, int bt_stride, int bt_width,
                                                 float* part_o, float* part_ml, int* counters, int nq, int nkv, int hd,
-                                                int page_size, float scale, float sink, int window, int rows, int ctas, int* err,
+                                                int page_size, float scale, const float* sinks, const void* gate, int gate_stride,
+                                                int window, int rows, int ctas, int* err,
                                                 cudaStream_t s) {
   return arle_paged_attention_decode_stream_prep(q, q_row_stride, out, k_cache, v_cache, cache_pages, q_indptr, kv_lens,
                                                  block_table, bt_stride, bt_width, part_o, part_ml, counters, nq, nkv, hd,
-                                                 page_size, scale, sink, window, rows, ctas, 0, nullptr, nullptr, nullptr, 0.f, nullptr,
-                                                 nullptr, err, s);
+                                                 page_size, scale, sinks, gate, gate_stride, window, rows, ctas, 0, nullptr, nullptr, nullptr, 0.f,
+                                                 nullptr, 0, nullptr, nullptr, err, s);
 }
 
 // Ints of a step's plan for this many rows and CTAs.
@@ -758,19 +774,25 @@ ARLE_API int arle_decode_stream_plan(const int* q_indptr, const int* kv_lens, co
 
 // The same with the fused preparation (fused != 0): q is the raw projection output of the step's tokens
 // ([q heads | k heads | v heads] per row, stride q_row_stride), every row a decoded token at position
-// kv_len - 1; q_weight / k_weight (float32 [hd], may be null: no norm), inv_freq (float32 [hd / 2], may be null: no
-// rotation; otherwise the whole head is rotated), slot_mapping int32 [tokens].  The new keys and values are
+// kv_len - 1; q_weight / k_weight (float32 [hd], may be null: no norm), inv_freq (float32 [rotary_dim / 2], may be null: no
+// rotation), rotary_dim (the first numbers of a head that turn: a multiple of hd / 16), bias (float32 [(nq + 2 nkv) * hd], added to q, k
+// and v first; may be null), slot_mapping int32 [tokens].  The new keys and values are
 // stored into the cache by this launch.
 ARLE_API int arle_paged_attention_decode_stream_prep(const void* q, int q_row_stride, void* out, const void* k_cache,
                                                      const void* v_cache, long long cache_pages, const int* q_indptr,
                                                      const int* kv_lens, const int* block_table, int bt_stride, int bt_width,
                                                      float* part_o, float* part_ml, int* counters, int nq, int nkv, int hd,
-                                                     int page_size, float scale, float sink, int window, int rows, int ctas, int fused,
+                                                     int page_size, float scale, const float* sinks, const void* gate, int gate_stride,
+                                                     int window, int rows, int ctas, int fused,
                                                      const int* slot_mapping, const float* q_weight, const float* k_weight,
-                                                     float eps, const float* inv_freq, const int* plan, int* err, cudaStream_t s) {
+                                                     float eps, const float* inv_freq, int rotary_dim, const float* bias, const int* plan, int* err,
+                                                     cudaStream_t s) {
   if (rows <= 0) return 0;
   if (fused && (!slot_mapping || ((uintptr_t)q & 15) || (q_row_stride % 8) != 0)) return ARLE_E_BADARG;
-  const Prep prep{fused ? 1 : 0, slot_mapping, q_weight, k_weight, eps, inv_freq, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache};
+  if (rotary_dim < 0 || rotary_dim > hd || (rotary_dim % (hd / 16 > 0 ? hd / 16 : 1)) != 0) return ARLE_E_UNSUPPORTED;
+  const Prep prep{fused ? 1 : 0, slot_mapping, q_weight, k_weight, eps, rotary_dim ? inv_freq : nullptr, rotary_dim, bias, (__nv_bfloat16*)k_cache,
+                  (__nv_bfloat16*)v_cache};
+  const HeadTail<__nv_bfloat16> tail{sinks, (const __nv_bfloat16*)gate, gate_stride};
   if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || nq / nkv > 16 || page_size <= 0 || page_size % 16 != 0) return ARLE_E_UNSUPPORTED;
   if (ctas < 1 || ctas > 1024 || rows > 2048 || !part_o || !part_ml || !counters) return ARLE_E_BADARG;
   if ((q_row_stride % 2) != 0 || ((uintptr_t)q & 3) || ((uintptr_t)k_cache & 15) || ((uintptr_t)v_cache & 15)) return ARLE_E_UNSUPPORTED;
@@ -786,7 +808,7 @@ ARLE_API int arle_paged_attention_decode_stream_prep(const void* q, int q_row_st
   if (rc) return rc;
   if (hd == 128)
     return launch_stream<128>(mk, mv, q, q_row_stride, out, q_indptr, kv_lens, block_table, bt_stride, part_o, part_ml, counters,
-                              rows, nq, nkv, bt_width, page_size, scale, sink, window, ctas, prep, plan, err, s);
+                              rows, nq, nkv, bt_width, page_size, scale, tail, window, ctas, prep, plan, err, s);
   return launch_stream<64>(mk, mv, q, q_row_stride, out, q_indptr, kv_lens, block_table, bt_stride, part_o, part_ml, counters,
-                           rows, nq, nkv, bt_width, page_size, scale, sink, window, ctas, prep, plan, err, s);
+                           rows, nq, nkv, bt_width, page_size, scale, tail, window, ctas, prep, plan, err, s);
 }

@@ -13,7 +13,8 @@
 //
 // Values may have another width than keys (vd; the value cache is [page][kv_head][slot][vd]).  With a sink the
 // softmax has one more term in its denominator, exp(sink_logit), that carries no value:
-// p_j = exp(s_j) / (exp(sink_logit) + sum exp(s_j)).
+// p_j = exp(s_j) / (exp(sink_logit) + sum exp(s_j)), one sink score per query head.  With a gate, head h's output is
+// multiplied by sigmoid(gate[t, h]).
 //
 // With sigmoid weights (pb: one number per query head, added to the scaled score) there is no softmax: a visible key's weight
 // is sigmoid(score + pb[h]) as it is, and the values' weighted sum is the result.  With chunks a query sees only the keys of
@@ -30,8 +31,8 @@ __global__ void paged_attention_plain_kernel(const T* __restrict__ q, int q_row_
                                              const int* __restrict__ positions,
                                              const int* __restrict__ row_of_token,
                                              const int* __restrict__ block_table, int bt_stride, int nq,
-                                             int nkv, int hd, int vd, int page_size, float scale, int window, int has_sink,
-                                             float sink_logit, int keep_first, float softcap, int chunk, const float* __restrict__ pb) {
+                                             int nkv, int hd, int vd, int page_size, float scale, int window,
+                                             HeadTail<T> tail, int keep_first, float softcap, int chunk, const float* __restrict__ pb) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float qs[256];
@@ -105,6 +106,8 @@ __global__ void paged_attention_plain_kernel(const T* __restrict__ q, int q_row_
     if (d < vd) acc_s[w][d] = acc[i];
   }
   __syncthreads();
+  const bool has_sink = tail.sinks != nullptr;
+  const float sink_logit = has_sink ? tail.sinks[h] : 0.f;
   float mm = has_sink ? sink_logit : m_s[0];
   for (int i = has_sink ? 0 : 1; i < kAttnWarps; ++i) mm = fmaxf(mm, m_s[i]);
   float f[kAttnWarps], ll = has_sink ? expf(sink_logit - mm) : 0.f;
@@ -113,11 +116,12 @@ __global__ void paged_attention_plain_kernel(const T* __restrict__ q, int q_row_
     ll += l_s[i] * f[i];
   }
   if (pb) ll = 1.f;
+  const float gate = tail.gate_of(t, h);
   T* op = out + ((size_t)t * nq + h) * vd;
   for (int d = threadIdx.x; d < vd; d += blockDim.x) {
     float o = 0.f;
     for (int i = 0; i < kAttnWarps; ++i) o += acc_s[i][d] * f[i];
-    op[d] = from_f32<T>(o / ll);
+    op[d] = from_f32<T>(o / ll * gate);
   }
 }
 
@@ -125,9 +129,10 @@ ARLE_API int arle_paged_attention_plain(const void* q, int q_row_stride, void* o
                                         const void* v_cache, int dtype, const int* positions,
                                         const int* row_of_token, const int* block_table, int bt_stride,
                                         int nq, int nkv, int hd, int vd, int page_size, float scale, int window,
-                                        int has_sink, float sink_logit, int keep_first, float softcap, int chunk, const float* pb, int num_tokens, cudaStream_t s) {
+                                        const float* sinks, const void* gate, int gate_stride, int keep_first, float softcap, int chunk, const float* pb,
+                                        int num_tokens, cudaStream_t s) {
   if (num_tokens <= 0) return 0;
-  if (chunk < 0 || (chunk > 0 && window > 0) || (pb && has_sink)) return ARLE_E_BADARG;
+  if (chunk < 0 || (chunk > 0 && window > 0) || (pb && sinks)) return ARLE_E_BADARG;
   if (vd <= 0 || vd > 256) return ARLE_E_UNSUPPORTED;
   if (hd <= 0 || hd > 256 || nq <= 0 || nkv <= 0 || nq % nkv != 0 || page_size <= 0) return ARLE_E_UNSUPPORTED;
   if (nq > 65535) return ARLE_E_UNSUPPORTED;
@@ -136,12 +141,13 @@ ARLE_API int arle_paged_attention_plain(const void* q, int q_row_stride, void* o
   if (dtype == 0)
     launch_kernel(paged_attention_plain_kernel<float>, dim3(grid), dim3(kAttnWarps * 32), 0, s, 1, 
         (const float*)q, q_row_stride, (float*)out, (const float*)k_cache, (const float*)v_cache, positions,
-        row_of_token, block_table, bt_stride, nq, nkv, hd, vd, page_size, scale, window, has_sink, sink_logit, keep_first, softcap, chunk, pb);
+        row_of_token, block_table, bt_stride, nq, nkv, hd, vd, page_size, scale, window,
+        HeadTail<float>{sinks, (const float*)gate, gate_stride}, keep_first, softcap, chunk, pb);
   else if (dtype == 1)
     launch_kernel(paged_attention_plain_kernel<__nv_bfloat16>, dim3(grid), dim3(kAttnWarps * 32), 0, s, 1, 
         (const __nv_bfloat16*)q, q_row_stride, (__nv_bfloat16*)out, (const __nv_bfloat16*)k_cache,
         (const __nv_bfloat16*)v_cache, positions, row_of_token, block_table, bt_stride, nq, nkv, hd, vd,
-        page_size, scale, window, has_sink, sink_logit, keep_first, softcap, chunk, pb);
+        page_size, scale, window, HeadTail<__nv_bfloat16>{sinks, (const __nv_bfloat16*)gate, gate_stride}, keep_first, softcap, chunk, pb);
   else
     return ARLE_E_BADARG;
   return launch_status();

@@ -39,7 +39,7 @@ __global__ void __launch_bounds__(kThreads, 3) paged_prefill_kernel(
     const __nv_bfloat16* __restrict__ q, int q_row_stride, __nv_bfloat16* __restrict__ out,
     const __nv_bfloat16* __restrict__ k_cache, const __nv_bfloat16* __restrict__ v_cache,
     const int* __restrict__ q_indptr, const int* __restrict__ kv_lens, const int* __restrict__ block_table,
-    int bt_stride, int nq, int nkv, int page_size, int ps_shift, float scale_log2, float sink_log2, int window, int skip_single,
+    int bt_stride, int nq, int nkv, int page_size, int ps_shift, float scale_log2, HeadTail<__nv_bfloat16> tail, int window, int skip_single,
     int keep_first_arg, float cap_arg, float scale_over_cap, int chunk_arg, const float* __restrict__ pb) {
   pdl_launch_dependents();
   pdl_wait();
@@ -259,9 +259,11 @@ __global__ void __launch_bounds__(kThreads, 3) paged_prefill_kernel(
   l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
-  // a sink's term in the denominator (its score in log2 units; -inf: none, and the sums stay as they are)
-  const float inv0 = SIG ? 1.0f : 1.0f / (l0 + exp2f(sink_log2 - m0)), inv1 = SIG ? 1.0f : 1.0f / (l1 + exp2f(sink_log2 - m1));
+  // a sink's term in the denominator (its score in log2 units; -inf: none, and the sums stay as they are), the head's gate
+  const float sink_log2 = tail.sink_log2(h);
   const int row0 = mbeg + warp * 16 + g, row1 = row0 + 8;
+  const float inv0 = (SIG ? 1.0f : 1.0f / (l0 + exp2f(sink_log2 - m0))) * (row0 < qlen ? tail.gate_of(t0 + row0, h) : 0.f);
+  const float inv1 = (SIG ? 1.0f : 1.0f / (l1 + exp2f(sink_log2 - m1))) * (row1 < qlen ? tail.gate_of(t0 + row1, h) : 0.f);
 #pragma unroll
   for (int i = 0; i < HD / 8; ++i) {
     if (row0 < qlen) {
@@ -278,7 +280,7 @@ __global__ void __launch_bounds__(kThreads, 3) paged_prefill_kernel(
 template <int HD>
 int launch_prefill(const void* q, int q_row_stride, void* out, const void* k_cache, const void* v_cache,
                    const int* q_indptr, const int* kv_lens, const int* block_table, int bt_stride, int nq, int nkv,
-                   int page_size, float scale, float sink, int window, int rows, int max_q_len, int skip_single, int keep_first, float softcap,
+                   int page_size, float scale, HeadTail<__nv_bfloat16> tail, int window, int rows, int max_q_len, int skip_single, int keep_first, float softcap,
                    int chunk, const float* pb, cudaStream_t s) {
   constexpr int ROW = HD + 8;
   int ps_shift = -1;
@@ -297,7 +299,7 @@ int launch_prefill(const void* q, int q_row_stride, void* out, const void* k_cac
   launch_kernel(kernel, dim3(grid), dim3(kThreads), smem, s, 1, 
       (const __nv_bfloat16*)q, q_row_stride, (__nv_bfloat16*)out, (const __nv_bfloat16*)k_cache,
       (const __nv_bfloat16*)v_cache, q_indptr, kv_lens, block_table, bt_stride, nq, nkv, page_size, ps_shift,
-      scale * 1.4426950408889634f, sink * 1.4426950408889634f, window, skip_single, window > 0 ? keep_first : 0,
+      scale * 1.4426950408889634f, tail, window, skip_single, window > 0 ? keep_first : 0,
       softcap > 0.f ? softcap * 1.4426950408889634f : 0.f, softcap > 0.f ? scale / softcap : 0.f, chunk, pb);
   return launch_status();
 }
@@ -307,18 +309,19 @@ int launch_prefill(const void* q, int q_row_stride, void* out, const void* k_cac
 ARLE_API int arle_paged_attention_prefill(const void* q, int q_row_stride, void* out, const void* k_cache,
                                           const void* v_cache, const int* q_indptr, const int* kv_lens,
                                           const int* block_table, int bt_stride, int nq, int nkv, int hd, int page_size,
-                                          float scale, float sink, int window, int rows, int max_q_len, int skip_single,
+                                          float scale, const float* sinks, const void* gate, int gate_stride, int window, int rows, int max_q_len, int skip_single,
                                           int keep_first, float softcap, int chunk, const float* pb, cudaStream_t s) {
   if (rows <= 0 || max_q_len <= 0) return 0;
   if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || page_size <= 0 || nq > 65535 || rows > 65535) return ARLE_E_UNSUPPORTED;
   if ((q_row_stride % 8) != 0) return ARLE_E_UNSUPPORTED;
   if (keep_first < 0 || softcap < 0.f || chunk < 0 || (chunk > 0 && window > 0)) return ARLE_E_BADARG;
   if (pb ? (keep_first > 0 || softcap > 0.f) : chunk > 0) return ARLE_E_UNSUPPORTED;      // the sigmoid form has neither; only it has chunks
+  const HeadTail<__nv_bfloat16> tail{sinks, (const __nv_bfloat16*)gate, gate_stride};
   if (hd == 128)
     return launch_prefill<128>(q, q_row_stride, out, k_cache, v_cache, q_indptr, kv_lens, block_table, bt_stride, nq,
-                               nkv, page_size, scale, sink, window, rows, max_q_len, skip_single, keep_first, softcap, chunk, pb, s);
+                               nkv, page_size, scale, tail, window, rows, max_q_len, skip_single, keep_first, softcap, chunk, pb, s);
   if (hd == 64)
     return launch_prefill<64>(q, q_row_stride, out, k_cache, v_cache, q_indptr, kv_lens, block_table, bt_stride, nq,
-                              nkv, page_size, scale, sink, window, rows, max_q_len, skip_single, keep_first, softcap, chunk, pb, s);
+                              nkv, page_size, scale, tail, window, rows, max_q_len, skip_single, keep_first, softcap, chunk, pb, s);
   return ARLE_E_UNSUPPORTED;
 }

@@ -196,7 +196,7 @@ __global__ void __launch_bounds__(kThreads, 1) paged_prefill_tc_kernel(
     const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
     const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* __restrict__ out, const int* __restrict__ q_indptr,
     const int* __restrict__ kv_lens, const int* __restrict__ block_table, int bt_stride, int bt_width, int nq, int nkv,
-    int page_size, float scale_log2, float sink_log2, int window, int skip_single, int nyb, int nblocks, int ticket_slot, int* __restrict__ err,
+    int page_size, float scale_log2, HeadTail<__nv_bfloat16> tail, int window, int skip_single, int nyb, int nblocks, int ticket_slot, int* __restrict__ err,
     int keep_arg, float cap_arg, float scale_over_cap, int chunk_arg, const float* __restrict__ pb) {
   pdl_launch_dependents();
   pdl_wait();
@@ -633,6 +633,9 @@ __global__ void __launch_bounds__(kThreads, 1) paged_prefill_tc_kernel(
         ++n;
         ++n_all;
       }
+      // asked for before the wait for the last product: a sink's score (log2 units; -inf: none), the head's gate
+      const float sink_log2 = SIG ? 0.f : tail.sink_log2(blk.h);
+      const float gate = row < rows_here ? tail.gate_of(blk.t0 + blk.mbeg + x * BQ + row, blk.h) : 1.0f;
       if (ok && n > 0) {
         const bool ready = mbar_wait_bounded(smem_addr(&o_full[x]), (uint32_t)(o_all & 1), aborted);
         if (__any_sync(0xffffffffu, !ready)) ok = false;
@@ -640,8 +643,7 @@ __global__ void __launch_bounds__(kThreads, 1) paged_prefill_tc_kernel(
       if (ok && n > 0) {
         ++o_all;
         tc_fence_after();
-        // a sink's term in the denominator (its score in log2 units; -inf: none, and the sum stays as it is)
-        const float inv = SIG ? 1.0f : 1.0f / (l + exp2f(sink_log2 - (m_used == -INFINITY ? 0.f : m_used)));
+        const float inv = (SIG ? 1.0f : 1.0f / (l + exp2f(sink_log2 - (m_used == -INFINITY ? 0.f : m_used)))) * gate;
         __nv_bfloat16* orow = out + ((size_t)(blk.t0 + blk.mbeg + x * BQ + row) * nq + blk.h) * HD;
 #pragma unroll 1
         for (int c = 0; c < 4; ++c) {
@@ -687,7 +689,8 @@ __global__ void __launch_bounds__(kThreads, 1) paged_prefill_tc_kernel(
 ARLE_API int arle_paged_attention_prefill_tc(const void* q, int q_row_stride, int num_tokens, void* out, const void* k_cache,
                                              const void* v_cache, long long cache_pages, const int* q_indptr,
                                              const int* kv_lens, const int* block_table, int bt_stride, int bt_width, int nq, int nkv,
-                                             int hd, int page_size, float scale, float sink, int window, int rows, int max_q_len,
+                                             int hd, int page_size, float scale, const float* sinks, const void* gate,
+                                             int gate_stride, int window, int rows, int max_q_len,
                                              int skip_single, int* err, int keep_first, float softcap, int chunk, const float* pb, cudaStream_t s) {
   if (rows <= 0 || max_q_len <= 0) return 0;
   if (bt_width < 1) return ARLE_E_BADARG;
@@ -726,7 +729,7 @@ ARLE_API int arle_paged_attention_prefill_tc(const void* q, int q_row_stride, in
   const int ticket_slot = (int)(launches++ % kTicketSlots);
   cudaError_t e = launch_kernel(kernel, dim3(ctas), dim3(kThreads), smem, s, 1, mq, mk, mv, (__nv_bfloat16*)out,
                                 q_indptr, kv_lens, block_table, bt_stride, bt_width, nq, nkv, page_size,
-                                scale * 1.4426950408889634f, sink * 1.4426950408889634f, window, skip_single, nyb, (int)nblocks, ticket_slot, err,
+                                scale * 1.4426950408889634f, HeadTail<__nv_bfloat16>{sinks, (const __nv_bfloat16*)gate, gate_stride}, window, skip_single, nyb, (int)nblocks, ticket_slot, err,
                                 window > 0 ? keep_first : 0, softcap > 0.f ? softcap * 1.4426950408889634f : 0.f,
                                 softcap > 0.f ? scale / softcap : 0.f, chunk, pb);
   if (e != cudaSuccess) return (int)e;

@@ -5,12 +5,15 @@
 //   q head: x <- rmsnorm_over_head(x; q_weight, eps) (if q_weight), rotate, store in place
 //   k head: the same with k_weight, then store into k_cache at the token's slot
 //   v head: copy into v_cache at the token's slot (no norm, no rotation)
+// A bias (float32, one number per element of a row, may be null) is added to q, k and v before everything else.
 // Norm statistics, the product x * inv * w and the rotation stay in float32; the
 // angle of pair i at position p is p * inv_freq[i], evaluated with sincosf in
 // float32.  Rotation pairs element i with i + rotary_dim/2 ("half split") inside
 // the first rotary_dim elements of the head; the rest passes through.
 // Cache layout: [page][kv_head][slot_in_page][head_dim]; slot_mapping[t] is
 // page * page_size + slot_in_page, negative = do not store.
+#include <type_traits>
+
 #include "common.cuh"
 using namespace arle;
 
@@ -25,7 +28,7 @@ __global__ void attention_prep_kernel(T* __restrict__ qkv, int row_stride,
                                       const float* __restrict__ k_weight, float eps,
                                       const float* __restrict__ inv_freq, int rotary_dim,
                                       T* __restrict__ k_cache, T* __restrict__ v_cache, int nq, int nkv,
-                                      int hd, int page_size, int num_tokens) {
+                                      int hd, int page_size, int num_tokens, const float* __restrict__ bias) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float bufs[kPrepWarps][kMaxHeadDim];
@@ -48,16 +51,17 @@ __global__ void attention_prep_kernel(T* __restrict__ qkv, int row_stride,
       store = true;
     }
   }
+  const float* bs = bias ? bias + (size_t)h * hd : nullptr;
   if (kind == 2) {
     if (store)
-      for (int e = lane; e < hd; e += 32) v_cache[cache_base + e] = src[e];
+      for (int e = lane; e < hd; e += 32) v_cache[cache_base + e] = bs ? from_f32<T>(to_f32(src[e]) + bs[e]) : src[e];
     return;
   }
   float* buf = bufs[w];
   const float* wt = kind == 0 ? q_weight : k_weight;
   float ss = 0.f;
   for (int e = lane; e < hd; e += 32) {
-    const float x = to_f32(src[e]);
+    const float x = to_f32(src[e]) + (bs ? bs[e] : 0.f);
     buf[e] = x;
     ss += x * x;
   }
@@ -86,18 +90,19 @@ __global__ void attention_prep_kernel(T* __restrict__ qkv, int row_stride,
   }
 }
 
-// Head sizes 64 and 128 with whole-head rotation, bfloat16: every lane keeps
-// hd/32 consecutive elements in registers (one 4- or 8-byte access), the norm's
-// sum is a warp reduction and the rotation partner (element i +- hd/2) lives in
-// lane ^ 16, so no shared memory is touched.  Same arithmetic as the general
-// kernel.
+// Head sizes 64 and 128, bfloat16, rotations of a multiple of hd/16 elements: every lane
+// keeps hd/32 consecutive elements in registers (one 4- or 8-byte access), the norm's
+// sum is a warp reduction and the rotation partner (element i +- rotary_dim/2) lives
+// rotary_dim/2 / (hd/32) lanes away, so no shared memory is touched.  Same arithmetic as
+// the general kernel.
 template <int HD>
 __global__ void attention_prep_bf16_kernel(__nv_bfloat16* __restrict__ qkv, int row_stride,
                                            const int* __restrict__ positions, const int* __restrict__ slot_mapping,
                                            const float* __restrict__ q_weight, const float* __restrict__ k_weight,
                                            float eps, const float* __restrict__ inv_freq,
                                            __nv_bfloat16* __restrict__ k_cache, __nv_bfloat16* __restrict__ v_cache,
-                                           int nq, int nkv, int page_size, int num_tokens) {
+                                           int nq, int nkv, int page_size, int num_tokens, int rotary_dim,
+                                           const float* __restrict__ bias) {
   pdl_launch_dependents();
   pdl_wait();
   constexpr int VE = HD / 32;                   // elements per lane: 2 or 4
@@ -127,7 +132,8 @@ __global__ void attention_prep_bf16_kernel(__nv_bfloat16* __restrict__ qkv, int 
   } else {
     raw[0] = *reinterpret_cast<const uint32_t*>(src);
   }
-  if (kind == 2) {
+  const float* bs = bias ? bias + (size_t)h * HD + lane * VE : nullptr;
+  if (kind == 2 && !bs) {
     if (store) {
       if (VE == 4) *reinterpret_cast<uint2*>(v_cache + cache_at) = make_uint2(raw[0], raw[VE / 2 - 1]);
       else *reinterpret_cast<uint32_t*>(v_cache + cache_at) = raw[0];
@@ -141,7 +147,11 @@ __global__ void attention_prep_bf16_kernel(__nv_bfloat16* __restrict__ qkv, int 
     x[2 * i] = __low2float(p);
     x[2 * i + 1] = __high2float(p);
   }
-  const float* wt = kind == 0 ? q_weight : k_weight;
+  if (bs) {
+#pragma unroll
+    for (int i = 0; i < VE; ++i) x[i] += bs[i];
+  }
+  const float* wt = kind == 0 ? q_weight : kind == 1 ? k_weight : nullptr;
   if (wt) {
     float ss = 0.f;
 #pragma unroll
@@ -153,13 +163,18 @@ __global__ void attention_prep_bf16_kernel(__nv_bfloat16* __restrict__ qkv, int 
   }
   const float pos = (float)positions[t];
   float o[VE];
+  const int hl = kind == 2 ? 0 : rotary_dim / (2 * VE);        // lanes with the pairs' first elements; the next hl have the second
+  const bool first = lane < hl, turns = lane < 2 * hl;
 #pragma unroll
   for (int i = 0; i < VE; ++i) {
-    const float other = __shfl_xor_sync(0xffffffffu, x[i], 16);
-    const int fi = (lane & 15) * VE + i;        // index of the pair
-    float sn, cs;
-    sincosf(pos * inv_freq[fi], &sn, &cs);
-    o[i] = lane < 16 ? x[i] * cs - other * sn : other * sn + x[i] * cs;
+    const float other = __shfl_sync(0xffffffffu, x[i], first ? lane + hl : turns ? lane - hl : lane);
+    o[i] = x[i];
+    if (turns) {
+      const int fi = (first ? lane : lane - hl) * VE + i;      // index of the pair
+      float sn, cs;
+      sincosf(pos * inv_freq[fi], &sn, &cs);
+      o[i] = first ? x[i] * cs - other * sn : other * sn + x[i] * cs;
+    }
   }
   uint32_t packed[VE / 2];
 #pragma unroll
@@ -167,7 +182,7 @@ __global__ void attention_prep_bf16_kernel(__nv_bfloat16* __restrict__ qkv, int 
     __nv_bfloat162 p = __floats2bfloat162_rn(o[2 * i], o[2 * i + 1]);
     packed[i] = *reinterpret_cast<uint32_t*>(&p);
   }
-  __nv_bfloat16* dst = kind == 0 ? src : (store ? k_cache + cache_at : nullptr);
+  __nv_bfloat16* dst = kind == 0 ? src : (store ? (kind == 1 ? k_cache : v_cache) + cache_at : nullptr);
   if (dst) {
     if (VE == 4) *reinterpret_cast<uint2*>(dst) = make_uint2(packed[0], packed[VE / 2 - 1]);
     else *reinterpret_cast<uint32_t*>(dst) = packed[0];
@@ -185,12 +200,14 @@ __global__ void attention_prep_bf16_kernel(__nv_bfloat16* __restrict__ qkv, int 
 constexpr int kPrepVecWarps = 8;
 constexpr int kPrepMaxPasses = 3;               // heads a warp takes, in passes, with its loads batched (more: in further rounds)
 
-template <int HD>
+// PART: only the first rotary_dim elements turn (a multiple of 8, at most hd / 2: both elements of a pair lie in the head's
+// first half, rotary_dim / 8 lanes apart, and are exchanged by shuffles).  BIAS: a bias is added first.
+template <int HD, bool PART, bool BIAS>
 __global__ void __launch_bounds__(kPrepVecWarps * 32, 4) attention_prep_bf16_token_kernel(
     __nv_bfloat16* __restrict__ qkv, int row_stride, const int* __restrict__ positions,
     const int* __restrict__ slot_mapping, const float* __restrict__ q_weight, const float* __restrict__ k_weight, float eps,
     const float* __restrict__ inv_freq, const float2* __restrict__ angles, __nv_bfloat16* __restrict__ k_cache,
-    __nv_bfloat16* __restrict__ v_cache, int nq, int nkv, int page_size, int num_tokens) {
+    __nv_bfloat16* __restrict__ v_cache, int nq, int nkv, int page_size, int num_tokens, int rotary_dim, const float* __restrict__ bias) {
   pdl_launch_dependents();
   pdl_wait();
   constexpr int LPH = HD / 8;                   // lanes per head: 16 or 8
@@ -199,7 +216,8 @@ __global__ void __launch_bounds__(kPrepVecWarps * 32, 4) attention_prep_bf16_tok
   __shared__ float cs_s[HALF], sn_s[HALF];
   const int t = blockIdx.x;
   const int w = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  if (!angles && threadIdx.x < HALF) {
+  const int pairs = PART ? rotary_dim / 2 : HALF;
+  if (!angles && threadIdx.x < pairs) {
     float sn, cs;
     sincosf((float)positions[t] * inv_freq[threadIdx.x], &sn, &cs);
     cs_s[threadIdx.x] = cs;
@@ -223,17 +241,20 @@ __global__ void __launch_bounds__(kPrepVecWarps * 32, 4) attention_prep_bf16_tok
     }
   };
   fetch(w * HPW + sub);                         // under way while the cosines and sines are fetched or computed
-  float cs[4], sn[4];
-  if (angles) {
+  const int pl = PART ? rotary_dim / 8 : 0;     // PART: lanes between the two elements of a pair
+  const bool first = l < pl, turns = !PART || l < 2 * pl;
+  const int a0 = PART ? (turns ? (first ? e0 : e0 - 4 * pl) : 0) : e0;      // this lane's first pair
+  float cs[4] = {1.f, 1.f, 1.f, 1.f}, sn[4] = {0.f, 0.f, 0.f, 0.f};
+  if (!angles) __syncthreads();
+  if (angles && turns) {
     // the step's table (the same for every layer): (cos, sin) of this token's hd / 2 angles
-    const float4* a4 = reinterpret_cast<const float4*>(angles + (size_t)t * HALF + e0);
+    const float4* a4 = reinterpret_cast<const float4*>(angles + (size_t)t * pairs + a0);
     const float4 v0 = a4[0], v1 = a4[1];
     cs[0] = v0.x, sn[0] = v0.y, cs[1] = v0.z, sn[1] = v0.w;
     cs[2] = v1.x, sn[2] = v1.y, cs[3] = v1.z, sn[3] = v1.w;
-  } else {
-    __syncthreads();
+  } else if (turns) {
 #pragma unroll
-    for (int i = 0; i < 4; ++i) cs[i] = cs_s[e0 + i], sn[i] = sn_s[e0 + i];
+    for (int i = 0; i < 4; ++i) cs[i] = cs_s[a0 + i], sn[i] = sn_s[a0 + i];
   }
   // the loop's condition is the same for all lanes of a warp: lanes without a head take part in the shuffles
   for (int hb = w * HPW; hb < heads; hb += stride_h * kPrepMaxPasses) {
@@ -246,11 +267,11 @@ __global__ void __launch_bounds__(kPrepVecWarps * 32, 4) attention_prep_bf16_tok
       const bool is_q = h < nq, is_v = h >= nq + nkv;
       const bool store = live && !is_q && slot >= 0;
       const size_t cache_at = store ? (((size_t)page * nkv + (is_v ? h - nq - nkv : h - nq)) * page_size + off) * HD + e0 : 0;
-      if (is_v && store) {
+      if (is_v && store && !BIAS) {
         *reinterpret_cast<uint2*>(v_cache + cache_at) = lo[p];
         *reinterpret_cast<uint2*>(v_cache + cache_at + HALF) = hi[p];
       }
-      if (__all_sync(0xffffffffu, is_v || !live)) continue;      // nothing to norm or rotate in this pass
+      if (__all_sync(0xffffffffu, (is_v && !BIAS) || !live)) continue;      // nothing to norm or rotate in this pass
       float a[4], b[4];                          // first half, second half
       {
         const __nv_bfloat162 a0 = *reinterpret_cast<const __nv_bfloat162*>(&lo[p].x), a1 = *reinterpret_cast<const __nv_bfloat162*>(&lo[p].y);
@@ -258,7 +279,12 @@ __global__ void __launch_bounds__(kPrepVecWarps * 32, 4) attention_prep_bf16_tok
         a[0] = __low2float(a0), a[1] = __high2float(a0), a[2] = __low2float(a1), a[3] = __high2float(a1);
         b[0] = __low2float(b0), b[1] = __high2float(b0), b[2] = __low2float(b1), b[3] = __high2float(b1);
       }
-      const float* wt = is_q ? q_weight : k_weight;
+      if (BIAS && live) {
+        const float4 ba = *reinterpret_cast<const float4*>(bias + (size_t)h * HD + e0), bb = *reinterpret_cast<const float4*>(bias + (size_t)h * HD + HALF + e0);
+        a[0] += ba.x, a[1] += ba.y, a[2] += ba.z, a[3] += ba.w;
+        b[0] += bb.x, b[1] += bb.y, b[2] += bb.z, b[3] += bb.w;
+      }
+      const float* wt = is_q ? q_weight : (BIAS && is_v) ? nullptr : k_weight;
       // The sum of squares in the order of the other preparation kernels (a warp per head, hd / 32 consecutive
       // elements per lane, butterfly over lane distances 16, 8, 4, 2, 1), so that a key prepared here has the
       // bits of one prepared there.  This lane holds the elements of 4 / VE of that warp's lanes in each half:
@@ -294,13 +320,23 @@ __global__ void __launch_bounds__(kPrepVecWarps * 32, 4) attention_prep_bf16_tok
         b[0] = b[0] * inv * gb.x, b[1] = b[1] * inv * gb.y, b[2] = b[2] * inv * gb.z, b[3] = b[3] * inv * gb.w;
       }
       float oa[4], ob[4];
+      if (PART) {
+        const int from = first ? lane + pl : turns ? lane - pl : lane;
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        oa[i] = a[i] * cs[i] - b[i] * sn[i];
-        ob[i] = a[i] * sn[i] + b[i] * cs[i];
+        for (int i = 0; i < 4; ++i) {
+          const float other = __shfl_sync(0xffffffffu, a[i], from);
+          oa[i] = (turns && !is_v) ? (first ? a[i] * cs[i] - other * sn[i] : other * sn[i] + a[i] * cs[i]) : a[i];
+          ob[i] = b[i];
+        }
+      } else {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          oa[i] = (BIAS && is_v) ? a[i] : a[i] * cs[i] - b[i] * sn[i];
+          ob[i] = (BIAS && is_v) ? b[i] : a[i] * sn[i] + b[i] * cs[i];
+        }
       }
-      if (live && !is_v) {
-        __nv_bfloat16* dst = is_q ? row + (size_t)h * HD : (store ? k_cache + cache_at : nullptr);
+      if (live && (!is_v || BIAS)) {
+        __nv_bfloat16* dst = is_q ? row + (size_t)h * HD : (store ? (is_v ? v_cache : k_cache) + cache_at : nullptr);
         if (dst) {
           __nv_bfloat162 p0 = __floats2bfloat162_rn(oa[0], oa[1]), p1 = __floats2bfloat162_rn(oa[2], oa[3]);
           __nv_bfloat162 q0 = __floats2bfloat162_rn(ob[0], ob[1]), q1 = __floats2bfloat162_rn(ob[2], ob[3]);
@@ -337,11 +373,11 @@ ARLE_API int arle_rotary_angles(const int* positions, const float* inv_freq, flo
 }
 
 // angles (may be null): the table of arle_rotary_angles for these positions and inv_freq; kernels that can use it
-// then skip the evaluation of the angles (16-byte aligned).
+// then skip the evaluation of the angles (16-byte aligned).  bias (may be null): float32 [(nq + 2 nkv) * hd], added to q, k, v first.
 ARLE_API int arle_attention_prep(void* qkv, int dtype, int row_stride, const int* positions,
                                  const int* slot_mapping, const float* q_weight, const float* k_weight,
                                  float eps, const float* inv_freq, const float* angles, int rotary_dim, void* k_cache,
-                                 void* v_cache, int nq, int nkv, int hd, int page_size, int num_tokens,
+                                 void* v_cache, int nq, int nkv, int hd, int page_size, int num_tokens, const float* bias,
                                  cudaStream_t s) {
   if (num_tokens <= 0) return 0;
   if (hd <= 0 || hd > kMaxHeadDim || nq < 0 || nkv < 0 || nq + nkv == 0) return ARLE_E_UNSUPPORTED;
@@ -351,41 +387,44 @@ ARLE_API int arle_attention_prep(void* qkv, int dtype, int row_stride, const int
   const long long units = (long long)num_tokens * (nq + 2 * nkv);
   const long long blocks = (units + kPrepWarps - 1) / kPrepWarps;
   if (blocks > 0x7fffffffLL) return ARLE_E_UNSUPPORTED;
-  if (dtype == 1 && (hd == 64 || hd == 128) && rotary_dim == hd && row_stride % 4 == 0 && ((uintptr_t)qkv & 7) == 0 &&
+  const bool whole = rotary_dim == hd;
+  if (dtype == 1 && (hd == 64 || hd == 128) && rotary_dim % (hd / 16) == 0 && row_stride % 4 == 0 && ((uintptr_t)qkv & 7) == 0 &&
       ((uintptr_t)k_cache & 7) == 0 && ((uintptr_t)v_cache & 7) == 0) {
     const bool wide = row_stride % 8 == 0 && ((uintptr_t)qkv & 15) == 0 && ((uintptr_t)k_cache & 15) == 0 &&
                       ((uintptr_t)v_cache & 15) == 0 && (!q_weight || ((uintptr_t)q_weight & 15) == 0) &&
-                      (!k_weight || ((uintptr_t)k_weight & 15) == 0);      // 16-byte accesses
-    if (num_tokens >= 32 && wide) {              // enough tokens to fill the GPU with one block each
+                      (!k_weight || ((uintptr_t)k_weight & 15) == 0) && (!bias || ((uintptr_t)bias & 15) == 0);      // 16-byte accesses
+    const bool part = rotary_dim <= hd / 2 && rotary_dim % 8 == 0;
+    if (num_tokens >= 32 && wide && (whole || part)) {              // enough tokens to fill the GPU with one block each
       const float2* tab = ((uintptr_t)angles & 15) == 0 ? reinterpret_cast<const float2*>(angles) : nullptr;
-      if (hd == 128)
-        launch_kernel(attention_prep_bf16_token_kernel<128>, dim3(num_tokens), dim3(kPrepVecWarps * 32), 0, s, 1,
-                      (__nv_bfloat16*)qkv, row_stride, positions, slot_mapping, q_weight, k_weight, eps, inv_freq, tab,
-                      (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, nq, nkv, page_size, num_tokens);
-      else
-        launch_kernel(attention_prep_bf16_token_kernel<64>, dim3(num_tokens), dim3(kPrepVecWarps * 32), 0, s, 1,
-                      (__nv_bfloat16*)qkv, row_stride, positions, slot_mapping, q_weight, k_weight, eps, inv_freq, tab,
-                      (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, nq, nkv, page_size, num_tokens);
+      auto pick = [&](auto has_bias) {
+        constexpr bool B = decltype(has_bias)::value;
+        return hd == 128 ? (whole ? attention_prep_bf16_token_kernel<128, false, B> : attention_prep_bf16_token_kernel<128, true, B>)
+                         : (whole ? attention_prep_bf16_token_kernel<64, false, B> : attention_prep_bf16_token_kernel<64, true, B>);
+      };
+      auto kern = bias ? pick(std::true_type{}) : pick(std::false_type{});
+      launch_kernel(kern, dim3(num_tokens), dim3(kPrepVecWarps * 32), 0, s, 1,
+                    (__nv_bfloat16*)qkv, row_stride, positions, slot_mapping, q_weight, k_weight, eps, inv_freq, tab,
+                    (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, nq, nkv, page_size, num_tokens, rotary_dim, bias);
       return launch_status();
     }
     if (hd == 128)
       launch_kernel(attention_prep_bf16_kernel<128>, dim3((int)blocks), dim3(kPrepWarps * 32), 0, s, 1, 
           (__nv_bfloat16*)qkv, row_stride, positions, slot_mapping, q_weight, k_weight, eps, inv_freq,
-          (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, nq, nkv, page_size, num_tokens);
+          (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, nq, nkv, page_size, num_tokens, rotary_dim, bias);
     else
       launch_kernel(attention_prep_bf16_kernel<64>, dim3((int)blocks), dim3(kPrepWarps * 32), 0, s, 1, 
           (__nv_bfloat16*)qkv, row_stride, positions, slot_mapping, q_weight, k_weight, eps, inv_freq,
-          (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, nq, nkv, page_size, num_tokens);
+          (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, nq, nkv, page_size, num_tokens, rotary_dim, bias);
     return launch_status();
   }
   if (dtype == 0)
     launch_kernel(attention_prep_kernel<float>, dim3((int)blocks), dim3(kPrepWarps * 32), 0, s, 1, 
         (float*)qkv, row_stride, positions, slot_mapping, q_weight, k_weight, eps, inv_freq, rotary_dim,
-        (float*)k_cache, (float*)v_cache, nq, nkv, hd, page_size, num_tokens);
+        (float*)k_cache, (float*)v_cache, nq, nkv, hd, page_size, num_tokens, bias);
   else if (dtype == 1)
     launch_kernel(attention_prep_kernel<__nv_bfloat16>, dim3((int)blocks), dim3(kPrepWarps * 32), 0, s, 1, 
         (__nv_bfloat16*)qkv, row_stride, positions, slot_mapping, q_weight, k_weight, eps, inv_freq,
-        rotary_dim, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, nq, nkv, hd, page_size, num_tokens);
+        rotary_dim, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, nq, nkv, hd, page_size, num_tokens, bias);
   else
     return ARLE_E_BADARG;
   return launch_status();

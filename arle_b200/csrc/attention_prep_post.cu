@@ -10,6 +10,7 @@
 //   v head: copied into v_cache at the token's slot
 // With norm_first the norm (and its weight) comes BEFORE the rotation instead: x <- x / sqrt(mean(x^2) + eps) * weight, then
 // the first rotary_dim numbers turn.
+// A bias (float32, one number per element of a row, may be null) is added to q, k and v before everything else.
 // Everything between load and store is float32; the angle is evaluated with sincosf in float32.
 // Cache layout: keys [page][kv_head][slot_in_page][hd], values [page][kv_head][slot_in_page][vd]; slot_mapping[t] is
 // page * page_size + slot_in_page, negative = do not store.  nkv = 0: the rows hold q only.
@@ -24,7 +25,7 @@ __global__ void attention_prep_post_kernel(T* __restrict__ qkv, int row_stride, 
                                            const int* __restrict__ slot_mapping, const float* __restrict__ q_weight,
                                            const float* __restrict__ k_weight, float eps, const float* __restrict__ inv_freq,
                                            int rotary_dim, T* __restrict__ k_cache, T* __restrict__ v_cache, int nq, int nkv, int hd,
-                                           int vd, int page_size, int num_tokens, int norm_first) {
+                                           int vd, int page_size, int num_tokens, int norm_first, const float* __restrict__ bias) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float bufs[kPostWarps][kPostMaxHead];
@@ -35,7 +36,9 @@ __global__ void attention_prep_post_kernel(T* __restrict__ qkv, int row_stride, 
   const int t = (int)(unit / heads), h = (int)(unit % heads);
   const int kind = h < nq ? 0 : (h < nq + nkv ? 1 : 2);
   const int kvh = kind == 1 ? h - nq : h - nq - nkv;
-  T* src = qkv + (size_t)t * row_stride + (kind < 2 ? (size_t)h * hd : (size_t)(nq + nkv) * hd + (size_t)kvh * vd);
+  const size_t at = kind < 2 ? (size_t)h * hd : (size_t)(nq + nkv) * hd + (size_t)kvh * vd;
+  T* src = qkv + (size_t)t * row_stride + at;
+  const float* bs = bias ? bias + at : nullptr;
 
   size_t cache_base = 0;
   bool store = false;
@@ -49,11 +52,11 @@ __global__ void attention_prep_post_kernel(T* __restrict__ qkv, int row_stride, 
   }
   if (kind == 2) {
     if (store)
-      for (int e = lane; e < vd; e += 32) v_cache[cache_base + e] = src[e];
+      for (int e = lane; e < vd; e += 32) v_cache[cache_base + e] = bs ? from_f32<T>(to_f32(src[e]) + bs[e]) : src[e];
     return;
   }
   float* buf = bufs[w];
-  for (int e = lane; e < hd; e += 32) buf[e] = to_f32(src[e]);
+  for (int e = lane; e < hd; e += 32) buf[e] = to_f32(src[e]) + (bs ? bs[e] : 0.f);
   __syncwarp();
   const float* wt = kind == 0 ? q_weight : k_weight;
   if (norm_first && eps >= 0.f) {
@@ -105,7 +108,7 @@ __global__ void attention_prep_post_kernel(T* __restrict__ qkv, int row_stride, 
 ARLE_API int arle_attention_prep_post(void* qkv, int dtype, int row_stride, const int* positions, const int* slot_mapping,
                                       const float* q_weight, const float* k_weight, float eps, const float* inv_freq, int rotary_dim,
                                       void* k_cache, void* v_cache, int nq, int nkv, int hd, int vd, int page_size, int num_tokens,
-                                      int norm_first, cudaStream_t s) {
+                                      int norm_first, const float* bias, cudaStream_t s) {
   if (num_tokens <= 0) return 0;
   if (hd <= 0 || hd > kPostMaxHead || vd <= 0 || nq <= 0 || nkv < 0 || page_size <= 0) return ARLE_E_UNSUPPORTED;
   if (rotary_dim < 0 || rotary_dim % 2 || rotary_dim > hd || (rotary_dim && !inv_freq)) return ARLE_E_BADARG;
@@ -116,11 +119,11 @@ ARLE_API int arle_attention_prep_post(void* qkv, int dtype, int row_stride, cons
   if (dtype == 0)
     launch_kernel(attention_prep_post_kernel<float>, dim3((unsigned)blocks), dim3(kPostWarps * 32), 0, s, 1, (float*)qkv, row_stride,
                   positions, slot_mapping, q_weight, k_weight, eps, inv_freq, rotary_dim, (float*)k_cache, (float*)v_cache, nq, nkv, hd,
-                  vd, page_size, num_tokens, norm_first);
+                  vd, page_size, num_tokens, norm_first, bias);
   else if (dtype == 1)
     launch_kernel(attention_prep_post_kernel<__nv_bfloat16>, dim3((unsigned)blocks), dim3(kPostWarps * 32), 0, s, 1, (__nv_bfloat16*)qkv,
                   row_stride, positions, slot_mapping, q_weight, k_weight, eps, inv_freq, rotary_dim, (__nv_bfloat16*)k_cache,
-                  (__nv_bfloat16*)v_cache, nq, nkv, hd, vd, page_size, num_tokens, norm_first);
+                  (__nv_bfloat16*)v_cache, nq, nkv, hd, vd, page_size, num_tokens, norm_first, bias);
   else
     return ARLE_E_BADARG;
   return launch_status();

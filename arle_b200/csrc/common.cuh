@@ -105,6 +105,19 @@ __device__ __forceinline__ int first_visible_key(int pos, int window, int chunk)
   return (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
 }
 
+// What the attention kernels apply behind a query head's sums: the score of a sink that the softmax's denominator counts besides
+// the keys (float32, one per query head; null: no sink) and an output gate, one number per (token, query head) that multiplies
+// the head's output as sigmoid(gate[t * gate_stride + head]) (null: none).
+template <typename T> struct HeadTail {
+  const float* sinks;
+  const T* gate;
+  int gate_stride;
+  __device__ __forceinline__ float sink_log2(int head) const { return sinks ? sinks[head] * 1.4426950408889634f : -INFINITY; }
+  __device__ __forceinline__ float gate_of(int t, int head) const {
+    return gate ? 1.0f / (1.0f + expf(-to_f32(gate[(size_t)t * gate_stride + head]))) : 1.0f;
+  }
+};
+
 // Programmatic dependent launch.  Every kernel of this library starts with
 // pdl_launch_dependents() (the next kernel of the stream may be scheduled as soon as
 // all CTAs of this one have started) and calls pdl_wait() before it first touches

@@ -25,7 +25,7 @@
 // Two optional fusions take the RMSNorm kernels out of a decode step (a norm between two
 // of these products is then no launch at all):
 //  * "sink": instead of storing its sums, the product adds them to the float32 residual,
-//    r = resid + sum, and stores resid = r and xs = bfloat16(r * gamma), the next norm's
+//    r = resid + branch_scale * sum (+ extra, rows that join the residual here), and stores resid = r and xs = bfloat16(r * gamma), the next norm's
 //    input without its per-row factor; every CTA also leaves the sum of r^2 over its
 //    columns in a slot of its own of a small table (no atomics, so the order of the
 //    additions is fixed);
@@ -70,6 +70,8 @@ struct Fusion {
   __nv_bfloat16* xs;           // [M, ldxs]
   int ldxs;
   float* out_ss;               // [kSsRows][kSsSlots]: this launch fills every slot (zeros beyond its own CTAs)
+  float branch_scale;          // with resid: what a sum is multiplied by before it is added
+  const float* extra;          // with resid: [M, ldr] float32 added to it as well, or null
   int act;                     // 1: the sums go through the square of relu on their way to out (not with resid)
 };
 
@@ -268,6 +270,7 @@ __global__ void __launch_bounds__(kThreads, 1) skinny_gemm_kernel(
     r = gn = 0.f;
     if (fu.resid && valid) {
       r = __ldcg(fu.resid + (size_t)m * fu.ldr + n);
+      if (fu.extra) r += __ldcg(fu.extra + (size_t)m * fu.ldr + n);
       gn = __ldg(fu.gamma + n);
     }
   };
@@ -282,7 +285,7 @@ __global__ void __launch_bounds__(kThreads, 1) skinny_gemm_kernel(
     }
     float r = 0.f;
     if (valid) {
-      r = r_old + v;
+      r = fmaf(fu.branch_scale, v, r_old);
       fu.resid[(size_t)m * fu.ldr + n] = r;
       fu.xs[(size_t)m * fu.ldxs + n] = __float2bfloat16_rn(r * gn);
     }
@@ -564,14 +567,14 @@ ARLE_API int arle_gemm_skinny_gated(const void* x, int ldx, const void* W, int l
 //    with a sink; the sums of this product are multiplied by rsqrt(sum(in_ss[m, :]) * inv_width + eps).
 //  gated: 0 plain product; 1 the gate is silu; 2 the gate is the tanh form of gelu; 3 no gate, out = max(sum, 0)^2.
 //  resid (may be null; not with gated): float32 [M, ldr].  When given, nothing goes to out (it may be
-//    null): resid[m, n] += sum, xs[m, n] = bfloat16(resid[m, n] * gamma[n]), and out_ss [16][192] gets
+//    null): resid[m, n] += branch_scale * sum (+ extra[m, n], float32 [M, ldr] or null), xs[m, n] = bfloat16(resid[m, n] * gamma[n]), and out_ss [16][192] gets
 //    the sums of squares of the new residual rows, every slot written.
 ARLE_API int arle_gemm_skinny_fused(const void* x, int ldx, const void* W, int ldw, void* out, int out_dtype, int ldo, int M,
                                     int N, int K, int gated, const float* in_ss, float inv_width, float eps, float* resid,
-                                    int ldr, const float* gamma, void* xs, int ldxs, float* out_ss, int* err,
-                                    cudaStream_t s) {
+                                    int ldr, const float* gamma, void* xs, int ldxs, float* out_ss, float branch_scale,
+                                    const float* extra, int* err, cudaStream_t s) {
   if (gated == 3 && resid) return ARLE_E_BADARG;
-  Fusion fu{in_ss, inv_width, eps, resid, ldr, gamma, (__nv_bfloat16*)xs, ldxs, out_ss, gated == 3 ? 1 : 0};
+  Fusion fu{in_ss, inv_width, eps, resid, ldr, gamma, (__nv_bfloat16*)xs, ldxs, out_ss, branch_scale, extra, gated == 3 ? 1 : 0};
   if (gated == 3) gated = 0;
   return skinny_entry(x, ldx, W, ldw, out, out_dtype, ldo, M, N, K, gated, fu, err, s);
 }

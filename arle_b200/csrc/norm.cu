@@ -1,7 +1,7 @@
 // RMSNorm over the 32-bit residual stream, fused with the residual sum.
 //
 // For output row i (source row r = rows ? rows[i] : i):
-//     x      = resid[r, :] (+ delta[r, :] when delta is given)      in float32
+//     x      = resid[r, :] (+ delta_scale * delta[r, :] when delta is given) (+ extra[r, :], float32, when given)    in float32
 //     resid[r, :] = x                      (when write_resid)
 //     out[i, :]   = x * rsqrt(mean(x^2) + eps) * weight
 // The sum of squares, the inverse and the product are float32; the only rounding
@@ -14,7 +14,8 @@ using namespace arle;
 template <typename TA>
 __global__ void rmsnorm_kernel(float* __restrict__ resid, const TA* __restrict__ delta,
                                const int* __restrict__ rows, const float* __restrict__ weight,
-                               TA* __restrict__ out, int hidden, float eps, int write_resid) {
+                               TA* __restrict__ out, int hidden, float eps, int write_resid, float delta_scale,
+                               const float* __restrict__ extra) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float xs[];
@@ -23,10 +24,12 @@ __global__ void rmsnorm_kernel(float* __restrict__ resid, const TA* __restrict__
   const int r = rows ? rows[i] : i;
   float* xr = resid + (size_t)r * hidden;
   const TA* dr = delta ? delta + (size_t)r * hidden : nullptr;
+  const float* er = extra ? extra + (size_t)r * hidden : nullptr;
   float ss = 0.f;
   for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
     float x = xr[c];
-    if (dr) x += to_f32(dr[c]);
+    if (dr) x = fmaf(delta_scale, to_f32(dr[c]), x);
+    if (er) x += er[c];
     xs[c] = x;
     if (write_resid) xr[c] = x;
     ss += x * x;
@@ -63,7 +66,8 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
 template <typename TA>
 __global__ void rmsnorm_vec_kernel(float* __restrict__ resid, const TA* __restrict__ delta,
                                    const int* __restrict__ rows, const float* __restrict__ weight,
-                                   TA* __restrict__ out, int hidden, float eps, int write_resid) {
+                                   TA* __restrict__ out, int hidden, float eps, int write_resid, float delta_scale,
+                               const float* __restrict__ extra) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float red[33];
@@ -71,6 +75,7 @@ __global__ void rmsnorm_vec_kernel(float* __restrict__ resid, const TA* __restri
   const int r = rows ? rows[i] : i;
   float* xr = resid + (size_t)r * hidden;
   const TA* dr = delta ? delta + (size_t)r * hidden : nullptr;
+  const float* er = extra ? extra + (size_t)r * hidden : nullptr;
   const int n4 = hidden >> 2;
   float4 x[kVecMax];
   float ss = 0.f;
@@ -81,9 +86,14 @@ __global__ void rmsnorm_vec_kernel(float* __restrict__ resid, const TA* __restri
       float4 v = load4(xr + 4 * c);
       if (dr) {
         const float4 d = load4(dr + 4 * c);
-        v.x += d.x; v.y += d.y; v.z += d.z; v.w += d.w;
-        if (write_resid) store4(xr + 4 * c, v);
+        v.x = fmaf(delta_scale, d.x, v.x), v.y = fmaf(delta_scale, d.y, v.y);
+        v.z = fmaf(delta_scale, d.z, v.z), v.w = fmaf(delta_scale, d.w, v.w);
       }
+      if (er) {
+        const float4 e = load4(er + 4 * c);
+        v.x += e.x; v.y += e.y; v.z += e.z; v.w += e.w;
+      }
+      if (write_resid && (dr || er)) store4(xr + 4 * c, v);
       x[k] = v;
       ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
     }
@@ -111,14 +121,14 @@ static bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 
 
 template <typename TA>
 static int launch(float* resid, const void* delta, const int* rows, const float* weight, void* out,
-                  int n_out, int hidden, float eps, int write_resid, cudaStream_t s) {
+                  int n_out, int hidden, float eps, int write_resid, float delta_scale, const float* extra, cudaStream_t s) {
   if (hidden % 4 == 0 && hidden <= 4 * kVecMax * 1024 && aligned16(resid) && aligned16(weight) && aligned16(out) &&
-      aligned16(delta)) {
+      aligned16(delta) && aligned16(extra)) {
     const int n4 = hidden / 4;
     int threads = (n4 + kVecMax - 1) / kVecMax;
     threads = threads <= 64 ? 64 : (threads <= 128 ? 128 : (threads <= 256 ? 256 : (threads <= 512 ? 512 : 1024)));
     launch_kernel(rmsnorm_vec_kernel<TA>, dim3(n_out), dim3(threads), 0, s, 1, resid, (const TA*)delta, rows, weight, (TA*)out, hidden, eps,
-                                                     write_resid);
+                                                     write_resid, delta_scale, extra);
     return launch_status();
   }
   const int threads = hidden >= 2048 ? 512 : (hidden >= 512 ? 256 : 128);
@@ -130,41 +140,41 @@ static int launch(float* resid, const void* delta, const int* rows, const float*
     if (e != cudaSuccess) return (int)e;
   }
   launch_kernel(rmsnorm_kernel<TA>, dim3(n_out), dim3(threads), smem, s, 1, resid, (const TA*)delta, rows, weight, (TA*)out, hidden,
-                                                  eps, write_resid);
+                                                  eps, write_resid, delta_scale, extra);
   return launch_status();
 }
 
 // act_dtype: type of delta and out.  The gain vector is float32 (norm gains are
 // widened once at load; they are a few KB).
 ARLE_API int arle_rmsnorm(float* resid, const void* delta, const int* rows, const float* weight,
-                          void* out, int act_dtype, int n_out, int hidden, float eps, int write_resid,
-                          cudaStream_t s) {
+                          void* out, int act_dtype, int n_out, int hidden, float eps, int write_resid, float delta_scale,
+                          const float* extra, cudaStream_t s) {
   if (n_out <= 0) return 0;
   if (hidden <= 0) return ARLE_E_BADARG;
-  if (act_dtype == 0) return launch<float>(resid, delta, rows, weight, out, n_out, hidden, eps, write_resid, s);
-  if (act_dtype == 1) return launch<__nv_bfloat16>(resid, delta, rows, weight, out, n_out, hidden, eps, write_resid, s);
+  if (act_dtype == 0) return launch<float>(resid, delta, rows, weight, out, n_out, hidden, eps, write_resid, delta_scale, extra, s);
+  if (act_dtype == 1) return launch<__nv_bfloat16>(resid, delta, rows, weight, out, n_out, hidden, eps, write_resid, delta_scale, extra, s);
   return ARLE_E_BADARG;
 }
 
-// resid[r, :] += delta[r, :] for all rows: the residual sum alone, for a branch
+// resid[r, :] += scale * delta[r, :] for all rows: the residual sum alone, for a branch
 // output that no norm follows directly.
 template <typename TA>
-__global__ void residual_add_kernel(float* __restrict__ resid, const TA* __restrict__ delta, size_t total) {
+__global__ void residual_add_kernel(float* __restrict__ resid, const TA* __restrict__ delta, size_t total, float scale) {
   pdl_launch_dependents();
   pdl_wait();
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x)
-    resid[i] += to_f32(delta[i]);
+    resid[i] = fmaf(scale, to_f32(delta[i]), resid[i]);
 }
 
-ARLE_API int arle_residual_add(float* resid, const void* delta, int act_dtype, int rows, int hidden, cudaStream_t s) {
+ARLE_API int arle_residual_add(float* resid, const void* delta, int act_dtype, int rows, int hidden, float scale, cudaStream_t s) {
   if (rows <= 0) return 0;
   const size_t total = (size_t)rows * hidden;
   size_t blocks = (total + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
   if (act_dtype == 0)
-    launch_kernel(residual_add_kernel<float>, dim3((int)blocks), dim3(256), 0, s, 1, resid, (const float*)delta, total);
+    launch_kernel(residual_add_kernel<float>, dim3((int)blocks), dim3(256), 0, s, 1, resid, (const float*)delta, total, scale);
   else if (act_dtype == 1)
-    launch_kernel(residual_add_kernel<__nv_bfloat16>, dim3((int)blocks), dim3(256), 0, s, 1, resid, (const __nv_bfloat16*)delta, total);
+    launch_kernel(residual_add_kernel<__nv_bfloat16>, dim3((int)blocks), dim3(256), 0, s, 1, resid, (const __nv_bfloat16*)delta, total, scale);
   else
     return ARLE_E_BADARG;
   return launch_status();

@@ -33,12 +33,14 @@ constexpr int kScanThreads = 256;
 
 // AHEAD: the variant that asks for the next chunk while this one's steps run (steps of prompt portions; it holds more registers,
 // which a step of decoded tokens, bound by reading and writing the memories, pays for in blocks per SM).
-template <typename T, int EPL, int CPT, bool AHEAD>
+// ROT: q and k turn first (half-split pairs of the first rotary_dim numbers, angle position * inv_freq), in float32 as they are staged.
+template <typename T, int EPL, int CPT, bool AHEAD, bool ROT>
 __global__ void __launch_bounds__(kScanThreads) decay_scan_kernel(
     const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, int q_stride, int k_stride, int v_stride,
     const float* __restrict__ a, const float* __restrict__ b, float* __restrict__ state, long slot_stride,
     const int* __restrict__ q_indptr, const int* __restrict__ state_slots, float* __restrict__ out, int H, int kq_heads,
-    int dim, int vdim, int ones_col, float q_scale, int lpc, int ab_stride, int act) {
+    int dim, int vdim, int ones_col, float q_scale, int lpc, int ab_stride, int act, const int* __restrict__ positions,
+    const float* __restrict__ inv_freq, int rotary_dim, int longest) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float sm[];
@@ -54,6 +56,7 @@ __global__ void __launch_bounds__(kScanThreads) decay_scan_kernel(
   const int cl0 = threadIdx.x / lpc * CPT, part = threadIdx.x % lpc;      // the thread's first column inside the block
   const int e0 = part * EPL;
   const int beg = q_indptr[r], end = q_indptr[r + 1];
+  if (longest > 0 && end - beg > longest) return;        // another kernel's row
   float* sp = state + (size_t)state_slots[r] * slot_stride + (size_t)h * vcols * dim;
   float S[CPT][EPL];
 #pragma unroll
@@ -119,6 +122,17 @@ __global__ void __launch_bounds__(kScanThreads) decay_scan_kernel(
         const bool in = e < dim;
         float qv = in ? to_f32(q[(size_t)(t0 + tt) * q_stride + (size_t)g * dim + e]) : 0.f;
         float kv = in ? to_f32(k[(size_t)(t0 + tt) * k_stride + (size_t)g * dim + e]) : 0.f;
+        if (ROT && e < rotary_dim) {
+          const int half = rotary_dim >> 1;
+          const bool first = e < half;
+          const int o = first ? e + half : e - half;
+          const float qo = to_f32(q[(size_t)(t0 + tt) * q_stride + (size_t)g * dim + o]);
+          const float ko = to_f32(k[(size_t)(t0 + tt) * k_stride + (size_t)g * dim + o]);
+          float sn, cs;
+          sincosf((float)positions[t0 + tt] * inv_freq[first ? e : o], &sn, &cs);
+          qv = first ? qv * cs - qo * sn : qv * cs + qo * sn;
+          kv = first ? kv * cs - ko * sn : kv * cs + ko * sn;
+        }
         if (act) {
           qv = qv / (1.0f + expf(-qv));
           kv = kv / (1.0f + expf(-kv));
@@ -198,13 +212,14 @@ template <typename T, int EPL, int CPT>
 static int launch_scan_as(const void* q, const void* k, const void* v, int q_stride, int k_stride, int v_stride, const float* a,
                           const float* b, float* state, long slot_stride, const int* q_indptr, const int* state_slots, float* out,
                           int R, int H, int kq_heads, int dim, int vdim, int ones_col, float q_scale, int lpc, int ab_stride, int act, bool ahead,
-                          cudaStream_t s) {
+                          const int* positions, const float* inv_freq, int rotary_dim, int longest, cudaStream_t s) {
   const int cpb = kScanThreads / lpc * CPT;
   const int vcols = vdim + ones_col;
   const size_t smem = ((size_t)2 * kScanChunk * lpc * EPL + (size_t)kScanChunk * cpb + kScanChunk) * sizeof(float);
   if (smem > 200 * 1024) return ARLE_E_UNSUPPORTED;
   // four numbers a lane (columns of up to 128) gain from asking ahead; eight a lane were measured slower with it
-  auto kernel = (ahead && EPL == 4) ? decay_scan_kernel<T, EPL, CPT, EPL == 4> : decay_scan_kernel<T, EPL, CPT, false>;
+  auto kernel = rotary_dim ? decay_scan_kernel<T, EPL, CPT, false, true>
+                : (ahead && EPL == 4) ? decay_scan_kernel<T, EPL, CPT, EPL == 4, false> : decay_scan_kernel<T, EPL, CPT, false, false>;
   if (smem > 40 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
@@ -212,7 +227,7 @@ static int launch_scan_as(const void* q, const void* k, const void* v, int q_str
   dim3 grid((vcols + cpb - 1) / cpb, H, R);
   launch_kernel(kernel, dim3(grid), dim3(kScanThreads), smem, s, 1, (const T*)q, (const T*)k, (const T*)v,
                 q_stride, k_stride, v_stride, a, b, state, slot_stride, q_indptr, state_slots, out, H, kq_heads, dim, vdim, ones_col,
-                q_scale, lpc, ab_stride, act);
+                q_scale, lpc, ab_stride, act, positions, inv_freq, rotary_dim, longest);
   return launch_status();
 }
 
@@ -221,34 +236,39 @@ static int launch_scan_as(const void* q, const void* k, const void* v, int q_str
 template <typename T, int EPL>
 static int launch_scan(const void* q, const void* k, const void* v, int q_stride, int k_stride, int v_stride, const float* a,
                        const float* b, float* state, long slot_stride, const int* q_indptr, const int* state_slots, float* out,
-                       int R, int H, int kq_heads, int dim, int vdim, int ones_col, float q_scale, int ab_stride, int act, bool ahead, cudaStream_t s) {
+                       int R, int H, int kq_heads, int dim, int vdim, int ones_col, float q_scale, int ab_stride, int act, bool ahead,
+                       const int* positions, const float* inv_freq, int rotary_dim, int longest, cudaStream_t s) {
   int lpc = 1;
   while (lpc * EPL < dim) lpc <<= 1;
   const int wide = kScanThreads / lpc * 4;
   const long blocks_wide = (long)((vdim + ones_col + wide - 1) / wide) * H * R;
   if (blocks_wide >= 148)
     return launch_scan_as<T, EPL, 4>(q, k, v, q_stride, k_stride, v_stride, a, b, state, slot_stride, q_indptr, state_slots, out, R, H,
-                                     kq_heads, dim, vdim, ones_col, q_scale, lpc, ab_stride, act, ahead, s);
+                                     kq_heads, dim, vdim, ones_col, q_scale, lpc, ab_stride, act, ahead, positions, inv_freq, rotary_dim, longest, s);
   return launch_scan_as<T, EPL, 1>(q, k, v, q_stride, k_stride, v_stride, a, b, state, slot_stride, q_indptr, state_slots, out, R, H,
-                                   kq_heads, dim, vdim, ones_col, q_scale, lpc, ab_stride, act, ahead, s);
+                                   kq_heads, dim, vdim, ones_col, q_scale, lpc, ab_stride, act, ahead, positions, inv_freq, rotary_dim, longest, s);
 }
 
 // q, k [T, kq_heads*dim] and v [T, H*vdim] in the activation type (row strides given); a, b float32 [T, H] (ab_stride = H), or
 // one number a head for all tokens (ab_stride = 0: a float32 [H], b float32 [H] or null for ones: a memory with a constant
 // decay per head); act 1: silu on q, k and v as they are staged; long_rows: the step's rows are mostly longer than a chunk of
 // 16 tokens (a hint: the variant that asks for the next chunk ahead is launched); state: float32,
+// rotary_dim > 0: positions int32 [T] and inv_freq float32 [rotary_dim / 2] (not with act); longest > 0: rows of more tokens than
+// that are left alone (another kernel runs them);
 // a slot every slot_stride numbers, [H][vdim + ones_col][dim] at its start; out float32 [T, H, vdim + ones_col].
 ARLE_API int arle_decay_scan(const void* q, const void* k, const void* v, int dtype, int q_stride, int k_stride, int v_stride,
                              const float* a, const float* b, float* state, long slot_stride, const int* q_indptr,
                              const int* state_slots, float* out, int R, int H, int kq_heads, int dim, int vdim, int ones_col,
-                             float q_scale, int ab_stride, int act, int long_rows, cudaStream_t s) {
+                             float q_scale, int ab_stride, int act, int long_rows, const int* positions, const float* inv_freq,
+                             int rotary_dim, int longest, cudaStream_t s) {
   if (R <= 0) return 0;
   if (!a || (ab_stride != 0 && ab_stride != H) || (act != 0 && act != 1)) return ARLE_E_BADARG;
   if (H <= 0 || kq_heads <= 0 || H % kq_heads || dim <= 0 || vdim <= 0 || H > 65535 || R > 65535) return ARLE_E_BADARG;
   if (dim > 32 * 16) return ARLE_E_UNSUPPORTED;
+  if (rotary_dim < 0 || rotary_dim % 2 || rotary_dim > dim || (rotary_dim && (!positions || !inv_freq || act))) return ARLE_E_BADARG;
 #define ARLE_SCAN(TT, E) \
   return launch_scan<TT, E>(q, k, v, q_stride, k_stride, v_stride, a, b, state, slot_stride, q_indptr, state_slots, out, R, H, \
-                            kq_heads, dim, vdim, ones_col, q_scale, ab_stride, act, long_rows != 0, s)
+                            kq_heads, dim, vdim, ones_col, q_scale, ab_stride, act, long_rows != 0, positions, inv_freq, rotary_dim, longest, s)
   // numbers of a column a lane holds: 4 up to 128 (eight at 128, with 16 lanes a column, measured 1.25 to 2 times slower)
   if (dtype == 0) {
     if (dim <= 128) ARLE_SCAN(float, 4);

@@ -39,9 +39,9 @@ def add_launches(n: int) -> None:
 
 _P, _I, _F = c_void_p, c_int, c_float
 _SIGNATURES = {
-    "arle_embedding": [_P, _P, _I, _P, _I, _I, _I, _P, _P, _P, _F, _P],
-    "arle_rmsnorm": [_P, _P, _P, _P, _P, _I, _I, _I, _F, _I, _P],
-    "arle_residual_add": [_P, _P, _I, _I, _I, _P],
+    "arle_embedding": [_P, _P, _I, _P, _I, _I, _I, _P, _P, _P, _F, _P, _I, _P, _P, _P],
+    "arle_rmsnorm": [_P, _P, _P, _P, _P, _I, _I, _I, _F, _I, _F, _P, _P],
+    "arle_residual_add": [_P, _P, _I, _I, _I, _F, _P],
     "arle_silu_mul": [_P, _P, _I, _I, _I, _P],
     "arle_act_mul": [_P, _P, _I, _I, _I, _I, _I, _P],
     "arle_attention_prep_row": [_P, _I, _I, _P, _P, _P, _P, _F, _P, _P, _I, _I, _I, _P, _P, _I, _I, _I, _I, _I, _I, _P],
@@ -51,10 +51,10 @@ _SIGNATURES = {
     "arle_gla_decay": [_P, _I, _I, _P, _P, _F, _P, _I, _I, _I, _I, _P],
     "arle_gla_scan": [_P, _P, _P, _I, _I, _P, _P, _P, ctypes.c_long, _P, _P, _P, _I, _I, _I, _I, _F, _I, _P],
     "arle_gla_out": [_P, _P, _I, _I, _P, _F, _F, _P, _I, _I, _I, _I, _I, _I, _P],
-    "arle_attention_prep": [_P, _I, _I, _P, _P, _P, _P, _F, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P],
+    "arle_attention_prep": [_P, _I, _I, _P, _P, _P, _P, _F, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P, _P],
     "arle_rotary_angles": [_P, _P, _P, _I, _I, _P],
-    "arle_paged_attention_plain": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _F, _I, _F, _I, _P, _I, _P],
-    "arle_attention_prep_post": [_P, _I, _I, _P, _P, _P, _P, _F, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
+    "arle_paged_attention_plain": [_P, _I, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P, _I, _I, _F, _I, _P, _I, _P],
+    "arle_attention_prep_post": [_P, _I, _I, _P, _P, _P, _P, _F, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P],
     "arle_branch_norm_add": [_P, _P, _I, _P, _P, _I, _I, _I, _F, _P],
     "arle_branch_norm_add_norm": [_P, _P, _I, _P, _P, _P, _I, _I, _I, _F, _F, _P],
     "arle_rms_rows": [_P, _I, _I, _P, _P, _I, _I, _I, _I, _F, _P],
@@ -65,21 +65,21 @@ _SIGNATURES = {
     "arle_delta_gates": [_P, _I, _P, _P, _P, _P, _I, _I, _P],
     "arle_delta_scan": [_P, _P, _P, _I, _I, _I, _I, _P, _P, _P, ctypes.c_long, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _P],
     "arle_clamped_glu": [_P, _P, _I, _I, _I, _I, _F, _F, _P],
-    "arle_paged_attention_decode": [_P, _I, _P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _F, _F, _I, _I, _I, _I, _F, _I, _P, _P],
+    "arle_paged_attention_decode": [_P, _I, _P, _P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _F, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P, _P],
     "arle_paged_attention_decode_stream": [_P, _I, _P, _P, _P, ctypes.c_longlong, _P, _P, _P, _I, _I, _P, _P, _P, _I, _I, _I, _I,
-                                           _F, _F, _I, _I, _I, _P, _P],
+                                           _F, _P, _P, _I, _I, _I, _I, _P, _P],
     "arle_paged_attention_decode_stream_prep": [_P, _I, _P, _P, _P, ctypes.c_longlong, _P, _P, _P, _I, _I, _P, _P, _P, _I, _I, _I, _I,
-                                                _F, _F, _I, _I, _I, _I, _P, _P, _P, _F, _P, _P, _P, _P],
+                                                _F, _P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _F, _P, _I, _P, _P, _P, _P],
     "arle_decode_stream_plan_ints": [_I, _I],
     "arle_decode_stream_plan": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P],
-    "arle_paged_attention_prefill": [_P, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _I, _I, _I, _I, _I, _F, _I, _P, _P],
-    "arle_paged_attention_prefill_tc": [_P, _I, _I, _P, _P, _P, ctypes.c_longlong, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _I,
+    "arle_paged_attention_prefill": [_P, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P],
+    "arle_paged_attention_prefill_tc": [_P, _I, _I, _P, _P, _P, ctypes.c_longlong, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _P, _P, _I, _I,
                                         _I, _I, _I, _P, _I, _F, _I, _P, _P],
     "arle_gemm_f32": [_P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _P],
     "arle_gemm_plain_bf16": [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
     "arle_gemm_skinny": [_P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _P, _P],
     "arle_gemm_skinny_gated": [_P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _P, _P],
-    "arle_gemm_skinny_fused": [_P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _P, _F, _F, _P, _I, _P, _P, _I, _P, _P, _P],
+    "arle_gemm_skinny_fused": [_P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _P, _F, _F, _P, _I, _P, _P, _I, _P, _F, _P, _P, _P],
     "arle_gemm_tcgen05": [_P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _P, _P],
     "arle_gemm_tcgen05_pair": [_P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _P, _P],
     "arle_argmax": [_P, _I, _I, _I, _P, _P, _P, _P, _P],
@@ -91,7 +91,7 @@ _SIGNATURES = {
     "arle_latent_prep": [_P, _I, _P, _I, _I, _P, _P, _P, _F, _P, _I, _I, _F, _P, _P, _I, _I, _I, _I, _I, _P],
     "arle_latent_attention_mma": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P],
     "arle_latent_attention": [_P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P],
-    "arle_decay_scan": [_P, _P, _P, _I, _I, _I, _I, _P, _P, _P, ctypes.c_long, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P],
+    "arle_decay_scan": [_P, _P, _P, _I, _I, _I, _I, _P, _P, _P, ctypes.c_long, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P, _P, _I, _I, _P],
     "arle_mlstm_gates": [_P, _I, _P, _P, _F, _P, _P, _P, ctypes.c_long, ctypes.c_long, _P, _P, _P, _I, _I, _P],
     "arle_mlstm_out": [_P, _P, _P, _I, _I, _P, _F, _P, _I, _I, _I, _I, _P],
     "arle_ssm_gates": [_P, _I, _P, _P, _P, _P, _I, _I, _P],
@@ -245,10 +245,12 @@ def _i32(t, name):
 
 # ------------------------------------------------------------------- embedding
 def embedding(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, err: torch.Tensor = None,
-              last_token: torch.Tensor = None, slot_of_token: torch.Tensor = None, scale: float = 1.0) -> None:
+              last_token: torch.Tensor = None, slot_of_token: torch.Tensor = None, scale: float = 1.0, pos_table: torch.Tensor = None,
+              positions: torch.Tensor = None, out2: torch.Tensor = None) -> None:
     """out[t, :] = float32(table[ids[t], :]) * scale.  ids int32 [T]; out float32 [T, H].  With
     ``last_token`` (int32, one entry per request slot) and ``slot_of_token`` (int32 [T]) a
-    negative id stands for last_token[slot_of_token[t]], the token the request sampled last."""
+    negative id stands for last_token[slot_of_token[t]], the token the request sampled last.  ``pos_table`` [positions, H] (the
+    table's type) with ``positions`` int32 [T]: pos_table[positions[t], :] is added (unscaled).  ``out2``: the same rows once more."""
     T, H = out.shape
     if out.dtype != torch.float32 or not out.is_contiguous() or not table.is_contiguous():
         raise KernelError("embedding: out must be contiguous float32 and the table contiguous")
@@ -259,15 +261,22 @@ def embedding(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, err: to
         _i32(last_token, "last_token"), _i32(slot_of_token, "slot_of_token")
         if slot_of_token is None or slot_of_token.numel() != T:
             raise KernelError("embedding: slot_of_token must name a slot for every token")
+    if pos_table is not None:
+        _i32(positions, "positions")
+        if pos_table.dtype != table.dtype or pos_table.dim() != 2 or pos_table.shape[1] != H or not pos_table.is_contiguous() or positions is None or positions.numel() != T:
+            raise KernelError("embedding: the position table must be contiguous [positions, H] in the table's type, with a position per token")
+    if out2 is not None and (out2.dtype != torch.float32 or out2.shape != out.shape or not out2.is_contiguous()):
+        raise KernelError("embedding: out2 must be like out")
     _check(library().arle_embedding(_ptr(ids), _ptr(table), _dt(table), _ptr(out), T, H, table.shape[0],
                                     _ptr(err), _ptr(last_token), _ptr(slot_of_token) if last_token is not None else None,
-                                    float(scale), _stream()), "embedding")
+                                    float(scale), _ptr(pos_table), pos_table.shape[0] if pos_table is not None else 0,
+                                    _ptr(positions) if pos_table is not None else None, _ptr(out2), _stream()), "embedding")
 
 
 # ------------------------------------------------------------------------ norm
-def rmsnorm(resid, delta, rows, weight, eps: float, out, write_resid: bool) -> None:
-    """For output row i (source row r = rows[i], or i): x = resid[r] (+ delta[r]);
-    resid[r] = x when write_resid; out[i] = x * rsqrt(mean(x^2) + eps) * weight.
+def rmsnorm(resid, delta, rows, weight, eps: float, out, write_resid: bool, delta_scale: float = 1.0, extra=None) -> None:
+    """For output row i (source row r = rows[i], or i): x = resid[r] (+ delta_scale * delta[r]) (+ extra[r], float32 like the
+    residual); resid[r] = x when write_resid; out[i] = x * rsqrt(mean(x^2) + eps) * weight.
     resid float32 [N, H]; delta and out in the activation type; weight float32 [H]."""
     H = resid.shape[1]
     n_out = out.shape[0]
@@ -277,6 +286,8 @@ def rmsnorm(resid, delta, rows, weight, eps: float, out, write_resid: bool) -> N
         raise KernelError("rmsnorm: bad shapes or strides")
     if delta is not None and (delta.dtype != out.dtype or delta.shape != resid.shape or not delta.is_contiguous()):
         raise KernelError("rmsnorm: delta must match the residual's shape and the output's type")
+    if extra is not None and (extra.dtype != torch.float32 or extra.shape != resid.shape or not extra.is_contiguous()):
+        raise KernelError("rmsnorm: extra must be float32 rows like the residual")
     if rows is not None:
         _i32(rows, "rows")
         if rows.numel() != n_out:
@@ -284,14 +295,14 @@ def rmsnorm(resid, delta, rows, weight, eps: float, out, write_resid: bool) -> N
     elif n_out != resid.shape[0]:
         raise KernelError("rmsnorm: output rows must match residual rows when no row list is given")
     _check(library().arle_rmsnorm(_ptr(resid), _ptr(delta), _ptr(rows), _ptr(weight), _ptr(out), _dt(out), n_out, H,
-                                  float(eps), int(bool(write_resid)), _stream()), "rmsnorm")
+                                  float(eps), int(bool(write_resid)), float(delta_scale), _ptr(extra), _stream()), "rmsnorm")
 
 
-def residual_add(resid, delta) -> None:
-    """resid += delta (float32 residual, delta in the activation type)."""
+def residual_add(resid, delta, scale: float = 1.0) -> None:
+    """resid += scale * delta (float32 residual, delta in the activation type or float32)."""
     if resid.dtype != torch.float32 or resid.shape != delta.shape or not (resid.is_contiguous() and delta.is_contiguous()):
         raise KernelError("residual_add: residual float32, same contiguous shape as delta")
-    _check(library().arle_residual_add(_ptr(resid), _ptr(delta), _dt(delta), resid.shape[0], resid.shape[1], _stream()),
+    _check(library().arle_residual_add(_ptr(resid), _ptr(delta), _dt(delta), resid.shape[0], resid.shape[1], float(scale), _stream()),
            "residual_add")
 
 
@@ -301,13 +312,14 @@ SS_TABLE_SHAPE = (16, 192)          # a sum-of-squares table of the fused produc
 
 class ResidualSink:
     """Where a product's result goes instead of an output tensor, so that the norm that follows
-    needs no kernel: the sums are added into ``resid`` (float32 [M, N], in place), ``xs`` gets
+    needs no kernel: ``scale`` times the sums (and ``extra``, float32 rows like the residual's, where given) are added into ``resid`` (float32 [M, N], in place), ``xs`` gets
     bfloat16(resid * gamma) (the norm's output without its per-row factor) and ``ss`` (float32
     ``SS_TABLE_SHAPE``) the sums of squares of the new residual rows, spread over slots that the
     reader adds up.  ``eps`` travels with it to the reader."""
 
-    def __init__(self, resid, gamma, eps, xs, ss):
+    def __init__(self, resid, gamma, eps, xs, ss, scale: float = 1.0, extra=None):
         self.resid, self.gamma, self.eps, self.xs, self.ss = resid, gamma, float(eps), xs, ss
+        self.scale, self.extra = float(scale), extra
         self.filled = False
 
 
@@ -356,6 +368,8 @@ def _fused_gemm(x, w, out, gated: bool, scaled: "ScaledRows", sink: "ResidualSin
         r, xs = sink.resid, sink.xs
         if (r.dtype != torch.float32 or tuple(r.shape) != (M, N) or r.stride(1) != 1 or xs.dtype != torch.bfloat16
                 or tuple(xs.shape) != (M, N) or xs.stride(1) != 1 or sink.gamma.dtype != torch.float32
+                or (sink.extra is not None and (sink.extra.dtype != torch.float32 or tuple(sink.extra.shape) != (M, N)
+                                                or sink.extra.stride() != r.stride()))
                 or sink.gamma.numel() != N or tuple(sink.ss.shape) != SS_TABLE_SHAPE or sink.ss.dtype != torch.float32):
             raise KernelError("gemm: residual sink does not fit the product")
     _check(library().arle_gemm_skinny_fused(
@@ -363,6 +377,7 @@ def _fused_gemm(x, w, out, gated: bool, scaled: "ScaledRows", sink: "ResidualSin
         out.stride(0) if out is not None else 0, M, N, K, int(gated), _ptr(in_ss), float(inv_w or 0.0), float(eps or 0.0),
         _ptr(sink.resid) if sink else None, sink.resid.stride(0) if sink else 0, _ptr(sink.gamma) if sink else None,
         _ptr(sink.xs) if sink else None, sink.xs.stride(0) if sink else 0, _ptr(sink.ss) if sink else None,
+        sink.scale if sink else 1.0, _ptr(sink.extra) if sink else None,
         _ptr(error_flag(x.device)), _stream()), "gemm_skinny_fused")
     if sink is not None:
         sink.filled = True
@@ -492,15 +507,18 @@ def rotary_angles(positions, inv_freq, out) -> None:
 def attention_prep_takes_angles(qkv, hd: int, rotary_dim: int) -> bool:
     """Whether ``attention_prep`` would use a table of ``rotary_angles`` for this input (the kernel for
     prompt portions does; the others evaluate the angles themselves)."""
-    return qkv.dtype == torch.bfloat16 and qkv.shape[0] >= 32 and hd in (64, 128) and rotary_dim == hd
+    return (qkv.dtype == torch.bfloat16 and qkv.shape[0] >= 32 and hd in (64, 128)
+            and (rotary_dim == hd or (0 < rotary_dim <= hd // 2 and rotary_dim % 8 == 0)))
 
 
 def attention_prep(qkv, positions, slot_mapping, q_weight, k_weight, eps, inv_freq, rotary_dim, k_cache, v_cache,
-                   nq: int, nkv: int, hd: int, page_size: int, angles=None) -> None:
+                   nq: int, nkv: int, hd: int, page_size: int, angles=None, bias=None) -> None:
     """Per-head q/k RMSNorm (weights float32 [hd] or None), rotary encoding, and the
     store of k and v into the paged cache, in place on qkv [T, (nq + 2 nkv) hd]
     (nkv = 0: the rows hold q only and nothing is stored).  ``angles``: the table of
-    ``rotary_angles`` for these positions and inv_freq, or None."""
+    ``rotary_angles`` for these positions and inv_freq, or None.  ``bias`` (float32 [(nq + 2 nkv) hd]): added to q, k and v first."""
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != (nq + 2 * nkv) * hd or not bias.is_contiguous()):
+        raise KernelError("attention_prep: bias must be float32 [(nq + 2 nkv) hd]")
     T = qkv.shape[0]
     if angles is not None and (angles.dtype != torch.float32 or tuple(angles.shape) != (T, rotary_dim // 2, 2)
                                or not angles.is_contiguous()):
@@ -527,12 +545,12 @@ def attention_prep(qkv, positions, slot_mapping, q_weight, k_weight, eps, inv_fr
         _ptr(qkv), _dt(qkv), qkv.stride(0), _ptr(positions), _ptr(slot_mapping), _ptr(q_weight), _ptr(k_weight),
         float(eps), _ptr(inv_freq) if rotary_dim else None, _ptr(angles) if rotary_dim else None, int(rotary_dim),
         _ptr(k_cache) if nkv else None,
-        _ptr(v_cache) if nkv else None, nq, nkv, hd, page_size, T, _stream()), "attention_prep")
+        _ptr(v_cache) if nkv else None, nq, nkv, hd, page_size, T, _ptr(bias), _stream()), "attention_prep")
 
 
 def paged_attention(q, out, k_cache, v_cache, positions, row_of_token, block_table, nq: int, nkv: int, hd: int,
-                    page_size: int, scale: float, window, batch=None, vd: int = None, sink: float = None, keep_first: int = 0,
-                    softcap: float = None, chunk: int = None, score_bias=None) -> None:
+                    page_size: int, scale: float, window, batch=None, vd: int = None, sink=None, keep_first: int = 0,
+                    softcap: float = None, chunk: int = None, score_bias=None, gate=None) -> None:
     """Causal attention of this step's queries over the paged cache.
 
     ``chunk``: a query sees only the keys of its own chunk of that many positions, counted from position 0 (in a window's
@@ -543,7 +561,9 @@ def paged_attention(q, out, k_cache, v_cache, positions, row_of_token, block_tab
 
     ``vd``: the values' width when it differs from the keys' (the value cache is then [pages, nkv, page_size, vd] and
     out [T, nq*vd]).  ``sink``: the score of a sink without a value that the softmax's denominator counts besides the
-    keys, p_j = exp(s_j) / (exp(sink) + sum exp(s_j)); None for the usual softmax.  Values of another width run on the
+    keys, p_j = exp(s_j) / (exp(sink) + sum exp(s_j)): a number, or a float32 tensor [nq] with one per query head; None for the
+    usual softmax.  ``gate`` ([T, nq], q's type, columns of a wider row are fine): head h's output is multiplied by
+    sigmoid(gate[t, h]).  Values of another width run on the
     general kernel; the sink is one more term at the end of every kernel's sums.
 
     q: [T, nq*hd] view (row stride free, unit inner stride); out: contiguous
@@ -566,6 +586,7 @@ def paged_attention(q, out, k_cache, v_cache, positions, row_of_token, block_tab
     _i32(positions, "positions"), _i32(row_of_token, "row_of_token"), _i32(block_table, "block_table")
     if block_table.stride(1) != 1:
         raise KernelError("paged_attention: block table rows must be contiguous")
+    sink, (gate_p, gate_stride) = _sinks(sink, nq, q.device), _gate_arg(gate, q, nq)
     keep_first = int(keep_first or 0) if window else 0
     chunk = int(chunk or 0)
     if chunk < 0 or (chunk and window) or (score_bias is not None and (sink is not None or score_bias.dtype != torch.float32
@@ -580,7 +601,7 @@ def paged_attention(q, out, k_cache, v_cache, positions, row_of_token, block_tab
             prefill = paged_attention_prefill_tc if tc_attention_supported(q, hd, page_size) else paged_attention_prefill
             prefill(q, out, k_cache, v_cache, batch.q_indptr, batch.kv_lens, block_table, nq, nkv, hd, page_size, scale,
                     window, batch.max_q_len, skip_single=batch.num_single > 0, sink=sink, keep_first=keep_first, softcap=softcap, chunk=chunk,
-                    score_bias=score_bias)
+                    score_bias=score_bias, gate=gate)
         if batch.num_single > 0 and not extended and stream_decode_supported(batch.num_rows, page_size, nq // nkv):
             ctas = sm_count(q.device)
             slots = (ctas + batch.num_rows * nkv) * (nq // nkv)
@@ -588,7 +609,7 @@ def paged_attention(q, out, k_cache, v_cache, positions, row_of_token, block_tab
                 q, out, k_cache, v_cache, batch.q_indptr, batch.kv_lens, block_table, nq, nkv, hd, page_size, scale, window,
                 batch.ws.get("attn_piece_o", (slots * hd,), torch.float32),
                 batch.ws.get("attn_piece_ml", (slots * 2,), torch.float32),
-                batch.ws.get_zeroed("attn_piece_counters", (batch.num_rows * nkv,), torch.int32), ctas, sink=sink)
+                batch.ws.get_zeroed("attn_piece_counters", (batch.num_rows * nkv,), torch.int32), ctas, sink=sink, gate=gate)
         elif batch.num_single > 0:
             bound = block_table.shape[1] * page_size
             if window:
@@ -603,19 +624,40 @@ def paged_attention(q, out, k_cache, v_cache, positions, row_of_token, block_tab
                 counters = batch.ws.get_zeroed("attn_split_counters", (batch.num_rows * nkv,), torch.int32)
             paged_attention_decode(q, out, k_cache, v_cache, batch.q_indptr, batch.kv_lens, block_table, nq, nkv, hd,
                                    page_size, scale, window, splits, part_o, part_ml, counters, sink=sink, keep_first=keep_first,
-                                   softcap=softcap, chunk=chunk, score_bias=score_bias)
+                                   softcap=softcap, chunk=chunk, score_bias=score_bias, gate=gate)
         return
     _check(library().arle_paged_attention_plain(
         _ptr(q), q.stride(0), _ptr(out), _ptr(k_cache), _ptr(v_cache), _dt(q), _ptr(positions), _ptr(row_of_token),
         _ptr(block_table), block_table.stride(0), nq, nkv, hd, vd, page_size, float(scale),
-        int(window) if window else 0, int(sink is not None), float(sink or 0.0), keep_first, float(softcap or 0.0), chunk,
+        int(window) if window else 0, _ptr(sink), gate_p, gate_stride, keep_first, float(softcap or 0.0), chunk,
         _ptr(score_bias), T, _stream()),
         "paged_attention")
 
 
-def _sink_arg(sink) -> float:
-    """The fast attention kernels take the sink's score as a number; minus infinity stands for no sink (its term is zero)."""
-    return float("-inf") if sink is None else float(sink)
+_SINKS: dict = {}
+
+
+def _sinks(sink, nq: int, device):
+    """The attention kernels take a float32 score per query head.  A number stands for the same score in every head (the tensor
+    is made once per device and kept); None for no sink."""
+    if sink is None:
+        return None
+    if isinstance(sink, torch.Tensor):
+        if sink.dtype != torch.float32 or sink.numel() != nq or not sink.is_contiguous():
+            raise KernelError("attention: sinks must be contiguous float32, one per query head")
+        return sink
+    key = (float(sink), nq, str(device))
+    if key not in _SINKS:
+        _SINKS[key] = torch.full((nq,), float(sink), dtype=torch.float32, device=device)
+    return _SINKS[key]
+
+
+def _gate_arg(gate, q, nq: int):
+    if gate is None:
+        return None, 0
+    if gate.dtype != q.dtype or tuple(gate.shape) != (q.shape[0], nq) or gate.stride(1) != 1:
+        raise KernelError("attention: gate must be [T, nq] in q's type with unit inner stride")
+    return _ptr(gate), gate.stride(0)
 
 
 def fast_attention_supported(q, nq: int, nkv: int, hd: int) -> bool:
@@ -632,8 +674,8 @@ def tc_attention_supported(q, hd: int, page_size: int) -> bool:
 
 
 def paged_attention_prefill_tc(q, out, k_cache, v_cache, q_indptr, kv_lens, block_table, nq, nkv, hd, page_size, scale,
-                               window, max_q_len: int, skip_single: bool = False, sink: float = None, keep_first: int = 0,
-                               softcap: float = None, chunk: int = 0, score_bias=None) -> None:
+                               window, max_q_len: int, skip_single: bool = False, sink=None, keep_first: int = 0,
+                               softcap: float = None, chunk: int = 0, score_bias=None, gate=None) -> None:
     """Flash attention over the paged cache on the tcgen05 tensor cores (TMA-fed, scores
     and output in tensor memory) for rows with several queries."""
     R = kv_lens.numel()
@@ -643,7 +685,8 @@ def paged_attention_prefill_tc(q, out, k_cache, v_cache, q_indptr, kv_lens, bloc
     _check(library().arle_paged_attention_prefill_tc(
         _ptr(q), q.stride(0), q.shape[0], _ptr(out), _ptr(k_cache), _ptr(v_cache), k_cache.shape[0], _ptr(q_indptr),
         _ptr(kv_lens), _ptr(block_table), block_table.stride(0), block_table.shape[1], nq, nkv, hd, page_size, float(scale),
-        _sink_arg(sink), int(window) if window else 0, R, int(max_q_len), int(bool(skip_single)), _ptr(error_flag(q.device)),
+        _ptr(_sinks(sink, nq, q.device)), *_gate_arg(gate, q, nq), int(window) if window else 0, R, int(max_q_len), int(bool(skip_single)),
+        _ptr(error_flag(q.device)),
         int(keep_first or 0), float(softcap or 0.0), int(chunk or 0), _ptr(score_bias), _stream()), "paged_attention_prefill_tc")
 
 
@@ -666,7 +709,7 @@ def stream_decode_supported(rows: int, page_size: int, group: int = 1) -> bool:
 
 
 def paged_attention_decode_stream(q, out, k_cache, v_cache, q_indptr, kv_lens, block_table, nq, nkv, hd, page_size, scale,
-                                  window, piece_o, piece_ml, counters, ctas: int, sink: float = None) -> None:
+                                  window, piece_o, piece_ml, counters, ctas: int, sink=None, gate=None) -> None:
     """Attention of the rows that have exactly one query (others are skipped), as a
     resident grid of ``ctas`` CTAs that share the batch's 64-key tiles evenly.
     Scratch: piece_o float32 [(ctas + R*nkv) * (nq/nkv) * hd], piece_ml float32
@@ -686,28 +729,34 @@ def paged_attention_decode_stream(q, out, k_cache, v_cache, q_indptr, kv_lens, b
     _check(library().arle_paged_attention_decode_stream(
         _ptr(q), q.stride(0), _ptr(out), _ptr(k_cache), _ptr(v_cache), k_cache.shape[0], _ptr(q_indptr), _ptr(kv_lens),
         _ptr(block_table), block_table.stride(0), block_table.shape[1], _ptr(piece_o), _ptr(piece_ml), _ptr(counters),
-        nq, nkv, hd, page_size, float(scale), _sink_arg(sink), int(window) if window else 0, R, int(ctas), _ptr(error_flag(q.device)),
-        _stream()), "paged_attention_decode_stream")
+        nq, nkv, hd, page_size, float(scale), _ptr(_sinks(sink, nq, q.device)), *_gate_arg(gate, q, nq), int(window) if window else 0, R,
+        int(ctas), _ptr(error_flag(q.device)), _stream()), "paged_attention_decode_stream")
 
 
 def fused_decode_supported(qkv, batch, cache_dtype, nq: int, nkv: int, hd: int, page_size: int, rotary_dim: int) -> bool:
     """Whether a step's attention can run as ONE launch that also prepares the queries and the new keys
     (``decode_attention_with_prep``): every row of the step one decoded token, bfloat16, the shapes the
-    streaming kernel takes, and a rotation of the whole head or none."""
+    streaming kernel takes, and a rotation of a multiple of head_dim / 16 numbers."""
     return (_KERNEL_SET == "fast" and batch is not None and batch.max_q_len == 1 and qkv.is_cuda
             and qkv.dtype == torch.bfloat16 and cache_dtype == torch.bfloat16 and hd in (64, 128) and nq % nkv == 0
-            and nq // nkv <= 16 and rotary_dim in (0, hd) and stream_decode_supported(batch.num_rows, page_size, nq // nkv)
+            and nq // nkv <= 16 and rotary_dim % (hd // 16) == 0 and stream_decode_supported(batch.num_rows, page_size, nq // nkv)
             and qkv.stride(1) == 1 and qkv.stride(0) % 8 == 0 and qkv.data_ptr() % 16 == 0)
 
 
 def decode_attention_with_prep(qkv, out, k_cache, v_cache, slot_mapping, q_weight, k_weight, eps: float, inv_freq,
-                               block_table, nq: int, nkv: int, hd: int, page_size: int, scale: float, window, batch) -> None:
+                               block_table, nq: int, nkv: int, hd: int, page_size: int, scale: float, window, batch, rotary_dim: int = None,
+                               bias=None, sink=None, gate=None) -> None:
     """Attention of a step in which every row is one decoded token, from the raw projection output
     qkv [T, (nq + 2 nkv) hd]: per-head norm and rotation of the queries and of the new keys, the store of
     the new keys and values into the cache, and the attention over the cache, in one launch of the
-    streaming kernel.  ``q_weight`` / ``k_weight`` None: no norm; ``inv_freq`` None: no rotation."""
+    streaming kernel.  ``q_weight`` / ``k_weight`` None: no norm; ``inv_freq`` None: no rotation; ``rotary_dim``: the first numbers
+    of a head that turn (None: all); ``bias`` (float32 [(nq + 2 nkv) hd]): added to q, k and v first; ``sink`` and ``gate`` as in
+    ``paged_attention``."""
     T = qkv.shape[0]
-    if not fused_decode_supported(qkv, batch, k_cache.dtype, nq, nkv, hd, page_size, hd if inv_freq is not None else 0):
+    rotary_dim = 0 if inv_freq is None else hd if rotary_dim is None else int(rotary_dim)
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != (nq + 2 * nkv) * hd or not bias.is_contiguous()):
+        raise KernelError("decode_attention_with_prep: bias must be float32 [(nq + 2 nkv) hd]")
+    if not fused_decode_supported(qkv, batch, k_cache.dtype, nq, nkv, hd, page_size, rotary_dim):
         raise KernelError("decode_attention_with_prep: this step or these shapes need the separate preparation kernel")
     if out.shape != (T, nq * hd) or not out.is_contiguous() or out.dtype != torch.bfloat16 or qkv.shape[1] < (nq + 2 * nkv) * hd:
         raise KernelError("decode_attention_with_prep: out must be contiguous bfloat16 [T, nq*hd] and qkv hold q, k and v heads")
@@ -717,8 +766,8 @@ def decode_attention_with_prep(qkv, out, k_cache, v_cache, slot_mapping, q_weigh
     for w_ in (q_weight, k_weight):
         if w_ is not None and (w_.dtype != torch.float32 or w_.numel() != hd):
             raise KernelError("decode_attention_with_prep: norm weights must be float32 [head_dim]")
-    if inv_freq is not None and (inv_freq.dtype != torch.float32 or inv_freq.numel() != hd // 2):
-        raise KernelError("decode_attention_with_prep: inv_freq must be float32 [head_dim / 2]")
+    if inv_freq is not None and (inv_freq.dtype != torch.float32 or inv_freq.numel() != rotary_dim // 2):
+        raise KernelError("decode_attention_with_prep: inv_freq must be float32 [rotary_dim / 2]")
     _i32(slot_mapping, "slot_mapping"), _i32(block_table, "block_table")
     R, G = batch.num_rows, nq // nkv
     ctas = sm_count(qkv.device)
@@ -745,8 +794,8 @@ def decode_attention_with_prep(qkv, out, k_cache, v_cache, slot_mapping, q_weigh
     _check(library().arle_paged_attention_decode_stream_prep(
         _ptr(qkv), qkv.stride(0), _ptr(out), _ptr(k_cache), _ptr(v_cache), k_cache.shape[0], _ptr(batch.q_indptr),
         _ptr(batch.kv_lens), _ptr(block_table), block_table.stride(0), block_table.shape[1], _ptr(piece_o), _ptr(piece_ml),
-        _ptr(counters), nq, nkv, hd, page_size, float(scale), _sink_arg(None), int(window) if window else 0, R, int(ctas), 1,
-        _ptr(slot_mapping), _ptr(q_weight), _ptr(k_weight), float(eps), _ptr(inv_freq), _ptr(plan),
+        _ptr(counters), nq, nkv, hd, page_size, float(scale), _ptr(_sinks(sink, nq, qkv.device)), *_gate_arg(gate, qkv, nq), int(window) if window else 0, R,
+        int(ctas), 1, _ptr(slot_mapping), _ptr(q_weight), _ptr(k_weight), float(eps), _ptr(inv_freq), rotary_dim, _ptr(bias), _ptr(plan),
         _ptr(error_flag(qkv.device)), _stream()), "decode_attention_with_prep")
 
 
@@ -762,8 +811,8 @@ def decode_splits(rows: int, nkv: int, kv_bound: int, device=None) -> int:
 
 
 def paged_attention_decode(q, out, k_cache, v_cache, q_indptr, kv_lens, block_table, nq, nkv, hd, page_size, scale,
-                           window, splits: int, part_o=None, part_ml=None, counters=None, sink: float = None, keep_first: int = 0,
-                           softcap: float = None, chunk: int = 0, score_bias=None) -> None:
+                           window, splits: int, part_o=None, part_ml=None, counters=None, sink=None, keep_first: int = 0,
+                           softcap: float = None, chunk: int = 0, score_bias=None, gate=None) -> None:
     """Split-KV attention of the rows that have exactly one query (others are
     skipped).  q_indptr int32 [R+1], kv_lens int32 [R] (keys after this step).
     When splits > 1: part_o / part_ml are float32 scratch of R*nq*splits*hd and
@@ -778,13 +827,14 @@ def paged_attention_decode(q, out, k_cache, v_cache, q_indptr, kv_lens, block_ta
     _check(library().arle_paged_attention_decode(
         _ptr(q), q.stride(0), _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(q_indptr), _ptr(kv_lens),
         _ptr(block_table), block_table.stride(0), _ptr(part_o), _ptr(part_ml), _ptr(counters), nq, nkv, hd, page_size,
-        float(scale), _sink_arg(sink), int(window) if window else 0, R, int(splits), int(keep_first or 0), float(softcap or 0.0),
+        float(scale), _ptr(_sinks(sink, nq, q.device)), *_gate_arg(gate, q, nq), int(window) if window else 0, R, int(splits),
+        int(keep_first or 0), float(softcap or 0.0),
         int(chunk or 0), _ptr(score_bias), _stream()), "paged_attention_decode")
 
 
 def paged_attention_prefill(q, out, k_cache, v_cache, q_indptr, kv_lens, block_table, nq, nkv, hd, page_size, scale,
-                            window, max_q_len: int, skip_single: bool = False, sink: float = None, keep_first: int = 0,
-                            softcap: float = None, chunk: int = 0, score_bias=None) -> None:
+                            window, max_q_len: int, skip_single: bool = False, sink=None, keep_first: int = 0,
+                            softcap: float = None, chunk: int = 0, score_bias=None, gate=None) -> None:
     """Flash-attention over the paged cache for rows with several queries (and,
     unless skip_single, for single-query rows too)."""
     R = kv_lens.numel()
@@ -792,7 +842,8 @@ def paged_attention_prefill(q, out, k_cache, v_cache, q_indptr, kv_lens, block_t
     _check(library().arle_paged_attention_prefill(
         _ptr(q), q.stride(0), _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(q_indptr), _ptr(kv_lens),
         _ptr(block_table), block_table.stride(0), nq, nkv, hd, page_size, float(scale),
-        _sink_arg(sink), int(window) if window else 0, R, int(max_q_len), int(bool(skip_single)), int(keep_first or 0),
+        _ptr(_sinks(sink, nq, q.device)), *_gate_arg(gate, q, nq), int(window) if window else 0, R, int(max_q_len), int(bool(skip_single)),
+        int(keep_first or 0),
         float(softcap or 0.0), int(chunk or 0), _ptr(score_bias), _stream()), "paged_attention_prefill")
 
 
@@ -1227,8 +1278,20 @@ def latent_attention(q_abs, out, cache, positions, row_of_token, block_table, ra
 
 
 # ------------------------------------------------------------------ matrix memories with a scalar decay
+def _rotation_args(rotation, T: int, dim: int, act: str):
+    if rotation is None:
+        return None, None, 0
+    positions, inv_freq, rdim = rotation
+    if not rdim:
+        return None, None, 0
+    _i32(positions, "positions")
+    if (positions.numel() != T or inv_freq.dtype != torch.float32 or inv_freq.numel() != rdim // 2 or rdim % 2 or rdim > dim or act != "none"):
+        raise KernelError("a memory's rotation takes a position per token, float32 frequencies [rotary_dim / 2], and goes without an activation")
+    return _ptr(positions), _ptr(inv_freq), int(rdim)
+
+
 def decay_scan(q, k, v, a, b, state, q_indptr, state_slots, out, heads: int, kq_heads: int, dim: int, vdim: int,
-               ones_column: bool, q_scale: float, act: str = "none") -> None:
+               ones_column: bool, q_scale: float, act: str = "none", rotation=None, longest: int = 0) -> None:
     """S_t = a_t S_(t-1) + b_t k_t v_t^T, o_t = S_t^T (q_t * q_scale) over the tokens of every row of the step (row r owns
     tokens q_indptr[r] .. q_indptr[r+1]-1), from and into state[state_slots[r]].  q, k [T, kq_heads*dim] (head h reads
     head h // (heads / kq_heads)), v [T, heads*vdim], in the activation type (views of wider rows are fine); a, b float32
@@ -1236,7 +1299,8 @@ def decay_scan(q, k, v, a, b, state, q_indptr, state_slots, out, heads: int, kq_
     ([heads][vcols][dim]); vcols = vdim + 1 with ``ones_column`` (a column of ones beside v: it carries sum a..b k, the
     normaliser of a matrix LSTM); out float32 [T, heads, vcols].  A memory whose decay is one constant per head gives a as
     float32 [heads] and b as float32 [heads] or None (ones).  ``act`` "silu": q, k and v go through silu as the kernel
-    reads them."""
+    reads them.  ``rotation`` (positions int32 [T], inv_freq float32, rotary_dim): q and k turn first (half-split pairs of a head's
+    first rotary_dim numbers), in float32 as the kernel reads them.  ``longest``: rows of more tokens are left alone (0: none)."""
     T = v.shape[0]
     R = state_slots.numel()
     vcols = vdim + int(bool(ones_column))
@@ -1261,7 +1325,7 @@ def decay_scan(q, k, v, a, b, state, q_indptr, state_slots, out, heads: int, kq_
     _check(library().arle_decay_scan(_ptr(q), _ptr(k), _ptr(v), _dt(q), q.stride(0), k.stride(0), v.stride(0), _ptr(a), _ptr(b),
                                      _ptr(state), state.stride(0), _ptr(q_indptr), _ptr(state_slots), _ptr(out), R, heads, kq_heads,
                                      dim, vdim, vcols - vdim, float(q_scale), 0 if per_head else heads, int(act == "silu"), int(T > 16 * R),
-                                     _stream()),
+                                     *_rotation_args(rotation, T, dim, act), int(longest), _stream()),
            "decay_scan")
 
 
@@ -1556,11 +1620,14 @@ def bias_add(x, bias) -> None:
 
 
 def attention_prep_post(qkv, positions, slot_mapping, q_weight, k_weight, eps, inv_freq, rotary_dim: int, k_cache, v_cache,
-                        nq: int, nkv: int, hd: int, vd: int, page_size: int, norm_first: bool = False) -> None:
+                        nq: int, nkv: int, hd: int, vd: int, page_size: int, norm_first: bool = False, bias=None) -> None:
     """(``norm_first``: the norm and its weight come before the rotation instead of after it.)  Rotation first, then the per-head norm x / sqrt(mean(x^2) + eps) (times a weight float32 [hd], or none), in place on
     the q heads of qkv [T, nq*hd + nkv*hd + nkv*vd]; the k heads go the same way into k_cache [pages, nkv, page_size, hd]
     and the v heads as they are into v_cache [pages, nkv, page_size, vd] (nkv = 0: the rows hold q only and nothing is
-    stored).  ``eps`` None: no norm.  Rotation as in ``attention_prep`` (number i with i + rotary_dim/2)."""
+    stored).  ``eps`` None: no norm.  Rotation as in ``attention_prep`` (number i with i + rotary_dim/2).  ``bias`` (float32
+    [(nq + nkv) hd + nkv vd]): added to q, k and v first."""
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != (nq + nkv) * hd + nkv * vd or not bias.is_contiguous()):
+        raise KernelError("attention_prep_post: bias must be float32 [(nq + nkv) hd + nkv vd]")
     T = qkv.shape[0]
     if qkv.stride(1) != 1 or qkv.shape[1] < nq * hd + nkv * (hd + vd):
         raise KernelError("attention_prep_post: qkv must be [T, >= nq*hd + nkv*(hd + vd)] with unit inner stride")
@@ -1583,7 +1650,7 @@ def attention_prep_post(qkv, positions, slot_mapping, q_weight, k_weight, eps, i
         _ptr(qkv), _dt(qkv), qkv.stride(0), _ptr(positions), _ptr(slot_mapping) if nkv else None, _ptr(q_weight), _ptr(k_weight),
         float(eps) if eps is not None else -1.0, _ptr(inv_freq) if rotary_dim else None, int(rotary_dim),
         _ptr(k_cache) if nkv else None, _ptr(v_cache) if nkv else None, nq, nkv, hd, vd, page_size, T, int(bool(norm_first)),
-        _stream()), "attention_prep_post")
+        _ptr(bias), _stream()), "attention_prep_post")
 
 
 def causal_conv(x, in_bias, weight, out_bias, act: str, state, conv_offset: int, q_indptr, row_of_token, state_slots, out) -> None:
@@ -1705,7 +1772,13 @@ def square_relu(x, out) -> None:
 
 def gemm_square_relu(x, w: torch.Tensor, out: torch.Tensor) -> None:
     """out = max(x . w^T, 0)^2: the first half of an ungated feed-forward.  Few rows of x take one launch of the
-    weight-streaming kernel (the activation on its float32 sums); otherwise the product is followed by the activation."""
+    weight-streaming kernel (the activation on its float32 sums; ``x`` may be ``ScaledRows``); otherwise the product is followed by the
+    activation."""
+    if isinstance(x, ScaledRows):
+        if not (fused_gemm_supported(x.rows, w) and tuple(out.shape) == (x.shape[0], w.shape[0])):
+            raise KernelError("gemm_square_relu: rows that lack their norm factor need the fused weight-streaming kernel")
+        _fused_gemm(x.rows, w, out, 3, x, None)
+        return
     if fused_gemm_supported(x, w) and skinny_gemm_supported(x, w, out) and w.shape[1] == x.shape[1] and tuple(out.shape) == (x.shape[0], w.shape[0]):
         _fused_gemm(x, w, out, 3, None, None)
         return

@@ -21,13 +21,17 @@ stored weight); ``value_dim`` gives values another width than keys; ``sink`` add
 softmax's denominator; ``cache_window`` is what the cache keeps when other runs read this run's keys through wider windows
 than its own.
 
-The general form (any of ``keep_first``, ``softcap``, ``bias``, ``conv_taps``, or a per-head norm before the rotation with
-values of another width): ``keep_first`` keeps the first tokens of a sequence visible after the window has passed them (at
+The general form (any of ``keep_first``, ``softcap``, ``bias``, ``conv_taps``, ``stored_sinks``, or a per-head norm before the
+rotation with values of another width or a gate per head): ``keep_first`` keeps the first tokens of a sequence visible after the window has passed them (at
 their true positions); ``softcap`` turns a score s into softcap * tanh(s / softcap); ``bias`` adds stored biases in the q, k, v
-and output projections (tensor name + ``bias_suffix``); ``conv_taps`` runs a short causal convolution over time on every
+and (``out_bias``) output projections (tensor name + ``bias_suffix``); ``stored_sinks`` gives the softmax's denominator one more
+term exp(sink_h) per query head, a stored number without a key and a value (tensor ``sink``); ``conv_taps`` runs a short causal convolution over time on every
 channel of q, k and v right after the projection (weights [channels, taps] under tensor name + ``conv_suffix``, zeros
 before a sequence's start; the last taps - 1 projected rows of a request are its state).  Its order is projection (+ bias)
--> convolution -> per-head norm -> rotation -> cache -> attention -> output projection (+ bias).
+-> convolution -> per-head norm -> rotation -> cache -> attention (with the sinks) -> gate per head -> output projection (+ bias).
+The biases are added by the preparation kernel (by the convolution where there is one), the sinks and the gate are applied by the
+attention kernels behind their sums; a step of decoded tokens runs preparation, cache store, attention and gate as one launch where
+the shapes allow it.
 
 With ``qk_norm`` "row": ``weights`` "sigmoid" has no softmax, a visible key's weight is sigmoid(score + b_h) with a stored number
 per query head (tensor ``score_bias``); ``chunk`` lets a position see only its own chunk of that many positions, counted from 0;
@@ -75,11 +79,14 @@ class AttentionSpec:
     weights: str = "softmax"        # "sigmoid": sigmoid(score + b_h) per key, not normalised
     chunk: Optional[int] = None     # a position sees its own chunk of this many positions only
     out_gate: bool = False          # the heads' outputs times sigmoid(W_g x), number by number
+    out_bias: bool = True           # with ``bias``: the output projection has one too
+    stored_sinks: bool = False      # a stored sink score per query head
     kind: ClassVar[str] = "attention"
 
 
 DEFAULT_NAMES = (("q", "q_proj.weight"), ("k", "k_proj.weight"), ("v", "v_proj.weight"), ("o", "o_proj.weight"),
-                 ("q_norm", "q_norm.weight"), ("k_norm", "k_norm.weight"), ("gate", "g_proj.weight"), ("score_bias", "score_bias"))
+                 ("q_norm", "q_norm.weight"), ("k_norm", "k_norm.weight"), ("gate", "g_proj.weight"), ("score_bias", "score_bias"),
+                 ("sink", "sink"))
 
 
 class Attention(Mixer):
@@ -109,14 +116,15 @@ class Attention(Mixer):
             raise ValueError("attention: sigmoid weights, chunks and a gate per number go with qk_norm 'row'")
         self.spec = spec
         self.own_keys = spec.own_keys
-        self.general_form = bool(spec.keep_first or spec.softcap is not None or spec.bias or spec.conv_taps
-                                 or (spec.qk_norm == "head" and (self.vd != spec.head_dim or spec.head_dim % 2)))
+        self.general_form = bool(spec.keep_first or spec.softcap is not None or spec.bias or spec.conv_taps or spec.stored_sinks
+                                 or (spec.qk_norm == "head" and (self.vd != spec.head_dim or spec.head_dim % 2
+                                                                 or (spec.head_gate and spec.qk_norm_eps is not None))))
         if spec.head_dim % 2 and not self.general_form and spec.qk_norm != "row":
             raise ValueError(f"head_dim {spec.head_dim} not supported by this form of attention (even sizes only)")
-        if self.general_form and (spec.qk_norm != "head" or spec.values != "projected" or spec.head_gate or spec.sink is not None
+        if self.general_form and (spec.qk_norm != "head" or spec.values != "projected" or spec.out_gate or spec.sink is not None
                                   or not spec.own_keys or not spec.qk_norm_weight):
-            raise ValueError("attention: kept first tokens, capped scores, biases and the convolution go with a per-head norm before "
-                             "the rotation (or none), projected values, keys of its own, no gate and no sink")
+            raise ValueError("attention: kept first tokens, capped scores, biases, the convolution and stored sinks go with a per-head norm "
+                             "before the rotation (or none), projected values, keys of its own, no gate per number and no constant sink")
         # rotation first and norm after it, values of another width, a sink: the later form, with kernels of its own
         self.post_form = spec.qk_norm == "head_after_rotation"
         if self.post_form and (spec.values != "projected" or spec.head_gate):
@@ -133,13 +141,13 @@ class Attention(Mixer):
             raise ValueError("attention: a norm after the rotation, and the general form, go with half-split rotation")
         self.plain_form = (spec.qk_norm == "head" and spec.values == "projected" and not spec.head_gate
                            and self.pairing == "half")
-        if not self.plain_form and spec.qk_norm == "head" and spec.qk_norm_eps is not None:
+        if not self.plain_form and not self.general_form and spec.qk_norm == "head" and spec.qk_norm_eps is not None:
             raise ValueError("attention: a per-head q/k norm goes with half-split rotation, projected values and no gate")
         self.names = dict(DEFAULT_NAMES)
         self.names.update(dict(spec.names or ()))
         self.w_qkv = self.w_o = self.q_norm = self.k_norm = None
         self.gate_at = None             # column of the packed projection where the gate numbers start
-        self.b_qkv = self.b_o = self.w_conv = self.score_bias = None
+        self.b_qkv = self.b_o = self.w_conv = self.score_bias = self.sinks = None
         self.channels = spec.num_heads * spec.head_dim + spec.num_kv_heads * (spec.head_dim + self.vd)   # q | k | v
 
     # ---------------------------------------------------------------- weights
@@ -155,7 +163,12 @@ class Attention(Mixer):
             decls.append(WeightDecl(self._name("o"), (s.hidden_size, s.num_heads * self.vd)))
             if s.bias:
                 decls += [WeightDecl(self._name(r) + s.bias_suffix, (n,), init="around_zero") for r, n in rows.items()]
-                decls.append(WeightDecl(self._name("o") + s.bias_suffix, (s.hidden_size,), init="around_zero"))
+                if s.out_bias:
+                    decls.append(WeightDecl(self._name("o") + s.bias_suffix, (s.hidden_size,), init="around_zero"))
+            if s.stored_sinks:
+                decls.append(WeightDecl(self._name("sink"), (s.num_heads,), init="around_zero"))
+            if s.head_gate:
+                decls.append(WeightDecl(self._name("gate"), (s.num_heads, s.hidden_size)))
             if s.conv_taps:
                 decls += [WeightDecl(self._name(r) + s.conv_suffix, (n, s.conv_taps), init="around_zero") for r, n in rows.items()]
             if s.qk_norm_eps is not None:
@@ -193,7 +206,7 @@ class Attention(Mixer):
             roles = ("q",)
         mats = [tensors[self._name(n)] for n in roles]
         if s.head_gate or s.out_gate:
-            gap = -sum(m.shape[0] for m in mats) % 8 if s.out_gate else 0
+            gap = -sum(m.shape[0] for m in mats) % 8 if s.out_gate or self.general_form else 0
             if gap:
                 mats.append(torch.zeros((gap, s.hidden_size), dtype=mats[0].dtype))
             self.gate_at = sum(m.shape[0] for m in mats)
@@ -215,7 +228,10 @@ class Attention(Mixer):
             self.position.load(tensors, dtype, device)
         if s.bias:
             self.b_qkv = torch.cat([tensors[self._name(r) + s.bias_suffix].to(device=device, dtype=torch.float32) for r in ("q", "k", "v")]).contiguous()
-            self.b_o = tensors[self._name("o") + s.bias_suffix].to(device=device, dtype=torch.float32).contiguous()
+            if s.out_bias:
+                self.b_o = tensors[self._name("o") + s.bias_suffix].to(device=device, dtype=torch.float32).contiguous()
+        if s.stored_sinks:
+            self.sinks = tensors[self._name("sink")].to(device=device, dtype=torch.float32).contiguous()
         if s.conv_taps:
             self.w_conv = torch.cat([tensors[self._name(r) + s.conv_suffix].to(device=device, dtype=torch.float32) for r in ("q", "k", "v")],
                                     dim=0).contiguous()
@@ -244,10 +260,10 @@ class Attention(Mixer):
         return None
 
     def takes_scaled_rows(self, num_rows):
-        return not self.post_form and not self.general_form and ops.fused_gemm_shape_ok(num_rows, self.w_qkv)
+        return not self.post_form and ops.fused_gemm_shape_ok(num_rows, self.w_qkv)
 
     def can_sink(self, num_rows):
-        return not self.post_form and not self.general_form and ops.fused_gemm_shape_ok(num_rows, self.w_o)
+        return not self.post_form and self.b_o is None and ops.fused_gemm_shape_ok(num_rows, self.w_o)
 
     def _angles(self, qkv, ctx, inv_freq, rdim, general=False):
         """Cosines and sines of the step's positions, evaluated once for all layers that rotate by the same
@@ -285,8 +301,8 @@ class Attention(Mixer):
         ops.gemm(attn, self.w_o, out)
         return out
 
-    # ------------------------------------------------- biases, convolution, kept first tokens, capped scores
-    def _forward_general(self, x, ctx, cache, state):
+    # ------------------------------------------------- biases, convolution, kept first tokens, capped scores, sinks
+    def _forward_general(self, x, ctx, cache, state, sink=None):
         s = self.spec
         T = x.shape[0]
         nq, nkv, hd, vd = s.num_heads, s.num_kv_heads, s.head_dim, self.vd
@@ -294,28 +310,39 @@ class Attention(Mixer):
         inv_freq, rdim = rot if rot is not None else (None, 0)
         if not cache.writable:
             raise RuntimeError("attention: this form keeps keys of its own")
-        proj = ctx.ws.get("qkv", (T, self.channels), x.dtype)
+        proj = ctx.ws.get("qkv", (T, self.w_qkv.shape[0]), x.dtype)
         ops.gemm(x, self.w_qkv, proj)
+        gate = proj[:, self.gate_at: self.gate_at + nq] if s.head_gate else None
+        attn = ctx.ws.get("attn_out", (T, nq * vd), x.dtype)
+        out = ctx.ws.get("mixer_out", (T, s.hidden_size), x.dtype)
+        if (vd == hd and not (s.conv_taps or s.keep_first or s.softcap)
+                and ops.fused_decode_supported(proj, ctx, cache.k.dtype, nq, nkv, hd, cache.page_size, rdim)):
+            ops.decode_attention_with_prep(proj, attn, cache.k, cache.v, cache.slot_mapping, self.q_norm, self.k_norm, s.qk_norm_eps or 0.0,
+                                           inv_freq if rdim else None, cache.block_table, nq, nkv, hd, cache.page_size, s.scale, s.window,
+                                           ctx, rotary_dim=rdim, bias=self.b_qkv, sink=self.sinks, gate=gate)
+            return self._output_general(attn, out, sink)
+        bias = self.b_qkv
         if s.conv_taps:
             # the biases ride into the convolution as its input bias: added to a request's rows, not to the zeros before them
             conv = ctx.ws.get("qkv_conv", (T, self.channels), x.dtype)
-            ops.causal_conv(proj, self.b_qkv, self.w_conv, None, "none", state if s.conv_taps > 1 else ctx.ws.get("conv_none", (ctx.cache.max_slots, 4), torch.float32),
+            ops.causal_conv(proj[:, : self.channels], bias, self.w_conv, None, "none", state if s.conv_taps > 1 else ctx.ws.get("conv_none", (ctx.cache.max_slots, 4), torch.float32),
                             0, ctx.q_indptr, ctx.row_of_token, ctx.state_slots, conv)
-            proj = conv
-        elif s.bias:
-            ops.bias_add(proj, self.b_qkv)
+            proj, bias = conv, None
         if vd == hd and hd % 2 == 0:
             ops.attention_prep(proj, ctx.positions, cache.slot_mapping, self.q_norm, self.k_norm, s.qk_norm_eps or 0.0, inv_freq, rdim,
-                               cache.k, cache.v, nq, nkv, hd, cache.page_size, angles=self._angles(proj, ctx, inv_freq, rdim))
+                               cache.k, cache.v, nq, nkv, hd, cache.page_size, angles=self._angles(proj, ctx, inv_freq, rdim), bias=bias)
         else:
             ops.attention_prep_post(proj, ctx.positions, cache.slot_mapping, self.q_norm, self.k_norm, s.qk_norm_eps, inv_freq, rdim,
-                                    cache.k, cache.v, nq, nkv, hd, vd, cache.page_size, norm_first=True)
-        attn = ctx.ws.get("attn_out", (T, nq * vd), x.dtype)
+                                    cache.k, cache.v, nq, nkv, hd, vd, cache.page_size, norm_first=True, bias=bias)
         ops.paged_attention(proj[:, : nq * hd], attn, cache.k, cache.v, ctx.positions, ctx.row_of_token, cache.block_table,
-                            nq, nkv, hd, cache.page_size, s.scale, s.window, batch=ctx, vd=vd, keep_first=s.keep_first, softcap=s.softcap)
-        out = ctx.ws.get("mixer_out", (T, s.hidden_size), x.dtype)
-        ops.gemm(attn, self.w_o, out)
-        if s.bias:
+                            nq, nkv, hd, cache.page_size, s.scale, s.window, batch=ctx, vd=vd, keep_first=s.keep_first, softcap=s.softcap,
+                            sink=self.sinks, gate=gate)
+        return self._output_general(attn, out, sink)
+
+    def _output_general(self, attn, out, sink):
+        if ops.gemm(attn, self.w_o, out, sink=sink):
+            return None
+        if self.b_o is not None:
             ops.bias_add(out, self.b_o)
         return out
 
@@ -364,7 +391,7 @@ class Attention(Mixer):
         s = self.spec
         T = x.shape[0]
         if self.general_form:
-            return self._forward_general(x, ctx, cache, state)
+            return self._forward_general(x, ctx, cache, state, sink)
         if self.post_form:
             return self._forward_post(x, ctx, cache)
         if not self.plain_form:

@@ -137,6 +137,7 @@ class Norm(Part):
 
     eps: float
     weight: torch.Tensor
+    takes_scaled_delta = False      # whether ``apply`` takes a factor on the pending branch and rows that join the residual with it
 
     def deferred(self):
         """(gain float32 [width], eps) when the norm is x * rsqrt(mean(x^2) + eps) * gain, so that its
@@ -206,6 +207,7 @@ class Block(Part):
     is its mixer's, unless the arrangement itself has a memory (a convolution in front of the mixer)."""
 
     mixer: Mixer
+    scales_branches = True          # False: what this arrangement adds to the residual cannot have the model's branch factor
 
     def state_need(self) -> Optional[StateNeed]:
         return self.mixer.state_need()

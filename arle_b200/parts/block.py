@@ -60,7 +60,7 @@ class PreNormBlock(Block):
         h = stream.normed(self.mixer_norm, "normed_a")
         if self.ffn is None:
             nxt = stream.next_entry
-            sink = stream.sink_for(nxt[0], nxt[1], "normed_a") if nxt is not None and self.mixer.can_sink(T) else None
+            sink = stream.sink_for(nxt[0], nxt[1], "normed_a", last=True) if nxt is not None and self.mixer.can_sink(T) else None
             stream.add(self.mixer.forward(h, ctx, cache, state, sink=sink) if sink is not None else self.mixer.forward(h, ctx, cache, state))
             return
         # where a branch's last product can add into the residual and leave the next norm's input behind,
@@ -72,7 +72,7 @@ class PreNormBlock(Block):
             stream.add(self.mixer.forward(h, ctx, cache, state))
         h = stream.normed(self.ffn_norm, "normed_b")
         nxt = stream.next_entry
-        sink = stream.sink_for(nxt[0], nxt[1], "normed_a") if nxt is not None and self.ffn.can_sink(T) else None
+        sink = stream.sink_for(nxt[0], nxt[1], "normed_a", last=True) if nxt is not None and self.ffn.can_sink(T) else None
         if sink is not None:
             stream.add(self.ffn.forward(h, ctx, sink=sink))
         else:
@@ -105,6 +105,8 @@ class OutputNormBlock(Block):
     The input convolution reads the 32-bit residual itself.  Its memory, a request's last taps - 1 residual rows in float32,
     stands in front of the mixer's state in one row per request slot (a mixer behind a convolution keeps a flat float32
     state).  In a step of decoded tokens only it runs inside the kernel that ends the block before."""
+
+    scales_branches = False
 
     def __init__(self, spec: OutputNormBlockSpec):
         self.spec = spec
@@ -195,6 +197,8 @@ class SandwichBlockSpec:
 class SandwichBlock(Block):
     """A sublayer's output norm, the sum into the 32-bit residual and the next sublayer's input norm are one kernel
     (``ResidualStream.add_normed_before_norm``): the stream keeps the branch until the next ``normed(...)``."""
+
+    scales_branches = False
 
     def __init__(self, spec: SandwichBlockSpec):
         self.spec = spec

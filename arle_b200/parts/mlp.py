@@ -129,6 +129,9 @@ class UngatedMlp(FeedForward):
     def scratch_elements_per_token(self):
         return self.spec.intermediate_size + self.spec.hidden_size
 
+    def takes_scaled_rows(self, num_rows):
+        return ops.fused_gemm_shape_ok(num_rows, self.w_up)
+
     def can_sink(self, num_rows):
         return ops.fused_gemm_shape_ok(num_rows, self.w_down)
 

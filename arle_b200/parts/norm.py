@@ -53,9 +53,11 @@ class RmsNorm(Norm):
     def deferred(self):
         return self.weight, self.eps
 
-    def apply(self, resid, delta, rows, out, write_resid: bool):
-        """out = norm(resid (+ delta)) on all rows or on ``rows``; see ops.rmsnorm."""
-        ops.rmsnorm(resid, delta, rows, self.weight, self.eps, out, write_resid)
+    takes_scaled_delta = True
+
+    def apply(self, resid, delta, rows, out, write_resid: bool, delta_scale: float = 1.0, extra=None):
+        """out = norm(resid (+ delta_scale * delta) (+ extra)) on all rows or on ``rows``; see ops.rmsnorm."""
+        ops.rmsnorm(resid, delta, rows, self.weight, self.eps, out, write_resid, delta_scale, extra)
         return out
 
     def add_normed(self, resid, branch, copy):

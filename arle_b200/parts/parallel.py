@@ -245,7 +245,7 @@ class ParallelBlock(Block):
         sink = None
         if nxt is not None and ops.fused_gemm_shape_ok(T, self.w_out):
             # every reader of this block's normed rows has run by now: their buffer can take the next block's
-            sink = stream.sink_for(nxt[0], nxt[1], "normed_a")
+            sink = stream.sink_for(nxt[0], nxt[1], "normed_a", last=True)
         out = ctx.ws.get("block_out", (T, stream.resid.shape[1]), n.dtype)
         stream.add(None if ops.gemm(pre, self.w_out, out, sink=sink) else out)
 

@@ -17,26 +17,32 @@ import torch
 F32 = torch.float32
 
 
-def embedding(ids, table, out, err=None, last_token=None, slot_of_token=None, scale=1.0):
+def embedding(ids, table, out, err=None, last_token=None, slot_of_token=None, scale=1.0, pos_table=None, positions=None, out2=None):
     ids = ids.long()
     if last_token is not None:
         ids = torch.where(ids < 0, last_token[slot_of_token.long()].long(), ids)
     out.copy_(table[ids].to(F32) * scale)
+    if pos_table is not None:
+        out += pos_table[positions.long()].to(F32)
+    if out2 is not None:
+        out2.copy_(out)
 
 
-def rmsnorm(resid, delta, rows, weight, eps, out, write_resid):
+def rmsnorm(resid, delta, rows, weight, eps, out, write_resid, delta_scale=1.0, extra=None):
     idx = rows.long() if rows is not None else torch.arange(resid.shape[0], device=resid.device)
     x = resid[idx].to(F32)
     if delta is not None:
-        x = x + delta[idx].to(F32)
+        x = x + delta_scale * delta[idx].to(F32)
+    if extra is not None:
+        x = x + extra[idx]
     if write_resid:
         resid[idx] = x
     inv = 1.0 / torch.sqrt((x * x).mean(dim=-1, keepdim=True) + eps)
     out.copy_((x * inv * weight).to(out.dtype))
 
 
-def residual_add(resid, delta):
-    resid += delta.to(F32)
+def residual_add(resid, delta, scale=1.0):
+    resid += scale * delta.to(F32)
 
 
 def gemm(x, w, out, sink=None):
@@ -58,12 +64,13 @@ def attention_prep_takes_angles(*args, **kwargs):
 
 
 def attention_prep(qkv, positions, slot_mapping, q_weight, k_weight, eps, inv_freq, rotary_dim, k_cache, v_cache,
-                   nq, nkv, hd, page_size, angles=None):
+                   nq, nkv, hd, page_size, angles=None, bias=None):
     T = qkv.shape[0]
     heads = qkv[:, : (nq + 2 * nkv) * hd].view(T, nq + 2 * nkv, hd)
+    b = bias.view(nq + 2 * nkv, hd) if bias is not None else torch.zeros(nq + 2 * nkv, hd)
 
-    def norm_rope(x, w):
-        x = x.to(F32)
+    def norm_rope(x, w, b):
+        x = x.to(F32) + b
         if w is not None:
             x = x * (1.0 / torch.sqrt((x * x).mean(dim=-1, keepdim=True) + eps)) * w
         if rotary_dim:
@@ -74,11 +81,11 @@ def attention_prep(qkv, positions, slot_mapping, q_weight, k_weight, eps, inv_fr
             x = torch.cat([lo * cos - hi * sin, lo * sin + hi * cos, x[..., rotary_dim:]], dim=-1)
         return x
 
-    q = norm_rope(heads[:, :nq], q_weight)
+    q = norm_rope(heads[:, :nq], q_weight, b[:nq])
     heads[:, :nq] = q.to(qkv.dtype)
     if nkv:
-        k = norm_rope(heads[:, nq:nq + nkv], k_weight).to(qkv.dtype)
-        v = heads[:, nq + nkv:]
+        k = norm_rope(heads[:, nq:nq + nkv], k_weight, b[nq:nq + nkv]).to(qkv.dtype)
+        v = (heads[:, nq + nkv:].to(F32) + b[nq + nkv:]).to(qkv.dtype)
         keep = slot_mapping >= 0
         page = (slot_mapping[keep] // page_size).long()
         off = (slot_mapping[keep] % page_size).long()
@@ -87,7 +94,7 @@ def attention_prep(qkv, positions, slot_mapping, q_weight, k_weight, eps, inv_fr
 
 
 def paged_attention(q, out, k_cache, v_cache, positions, row_of_token, block_table, nq, nkv, hd, page_size, scale,
-                    window, batch=None, vd=None, sink=None, keep_first=0, softcap=None, chunk=None, score_bias=None):
+                    window, batch=None, vd=None, sink=None, keep_first=0, softcap=None, chunk=None, score_bias=None, gate=None):
     T = q.shape[0]
     g = nq // nkv
     vd = hd if vd is None else vd
@@ -109,8 +116,9 @@ def paged_attention(q, out, k_cache, v_cache, positions, row_of_token, block_tab
             elif sink is None:
                 pr = torch.softmax(s, dim=0)
             else:                                            # one more term in the denominator, without a value
-                pr = torch.softmax(torch.cat([s, torch.tensor([float(sink)])]), dim=0)[:-1]
-            out[t, h * vd:(h + 1) * vd] = (pr @ v[:, h // g]).to(out.dtype)
+                pr = torch.softmax(torch.cat([s, torch.tensor([float(sink[h] if isinstance(sink, torch.Tensor) else sink)])]), dim=0)[:-1]
+            g_ = torch.sigmoid(gate[t, h].to(F32)) if gate is not None else 1.0
+            out[t, h * vd:(h + 1) * vd] = (pr @ v[:, h // g] * g_).to(out.dtype)
 
 
 def silu_mul(gate_up, out):
@@ -344,7 +352,8 @@ def latent_attention(q_abs, out, cache, positions, row_of_token, block_table, ra
 
 
 # ---------------------------------------------------------------- matrix memories with a scalar decay
-def decay_scan(q, k, v, a, b, state, q_indptr, state_slots, out, heads, kq_heads, dim, vdim, ones_column, q_scale, act="none"):
+def decay_scan(q, k, v, a, b, state, q_indptr, state_slots, out, heads, kq_heads, dim, vdim, ones_column, q_scale, act="none", rotation=None,
+               longest=0):
     vcols = vdim + int(bool(ones_column))
     rep = heads // kq_heads
     T = v.shape[0]
@@ -353,7 +362,12 @@ def decay_scan(q, k, v, a, b, state, q_indptr, state_slots, out, heads, kq_heads
         b = torch.ones(T, heads) if b is None else b[None, :].expand(T, heads)
     if act == "silu":
         q, k, v = (x.to(F32) / (1.0 + torch.exp(-x.to(F32))) for x in (q, k, v))
+    if rotation is not None and rotation[2]:
+        positions, inv_freq, rdim = rotation
+        q, k = (_turn_half(x.to(F32).view(T, kq_heads, dim), positions, inv_freq, rdim).reshape(T, -1) for x in (q, k))
     for r in range(state_slots.numel()):
+        if longest and int(q_indptr[r + 1]) - int(q_indptr[r]) > longest:
+            continue
         S = state[int(state_slots[r]), : heads * vcols * dim].view(heads, vcols, dim)
         for t in range(int(q_indptr[r]), int(q_indptr[r + 1])):
             qt = q[t].to(F32).view(kq_heads, dim).repeat_interleave(rep, dim=0) * q_scale
@@ -517,12 +531,13 @@ def bias_add(x, bias):
 
 
 def attention_prep_post(qkv, positions, slot_mapping, q_weight, k_weight, eps, inv_freq, rotary_dim, k_cache, v_cache,
-                        nq, nkv, hd, vd, page_size, norm_first=False):
+                        nq, nkv, hd, vd, page_size, norm_first=False, bias=None):
     T = qkv.shape[0]
     pos = positions.to(F32)
+    b = bias if bias is not None else torch.zeros((nq + nkv) * hd + nkv * vd)
 
-    def prepared(x, weight):                         # x [T, heads, hd]
-        x = x.to(F32).clone()
+    def prepared(x, weight, b):                      # x [T, heads, hd]
+        x = x.to(F32) + b.view(-1, hd)
         if norm_first:
             if eps is not None:
                 x = x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps)
@@ -534,11 +549,11 @@ def attention_prep_post(qkv, positions, slot_mapping, q_weight, k_weight, eps, i
             x = x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps)
         return x * weight if weight is not None else x
 
-    q = prepared(qkv[:, : nq * hd].view(T, nq, hd), q_weight)
+    q = prepared(qkv[:, : nq * hd].view(T, nq, hd), q_weight, b[: nq * hd])
     qkv[:, : nq * hd] = q.reshape(T, nq * hd).to(qkv.dtype)
     if nkv:
-        k = prepared(qkv[:, nq * hd: (nq + nkv) * hd].view(T, nkv, hd), k_weight).to(qkv.dtype)
-        v = qkv[:, (nq + nkv) * hd: (nq + nkv) * hd + nkv * vd].view(T, nkv, vd)
+        k = prepared(qkv[:, nq * hd: (nq + nkv) * hd].view(T, nkv, hd), k_weight, b[nq * hd: (nq + nkv) * hd]).to(qkv.dtype)
+        v = (qkv[:, (nq + nkv) * hd: (nq + nkv) * hd + nkv * vd].to(F32) + b[(nq + nkv) * hd:]).to(qkv.dtype).view(T, nkv, vd)
         keep = slot_mapping >= 0
         page, off = (slot_mapping[keep] // page_size).long(), (slot_mapping[keep] % page_size).long()
         k_cache[page, :, off] = k[keep]
