@@ -1,0 +1,384 @@
+// Matrix memories with one constant decay per head, over long rows of a step, in chunks of tokens that run side by side:
+//
+//     S_t = a S_(t-1) + k_t v_t^T,        o_t = S_t^T (q_scale q_t)          (S: dim x vdim, float32; a = decay[h])
+//
+// With S_0 the memory before a chunk of n tokens (0-based places i, j in the chunk),
+//     o_i = sum_(j <= i) a^(i - j) (q_i . k_j) v_j + a^(i + 1) S_0^T q_i,
+//     S_n = a^n S_0 + sum_j a^(n - 1 - j) k_j v_j^T,
+// so only the carry from chunk to chunk is serial.  Three kernels over the chunks of all long rows of the step:
+//  * chunk_own: U_c = sum_j a^(n - 1 - j) k_j v_j^T of every chunk (a block per chunk, head, tile of 64 columns of v);
+//  * chunk_carry: walks a row's chunks in order, S_c = a^n S_(c-1) + U_c element by element; leaves the memory BEFORE every chunk
+//    in U_c's place and the row's last memory in its state slot;
+//  * chunk_out: scores of the chunk's queries against its own keys with the decay's powers as a mask, times v, plus the read-out
+//    of the memory before the chunk.
+// Everything is float32 (FFMA) whatever the activation type.  q and k may be rotated (half-split pairs, cosines and sines from the
+// step's table) or go through silu (then v too) as they are staged.  The powers are powf(a, n).  A chunk is 64 tokens counted from
+// the row's first token of the step, so the order of a token's sums depends on where its portion starts: within rounding.
+// chunk_plan lists the chunks of the step once for all layers.  Rows of up to `longest` tokens are left alone (the scan in
+// recurrent.cu runs them).
+#include "common.cuh"
+using namespace arle;
+
+namespace {
+
+constexpr int kC = 64;                  // tokens of a chunk
+constexpr int kThreads = 256;
+constexpr int kVT = 64;                 // columns of v a block takes
+constexpr int kPad = 4;                 // floats behind a row in shared memory: rows fall on different banks, 16-byte aligned
+
+struct Chunk {
+  int t0, n, row, index;                // first token, tokens, row of the step, place among the row's chunks
+};
+
+// plan: first [R + 1] (a row's first chunk; the total at the end), padded to a multiple of 4, then a Chunk each.
+__global__ void __launch_bounds__(kThreads) chunk_plan_kernel(const int* __restrict__ q_indptr, int R, int longest, int* __restrict__ plan) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ int sums[kThreads];
+  Chunk* list = reinterpret_cast<Chunk*>(plan + ((R + 1 + 3) & ~3));
+  int carry = 0;
+  for (int base = 0; base < R; base += kThreads) {
+    const int r = base + threadIdx.x;
+    const int beg = r < R ? q_indptr[r] : 0, len = r < R ? q_indptr[r + 1] - beg : 0;
+    const int mine = len > longest ? (len + kC - 1) / kC : 0;
+    sums[threadIdx.x] = mine;
+    __syncthreads();
+    for (int o = 1; o < kThreads; o <<= 1) {
+      const int v = threadIdx.x >= o ? sums[threadIdx.x - o] : 0;
+      __syncthreads();
+      sums[threadIdx.x] += v;
+      __syncthreads();
+    }
+    const int first = carry + sums[threadIdx.x] - mine;
+    if (r < R) plan[r] = first;
+    for (int c = 0; c < mine; ++c) list[first + c] = Chunk{beg + c * kC, min(kC, len - c * kC), r, c};
+    carry += sums[kThreads - 1];
+    __syncthreads();
+  }
+  if (threadIdx.x == 0) plan[R] = carry;
+}
+
+struct Stage {                          // how q and k are read
+  const float2* angles;                 // [T, rotary_dim / 2] (cos, sin), or null: no rotation
+  int rotary_dim, act;                  // act 1: silu
+};
+
+__device__ __forceinline__ float silu(float x) { return x / (1.0f + expf(-x)); }
+
+// rows 0 .. n-1 of x (row stride `stride`, dim numbers), rotated, times scale (and w[row], if given), into dst [kC][DP + kPad];
+// zeros past dim and past n.
+template <typename T, int DP, bool VEC>
+__device__ __forceinline__ void stage_rows(const T* __restrict__ x, long stride, int t0, int n, int dim, const Stage& st, float scale,
+                                           const float* w, float* dst) {
+  constexpr int PITCH = DP + kPad;
+  constexpr int G = VEC ? 4 : 1;
+  const int half = st.rotary_dim >> 1;
+  for (int idx = threadIdx.x; idx < kC * (DP / G); idx += kThreads) {
+    const int tt = idx / (DP / G), e = (idx - tt * (DP / G)) * G;
+    float v[G];
+#pragma unroll
+    for (int g = 0; g < G; ++g) v[g] = 0.f;
+    if (tt < n && e < dim) {
+      const T* row = x + (size_t)(t0 + tt) * stride;
+      load_vec<T, G>(row + e, v);
+      if (e < st.rotary_dim) {
+        const bool first = e < half;
+        const int i0 = first ? e : e - half;
+        float o[G], cs[2 * G];
+        load_vec<T, G>(row + (first ? e + half : i0), o);
+        const float* a = reinterpret_cast<const float*>(st.angles + (size_t)(t0 + tt) * half + i0);
+#pragma unroll
+        for (int g = 0; g < 2 * G; g += G == 1 ? 1 : 4) {
+          if constexpr (G == 1) cs[g] = a[g];
+          else {
+            const float4 f = *reinterpret_cast<const float4*>(a + g);
+            cs[g] = f.x, cs[g + 1] = f.y, cs[g + 2] = f.z, cs[g + 3] = f.w;
+          }
+        }
+#pragma unroll
+        for (int g = 0; g < G; ++g) v[g] = first ? v[g] * cs[2 * g] - o[g] * cs[2 * g + 1] : v[g] * cs[2 * g] + o[g] * cs[2 * g + 1];
+      }
+      const float f = w ? scale * w[tt] : scale;
+#pragma unroll
+      for (int g = 0; g < G; ++g) v[g] = (st.act ? silu(v[g]) : v[g]) * f;
+    }
+#pragma unroll
+    for (int g = 0; g < G; ++g) dst[tt * PITCH + e + g] = v[g];
+  }
+}
+
+// U[chunk][h][v][d] = sum_j a^(n - 1 - j) k_j[d] v_j[v]
+template <typename T, int DP, bool VEC>
+__global__ void __launch_bounds__(kThreads) chunk_own_kernel(const T* __restrict__ k, const T* __restrict__ v, long k_stride, long v_stride,
+                                                             const float* __restrict__ decay, const int* __restrict__ plan, int R,
+                                                             Stage st, float* __restrict__ own, int H, int dim, int vdim) {
+  pdl_launch_dependents();
+  pdl_wait();
+  constexpr int PITCH = DP + kPad;
+  constexpr int ND = DP / 16;                           // numbers of d a thread holds: groups of min(4, ND), 64 apart
+  constexpr int GD = ND < 4 ? ND : 4;
+  extern __shared__ __align__(16) float sm[];
+  float* ks = sm;                                       // [kC][PITCH], times the decay's power
+  float* vs = ks + kC * PITCH;                          // [kC][kVT]
+  float* pw = vs + kC * kVT;                            // [kC]
+  const Chunk ch = reinterpret_cast<const Chunk*>(plan + ((R + 1 + 3) & ~3))[blockIdx.z];
+  const int h = blockIdx.y, v0 = blockIdx.x * kVT;
+  const float a = decay[h];
+  if (threadIdx.x < kC) pw[threadIdx.x] = threadIdx.x < ch.n ? powf(a, (float)(ch.n - 1 - threadIdx.x)) : 0.f;
+  __syncthreads();
+  stage_rows<T, DP, VEC>(k + (size_t)h * dim, k_stride, ch.t0, ch.n, dim, st, 1.0f, pw, ks);
+  for (int idx = threadIdx.x; idx < kC * kVT; idx += kThreads) {
+    const int tt = idx / kVT, c = v0 + idx - tt * kVT;
+    float x = (tt < ch.n && c < vdim) ? to_f32(v[(size_t)(ch.t0 + tt) * v_stride + (size_t)h * vdim + c]) : 0.f;
+    vs[idx] = st.act ? silu(x) : x;
+  }
+  __syncthreads();
+  const int td = threadIdx.x & 15, tv = threadIdx.x >> 4;
+  float acc[4][ND];
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int d = 0; d < ND; ++d) acc[i][d] = 0.f;
+  for (int j = 0; j < ch.n; ++j) {
+    const float4 vv = *reinterpret_cast<const float4*>(vs + j * kVT + tv * 4);
+    const float vr[4] = {vv.x, vv.y, vv.z, vv.w};
+#pragma unroll
+    for (int g = 0; g < ND / GD; ++g) {
+      float kr[GD];
+      load_vec<float, GD>(ks + j * PITCH + g * 16 * GD + td * GD, kr);
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int d = 0; d < GD; ++d) acc[i][g * GD + d] = fmaf(vr[i], kr[d], acc[i][g * GD + d]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int c = v0 + tv * 4 + i;
+    if (c >= vdim) break;
+    float* o = own + (((size_t)blockIdx.z * H + h) * vdim + c) * dim;
+#pragma unroll
+    for (int g = 0; g < ND / GD; ++g) {
+      const int d0 = g * 16 * GD + td * GD;
+      if (VEC && GD == 4) {
+        if (d0 < dim) *reinterpret_cast<float4*>(o + d0) = make_float4(acc[i][g * GD], acc[i][g * GD + 1], acc[i][g * GD + GD - 2], acc[i][g * GD + GD - 1]);
+      } else {
+#pragma unroll
+        for (int d = 0; d < GD; ++d)
+          if (d0 + d < dim) o[d0 + d] = acc[i][g * GD + d];
+      }
+    }
+  }
+}
+
+// A thread walks G numbers of a row's memories through the row's chunks.
+template <int G>
+__global__ void __launch_bounds__(kThreads) chunk_carry_kernel(float* __restrict__ own, const float* __restrict__ decay, const int* __restrict__ plan,
+                                                               int R, float* __restrict__ state, long slot_stride,
+                                                               const int* __restrict__ state_slots, long per_head, long total) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int r = blockIdx.y;
+  const int first = plan[r], count = plan[r + 1] - first;
+  const long e = ((long)blockIdx.x * kThreads + threadIdx.x) * G;
+  if (count == 0 || e >= total) return;
+  const Chunk* list = reinterpret_cast<const Chunk*>(plan + ((R + 1 + 3) & ~3));
+  const float a = decay[e / per_head];
+  const float whole = powf(a, (float)kC), last = powf(a, (float)list[first + count - 1].n);
+  float* sp = state + (size_t)state_slots[r] * slot_stride + e;
+  float* up = own + (size_t)first * total + e;
+  float S[G];
+  load_vec<float, G>(sp, S);
+  constexpr int B = 8;                                  // chunks asked for together
+  for (int c0 = 0; c0 < count; c0 += B) {
+    float U[B][G];
+#pragma unroll
+    for (int b = 0; b < B; ++b)
+      if (c0 + b < count) load_vec<float, G>(up + (size_t)(c0 + b) * total, U[b]);
+#pragma unroll
+    for (int b = 0; b < B; ++b) {
+      if (c0 + b < count) {
+        store_vec<float, G>(up + (size_t)(c0 + b) * total, S);
+        const float p = c0 + b == count - 1 ? last : whole;
+#pragma unroll
+        for (int g = 0; g < G; ++g) S[g] = fmaf(p, S[g], U[b][g]);
+      }
+    }
+  }
+  store_vec<float, G>(sp, S);
+}
+
+template <typename T, int DP, bool VEC>
+__global__ void __launch_bounds__(kThreads, DP == 128 ? 2 : 3) chunk_out_kernel(
+    const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, long q_stride, long k_stride, long v_stride,
+    const float* __restrict__ decay, const int* __restrict__ plan, int R, Stage st, const float* __restrict__ before,
+    float* __restrict__ out, int H, int dim, int vdim, float q_scale) {
+  pdl_launch_dependents();
+  pdl_wait();
+  constexpr int PITCH = DP + kPad, AP = kC + kPad;
+  extern __shared__ __align__(16) float sm[];
+  float* qs = sm;                                       // [kC][PITCH]
+  float* ks = qs + kC * PITCH;                          // [kC][PITCH]; the memory's columns [kVT][PITCH] once the scores are formed
+  float* as = ks + kC * PITCH;                          // [kC][AP] scores with the decay's powers
+  float* vt = as + kC * AP;                             // [kVT][AP] v transposed
+  float* pw = vt + kVT * AP;                            // [kC + 1]
+  const Chunk ch = reinterpret_cast<const Chunk*>(plan + ((R + 1 + 3) & ~3))[blockIdx.z];
+  const int h = blockIdx.y, v0 = blockIdx.x * kVT, n = ch.n;
+  const float a = decay[h];
+  if (threadIdx.x <= kC) pw[threadIdx.x] = powf(a, (float)threadIdx.x);
+  stage_rows<T, DP, VEC>(q + (size_t)h * dim, q_stride, ch.t0, n, dim, st, q_scale, nullptr, qs);
+  stage_rows<T, DP, VEC>(k + (size_t)h * dim, k_stride, ch.t0, n, dim, st, 1.0f, nullptr, ks);
+  for (int idx = threadIdx.x; idx < kVT * (kC / 4); idx += kThreads) {        // a column, four tokens
+    const int c = idx & (kVT - 1), j0 = (idx / kVT) * 4;
+    float x[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      x[i] = (j0 + i < n && v0 + c < vdim) ? to_f32(v[(size_t)(ch.t0 + j0 + i) * v_stride + (size_t)h * vdim + v0 + c]) : 0.f;
+      if (st.act) x[i] = silu(x[i]);
+    }
+    *reinterpret_cast<float4*>(vt + c * AP + j0) = make_float4(x[0], x[1], x[2], x[3]);
+  }
+  __syncthreads();
+  const int tc = threadIdx.x & 15, ti = threadIdx.x >> 4;
+  float acc[4][4];
+  // acc[i][c] += sum_e x[ti * 4 + i][e] y[tc + 16 c][e]
+  auto product = [&](const float* x, const float* y, int xp, int yp, int len) {
+    for (int e = 0; e < len; e += 4) {
+      float4 xr[4], yr[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        xr[i] = *reinterpret_cast<const float4*>(x + (ti * 4 + i) * xp + e);
+        yr[i] = *reinterpret_cast<const float4*>(y + (tc + 16 * i) * yp + e);
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          acc[i][c] = fmaf(xr[i].x, yr[c].x, acc[i][c]);
+          acc[i][c] = fmaf(xr[i].y, yr[c].y, acc[i][c]);
+          acc[i][c] = fmaf(xr[i].z, yr[c].z, acc[i][c]);
+          acc[i][c] = fmaf(xr[i].w, yr[c].w, acc[i][c]);
+        }
+    }
+  };
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) acc[i][c] = 0.f;
+  product(qs, ks, PITCH, PITCH, DP);
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+      const int row = ti * 4 + i, col = tc + 16 * c;
+      as[row * AP + col] = col <= row ? acc[i][c] * pw[row - col] : 0.f;
+      acc[i][c] = 0.f;
+    }
+  __syncthreads();                                      // the keys have been read
+  const float* bp = before + (((size_t)blockIdx.z * H + h) * vdim + v0) * dim;
+  constexpr int G = VEC ? 4 : 1;
+  for (int idx = threadIdx.x; idx < kVT * (DP / G); idx += kThreads) {
+    const int c = idx / (DP / G), e = (idx - c * (DP / G)) * G;
+    float x[G];
+#pragma unroll
+    for (int g = 0; g < G; ++g) x[g] = 0.f;
+    if (v0 + c < vdim && e < dim) load_vec<float, G>(bp + (size_t)c * dim + e, x);
+#pragma unroll
+    for (int g = 0; g < G; ++g) ks[c * PITCH + e + g] = x[g];
+  }
+  __syncthreads();
+  product(qs, ks, PITCH, PITCH, DP);
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) acc[i][c] *= pw[ti * 4 + i + 1];
+  product(as, vt, AP, AP, (min(n, ti * 4 + 4) + 3) & ~3);        // scores beyond the query's own place are zero
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    if (ti * 4 + i >= n) break;
+    float* o = out + ((size_t)(ch.t0 + ti * 4 + i) * H + h) * vdim + v0;
+#pragma unroll
+    for (int c = 0; c < 4; ++c)
+      if (v0 + tc + 16 * c < vdim) o[tc + 16 * c] = acc[i][c];
+  }
+}
+
+template <typename T, int DP, bool VEC>
+int launch_as(const void* q, const void* k, const void* v, int q_stride, int k_stride, int v_stride, const float* decay, float* state,
+              long slot_stride, const int* state_slots, const int* plan, int chunks, const Stage& st, float* own, float* out, int R, int H,
+              int dim, int vdim, float q_scale, cudaStream_t s) {
+  const dim3 grid((vdim + kVT - 1) / kVT, H, chunks);
+  const size_t smem1 = (size_t)(kC * (DP + kPad) + kC * kVT + kC) * sizeof(float);
+  const size_t smem3 = (size_t)(2 * kC * (DP + kPad) + 2 * kC * (kC + kPad) + kC + 4) * sizeof(float);
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(chunk_own_kernel<T, DP, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(chunk_out_kernel<T, DP, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem3);
+    if (e != cudaSuccess) return (int)e;
+    configured = true;
+  }
+  launch_kernel(chunk_own_kernel<T, DP, VEC>, grid, dim3(kThreads), smem1, s, 1, (const T*)k, (const T*)v, (long)k_stride, (long)v_stride, decay,
+                plan, R, st, own, H, dim, vdim);
+  const long total = (long)H * vdim * dim;
+  if (dim % 4 == 0 && slot_stride % 4 == 0 && vec_aligned<4>(state, 4) && vec_aligned<4>(own, 4))
+    launch_kernel(chunk_carry_kernel<4>, dim3((unsigned)((total / 4 + kThreads - 1) / kThreads), R), dim3(kThreads), 0, s, 1, own, decay, plan, R,
+                  state, slot_stride, state_slots, (long)vdim * dim, total);
+  else
+    launch_kernel(chunk_carry_kernel<1>, dim3((unsigned)((total + kThreads - 1) / kThreads), R), dim3(kThreads), 0, s, 1, own, decay, plan, R,
+                  state, slot_stride, state_slots, (long)vdim * dim, total);
+  launch_kernel(chunk_out_kernel<T, DP, VEC>, grid, dim3(kThreads), smem3, s, 1, (const T*)q, (const T*)k, (const T*)v, (long)q_stride,
+                (long)k_stride, (long)v_stride, decay, plan, R, st, own, out, H, dim, vdim, q_scale);
+  return launch_status();
+}
+
+}  // namespace
+
+// Ints of a step's plan for this many rows and chunks, and the chunks of a row of this many tokens.
+ARLE_API int arle_decay_chunk_plan_ints(int rows, int chunks) { return ((rows + 1 + 3) & ~3) + 4 * chunks; }
+ARLE_API int arle_decay_chunk_tokens() { return kC; }
+
+ARLE_API int arle_decay_chunk_plan(const int* q_indptr, int rows, int longest, int* plan, cudaStream_t s) {
+  if (rows <= 0) return 0;
+  if (longest < 0 || !plan || ((uintptr_t)plan & 15)) return ARLE_E_BADARG;
+  launch_kernel(chunk_plan_kernel, dim3(1), dim3(kThreads), 0, s, 1, q_indptr, rows, longest, plan);
+  return launch_status();
+}
+
+// q, k [T, H*dim], v [T, H*vdim] in the activation type (row strides given); decay float32 [H]; state float32, a slot every
+// slot_stride numbers, [H][vdim][dim] at its start; plan: arle_decay_chunk_plan's, with `chunks` chunks in all; angles: float32
+// [T, rotary_dim / 2, 2] or null; act 1: silu on q, k and v; own: float32 scratch [chunks, H, vdim, dim]; out float32 [T, H, vdim]
+// (rows that have no chunk are not written).  dim at most 128.
+ARLE_API int arle_decay_chunks(const void* q, const void* k, const void* v, int dtype, int q_stride, int k_stride, int v_stride,
+                               const float* decay, float* state, long slot_stride, const int* state_slots, const int* plan, int chunks,
+                               const float* angles, int rotary_dim, int act, float* own, float* out, int R, int H, int dim, int vdim,
+                               float q_scale, cudaStream_t s) {
+  if (R <= 0 || chunks <= 0) return 0;
+  if (!decay || !state || !plan || !own || !out || H <= 0 || dim <= 0 || vdim <= 0 || rotary_dim < 0 || rotary_dim % 2 || rotary_dim > dim ||
+      (rotary_dim && (!angles || act)))
+    return ARLE_E_BADARG;
+  if (dim > 128 || H > 65535 || chunks > 65535 || R > 65535) return ARLE_E_UNSUPPORTED;
+  const Stage st{reinterpret_cast<const float2*>(angles), rotary_dim, act};
+  const size_t el = dtype == 0 ? 4 : 2;
+  const bool vec = dim % 4 == 0 && rotary_dim % 8 == 0 && q_stride % 4 == 0 && k_stride % 4 == 0 && vec_aligned<4>(q, el) && vec_aligned<4>(k, el) &&
+                   vec_aligned<4>(angles, 4) && vec_aligned<4>(own, 4);
+#define ARLE_CHUNKS(TT, D, V) \
+  return launch_as<TT, D, V>(q, k, v, q_stride, k_stride, v_stride, decay, state, slot_stride, state_slots, plan, chunks, st, own, out, R, H, dim, \
+                             vdim, q_scale, s)
+#define ARLE_CHUNKS_D(TT, V) \
+  do { \
+    if (dim <= 32) ARLE_CHUNKS(TT, 32, V); \
+    if (dim <= 64) ARLE_CHUNKS(TT, 64, V); \
+    ARLE_CHUNKS(TT, 128, V); \
+  } while (0)
+  if (dtype == 0) {
+    if (vec) ARLE_CHUNKS_D(float, true);
+    ARLE_CHUNKS_D(float, false);
+  }
+  if (dtype == 1) {
+    if (vec) ARLE_CHUNKS_D(__nv_bfloat16, true);
+    ARLE_CHUNKS_D(__nv_bfloat16, false);
+  }
+#undef ARLE_CHUNKS_D
+#undef ARLE_CHUNKS
+  return ARLE_E_BADARG;
+}

@@ -92,6 +92,10 @@ _SIGNATURES = {
     "arle_latent_attention_mma": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P],
     "arle_latent_attention": [_P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P],
     "arle_decay_scan": [_P, _P, _P, _I, _I, _I, _I, _P, _P, _P, ctypes.c_long, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P, _P, _I, _I, _P],
+    "arle_decay_chunk_plan_ints": [_I, _I],
+    "arle_decay_chunk_tokens": [],
+    "arle_decay_chunk_plan": [_P, _I, _I, _P, _P],
+    "arle_decay_chunks": [_P, _P, _P, _I, _I, _I, _I, _P, _P, ctypes.c_long, _P, _P, _I, _P, _I, _I, _P, _P, _I, _I, _I, _I, _F, _P],
     "arle_mlstm_gates": [_P, _I, _P, _P, _F, _P, _P, _P, ctypes.c_long, ctypes.c_long, _P, _P, _P, _I, _I, _P],
     "arle_mlstm_out": [_P, _P, _P, _I, _I, _P, _F, _P, _I, _I, _I, _I, _P],
     "arle_ssm_gates": [_P, _I, _P, _P, _P, _P, _I, _I, _P],
@@ -1327,6 +1331,63 @@ def decay_scan(q, k, v, a, b, state, q_indptr, state_slots, out, heads: int, kq_
                                      dim, vdim, vcols - vdim, float(q_scale), 0 if per_head else heads, int(act == "silu"), int(T > 16 * R),
                                      *_rotation_args(rotation, T, dim, act), int(longest), _stream()),
            "decay_scan")
+
+
+DECAY_CHUNK = 64                    # tokens of a chunk
+DECAY_CHUNK_LONGEST = 32            # rows of up to this many tokens stay with the scan
+
+
+def decay_chunk_count(q_lens, dim: int, dtype) -> int:
+    """Chunks that ``decay_chunks`` would run for rows of these lengths (those of more than DECAY_CHUNK_LONGEST tokens); 0: none, the
+    scan runs every row."""
+    if _KERNEL_SET != "fast" or dim > 128:
+        return 0
+    return sum(-(-n // DECAY_CHUNK) for n in q_lens if n > DECAY_CHUNK_LONGEST)
+
+
+def decay_chunks(q, k, v, decay, state, batch, out, heads: int, dim: int, vdim: int, q_scale: float, act: str = "none", rotation=None,
+                 chunks: int = None) -> None:
+    """What ``decay_scan`` does with one constant decay per head (float32 [heads], one key head per head, no column of ones), for the
+    rows of the step with more than DECAY_CHUNK_LONGEST tokens: their tokens run in chunks side by side, with one carry from
+    chunk to chunk.  Other rows are left alone.  ``batch``: the StepContext (rows, slots, workspace, the step's memo: the list of chunks
+    and the table of angles are made once for all layers).  ``chunks``: ``decay_chunk_count`` of the step.  dim at most 128."""
+    T = v.shape[0]
+    R = batch.num_rows
+    if (q.shape != (T, heads * dim) or k.shape != q.shape or v.shape != (T, heads * vdim) or q.dtype != k.dtype
+            or q.dtype != v.dtype or q.stride(1) != 1 or k.stride(1) != 1 or v.stride(1) != 1):
+        raise KernelError("decay_chunks: q, k [T, heads*dim] and v [T, heads*vdim] of one type with unit inner stride")
+    if decay.dtype != torch.float32 or decay.numel() != heads or not decay.is_contiguous() or act not in ("none", "silu"):
+        raise KernelError("decay_chunks: decay must be float32 [heads]; act none or silu")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.shape[1] < heads * vdim * dim or state.stride(1) != 1:
+        raise KernelError(f"decay_chunks: state {tuple(state.shape)} must be float32 [slots, >= {heads * vdim * dim}]")
+    if out.dtype != torch.float32 or tuple(out.shape) != (T, heads, vdim) or not out.is_contiguous():
+        raise KernelError("decay_chunks: out must be contiguous float32 [T, heads, vdim]")
+    if chunks is None:
+        chunks = decay_chunk_count(batch.q_lens, dim, q.dtype)
+    if chunks <= 0:
+        return
+    lib = library()
+    memo = batch.memo
+    plan = memo.get("decay_chunk_plan")
+    if plan is None:
+        plan = batch.ws.get("decay_chunk_plan", (lib.arle_decay_chunk_plan_ints(R, chunks),), torch.int32)
+        _check(lib.arle_decay_chunk_plan(_ptr(batch.q_indptr), R, DECAY_CHUNK_LONGEST, _ptr(plan), _stream()), "decay_chunk_plan")
+        memo["decay_chunk_plan"] = plan
+    _, _, rdim = _rotation_args(rotation, T, dim, act)
+    angles = None
+    if rdim:
+        positions, inv_freq, _ = rotation
+        key = ("decay_angles", inv_freq.data_ptr(), rdim)
+        angles = memo.get(key)
+        if angles is None:
+            angles = batch.ws.get(f"decay_angles_{len(memo)}", (T, rdim // 2, 2), torch.float32)
+            rotary_angles(positions, inv_freq, angles)
+            memo[key] = angles
+    own = batch.ws.get("decay_chunk_memories", (chunks, heads, vdim, dim), torch.float32)
+    _check(lib.arle_decay_chunks(_ptr(q), _ptr(k), _ptr(v), _dt(q), q.stride(0), k.stride(0), v.stride(0), _ptr(decay), _ptr(state),
+                                 state.stride(0), _ptr(batch.state_slots), _ptr(plan), int(chunks), _ptr(angles), rdim, int(act == "silu"),
+                                 _ptr(own), _ptr(out), R, heads, dim, vdim, float(q_scale), _stream()), "decay_chunks")
+    add_launches(2)
 
 
 def mlstm_gates(pre, bias_i, bias_f, cap: float, q_indptr, state_slots, state, m_offset: int, a, b, floor) -> None:

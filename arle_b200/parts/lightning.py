@@ -11,7 +11,7 @@ k).  ``norm`` "head" norms each head's o alone, without a weight when ``norm_wei
 No softmax, no cache that grows: what a request keeps is the heads' memories, one float32 row per request
 slot that the cache manager zeroes when a request gets the slot.  The four input projections are one packed product;
 the silu (or the rotation) of q and k is applied by the scan as it stages them; the recurrence is the package's scalar-decay scan with the
-decays as one number per head; the norm over all heads, its weight and the gate are one kernel.  ``decay`` are the heads'
+decays as one number per head, or, for long rows of a prompt, its form in chunks of tokens that run side by side; the norm over all heads, its weight and the gate are one kernel.  ``decay`` are the heads'
 constants (usually in (0, 1]).
 """
 from __future__ import annotations
@@ -99,7 +99,8 @@ class ConstantDecayAttention(Mixer):
         return sum(t.numel() * t.element_size() for t in (self.w_in, self.w_o))
 
     def scratch_elements_per_token(self):
-        return 2 * self.dqk + 6 * self.inner + self.spec.hidden_size
+        # a chunk of 64 tokens keeps a float32 copy of the memories (two elements of the activation type each)
+        return 2 * self.dqk + 6 * self.inner + self.spec.hidden_size + 2 * self.spec.num_heads * self.spec.key_dim * self.spec.value_dim // 64
 
     def state_need(self):
         n = self.spec.num_heads * self.spec.value_dim * self.spec.key_dim
@@ -118,9 +119,15 @@ class ConstantDecayAttention(Mixer):
         proj = ctx.ws.get("lightning_in", (T, 2 * dqk + 2 * inner), x.dtype)                # q | k | v | gate
         ops.gemm(x, self.w_in, proj)
         o = ctx.ws.get("lightning_o", (T, H, s.value_dim), torch.float32)
-        ops.decay_scan(proj[:, :dqk], proj[:, dqk: 2 * dqk], proj[:, 2 * dqk: 2 * dqk + inner], self.decay, None, state, ctx.q_indptr,
-                       ctx.state_slots, o, H, H, s.key_dim, s.value_dim, False, s.q_scale, act=s.activation,
-                       rotation=(ctx.positions, *self.position.rotary()) if self.position is not None else None)
+        q, k, v = proj[:, :dqk], proj[:, dqk: 2 * dqk], proj[:, 2 * dqk: 2 * dqk + inner]
+        rotation = (ctx.positions, *self.position.rotary()) if self.position is not None else None
+        chunks = ops.decay_chunk_count(ctx.q_lens, s.key_dim, x.dtype)
+        if chunks:
+            ops.decay_chunks(q, k, v, self.decay, state, ctx, o, H, s.key_dim, s.value_dim, s.q_scale, act=s.activation, rotation=rotation,
+                             chunks=chunks)
+        if not chunks or min(ctx.q_lens) <= ops.DECAY_CHUNK_LONGEST:
+            ops.decay_scan(q, k, v, self.decay, None, state, ctx.q_indptr, ctx.state_slots, o, H, H, s.key_dim, s.value_dim, False, s.q_scale,
+                           act=s.activation, rotation=rotation, longest=ops.DECAY_CHUNK_LONGEST if chunks else 0)
         gated = ctx.ws.get("lightning_gated", (T, inner), x.dtype)
         # one norm over all heads at once is a single "head" as wide as the row
         heads, width = (1, inner) if s.norm == "all" else (H, s.value_dim)

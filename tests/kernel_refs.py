@@ -67,7 +67,7 @@ def attention_prep(qkv, positions, slot_mapping, q_weight, k_weight, eps, inv_fr
                    nq, nkv, hd, page_size, angles=None, bias=None):
     T = qkv.shape[0]
     heads = qkv[:, : (nq + 2 * nkv) * hd].view(T, nq + 2 * nkv, hd)
-    b = bias.view(nq + 2 * nkv, hd) if bias is not None else torch.zeros(nq + 2 * nkv, hd)
+    b = bias.view(nq + 2 * nkv, hd) if bias is not None else torch.zeros(nq + 2 * nkv, hd, device=qkv.device)
 
     def norm_rope(x, w, b):
         x = x.to(F32) + b
@@ -379,6 +379,24 @@ def decay_scan(q, k, v, a, b, state, q_indptr, state_slots, out, heads, kq_heads
             out[t] = torch.einsum("hvd,hd->hv", S, qt)
 
 
+def decay_chunk_count(q_lens, dim, dtype):
+    import arle_b200.ops as ops
+
+    return sum(-(-n // ops.DECAY_CHUNK) for n in q_lens if n > ops.DECAY_CHUNK_LONGEST)
+
+
+def decay_chunks(q, k, v, decay, state, batch, out, heads, dim, vdim, q_scale, act="none", rotation=None, chunks=None):
+    """The same memories token by token, for the long rows alone."""
+    import arle_b200.ops as ops
+
+    for r in range(batch.num_rows):
+        lo, hi = int(batch.q_indptr[r]), int(batch.q_indptr[r + 1])
+        if hi - lo > ops.DECAY_CHUNK_LONGEST:
+            rot = (rotation[0][lo:hi],) + tuple(rotation[1:]) if rotation is not None else None
+            decay_scan(q[lo:hi], k[lo:hi], v[lo:hi], decay, None, state, torch.tensor([0, hi - lo]), batch.state_slots[r: r + 1], out[lo:hi],
+                       heads, heads, dim, vdim, False, q_scale, act=act, rotation=rot)
+
+
 def mlstm_gates(pre, bias_i, bias_f, cap, q_indptr, state_slots, state, m_offset, a, b, floor):
     H = pre.shape[1] // 2
     gi = cap * torch.tanh((pre[:, :H] + bias_i) / cap)
@@ -534,7 +552,7 @@ def attention_prep_post(qkv, positions, slot_mapping, q_weight, k_weight, eps, i
                         nq, nkv, hd, vd, page_size, norm_first=False, bias=None):
     T = qkv.shape[0]
     pos = positions.to(F32)
-    b = bias if bias is not None else torch.zeros((nq + nkv) * hd + nkv * vd)
+    b = bias if bias is not None else torch.zeros((nq + nkv) * hd + nkv * vd, device=qkv.device)
 
     def prepared(x, weight, b):                      # x [T, heads, hd]
         x = x.to(F32) + b.view(-1, hd)
@@ -693,5 +711,5 @@ ALL = ("rotary_angles", "embedding", "rmsnorm", "residual_add", "gemm", "fused_g
        "act_mul", "gemm_act_mul", "attention_prep_row", "head_gate", "weighted_sum", "logit_cap", "gla_decay", "gla_scan", "gla_out",
        "dyt_norm", "gemm_heads", "latent_prep", "latent_attention", "decay_scan", "mlstm_gates", "mlstm_out", "ssm_gates", "conv_silu",
        "gated_group_norm", "moe_select", "moe_plan_size", "moe_plan", "moe_gemm", "moe_combine", "clamped_glu", "branch_norm_add",
-       "attention_prep_post", "causal_conv", "rglru_scan", "delta_gates", "delta_scan", "branch_norm_add_norm", "rms_rows", "normed_sum",
+       "attention_prep_post", "causal_conv", "rglru_scan", "delta_gates", "delta_scan", "decay_chunk_count", "decay_chunks", "branch_norm_add_norm", "rms_rows", "normed_sum",
        "bias_add", "gate_mul", "square_relu", "gemm_square_relu", "layernorm", "branch_layernorm_add", "input_conv", "token_shift")
