@@ -27,6 +27,8 @@ attention with sigmoid weights, RWKV-style time mixing, in turn, all with routed
 ``--design lasupel`` does the same for Lasupel layers (an attention with a sliding window and a sink, an RG-LRU layer, an
 attention that reads the first one's keys and values, a gated delta rule layer, in turn; the first feed-forward of four
 dense, the others routed experts) beside Zuderax and Qwen3 layers of equal width.
+``--design virorax`` does the same for Virorax layers (a windowed attention with biases, sinks and gates per head, and a retention, in
+turn, all with dense feed-forwards; two of the stored layers run twice) beside Kolodra and Qwen3 layers of equal width.
 """
 import argparse
 import json
@@ -268,6 +270,20 @@ def dabilorn_config(z, dd, L, chunk):
     return {"architecture": "Dabilorn", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "canon": {"taps": 4}, "layers": layers}
 
 
+# Mixer sizes for ``--design virorax`` at the same widths: the attention's heads are the Qwen3 layer's (a window of half the
+# benchmark's context, half of a head rotated), the retention has Kolodra's memories of 128 x 128, and the feed-forward's two
+# matrices are together as large as the three of the Qwen3 layer.  L layer runs of L - 2 stored layers: two of them run twice.
+def virorax_config(z, L, window, positions):
+    h = z["rheads"]
+    ff = {"kind": "dense", "ff": z["ff"] * 3 // 2}
+    attn = {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["hd"], "vdim": z["hd"], "scale": z["hd"] ** -0.5, "mask": {"size": window},
+            "rot": {"base": 1e6, "dims": z["hd"] // 2}}
+    ret = {"heads": h, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** -(5 + 7 * i / max(1, h - 1)) for i in range(h)], "rot": {"base": 1e6, "dims": 128}}
+    layers = [{"type": "retention" if i % 2 else "attention", "mixer": dict(ret if i % 2 else attn), "mlp": ff} for i in range(L - 2)]
+    return {"architecture": "Virorax", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "residual_mult": 0.5, "logit_softcap": 30.0,
+            "max_positions": positions, "loop": {"start": 2, "stop": 4, "times": 2}, "layers": layers}
+
+
 def design_table(args, torch, ops, pk) -> int:
     """``--design kolodra``: prefill and decode throughput of a few Kolodra layers beside the same number of Qwen3
     layers of equal width, heads and feed-forward, with the device time of every kernel of one step (profiler
@@ -277,7 +293,7 @@ def design_table(args, torch, ops, pk) -> int:
     from arle_b200.engine import ModelRunner, StepEntry, random_model
 
     dev = torch.device("cuda:0")
-    L, T, C = args.layers or (6 if args.design == "zuderax" else 12 if args.design == "dabilorn" else (8 if args.design in ("lasupel", "lukinex") else 4)), args.prefill_tokens, args.context
+    L, T, C = args.layers or (6 if args.design == "zuderax" else 12 if args.design == "dabilorn" else (8 if args.design in ("lasupel", "lukinex", "virorax") else 4)), args.prefill_tokens, args.context
     gen = torch.Generator().manual_seed(1)
     out = {"design": args.design, "layers": L, "prefill_tokens": T, "context": C, "dtype": "bf16", "peaks": pk, "sizes": {}}
 
@@ -399,6 +415,10 @@ def design_table(args, torch, ops, pk) -> int:
                 # twelve layers by default: whole rounds of Dabilorn's three kinds of layers and of Lukinex's four
                 out["sizes"][name].update({"lukinex": measure(lukinex_config(z, LUKINEX_SIZES[name], L, max(C // 2, 16))),
                                            "kolodra": measure(kolodra_config(z))})
+        elif args.design == "virorax":
+            out["sizes"][name]["virorax"] = measure(virorax_config(z, L, max(C // 2, 16), 4 * max(C, T)))
+            if not args.design_alone:
+                out["sizes"][name].update({"kolodra": measure(kolodra_config(z)), "qwen3": measure(qwen_config(z))})
         elif not args.design_alone:
             out["sizes"][name].update({"kolodra": measure(kolodra_config(z)), "qwen3": measure(qwen_config(z))})
     print(json.dumps(out))
@@ -427,8 +447,8 @@ def main() -> int:
     ap.add_argument("--no-cuda-graph", action="store_true")
     ap.add_argument("--no-kernel-times", action="store_true",
                     help="with --design: leave out the per-kernel times (they come from torch's profiler, which cannot run under another profiler)")
-    ap.add_argument("--design-alone", action="store_true", help="with --design zuderax, lasupel, lukinex or dabilorn: leave out the models it stands beside")
-    ap.add_argument("--design", default=None, choices=["kolodra", "zuderax", "lasupel", "lukinex", "dabilorn"],
+    ap.add_argument("--design-alone", action="store_true", help="with --design zuderax, lasupel, lukinex, dabilorn or virorax: leave out the models it stands beside")
+    ap.add_argument("--design", default=None, choices=["kolodra", "zuderax", "lasupel", "lukinex", "dabilorn", "virorax"],
                     help="instead of the default workload: a few layers of this design beside as many Qwen3 layers of equal "
                          "sizes, prefill and decode, with every kernel's time (uses --layers, --steps, --context, --prefill-tokens)")
     ap.add_argument("--timeline", action="store_true",
