@@ -6,7 +6,7 @@
 //     o_i = sum_(j <= i) a^(i - j) (q_i . k_j) v_j + a^(i + 1) S_0^T q_i,
 //     S_n = a^n S_0 + sum_j a^(n - 1 - j) k_j v_j^T,
 // so only the carry from chunk to chunk is serial.  Three kernels over the chunks of all long rows of the step:
-//  * chunk_own: U_c = sum_j a^(n - 1 - j) k_j v_j^T of every chunk (a block per chunk, head, tile of 64 columns of v);
+//  * chunk_own: U_c = sum_j a^(n - 1 - j) k_j v_j^T of every chunk (a block per chunk, head, tile of 64 or 128 columns of v);
 //  * chunk_carry: walks a row's chunks in order, S_c = a^n S_(c-1) + U_c element by element; leaves the memory BEFORE every chunk
 //    in U_c's place and the row's last memory in its state slot;
 //  * chunk_out: scores of the chunk's queries against its own keys with the decay's powers as a mask, times v, plus the read-out
@@ -23,7 +23,6 @@ namespace {
 
 constexpr int kC = 64;                  // tokens of a chunk
 constexpr int kThreads = 256;
-constexpr int kVT = 64;                 // columns of v a block takes
 constexpr int kPad = 4;                 // floats behind a row in shared memory: rows fall on different banks, 16-byte aligned
 
 struct Chunk {
@@ -108,8 +107,8 @@ __device__ __forceinline__ void stage_rows(const T* __restrict__ x, long stride,
 }
 
 // U[chunk][h][v][d] = sum_j a^(n - 1 - j) k_j[d] v_j[v]
-template <typename T, int DP, bool VEC>
-__global__ void __launch_bounds__(kThreads) chunk_own_kernel(const T* __restrict__ k, const T* __restrict__ v, long k_stride, long v_stride,
+template <typename T, int DP, int VT, bool VEC>
+__global__ void __launch_bounds__(kThreads, DP == 128 && VT == 128 ? 2 : 3) chunk_own_kernel(const T* __restrict__ k, const T* __restrict__ v, long k_stride, long v_stride,
                                                              const float* __restrict__ decay, const int* __restrict__ plan, int R,
                                                              Stage st, float* __restrict__ own, int H, int dim, int vdim) {
   pdl_launch_dependents();
@@ -117,44 +116,50 @@ __global__ void __launch_bounds__(kThreads) chunk_own_kernel(const T* __restrict
   constexpr int PITCH = DP + kPad;
   constexpr int ND = DP / 16;                           // numbers of d a thread holds: groups of min(4, ND), 64 apart
   constexpr int GD = ND < 4 ? ND : 4;
+  constexpr int NV = VT / 16;                           // columns of v a thread holds: groups of four, 64 apart
   extern __shared__ __align__(16) float sm[];
   float* ks = sm;                                       // [kC][PITCH], times the decay's power
-  float* vs = ks + kC * PITCH;                          // [kC][kVT]
-  float* pw = vs + kC * kVT;                            // [kC]
+  float* vs = ks + kC * PITCH;                          // [kC][VT]
+  float* pw = vs + kC * VT;                             // [kC]
   const Chunk ch = reinterpret_cast<const Chunk*>(plan + ((R + 1 + 3) & ~3))[blockIdx.z];
-  const int h = blockIdx.y, v0 = blockIdx.x * kVT;
+  const int h = blockIdx.y, v0 = blockIdx.x * VT;
   const float a = decay[h];
   if (threadIdx.x < kC) pw[threadIdx.x] = threadIdx.x < ch.n ? powf(a, (float)(ch.n - 1 - threadIdx.x)) : 0.f;
   __syncthreads();
   stage_rows<T, DP, VEC>(k + (size_t)h * dim, k_stride, ch.t0, ch.n, dim, st, 1.0f, pw, ks);
-  for (int idx = threadIdx.x; idx < kC * kVT; idx += kThreads) {
-    const int tt = idx / kVT, c = v0 + idx - tt * kVT;
+  for (int idx = threadIdx.x; idx < kC * VT; idx += kThreads) {
+    const int tt = idx / VT, c = v0 + idx - tt * VT;
     float x = (tt < ch.n && c < vdim) ? to_f32(v[(size_t)(ch.t0 + tt) * v_stride + (size_t)h * vdim + c]) : 0.f;
     vs[idx] = st.act ? silu(x) : x;
   }
   __syncthreads();
   const int td = threadIdx.x & 15, tv = threadIdx.x >> 4;
-  float acc[4][ND];
+  float acc[NV][ND];
 #pragma unroll
-  for (int i = 0; i < 4; ++i)
+  for (int i = 0; i < NV; ++i)
 #pragma unroll
     for (int d = 0; d < ND; ++d) acc[i][d] = 0.f;
+#pragma unroll 2
   for (int j = 0; j < ch.n; ++j) {
-    const float4 vv = *reinterpret_cast<const float4*>(vs + j * kVT + tv * 4);
-    const float vr[4] = {vv.x, vv.y, vv.z, vv.w};
+    float vr[NV];
+#pragma unroll
+    for (int g = 0; g < NV / 4; ++g) {
+      const float4 vv = *reinterpret_cast<const float4*>(vs + j * VT + g * 64 + tv * 4);
+      vr[4 * g] = vv.x, vr[4 * g + 1] = vv.y, vr[4 * g + 2] = vv.z, vr[4 * g + 3] = vv.w;
+    }
 #pragma unroll
     for (int g = 0; g < ND / GD; ++g) {
       float kr[GD];
       load_vec<float, GD>(ks + j * PITCH + g * 16 * GD + td * GD, kr);
 #pragma unroll
-      for (int i = 0; i < 4; ++i)
+      for (int i = 0; i < NV; ++i)
 #pragma unroll
         for (int d = 0; d < GD; ++d) acc[i][g * GD + d] = fmaf(vr[i], kr[d], acc[i][g * GD + d]);
     }
   }
 #pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const int c = v0 + tv * 4 + i;
+  for (int i = 0; i < NV; ++i) {
+    const int c = v0 + (i >> 2) * 64 + tv * 4 + (i & 3);
     if (c >= vdim) break;
     float* o = own + (((size_t)blockIdx.z * H + h) * vdim + c) * dim;
 #pragma unroll
@@ -208,28 +213,48 @@ __global__ void __launch_bounds__(kThreads) chunk_carry_kernel(float* __restrict
   store_vec<float, G>(sp, S);
 }
 
-template <typename T, int DP, bool VEC>
-__global__ void __launch_bounds__(kThreads, DP == 128 ? 2 : 3) chunk_out_kernel(
+__device__ __forceinline__ void copy16(float* dst, const float* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+
+template <typename T, int DP, int VT, bool VEC>
+__global__ void __launch_bounds__(kThreads, VT == 128 ? 1 : 2) chunk_out_kernel(
     const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, long q_stride, long k_stride, long v_stride,
     const float* __restrict__ decay, const int* __restrict__ plan, int R, Stage st, const float* __restrict__ before,
     float* __restrict__ out, int H, int dim, int vdim, float q_scale) {
   pdl_launch_dependents();
   pdl_wait();
   constexpr int PITCH = DP + kPad, AP = kC + kPad;
+  constexpr int NC = VT / 16;                           // columns a thread holds, 16 apart
   extern __shared__ __align__(16) float sm[];
   float* qs = sm;                                       // [kC][PITCH]
-  float* ks = qs + kC * PITCH;                          // [kC][PITCH]; the memory's columns [kVT][PITCH] once the scores are formed
-  float* as = ks + kC * PITCH;                          // [kC][AP] scores with the decay's powers
-  float* vt = as + kC * AP;                             // [kVT][AP] v transposed
-  float* pw = vt + kVT * AP;                            // [kC + 1]
+  float* ks = qs + kC * PITCH;                          // [kC][PITCH]
+  float* ms = ks + kC * PITCH;                          // [VT][PITCH] the memory's columns
+  float* as = ms + VT * PITCH;                          // [kC][AP] scores with the decay's powers
+  float* vt = as + kC * AP;                             // [VT][AP] v transposed
+  float* pw = vt + VT * AP;                             // [kC + 1]
   const Chunk ch = reinterpret_cast<const Chunk*>(plan + ((R + 1 + 3) & ~3))[blockIdx.z];
-  const int h = blockIdx.y, v0 = blockIdx.x * kVT, n = ch.n;
+  const int h = blockIdx.y, v0 = blockIdx.x * VT, n = ch.n;
   const float a = decay[h];
   if (threadIdx.x <= kC) pw[threadIdx.x] = powf(a, (float)threadIdx.x);
+  // the memory before the chunk: on its way while q, k and v are staged and the scores are formed
+  const float* bp = before + (((size_t)blockIdx.z * H + h) * vdim + v0) * dim;
+  constexpr int G = VEC ? 4 : 1;
+  for (int idx = threadIdx.x; idx < VT * (DP / G); idx += kThreads) {
+    const int c = idx / (DP / G), e = (idx - c * (DP / G)) * G;
+    float* dst = ms + c * PITCH + e;
+    if (v0 + c < vdim && e < dim) {
+      if (VEC) copy16(dst, bp + (size_t)c * dim + e);
+      else *dst = bp[(size_t)c * dim + e];
+    } else {
+#pragma unroll
+      for (int g = 0; g < G; ++g) dst[g] = 0.f;
+    }
+  }
   stage_rows<T, DP, VEC>(q + (size_t)h * dim, q_stride, ch.t0, n, dim, st, q_scale, nullptr, qs);
   stage_rows<T, DP, VEC>(k + (size_t)h * dim, k_stride, ch.t0, n, dim, st, 1.0f, nullptr, ks);
-  for (int idx = threadIdx.x; idx < kVT * (kC / 4); idx += kThreads) {        // a column, four tokens
-    const int c = idx & (kVT - 1), j0 = (idx / kVT) * 4;
+  for (int idx = threadIdx.x; idx < VT * (kC / 4); idx += kThreads) {        // a column, four tokens
+    const int c = idx & (VT - 1), j0 = (idx / VT) * 4;
     float x[4];
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
@@ -240,20 +265,20 @@ __global__ void __launch_bounds__(kThreads, DP == 128 ? 2 : 3) chunk_out_kernel(
   }
   __syncthreads();
   const int tc = threadIdx.x & 15, ti = threadIdx.x >> 4;
-  float acc[4][4];
   // acc[i][c] += sum_e x[ti * 4 + i][e] y[tc + 16 c][e]
-  auto product = [&](const float* x, const float* y, int xp, int yp, int len) {
+  auto product = [&](auto& acc, const float* x, const float* y, int xp, int yp, int len) {
+    constexpr int N = sizeof(acc[0]) / sizeof(float);
+#pragma unroll 2
     for (int e = 0; e < len; e += 4) {
-      float4 xr[4], yr[4];
+      float4 xr[4], yr[N];
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        xr[i] = *reinterpret_cast<const float4*>(x + (ti * 4 + i) * xp + e);
-        yr[i] = *reinterpret_cast<const float4*>(y + (tc + 16 * i) * yp + e);
-      }
+      for (int i = 0; i < 4; ++i) xr[i] = *reinterpret_cast<const float4*>(x + (ti * 4 + i) * xp + e);
+#pragma unroll
+      for (int c = 0; c < N; ++c) yr[c] = *reinterpret_cast<const float4*>(y + (tc + 16 * c) * yp + e);
 #pragma unroll
       for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
+        for (int c = 0; c < N; ++c) {
           acc[i][c] = fmaf(xr[i].x, yr[c].x, acc[i][c]);
           acc[i][c] = fmaf(xr[i].y, yr[c].y, acc[i][c]);
           acc[i][c] = fmaf(xr[i].z, yr[c].z, acc[i][c]);
@@ -261,63 +286,59 @@ __global__ void __launch_bounds__(kThreads, DP == 128 ? 2 : 3) chunk_out_kernel(
         }
     }
   };
+  {
+    float sc[4][kC / 16];
 #pragma unroll
-  for (int i = 0; i < 4; ++i)
+    for (int i = 0; i < 4; ++i)
 #pragma unroll
-    for (int c = 0; c < 4; ++c) acc[i][c] = 0.f;
-  product(qs, ks, PITCH, PITCH, DP);
+      for (int c = 0; c < kC / 16; ++c) sc[i][c] = 0.f;
+    product(sc, qs, ks, PITCH, PITCH, DP);
 #pragma unroll
-  for (int i = 0; i < 4; ++i)
+    for (int i = 0; i < 4; ++i)
 #pragma unroll
-    for (int c = 0; c < 4; ++c) {
-      const int row = ti * 4 + i, col = tc + 16 * c;
-      as[row * AP + col] = col <= row ? acc[i][c] * pw[row - col] : 0.f;
-      acc[i][c] = 0.f;
-    }
-  __syncthreads();                                      // the keys have been read
-  const float* bp = before + (((size_t)blockIdx.z * H + h) * vdim + v0) * dim;
-  constexpr int G = VEC ? 4 : 1;
-  for (int idx = threadIdx.x; idx < kVT * (DP / G); idx += kThreads) {
-    const int c = idx / (DP / G), e = (idx - c * (DP / G)) * G;
-    float x[G];
-#pragma unroll
-    for (int g = 0; g < G; ++g) x[g] = 0.f;
-    if (v0 + c < vdim && e < dim) load_vec<float, G>(bp + (size_t)c * dim + e, x);
-#pragma unroll
-    for (int g = 0; g < G; ++g) ks[c * PITCH + e + g] = x[g];
+      for (int c = 0; c < kC / 16; ++c) {
+        const int row = ti * 4 + i, col = tc + 16 * c;
+        as[row * AP + col] = col <= row ? sc[i][c] * pw[row - col] : 0.f;
+      }
   }
+  if (VEC) asm volatile("cp.async.wait_all;\n" ::: "memory");
   __syncthreads();
-  product(qs, ks, PITCH, PITCH, DP);
+  float acc[4][NC];
 #pragma unroll
   for (int i = 0; i < 4; ++i)
 #pragma unroll
-    for (int c = 0; c < 4; ++c) acc[i][c] *= pw[ti * 4 + i + 1];
-  product(as, vt, AP, AP, (min(n, ti * 4 + 4) + 3) & ~3);        // scores beyond the query's own place are zero
+    for (int c = 0; c < NC; ++c) acc[i][c] = 0.f;
+  product(acc, qs, ms, PITCH, PITCH, DP);
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int c = 0; c < NC; ++c) acc[i][c] *= pw[ti * 4 + i + 1];
+  product(acc, as, vt, AP, AP, (min(n, ti * 4 + 4) + 3) & ~3);        // scores beyond the query's own place are zero
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
     if (ti * 4 + i >= n) break;
     float* o = out + ((size_t)(ch.t0 + ti * 4 + i) * H + h) * vdim + v0;
 #pragma unroll
-    for (int c = 0; c < 4; ++c)
+    for (int c = 0; c < NC; ++c)
       if (v0 + tc + 16 * c < vdim) o[tc + 16 * c] = acc[i][c];
   }
 }
 
-template <typename T, int DP, bool VEC>
+template <typename T, int DP, int VT, bool VEC>
 int launch_as(const void* q, const void* k, const void* v, int q_stride, int k_stride, int v_stride, const float* decay, float* state,
               long slot_stride, const int* state_slots, const int* plan, int chunks, const Stage& st, float* own, float* out, int R, int H,
               int dim, int vdim, float q_scale, cudaStream_t s) {
-  const dim3 grid((vdim + kVT - 1) / kVT, H, chunks);
-  const size_t smem1 = (size_t)(kC * (DP + kPad) + kC * kVT + kC) * sizeof(float);
-  const size_t smem3 = (size_t)(2 * kC * (DP + kPad) + 2 * kC * (kC + kPad) + kC + 4) * sizeof(float);
+  const dim3 grid((vdim + VT - 1) / VT, H, chunks);
+  const size_t smem1 = (size_t)(kC * (DP + kPad) + kC * VT + kC) * sizeof(float);
+  const size_t smem3 = (size_t)((2 * kC + VT) * (DP + kPad) + (kC + VT) * (kC + kPad) + kC + 4) * sizeof(float);
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(chunk_own_kernel<T, DP, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(chunk_out_kernel<T, DP, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem3);
+    cudaError_t e = cudaFuncSetAttribute(chunk_own_kernel<T, DP, VT, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(chunk_out_kernel<T, DP, VT, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem3);
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
-  launch_kernel(chunk_own_kernel<T, DP, VEC>, grid, dim3(kThreads), smem1, s, 1, (const T*)k, (const T*)v, (long)k_stride, (long)v_stride, decay,
+  launch_kernel(chunk_own_kernel<T, DP, VT, VEC>, grid, dim3(kThreads), smem1, s, 1, (const T*)k, (const T*)v, (long)k_stride, (long)v_stride, decay,
                 plan, R, st, own, H, dim, vdim);
   const long total = (long)H * vdim * dim;
   if (dim % 4 == 0 && slot_stride % 4 == 0 && vec_aligned<4>(state, 4) && vec_aligned<4>(own, 4))
@@ -326,7 +347,7 @@ int launch_as(const void* q, const void* k, const void* v, int q_stride, int k_s
   else
     launch_kernel(chunk_carry_kernel<1>, dim3((unsigned)((total + kThreads - 1) / kThreads), R), dim3(kThreads), 0, s, 1, own, decay, plan, R,
                   state, slot_stride, state_slots, (long)vdim * dim, total);
-  launch_kernel(chunk_out_kernel<T, DP, VEC>, grid, dim3(kThreads), smem3, s, 1, (const T*)q, (const T*)k, (const T*)v, (long)q_stride,
+  launch_kernel(chunk_out_kernel<T, DP, VT, VEC>, grid, dim3(kThreads), smem3, s, 1, (const T*)q, (const T*)k, (const T*)v, (long)q_stride,
                 (long)k_stride, (long)v_stride, decay, plan, R, st, own, out, H, dim, vdim, q_scale);
   return launch_status();
 }
@@ -361,14 +382,15 @@ ARLE_API int arle_decay_chunks(const void* q, const void* k, const void* v, int 
   const size_t el = dtype == 0 ? 4 : 2;
   const bool vec = dim % 4 == 0 && rotary_dim % 8 == 0 && q_stride % 4 == 0 && k_stride % 4 == 0 && vec_aligned<4>(q, el) && vec_aligned<4>(k, el) &&
                    vec_aligned<4>(angles, 4) && vec_aligned<4>(own, 4);
-#define ARLE_CHUNKS(TT, D, V) \
-  return launch_as<TT, D, V>(q, k, v, q_stride, k_stride, v_stride, decay, state, slot_stride, state_slots, plan, chunks, st, own, out, R, H, dim, \
-                             vdim, q_scale, s)
+#define ARLE_CHUNKS(TT, D, VT, V) \
+  return launch_as<TT, D, VT, V>(q, k, v, q_stride, k_stride, v_stride, decay, state, slot_stride, state_slots, plan, chunks, st, own, out, R, H, \
+                                 dim, vdim, q_scale, s)
 #define ARLE_CHUNKS_D(TT, V) \
   do { \
-    if (dim <= 32) ARLE_CHUNKS(TT, 32, V); \
-    if (dim <= 64) ARLE_CHUNKS(TT, 64, V); \
-    ARLE_CHUNKS(TT, 128, V); \
+    if (dim <= 32) ARLE_CHUNKS(TT, 32, 64, V); \
+    if (dim <= 64) ARLE_CHUNKS(TT, 64, 64, V); \
+    if (vdim <= 64) ARLE_CHUNKS(TT, 128, 64, V); \
+    ARLE_CHUNKS(TT, 128, 128, V); \
   } while (0)
   if (dtype == 0) {
     if (vec) ARLE_CHUNKS_D(float, true);

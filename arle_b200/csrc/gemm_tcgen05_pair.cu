@@ -2,7 +2,7 @@
 //     out[M, N] = x[M, K] . W[N, K]^T      (float32 accumulation, bfloat16 or float32 out)
 // or, gated, out[M, N / 2] = silu(x . W[2i]) * (x . W[2i + 1]) for a weight whose rows 2i and 2i + 1 are
 // gate_i and up_i (the first half of a gated feed-forward without the round trip of the product through
-// memory and without the kernel that applies the gate).
+// memory and without the kernel that applies the gate), or out = max(sum, 0)^2 for an ungated feed-forward's first half.
 //
 // Why two SMs: a 128 x 256 tile fed from one SM's shared memory needs 48 KB per 64 elements of K, and at
 // the tensor cores' pace that is more than an SM can take in from L2 (the one-SM kernel, gemm_tcgen05.cu,
@@ -247,6 +247,13 @@ __global__ void __launch_bounds__(kThreads, 1) gemm_tcgen05_pair_kernel(const __
           }
         } else {
           OutT* dst = out + (size_t)row * ldo + col;
+          if (act == 3) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) {
+              const float z = fmaxf(__uint_as_float(r[i]), 0.f);
+              r[i] = __float_as_uint(z * z);
+            }
+          }
           if (sizeof(OutT) == 2) {
             if (col + 32 <= N && (((uintptr_t)dst) & 15) == 0) {
               uint32_t p[16];
@@ -325,18 +332,19 @@ int launch(const void* x, int ldx, const void* W, int ldw, void* out, int ldo, i
 }  // namespace
 
 // out_dtype: 0 float32, 1 bfloat16.  gated != 0: W holds (gate_i, up_i) in rows 2i and 2i + 1 and out is bfloat16
-// [M, N / 2] (N even); gated 1: the gate is silu, 2: the tanh form of gelu.  Needs K, ldx, ldw multiples of 8 and 16-byte aligned x and W.  err: set to 3 if a bounded
+// [M, N / 2] (N even); gated 1: the gate is silu, 2: the tanh form of gelu; 3: not gated, out [M, N] = max(sum, 0)^2.  Needs K, ldx, ldw multiples of 8 and 16-byte aligned x and W.  err: set to 3 if a bounded
 // wait ran out.
 ARLE_API int arle_gemm_tcgen05_pair(const void* x, int ldx, const void* W, int ldw, void* out, int out_dtype, int ldo, int M,
                                     int N, int K, int gated, int* err, cudaStream_t s) {
   if (M <= 0 || N <= 0) return 0;
+  if (gated < 0 || gated > 3) return ARLE_E_BADARG;
   if (K <= 0 || K % 8 != 0 || ldx % 8 != 0 || ldw % 8 != 0) return ARLE_E_UNSUPPORTED;
   if (((uintptr_t)x & 15) || ((uintptr_t)W & 15)) return ARLE_E_UNSUPPORTED;
-  if (gated) {
+  if (gated == 1 || gated == 2) {
     if (N % 2 != 0 || out_dtype != 1) return ARLE_E_BADARG;
     return launch<6, true, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, M, N, K, gated, err, s);
   }
-  if (out_dtype == 1) return launch<6, false, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, M, N, K, 0, err, s);
-  if (out_dtype == 0) return launch<6, false, float>(x, ldx, W, ldw, out, ldo, M, N, K, 0, err, s);
+  if (out_dtype == 1) return launch<6, false, __nv_bfloat16>(x, ldx, W, ldw, out, ldo, M, N, K, gated, err, s);
+  if (out_dtype == 0) return launch<6, false, float>(x, ldx, W, ldw, out, ldo, M, N, K, gated, err, s);
   return ARLE_E_BADARG;
 }

@@ -59,10 +59,23 @@ __global__ void __launch_bounds__(kScanThreads) decay_scan_kernel(
   if (longest > 0 && end - beg > longest) return;        // another kernel's row
   float* sp = state + (size_t)state_slots[r] * slot_stride + (size_t)h * vcols * dim;
   float S[CPT][EPL];
+  // columns on 16-byte boundaries: four numbers an access
+  const bool vec = (dim & 3) == 0 && (slot_stride & 3) == 0 && ((uintptr_t)state & 15) == 0;
+  if (vec) {
 #pragma unroll
-  for (int j = 0; j < CPT; ++j)
+    for (int j = 0; j < CPT; ++j)
 #pragma unroll
-    for (int i = 0; i < EPL; ++i) S[j][i] = (c0 + cl0 + j < vcols && e0 + i < dim) ? sp[(size_t)(c0 + cl0 + j) * dim + e0 + i] : 0.f;
+      for (int i = 0; i < EPL; i += 4) {
+        const float4 f = (c0 + cl0 + j < vcols && e0 + i < dim) ? *reinterpret_cast<const float4*>(sp + (size_t)(c0 + cl0 + j) * dim + e0 + i)
+                                                                : make_float4(0.f, 0.f, 0.f, 0.f);
+        S[j][i] = f.x, S[j][i + 1] = f.y, S[j][i + 2] = f.z, S[j][i + 3] = f.w;
+      }
+  } else {
+#pragma unroll
+    for (int j = 0; j < CPT; ++j)
+#pragma unroll
+      for (int i = 0; i < EPL; ++i) S[j][i] = (c0 + cl0 + j < vcols && e0 + i < dim) ? sp[(size_t)(c0 + cl0 + j) * dim + e0 + i] : 0.f;
+  }
 
   // Rows of more than one chunk: the NEXT chunk's q, k, v, a and b are asked for before this chunk's steps run and wait in
   // registers (as they lie in memory) until the steps are done; the chain of steps then never waits for memory.  A thread
@@ -200,6 +213,15 @@ __global__ void __launch_bounds__(kScanThreads) decay_scan_kernel(
           if (c0 + cl0 + j < vcols) op[j] = p[j];
       }
     }
+  }
+  if (vec) {
+#pragma unroll
+    for (int j = 0; j < CPT; ++j)
+#pragma unroll
+      for (int i = 0; i < EPL; i += 4)
+        if (c0 + cl0 + j < vcols && e0 + i < dim)
+          *reinterpret_cast<float4*>(sp + (size_t)(c0 + cl0 + j) * dim + e0 + i) = make_float4(S[j][i], S[j][i + 1], S[j][i + 2], S[j][i + 3]);
+    return;
   }
 #pragma unroll
   for (int j = 0; j < CPT; ++j)

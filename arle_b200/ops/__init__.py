@@ -475,7 +475,7 @@ def gemm_tcgen05_pair(x, w, out, gated: bool = False, activation: str = "silu") 
     """out[M, N] = x[M, K] . w[N, K]^T on the tcgen05 tensor cores with two SMs to a 256 x 256 tile
     (``cta_group::2``).  ``gated``: w holds (gate_i, up_i) in rows 2i and 2i + 1 and out [M, N / 2] gets
     act(gate) * up (``activation`` "silu" or "gelu_tanh"), the gate applied to the float32 sums in the kernel's
-    epilogue."""
+    epilogue.  Not gated, ``activation`` may be "square_relu": out = max(sum, 0)^2 ("silu": none)."""
     M, K = x.shape
     N = w.shape[0]
     No = N // 2 if gated else N
@@ -483,8 +483,8 @@ def gemm_tcgen05_pair(x, w, out, gated: bool = False, activation: str = "silu") 
             or (gated and (N % 2 or out.dtype != torch.bfloat16))):
         raise KernelError(f"gemm_tcgen05_pair: unsupported operands x {tuple(x.shape)} w {tuple(w.shape)} out {tuple(out.shape)}")
     _check(library().arle_gemm_tcgen05_pair(_ptr(x), x.stride(0), _ptr(w), w.stride(0), _ptr(out), _dt(out), out.stride(0), M,
-                                            N, K, (1 + ACTIVATIONS[activation]) if gated else 0, _ptr(error_flag(x.device)),
-                                            _stream()), "gemm_tcgen05_pair")
+                                            N, K, (1 + ACTIVATIONS[activation]) if gated else 3 * int(activation == "square_relu"),
+                                            _ptr(error_flag(x.device)), _stream()), "gemm_tcgen05_pair")
 
 
 def skinny_gemm_supported(x, w, out) -> bool:
@@ -1833,8 +1833,8 @@ def square_relu(x, out) -> None:
 
 def gemm_square_relu(x, w: torch.Tensor, out: torch.Tensor) -> None:
     """out = max(x . w^T, 0)^2: the first half of an ungated feed-forward.  Few rows of x take one launch of the
-    weight-streaming kernel (the activation on its float32 sums; ``x`` may be ``ScaledRows``); otherwise the product is followed by the
-    activation."""
+    weight-streaming kernel (the activation on its float32 sums; ``x`` may be ``ScaledRows``), many rows (1,024 and more)
+    the two-SM tcgen05 kernel, which squares in its epilogue; otherwise the product is followed by the activation."""
     if isinstance(x, ScaledRows):
         if not (fused_gemm_supported(x.rows, w) and tuple(out.shape) == (x.shape[0], w.shape[0])):
             raise KernelError("gemm_square_relu: rows that lack their norm factor need the fused weight-streaming kernel")
@@ -1842,6 +1842,10 @@ def gemm_square_relu(x, w: torch.Tensor, out: torch.Tensor) -> None:
         return
     if fused_gemm_supported(x, w) and skinny_gemm_supported(x, w, out) and w.shape[1] == x.shape[1] and tuple(out.shape) == (x.shape[0], w.shape[0]):
         _fused_gemm(x, w, out, 3, None, None)
+        return
+    if (_KERNEL_SET == "fast" and x.shape[0] >= _GATED_TCGEN05_MIN_ROWS and x.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
+            and w.shape[1] == x.shape[1] and tcgen05_gemm_supported(x, w, out)):
+        gemm_tcgen05_pair(x, w, out, activation="square_relu")
         return
     gemm(x, w, out)
     square_relu(out, out)

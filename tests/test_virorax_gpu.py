@@ -171,6 +171,18 @@ def test_product_into_the_residual_with_a_factor_and_joining_rows(M, N, K):
     ops.check_errors(DEV)
 
 
+@pytest.mark.parametrize("M,N,K", [(1024, 320, 128), (1100, 1000, 256), (2048, 96, 72)])
+def test_first_half_of_an_ungated_feed_forward_on_the_two_sm_kernel(M, N, K):
+    g = torch.Generator().manual_seed(N)
+    x, w = torch.randn(M, K, generator=g).to(torch.bfloat16), (torch.randn(N, K, generator=g) / math.sqrt(K)).to(torch.bfloat16)
+    want = torch.relu(x.double() @ w.double().t()) ** 2
+    for fn in (lambda out: ops.gemm_tcgen05_pair(x.to(DEV), w.to(DEV), out, activation="square_relu"), lambda out: ops.gemm_square_relu(x.to(DEV), w.to(DEV), out)):
+        out = torch.full((M, N), float("nan"), dtype=torch.bfloat16, device=DEV)
+        fn(out)
+        ops.check_errors(DEV)
+        torch.testing.assert_close(out.double().cpu(), want, rtol=1e-2, atol=1e-2)
+
+
 @pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
 @pytest.mark.parametrize("nq,nkv,hd,vd,window,ps", [(4, 2, 16, 24, 7, 4), (1, 1, 12, 40, 5, 8), (6, 2, 8, 4, 1, 16), (3, 1, 48, 48, 33, 16),
                                                     (2, 2, 80, 32, 0, 4), (5, 5, 20, 20, 40, 16)])
