@@ -64,51 +64,90 @@ struct Stage {                          // how q and k are read
 
 __device__ __forceinline__ float silu(float x) { return x / (1.0f + expf(-x)); }
 
-// rows 0 .. n-1 of x (row stride `stride`, dim numbers), rotated, times scale (and w[row], if given), into dst [kC][DP + kPad];
-// zeros past dim and past n.
-template <typename T, int DP, bool VEC>
-__device__ __forceinline__ void stage_rows(const T* __restrict__ x, long stride, int t0, int n, int dim, const Stage& st, float scale,
-                                           const float* w, float* dst) {
-  constexpr int PITCH = DP + kPad;
-  constexpr int G = VEC ? 4 : 1;
+// rows 0 .. n-1 of NS arrays (row strides given, dim numbers), rotated, times scale (and w[row], if given), into dst [kC][DP + kPad];
+// zeros past dim and past n.  Four numbers an access; a thread's loads of up to four places are asked for together.
+template <typename T, int DP, int NS>
+__device__ __forceinline__ void stage_rows_vec(const T* const (&x)[NS], const long (&stride)[NS], int t0, int n, int dim, const Stage& st,
+                                               const float (&scale)[NS], const float* w, float* const (&dst)[NS]) {
+  constexpr int PITCH = DP + kPad, Q = DP / 4, ITEMS = kC * Q / kThreads, B = ITEMS < 4 ? ITEMS : 4;
+  typedef Pack<T, 4> P4;
   const int half = st.rotary_dim >> 1;
-  for (int idx = threadIdx.x; idx < kC * (DP / G); idx += kThreads) {
-    const int tt = idx / (DP / G), e = (idx - tt * (DP / G)) * G;
-    float v[G];
 #pragma unroll
-    for (int g = 0; g < G; ++g) v[g] = 0.f;
-    if (tt < n && e < dim) {
-      const T* row = x + (size_t)(t0 + tt) * stride;
-      load_vec<T, G>(row + e, v);
-      if (e < st.rotary_dim) {
-        const bool first = e < half;
-        const int i0 = first ? e : e - half;
-        float o[G], cs[2 * G];
-        load_vec<T, G>(row + (first ? e + half : i0), o);
-        const float* a = reinterpret_cast<const float*>(st.angles + (size_t)(t0 + tt) * half + i0);
+  for (int b0 = 0; b0 < ITEMS; b0 += B) {
+    P4 own[NS][B], other[NS][B];
+    float4 ca[B], cb[B];
 #pragma unroll
-        for (int g = 0; g < 2 * G; g += G == 1 ? 1 : 4) {
-          if constexpr (G == 1) cs[g] = a[g];
-          else {
-            const float4 f = *reinterpret_cast<const float4*>(a + g);
-            cs[g] = f.x, cs[g + 1] = f.y, cs[g + 2] = f.z, cs[g + 3] = f.w;
-          }
-        }
+    for (int b = 0; b < B; ++b) {
+      const int idx = threadIdx.x + (b0 + b) * kThreads;
+      const int tt = idx / Q, e = (idx - tt * Q) * 4;
+      const bool in = tt < n && e < dim;
+      const bool turns = in && e < st.rotary_dim, first = e < half;
+      ca[b] = cb[b] = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-        for (int g = 0; g < G; ++g) v[g] = first ? v[g] * cs[2 * g] - o[g] * cs[2 * g + 1] : v[g] * cs[2 * g] + o[g] * cs[2 * g + 1];
+      for (int m = 0; m < NS; ++m) {
+        const T* p = x[m] + (size_t)(t0 + tt) * stride[m] + e;
+#pragma unroll
+        for (int g = 0; g < 4; ++g) own[m][b].e[g] = other[m][b].e[g] = from_f32<T>(0.f);
+        if (in) own[m][b] = *reinterpret_cast<const P4*>(p);
+        if (turns) other[m][b] = *reinterpret_cast<const P4*>(first ? p + half : p - half);
       }
-      const float f = w ? scale * w[tt] : scale;
-#pragma unroll
-      for (int g = 0; g < G; ++g) v[g] = (st.act ? silu(v[g]) : v[g]) * f;
+      if (turns) {
+        const float4* a = reinterpret_cast<const float4*>(st.angles + (size_t)(t0 + tt) * half + (first ? e : e - half));
+        ca[b] = a[0];
+        cb[b] = a[1];
+      }
     }
 #pragma unroll
-    for (int g = 0; g < G; ++g) dst[tt * PITCH + e + g] = v[g];
+    for (int b = 0; b < B; ++b) {
+      const int idx = threadIdx.x + (b0 + b) * kThreads;
+      const int tt = idx / Q, e = (idx - tt * Q) * 4;
+      const bool turns = tt < n && e < st.rotary_dim;
+      const float side = e < half ? -1.f : 1.f;
+      const float cs[4] = {ca[b].x, ca[b].z, cb[b].x, cb[b].z}, sn[4] = {ca[b].y, ca[b].w, cb[b].y, cb[b].w};
+#pragma unroll
+      for (int m = 0; m < NS; ++m) {
+        const float f = w ? scale[m] * w[tt] : scale[m];
+        float v[4];
+#pragma unroll
+        for (int g = 0; g < 4; ++g) {
+          v[g] = to_f32(own[m][b].e[g]);
+          if (turns) v[g] = v[g] * cs[g] + side * (to_f32(other[m][b].e[g]) * sn[g]);
+          v[g] = (st.act ? silu(v[g]) : v[g]) * f;
+        }
+        *reinterpret_cast<float4*>(dst[m] + tt * PITCH + e) = make_float4(v[0], v[1], v[2], v[3]);
+      }
+    }
+  }
+}
+
+// The same number by number, for rows that are not on the boundaries the other needs.
+template <typename T, int DP>
+__device__ __forceinline__ void stage_rows_any(const T* __restrict__ x, long stride, int t0, int n, int dim, const Stage& st, float scale,
+                                               const float* w, float* dst) {
+  constexpr int PITCH = DP + kPad;
+  const int half = st.rotary_dim >> 1;
+  for (int idx = threadIdx.x; idx < kC * DP; idx += kThreads) {
+    const int tt = idx / DP, e = idx - tt * DP;
+    float v = 0.f;
+    if (tt < n && e < dim) {
+      const T* row = x + (size_t)(t0 + tt) * stride;
+      v = to_f32(row[e]);
+      if (e < st.rotary_dim) {
+        const bool first = e < half;
+        const int i = first ? e : e - half;
+        const float2 a = st.angles[(size_t)(t0 + tt) * half + i];
+        const float o = to_f32(row[first ? e + half : i]);
+        v = first ? v * a.x - o * a.y : v * a.x + o * a.y;
+      }
+      v = (st.act ? silu(v) : v) * (w ? scale * w[tt] : scale);
+    }
+    dst[tt * PITCH + e] = v;
   }
 }
 
 // U[chunk][h][v][d] = sum_j a^(n - 1 - j) k_j[d] v_j[v]
 template <typename T, int DP, int VT, bool VEC>
-__global__ void __launch_bounds__(kThreads, DP == 128 && VT == 128 ? 2 : 3) chunk_own_kernel(const T* __restrict__ k, const T* __restrict__ v, long k_stride, long v_stride,
+__global__ void __launch_bounds__(kThreads, 2) chunk_own_kernel(const T* __restrict__ k, const T* __restrict__ v, long k_stride, long v_stride,
                                                              const float* __restrict__ decay, const int* __restrict__ plan, int R,
                                                              Stage st, float* __restrict__ own, int H, int dim, int vdim) {
   pdl_launch_dependents();
@@ -126,11 +165,36 @@ __global__ void __launch_bounds__(kThreads, DP == 128 && VT == 128 ? 2 : 3) chun
   const float a = decay[h];
   if (threadIdx.x < kC) pw[threadIdx.x] = threadIdx.x < ch.n ? powf(a, (float)(ch.n - 1 - threadIdx.x)) : 0.f;
   __syncthreads();
-  stage_rows<T, DP, VEC>(k + (size_t)h * dim, k_stride, ch.t0, ch.n, dim, st, 1.0f, pw, ks);
-  for (int idx = threadIdx.x; idx < kC * VT; idx += kThreads) {
-    const int tt = idx / VT, c = v0 + idx - tt * VT;
-    float x = (tt < ch.n && c < vdim) ? to_f32(v[(size_t)(ch.t0 + tt) * v_stride + (size_t)h * vdim + c]) : 0.f;
-    vs[idx] = st.act ? silu(x) : x;
+  if constexpr (VEC) {
+    constexpr int Q = VT / 4, ITEMS = kC * Q / kThreads;
+    Pack<T, 4> x[ITEMS];
+#pragma unroll
+    for (int i = 0; i < ITEMS; ++i) {
+      const int idx = threadIdx.x + i * kThreads;
+      const int tt = idx / Q, c = v0 + (idx - tt * Q) * 4;
+#pragma unroll
+      for (int g = 0; g < 4; ++g) x[i].e[g] = from_f32<T>(0.f);
+      if (tt < ch.n && c < vdim) x[i] = *reinterpret_cast<const Pack<T, 4>*>(v + (size_t)(ch.t0 + tt) * v_stride + (size_t)h * vdim + c);
+    }
+    const T* const src[1] = {k + (size_t)h * dim};
+    const long strides[1] = {k_stride};
+    const float one[1] = {1.0f};
+    float* const dst[1] = {ks};
+    stage_rows_vec<T, DP, 1>(src, strides, ch.t0, ch.n, dim, st, one, pw, dst);
+#pragma unroll
+    for (int i = 0; i < ITEMS; ++i) {
+      float y[4];
+#pragma unroll
+      for (int g = 0; g < 4; ++g) y[g] = st.act ? silu(to_f32(x[i].e[g])) : to_f32(x[i].e[g]);
+      *reinterpret_cast<float4*>(vs + (threadIdx.x + i * kThreads) * 4) = make_float4(y[0], y[1], y[2], y[3]);
+    }
+  } else {
+    stage_rows_any<T, DP>(k + (size_t)h * dim, k_stride, ch.t0, ch.n, dim, st, 1.0f, pw, ks);
+    for (int idx = threadIdx.x; idx < kC * VT; idx += kThreads) {
+      const int tt = idx / VT, c = v0 + idx - tt * VT;
+      const float x = (tt < ch.n && c < vdim) ? to_f32(v[(size_t)(ch.t0 + tt) * v_stride + (size_t)h * vdim + c]) : 0.f;
+      vs[idx] = st.act ? silu(x) : x;
+    }
   }
   __syncthreads();
   const int td = threadIdx.x & 15, tv = threadIdx.x >> 4;
@@ -251,17 +315,47 @@ __global__ void __launch_bounds__(kThreads, VT == 128 ? 1 : 2) chunk_out_kernel(
       for (int g = 0; g < G; ++g) dst[g] = 0.f;
     }
   }
-  stage_rows<T, DP, VEC>(q + (size_t)h * dim, q_stride, ch.t0, n, dim, st, q_scale, nullptr, qs);
-  stage_rows<T, DP, VEC>(k + (size_t)h * dim, k_stride, ch.t0, n, dim, st, 1.0f, nullptr, ks);
-  for (int idx = threadIdx.x; idx < VT * (kC / 4); idx += kThreads) {        // a column, four tokens
-    const int c = idx & (VT - 1), j0 = (idx / VT) * 4;
-    float x[4];
+  if constexpr (VEC) {
+    // v: four columns of four tokens a thread, turned round in registers; eight lanes write a column's tokens side by side
+    constexpr int CG = VT / 4, ITEMS = CG * (kC / 4) / kThreads;
+    Pack<T, 4> x[ITEMS][4];
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      x[i] = (j0 + i < n && v0 + c < vdim) ? to_f32(v[(size_t)(ch.t0 + j0 + i) * v_stride + (size_t)h * vdim + v0 + c]) : 0.f;
-      if (st.act) x[i] = silu(x[i]);
+    for (int it = 0; it < ITEMS; ++it) {
+      const int idx = threadIdx.x + it * kThreads;
+      const int j0 = ((idx & 7) + idx / (8 * CG) * 8) * 4, c = (idx / 8) % CG * 4;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+#pragma unroll
+        for (int g = 0; g < 4; ++g) x[it][i].e[g] = from_f32<T>(0.f);
+        if (j0 + i < n && v0 + c < vdim)
+          x[it][i] = *reinterpret_cast<const Pack<T, 4>*>(v + (size_t)(ch.t0 + j0 + i) * v_stride + (size_t)h * vdim + v0 + c);
+      }
     }
-    *reinterpret_cast<float4*>(vt + c * AP + j0) = make_float4(x[0], x[1], x[2], x[3]);
+    const T* const src[2] = {q + (size_t)h * dim, k + (size_t)h * dim};
+    const long strides[2] = {q_stride, k_stride};
+    const float scales[2] = {q_scale, 1.0f};
+    float* const dst[2] = {qs, ks};
+    stage_rows_vec<T, DP, 2>(src, strides, ch.t0, n, dim, st, scales, nullptr, dst);
+#pragma unroll
+    for (int it = 0; it < ITEMS; ++it) {
+      const int idx = threadIdx.x + it * kThreads;
+      const int j0 = ((idx & 7) + idx / (8 * CG) * 8) * 4, c = (idx / 8) % CG * 4;
+#pragma unroll
+      for (int g = 0; g < 4; ++g) {
+        float y[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) y[i] = st.act ? silu(to_f32(x[it][i].e[g])) : to_f32(x[it][i].e[g]);
+        *reinterpret_cast<float4*>(vt + (c + g) * AP + j0) = make_float4(y[0], y[1], y[2], y[3]);
+      }
+    }
+  } else {
+    stage_rows_any<T, DP>(q + (size_t)h * dim, q_stride, ch.t0, n, dim, st, q_scale, nullptr, qs);
+    stage_rows_any<T, DP>(k + (size_t)h * dim, k_stride, ch.t0, n, dim, st, 1.0f, nullptr, ks);
+    for (int idx = threadIdx.x; idx < VT * kC; idx += kThreads) {
+      const int c = idx & (VT - 1), j = idx / VT;
+      const float x = (j < n && v0 + c < vdim) ? to_f32(v[(size_t)(ch.t0 + j) * v_stride + (size_t)h * vdim + v0 + c]) : 0.f;
+      vt[c * AP + j] = st.act ? silu(x) : x;
+    }
   }
   __syncthreads();
   const int tc = threadIdx.x & 15, ti = threadIdx.x >> 4;
@@ -380,7 +474,8 @@ ARLE_API int arle_decay_chunks(const void* q, const void* k, const void* v, int 
   if (dim > 128 || H > 65535 || chunks > 65535 || R > 65535) return ARLE_E_UNSUPPORTED;
   const Stage st{reinterpret_cast<const float2*>(angles), rotary_dim, act};
   const size_t el = dtype == 0 ? 4 : 2;
-  const bool vec = dim % 4 == 0 && rotary_dim % 8 == 0 && q_stride % 4 == 0 && k_stride % 4 == 0 && vec_aligned<4>(q, el) && vec_aligned<4>(k, el) &&
+  const bool vec = dim % 4 == 0 && vdim % 4 == 0 && rotary_dim % 8 == 0 && q_stride % 4 == 0 && k_stride % 4 == 0 && v_stride % 4 == 0 &&
+                   vec_aligned<4>(q, el) && vec_aligned<4>(k, el) && vec_aligned<4>(v, el) &&
                    vec_aligned<4>(angles, 4) && vec_aligned<4>(own, 4);
 #define ARLE_CHUNKS(TT, D, VT, V) \
   return launch_as<TT, D, VT, V>(q, k, v, q_stride, k_stride, v_stride, decay, state, slot_stride, state_slots, plan, chunks, st, own, out, R, H, \
