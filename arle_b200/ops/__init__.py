@@ -1831,9 +1831,14 @@ def square_relu(x, out) -> None:
     _check(library().arle_square_relu(_ptr(x), x.stride(0), _ptr(out), out.stride(0), _dt(x), T, width, _stream()), "square_relu")
 
 
+# Rows from which the product with the square in its epilogue beats cuBLAS followed by the activation: 6 to 13 % at 4,096 and 8,192
+# rows of 3,072 x 1,024 to 18,432 x 4,096 weights; level at 2,048, behind below.
+SQUARE_RELU_TCGEN05_MIN_ROWS = 4096
+
+
 def gemm_square_relu(x, w: torch.Tensor, out: torch.Tensor) -> None:
     """out = max(x . w^T, 0)^2: the first half of an ungated feed-forward.  Few rows of x take one launch of the
-    weight-streaming kernel (the activation on its float32 sums; ``x`` may be ``ScaledRows``), many rows (1,024 and more)
+    weight-streaming kernel (the activation on its float32 sums; ``x`` may be ``ScaledRows``), many rows (4,096 and more)
     the two-SM tcgen05 kernel, which squares in its epilogue; otherwise the product is followed by the activation."""
     if isinstance(x, ScaledRows):
         if not (fused_gemm_supported(x.rows, w) and tuple(out.shape) == (x.shape[0], w.shape[0])):
@@ -1843,7 +1848,7 @@ def gemm_square_relu(x, w: torch.Tensor, out: torch.Tensor) -> None:
     if fused_gemm_supported(x, w) and skinny_gemm_supported(x, w, out) and w.shape[1] == x.shape[1] and tuple(out.shape) == (x.shape[0], w.shape[0]):
         _fused_gemm(x, w, out, 3, None, None)
         return
-    if (_KERNEL_SET == "fast" and x.shape[0] >= _GATED_TCGEN05_MIN_ROWS and x.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
+    if (_KERNEL_SET == "fast" and x.shape[0] >= SQUARE_RELU_TCGEN05_MIN_ROWS and x.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
             and w.shape[1] == x.shape[1] and tcgen05_gemm_supported(x, w, out)):
         gemm_tcgen05_pair(x, w, out, activation="square_relu")
         return

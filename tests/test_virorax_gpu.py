@@ -171,7 +171,7 @@ def test_product_into_the_residual_with_a_factor_and_joining_rows(M, N, K):
     ops.check_errors(DEV)
 
 
-@pytest.mark.parametrize("M,N,K", [(1024, 320, 128), (1100, 1000, 256), (2048, 96, 72)])
+@pytest.mark.parametrize("M,N,K", [(1024, 320, 128), (1100, 1000, 256), (4096, 96, 72)])
 def test_first_half_of_an_ungated_feed_forward_on_the_two_sm_kernel(M, N, K):
     g = torch.Generator().manual_seed(N)
     x, w = torch.randn(M, K, generator=g).to(torch.bfloat16), (torch.randn(N, K, generator=g) / math.sqrt(K)).to(torch.bfloat16)
